@@ -6,7 +6,8 @@ repository carries them:
 
 * ``lib/libb200_kernels.so``  - every ``csrc/kernels/*.cu`` and ``csrc/comm/*.cu``;
   plain C entry points, loaded with ctypes (no torch headers, so a kernel edit
-  rebuilds in seconds).
+  rebuilds in seconds).  ``build_kernel_subset`` makes ``lib/libb200_<name>.so`` from
+  the sources one model family needs, for a checkout that has not been built.
 * ``lib/libb200_core.so`` + ``pocketllm_cpp`` pybind module - the C++ runtime
   (block pool/table, scheduler, command channel, readers, tokenizer, sampler).
 * ``lib/libb200_cpu.so`` - AVX2 multi-threaded host kernels (FP4 and INT8 routed experts on the CPU).
@@ -37,6 +38,8 @@ CXX = os.environ.get("CXX", "g++")
 ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]
 NVCC_FLAGS = ARCH + ["-lineinfo", "-O3", "-std=c++17", "--use_fast_math", "-Xcompiler", "-fPIC",
                      "-Xcompiler", "-fvisibility=default", "--expt-relaxed-constexpr"]
+# Kernels that also serve the fp32 runtimes: exact division, square root and exponentials instead of the fast variants.
+PRECISE = {"residual_norm.cu", "bias_act.cu", "qk_row_prep.cu", "attn_mix_rows.cu", "gemm_f32.cu"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-pthread"]
 # A compiler that links its C++ runtime statically would otherwise export that runtime's symbols from every module;
 # in a process that has already loaded another libstdc++ (torch) the dynamic linker then binds half of a stream or
@@ -68,7 +71,8 @@ def _needs(src: Path, obj: Path) -> bool:
 def _compile_cu(src: Path) -> Path:
     obj = OBJ / (src.stem + ".cu.o")
     if _needs(src, obj):
-        _run([NVCC, *NVCC_FLAGS, "-I", str(CSRC), "-c", str(src), "-o", str(obj)])
+        flags = [f for f in NVCC_FLAGS if f != "--use_fast_math" or src.name not in PRECISE]
+        _run([NVCC, *flags, "-I", str(CSRC), "-c", str(src), "-o", str(obj)])
     return obj
 
 
@@ -90,6 +94,25 @@ def build_kernels(jobs: int | None = None) -> Path:
     if (not out.exists()) or any(o.stat().st_mtime > out.stat().st_mtime for o in objs):
         _run([NVCC, *ARCH, "-shared", "-o", str(out), *map(str, objs), "-lcudart_static", "-lpthread",
               "-ldl", "-lrt"])
+    return out
+
+
+def build_kernel_subset(name: str, sources, jobs: int | None = None) -> Path:
+    """``lib/libb200_<name>.so`` from the given ``csrc/kernels`` files only (every symbol must resolve among them).
+    Serialised by a lock file: several processes may start in the same fresh checkout."""
+    import fcntl
+    OBJ.mkdir(exist_ok=True)
+    LIB.mkdir(exist_ok=True)
+    out = LIB / f"libb200_{name}.so"
+    with open(OBJ / f"{name}.lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        with cf.ThreadPoolExecutor(max_workers=jobs or os.cpu_count() or 4) as ex:
+            objs = list(ex.map(_compile_cu, [CSRC / "kernels" / s for s in sources]))
+        if (not out.exists()) or any(o.stat().st_mtime > out.stat().st_mtime for o in objs):
+            part = out.with_suffix(f".so.{os.getpid()}")
+            _run([NVCC, *ARCH, "-shared", "-Xlinker", "-z,defs", "-o", str(part), *map(str, objs), "-lcudart_static", "-lpthread",
+                  "-ldl", "-lrt"])
+            os.replace(part, out)
     return out
 
 

@@ -1,0 +1,49 @@
+// y = xIELU(z + bias) over rows: for z > 0  ap z^2 + z / 2,  otherwise  an (exp(z) - 1 - z) + z / 2, with the two
+// positive coefficients given as numbers.  bf16 or fp32 data, fp32 arithmetic; `ld` (a multiple of 8) columns per row,
+// columns whose input and bias are zero stay zero.
+#include "launch.h"
+#include "ops.h"
+#include "vec8.cuh"
+
+namespace {
+using namespace b200;
+
+template <typename T>
+__global__ void bias_xielu_kernel(const T* __restrict__ in, const float* __restrict__ bias, T* __restrict__ out,
+                                  long long nvec_total, int nvec, float ap, float an) {
+  pdl_grid_trigger();
+  pdl_grid_wait();
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < nvec_total; i += (long long)gridDim.x * blockDim.x) {
+    float z[8];
+    load8(in + i * 8, z);
+    if (bias) {
+      float b[8];
+      load8(bias + (i % nvec) * 8, b);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) z[j] += b[j];
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const float v = z[j];
+      z[j] = (v > 0.f ? ap * v * v : an * (expm1f(v) - v)) + 0.5f * v;
+    }
+    store8(out + i * 8, z);
+  }
+}
+
+}  // namespace
+
+extern "C" int b200_bias_xielu(const void* in, const float* bias, void* out, long long rows, int ld, float ap, float an,
+                               int f32, cudaStream_t stream) {
+  if (rows <= 0 || ld <= 0 || (ld & 7)) return -6;
+  const int nvec = ld >> 3;
+  const long long total = rows * nvec;
+  const long long blocks = (total + 255) / 256;
+  const dim3 grid((unsigned)(blocks < 148 * 16 ? blocks : 148 * 16));
+  if (f32)
+    return (int)launch_pdl(bias_xielu_kernel<float>, grid, dim3(256), 0, stream, reinterpret_cast<const float*>(in), bias,
+                           reinterpret_cast<float*>(out), total, nvec, ap, an);
+  return (int)launch_pdl(bias_xielu_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream,
+                         reinterpret_cast<const __nv_bfloat16*>(in), bias, reinterpret_cast<__nv_bfloat16*>(out), total, nvec,
+                         ap, an);
+}

@@ -170,6 +170,28 @@ int b200_kv8_dequantize(const void* k8, const void* v8, const float* k_scale, co
                         const int* block_table_row, void* stage_k, void* stage_v, int bs, int n_tokens, int Hkv, int fmt,
                         cudaStream_t stream);
 
+// Decoder layers with norms around each sublayer, an fp32 residual and score mixing across heads (residual_norm.cu,
+// bias_act.cu, qk_row_prep.cu, attn_mix_prefill.cu, attn_mix_rows.cu) and the fp32 projection GEMM (gemm_f32.cu)
+int b200_residual_norm(float* x, const int* ids, const void* table, int vocab, const void* delta, const float* bias,
+                       const float* post_w, const float* step, const float* pre_w, void* out, const int* rows, int n, int ld,
+                       int cols, float eps, int rms, int unit_offset, int write_x, int f32, cudaStream_t stream);
+int b200_bias_xielu(const void* in, const float* bias, void* out, long long rows, int ld, float ap, float an, int f32,
+                    cudaStream_t stream);
+int b200_qk_row_prep(const void* proj, int ld, int q_off, int k_off, int v_off, const float* q_w, const float* k_w,
+                     int q_count, int k_count, float eps, const double* freq, int rot, float mscale, const float* talk_t,
+                     const int* positions, const int* slots, void* q_mix, float* q_row, void* k_cache, void* v_cache, int T,
+                     int n_mix, int H, int G, int D, int f32, cudaStream_t stream);
+int b200_attn_mix_rows(const float* q, const void* k_cache, const void* v_cache, void* out, const float* talk_t,
+                       const int* block_table, const int* seq, const int* positions, float* partial, int rows, int max_blocks,
+                       int block_size, int H, int G, int D, int chunk, int splits, int ldo, float scale, int f32,
+                       cudaStream_t stream);
+int b200_attn_mix_prefill_supported(int H, int G, int D, int block_size);
+int b200_attn_mix_prefill(const void* q_mix, const void* k_cache, const void* v_cache, void* out, const int* block_table,
+                          const int* seq, const int* q_start, const int* q_len, const int* kv_len, int batch, int max_q_len,
+                          int q_rows, int max_blocks, int num_blocks, int block_size, int H, int G, int D, int chunk, int ldo,
+                          float scale, int* status, cudaStream_t stream);
+int b200_gemm_f32(const float* x, const float* w, float* y, int T, int N, int K, cudaStream_t stream);
+
 #ifdef __cplusplus
 }
 #endif

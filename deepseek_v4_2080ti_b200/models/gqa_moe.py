@@ -12,13 +12,14 @@ transformer :443-472), tensor names src/loader/mappings/minimax_m2.py:7-27, meta
 from __future__ import annotations
 
 import math
-from dataclasses import dataclass, field
+from dataclasses import dataclass
 from typing import Any, Iterator
 
 import torch
 
 from ..formats import gguf as G
 from ..formats.gguf import GGMLType
+from .paged import PagedRuntime
 
 ARCH = "minimax-m2"
 
@@ -309,71 +310,38 @@ class GqaMoeGpuWeights:
         return n
 
 
-class _NoComm:
-    world, rank = 1, 0
-
-    def all_reduce(self, t):
-        return t
-
-    def argmax_merge(self, idx, val):
-        return idx
-
-
-@dataclass
-class _Seq:
-    slot: int
-    blocks: list[int] = field(default_factory=list)
-    length: int = 0
-
-
-class GqaMoeRuntime:
-    """Paged-KV runtime: chunked prefill of one sequence, batched decode (CUDA-graph replay per batch size)."""
+class GqaMoeRuntime(PagedRuntime):
+    """Paged-KV runtime of the family (slots, pages, step / prefill / decode: ``models/paged.py``)."""
 
     def __init__(self, cfg: GqaMoeConfig, weights: GqaMoeGpuWeights, max_slots: int = 1, max_context: int = 4096 + 512,
-                 block_size: int = 64, comm=None):
+                 block_size: int = 64, comm=None, num_blocks: int | None = None):
         from ..ops import attention
-        self.cfg, self.w, self.device = cfg, weights, weights.device
-        self.comm = comm or _NoComm()
+        super().__init__(weights.device, max_slots, max_context, block_size, num_blocks, comm)
+        self.cfg, self.w = cfg, weights
         assert self.comm.world == weights.world
-        self.block_size, self.max_slots = block_size, max_slots
-        self.max_blocks = (max_context + block_size - 1) // block_size
-        self.num_blocks = self.max_blocks * max_slots + 1
         dev = self.device
         self.k_cache = torch.zeros(cfg.n_layers, self.num_blocks, weights.hkv, block_size, 128, dtype=torch.bfloat16, device=dev)
         self.v_cache = torch.zeros_like(self.k_cache)
         self.inv_freq = attention.rope_inv_freq(cfg.rope_dim, cfg.rope_base, dev)
-        self.free_blocks = list(range(self.num_blocks - 1, 0, -1))
-        self.free_slots = list(range(max_slots - 1, -1, -1))
-        self.seqs: dict[int, _Seq] = {}
-        self.block_table = torch.zeros(max_slots, self.max_blocks, dtype=torch.int32, device=dev)
-        self._bt_host = torch.zeros(max_slots, self.max_blocks, dtype=torch.int32)
-        self._graphs: dict[tuple, dict] = {}
-        self.launches = 0
+        # the whole vocabulary of a step's logits is on this rank: log-probabilities and sampling can use it
+        self.exposes_logits = self.comm.world == 1
 
-    def allocate(self) -> int:
-        s = self.free_slots.pop()
-        self.seqs[s] = _Seq(s)
-        return s
-
-    def free(self, slot: int) -> None:
-        st = self.seqs.pop(slot)
-        self.free_blocks.extend(reversed(st.blocks))
-        self.free_slots.append(slot)
-
-    def _ensure(self, st: _Seq, new_len: int) -> None:
-        need = (new_len + self.block_size - 1) // self.block_size
-        if need > self.max_blocks:
-            raise RuntimeError("sequence exceeds max_context")
-        grown = False
-        while len(st.blocks) < need:
-            if not self.free_blocks:
-                raise RuntimeError("KV cache exhausted")
-            b = self.free_blocks.pop()
-            self._bt_host[st.slot, len(st.blocks)] = b
-            st.blocks.append(b)
-            grown = True
-        if grown:
-            self.block_table[st.slot].copy_(self._bt_host[st.slot], non_blocking=True)
+    def _attend(self, q: torch.Tensor, i: int, meta: dict) -> torch.Tensor:
+        """Attention of the batch's rows over layer ``i``'s cache: portions on the tile kernel, single rows on the
+        split-context kernel."""
+        from ..ops import attention
+        k, v = self.k_cache[i], self.v_cache[i]
+        if meta["mode"] == "prefill":
+            return attention.prefill(q, k, v, meta["block_table"], meta["q_start"], meta["q_len"], meta["kv_len"], meta["max_q_len"])
+        if meta["mode"] == "decode":
+            return attention.decode(q, k, v, meta["block_table"], meta["kv_len"], max_kv_len=meta["max_kv_len"])
+        n, parts = meta["tile_rows"], []
+        if n:
+            parts.append(attention.prefill(q[:n], k, v, meta["tile_table"], meta["q_start"], meta["q_len"], meta["kv_len"],
+                                           meta["max_q_len"]))
+        if n < q.shape[0]:
+            parts.append(attention.decode(q[n:], k, v, meta["row_table"], meta["row_kv_len"], max_kv_len=meta["max_kv_len"]))
+        return parts[0] if len(parts) == 1 else torch.cat(parts)
 
     # ---- one forward pass over T rows
     def _forward(self, ids, positions, kv_slots, meta, last_rows: torch.Tensor | None) -> torch.Tensor:
@@ -382,6 +350,11 @@ class GqaMoeRuntime:
         t = ids.numel()
         d = 128
         qw, kw = w.hq * d, w.hkv * d
+        if meta["mode"] == "mixed":
+            n = meta["tile_rows"]
+            meta = dict(meta, tile_table=self.block_table[meta["tile_seq"].long()] if n else None,
+                        row_table=self.block_table[meta["row_seq"][n:].long()] if n < t else None,
+                        row_kv_len=positions[n:] + 1)
         h = basic.embedding(ids, w.embed, 0, cfg.vocab)
         delta = None
         for i, L in enumerate(w.layers):
@@ -394,12 +367,7 @@ class GqaMoeRuntime:
             q = attention.qk_fullnorm_rope_append(proj, 0, qw, qw + kw, L.q_gamma, L.k_gamma, ss, cfg.n_heads * d,
                                                   cfg.n_kv_heads * d, cfg.norm_eps, self.inv_freq, cfg.rope_dim, positions,
                                                   kv_slots, self.k_cache[i], self.v_cache[i], w.hq, w.hkv)
-            if meta["mode"] == "prefill":
-                o = attention.prefill(q, self.k_cache[i], self.v_cache[i], meta["block_table"], meta["q_start"],
-                                      meta["q_len"], meta["kv_len"], meta["max_q_len"])
-            else:
-                o = attention.decode(q, self.k_cache[i], self.v_cache[i], meta["block_table"], meta["kv_len"],
-                                     max_kv_len=meta["max_kv_len"])
+            o = self._attend(q, i, meta)
             d_attn = comm.all_reduce(gguf_gemm.linear(o.view(t, qw), L.o))
             xn = basic.add_rmsnorm(h, d_attn, L.ffn_norm, cfg.norm_eps, False)      # h += d_attn
             logits = gemm.linear(xn, L.gate, out_f32=True)
@@ -409,6 +377,8 @@ class GqaMoeRuntime:
                                     residual=h)
             delta = None
         if last_rows is not None:
+            if last_rows.numel() == 0:
+                return None
             h = h.index_select(0, last_rows)
         x = basic.rmsnorm(h, w.final_norm, cfg.norm_eps, False)
         return gguf_gemm.linear(x, w.head, out_f32=True)
@@ -417,84 +387,3 @@ class GqaMoeRuntime:
         from ..ops import basic
         idx, val = basic.argmax(logits, self.w.head_lo, True)
         return self.comm.argmax_merge(idx, val)
-
-    @torch.no_grad()
-    def prefill(self, slot: int, token_ids: torch.Tensor, chunk: int = 4096) -> torch.Tensor:
-        from ..ops import _lib
-        st = self.seqs[slot]
-        l0 = _lib.LAUNCHES
-        nxt, total, dev = None, token_ids.numel(), self.device
-        i32 = lambda v: torch.tensor([v], dtype=torch.int32, device=dev)
-        for s in range(0, total, chunk):
-            ids = token_ids[s:s + chunk]
-            t = ids.numel()
-            self._ensure(st, st.length + t)
-            pos = torch.arange(st.length, st.length + t, dtype=torch.int32, device=dev)
-            row = self.block_table[slot]
-            kv_slots = (row[(pos // self.block_size).long()] * self.block_size + pos % self.block_size).to(torch.int32)
-            meta = {"mode": "prefill", "block_table": self.block_table[slot:slot + 1], "q_start": i32(0), "q_len": i32(t),
-                    "kv_len": i32(st.length + t), "max_q_len": t}
-            logits = self._forward(ids, pos, kv_slots, meta, torch.tensor([t - 1], dtype=torch.int64, device=dev))
-            st.length += t
-            if s + t >= total:
-                nxt = self._next(logits)
-        self.launches = _lib.LAUNCHES - l0
-        return nxt
-
-    def _decode_body(self, buf, bucket: int) -> torch.Tensor:
-        meta = {"mode": "decode", "block_table": buf["bt"], "kv_len": buf["kv_len"], "max_kv_len": bucket}
-        return self._next(self._forward(buf["ids"], buf["pos"], buf["kv_slots"], meta, None))
-
-    @torch.no_grad()
-    def decode(self, slots: list[int], token_ids: torch.Tensor, use_graph: bool = True) -> torch.Tensor:
-        from ..ops import _lib
-        b, dev = len(slots), self.device
-        sts = [self.seqs[s] for s in slots]
-        for st in sts:
-            self._ensure(st, st.length + 1)
-        bucket = 1 << max(10, max(st.length for st in sts).bit_length())
-        entry = self._graphs.setdefault((b, bucket), {"buf": None, "graph": None})
-        if entry["buf"] is None:
-            z = lambda *s: torch.zeros(*s, dtype=torch.int32, device=dev)
-            entry["buf"] = {"ids": z(b), "pos": z(b), "kv_slots": z(b), "kv_len": z(b) + 1, "bt": z(b, self.max_blocks)}
-        buf = entry["buf"]
-        host = torch.tensor([[st.length, st.length + 1, st.slot,
-                              st.blocks[st.length // self.block_size] * self.block_size + st.length % self.block_size]
-                             for st in sts], dtype=torch.int32).to(dev, non_blocking=True)
-        buf["ids"].copy_(token_ids)
-        buf["pos"].copy_(host[:, 0])
-        buf["kv_len"].copy_(host[:, 1])
-        buf["kv_slots"].copy_(host[:, 3])
-        buf["bt"].copy_(self.block_table[host[:, 2].long()])
-        if not use_graph:
-            l0 = _lib.LAUNCHES
-            out = self._decode_body(buf, bucket)
-            self.launches = _lib.LAUNCHES - l0
-        else:
-            if entry["graph"] is None:
-                self._decode_body(buf, bucket)          # warm-up: the K/V row written here is rewritten by the replay
-                torch.cuda.synchronize()
-                g = torch.cuda.CUDAGraph()
-                l0 = _lib.LAUNCHES
-                with torch.cuda.graph(g):
-                    entry["out"] = self._decode_body(buf, bucket)
-                entry["graph"], entry["launches"] = g, _lib.LAUNCHES - l0
-            entry["graph"].replay()
-            self.launches = entry["launches"]
-            out = entry["out"]
-        for st in sts:
-            st.length += 1
-        return out
-
-    @torch.no_grad()
-    def generate(self, prompt: torch.Tensor, max_new_tokens: int, chunk: int = 4096, use_graph: bool = True) -> list[int]:
-        slot = self.allocate()
-        try:
-            tok = self.prefill(slot, prompt.to(self.device, torch.int32), chunk)
-            out = [int(tok.item())]
-            while len(out) < max_new_tokens:
-                tok = self.decode([slot], tok.to(torch.int32), use_graph)
-                out.append(int(tok.item()))
-            return out
-        finally:
-            self.free(slot)

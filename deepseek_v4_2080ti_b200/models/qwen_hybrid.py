@@ -22,6 +22,7 @@ from ..utils import canary
 from ..utils.phase_profile import PROFILER
 from ..ops import _lib, attention, basic, gdn, gemm
 from ..ops.gemm import PackedLinear
+from .paged import NoComm, PagedSequences, SeqState
 
 
 # ------------------------------------------------------------------ config
@@ -413,28 +414,7 @@ class QwenHybridWeights:
 
 
 # ------------------------------------------------------------------ runtime
-class NoComm:
-    """Single-rank stand-in for the tensor-parallel communicator."""
-    world, rank = 1, 0
-
-    def all_reduce(self, t: torch.Tensor) -> torch.Tensor:
-        return t
-
-    def argmax_merge(self, idx: torch.Tensor, val: torch.Tensor) -> torch.Tensor:
-        return idx
-
-    def all_gather(self, t: torch.Tensor) -> torch.Tensor:
-        return t.unsqueeze(0)
-
-
-@dataclass
-class SeqState:
-    slot: int
-    blocks: list[int] = field(default_factory=list)
-    length: int = 0
-
-
-class QwenHybridRuntime:
+class QwenHybridRuntime(PagedSequences):
     """Owns weights, the paged KV pool, per-slot recurrent state and the forward passes."""
 
     def __init__(self, cfg: QwenHybridConfig, weights: QwenHybridWeights, max_slots: int = 1,
@@ -463,10 +443,7 @@ class QwenHybridRuntime:
         self.hk_lin = cfg.linear_num_key_heads // W
         self.hv_lin = cfg.linear_num_value_heads // W
         self.kd, self.vd = self.hk_lin * 128, self.hv_lin * 128
-        self.block_size = block_size
-        self.max_slots = max_slots
-        self.max_blocks_per_seq = (max_context + block_size - 1) // block_size
-        self.num_blocks = num_blocks or (self.max_blocks_per_seq * max_slots + 1)
+        super().__init__(weights.device, max_slots, max_context, block_size, num_blocks)
         self.full_layers = [i for i, t in enumerate(cfg.layer_types) if t == "full_attention"]
         self.lin_layers = [i for i, t in enumerate(cfg.layer_types) if t == "linear_attention"]
         dev = self.device
@@ -501,14 +478,8 @@ class QwenHybridRuntime:
         self.tails = torch.zeros(max_slots, nl, cfg.linear_conv_kernel_dim - 1, 2 * self.kd + self.vd,
                                  dtype=torch.bfloat16, device=dev)
         self.inv_freq = attention.rope_inv_freq(cfg.rotary_dim, cfg.rope_theta, dev)
-        self.free_blocks = list(range(self.num_blocks - 1, 0, -1))
-        self.block_refs = [0] * self.num_blocks        # sequences + prefix-cache entries holding each block
         self.prefix_cache = None
         self.prefill_tokens_computed = 0               # prompt tokens actually run through the model (cache hits skip)
-        self.free_slots = list(range(max_slots - 1, -1, -1))
-        self.seqs: dict[int, SeqState] = {}
-        self.block_table = torch.zeros(max_slots, self.max_blocks_per_seq, dtype=torch.int32, device=dev)
-        self._bt_host = torch.zeros(max_slots, self.max_blocks_per_seq, dtype=torch.int32)
         self._graphs: dict[int, tuple] = {}
         self.launches = 0  # kernels launched by the last forward (for the bench record)
         self._sp = False   # set while a sequence-parallel prefill chunk is in flight
@@ -521,22 +492,10 @@ class QwenHybridRuntime:
 
     # ---- slot / block management (host side)
     def allocate(self) -> int:
-        slot = self.free_slots.pop()
-        self.seqs[slot] = SeqState(slot)
+        slot = super().allocate()
         self.states[slot].zero_()
         self.tails[slot].zero_()
         return slot
-
-    def free(self, slot: int) -> None:
-        st = self.seqs.pop(slot)
-        self._release_blocks(st.blocks)
-        self.free_slots.append(slot)
-
-    def _release_blocks(self, blocks: list[int]) -> None:
-        for b in reversed(blocks):
-            self.block_refs[b] -= 1
-            if self.block_refs[b] == 0:
-                self.free_blocks.append(b)
 
     def enable_prefix_cache(self, interval: int = 256, max_entries: int = 8, max_bytes: int = 8 << 30):
         """Re-use KV blocks and recurrent-state snapshots of already-seen prompt prefixes (runtime/prefix_cache.py).
@@ -570,22 +529,6 @@ class QwenHybridRuntime:
         if self.prefix_cache.insert(tokens, n, blocks, snap, nbytes):
             for b in blocks:
                 self.block_refs[b] += 1
-
-    def _ensure_blocks(self, st: SeqState, new_len: int) -> None:
-        need = (new_len + self.block_size - 1) // self.block_size
-        if need > self.max_blocks_per_seq:
-            raise RuntimeError("sequence exceeds max_context")
-        changed = False
-        while len(st.blocks) < need:
-            if not self.free_blocks:
-                raise RuntimeError("KV cache exhausted")
-            b = self.free_blocks.pop()
-            self.block_refs[b] = 1
-            self._bt_host[st.slot, len(st.blocks)] = b
-            st.blocks.append(b)
-            changed = True
-        if changed:
-            self.block_table[st.slot].copy_(self._bt_host[st.slot], non_blocking=True)
 
     def recover_collectives(self) -> None:
         """After a collective timed out: re-synchronise the communicator (all ranks call this) and drop the captured

@@ -1,6 +1,9 @@
-"""Model-family registry for GGUF checkpoints: detect the family from ``general.architecture``, parse its
-hyper-parameters, check the tensor inventory against the family's naming, report which tensor types the runtime can
-execute, and plan placement on a B200 box (everything resident; experts sharded by range).
+"""Model-family registry.
+
+GGUF checkpoints: detect the family from ``general.architecture``, parse its hyper-parameters, check the tensor inventory
+against the family's naming, report which tensor types the runtime can execute, and plan placement on a B200 box
+(everything resident; experts sharded by range).  Checkpoint folders (config.json + safetensors): ``CheckpointSpec``
+recognises a family by its configuration and builds its runtime.
 
 Reference behaviour: the MoE spec registry (src/components/moe/spec.py:80-98, registry.py:10-47), the capability table
 (capability.py:7-63) and the placement decisions (placement.py:9-56)."""
@@ -333,3 +336,93 @@ register(ModelSpec(
                     "output_hc_base.weight", "output_hc_scale.weight"),
     layer_tensors=_v4_layer_tensors, n_layers=lambda p: p.n_layers + (1 if p.mtp else 0),
     routed_suffixes=("ffn_gate_exps.weight", "ffn_up_exps.weight", "ffn_down_exps.weight"), build_runtime=_v4_runtime))
+
+
+# ---------------------------------------------------------------------------------------------- checkpoint folders
+@dataclass(frozen=True)
+class CheckpointSpec:
+    """A family stored as config.json + safetensors.  ``build(raw_config, directory, device, rank=, world=, dtype=,
+    max_slots=, max_context=, num_blocks=, make_comm=)`` returns (config, runtime behind the slot interface)."""
+    name: str
+    display_name: str
+    matches: Callable[[Any], bool]               # parsed config.json -> is it this family?
+    build: Callable[..., Any]
+    chat_family: str | None = None
+    dtypes: tuple[str, ...] = ("bfloat16",)      # activation dtypes the runtime serves in
+    kernel_sources: tuple[str, ...] = ()         # csrc/kernels files it needs (empty: the whole library)
+
+
+_CHECKPOINTS: list[CheckpointSpec] = []
+
+
+def register_checkpoint(spec: CheckpointSpec) -> None:
+    _CHECKPOINTS.append(spec)
+
+
+def detect_checkpoint(raw_config: Any) -> CheckpointSpec | None:
+    """The registered family of a parsed config.json; None when no registered family claims it."""
+    return next((s for s in _CHECKPOINTS if s.matches(raw_config)), None)
+
+
+def checkpoint_families() -> list[str]:
+    return sorted(s.name for s in _CHECKPOINTS)
+
+
+def _torch_dtype(name: str | None, allowed: tuple[str, ...]):
+    import torch
+    name = {None: "bfloat16", "": "bfloat16", "auto": "bfloat16", "bf16": "bfloat16", "fp32": "float32"}.get(name, name)
+    if name not in allowed:
+        raise ValueError(f"dtype {name!r} is not served by this family (available: {', '.join(allowed)})")
+    return getattr(torch, name)
+
+
+def _mla_matches(raw) -> bool:
+    from .mla_moe import MlaMoeConfig
+    return MlaMoeConfig.is_mla_moe_json(raw)
+
+
+def _mla_build(raw, directory, device, rank=0, world=1, dtype=None, max_slots=1, max_context=4096, num_blocks=None,
+               make_comm=None):
+    """MLA + routed-expert checkpoints (DeepSeek inference layout: FP8 block-128 or bf16 dense matrices, FP4 or bf16
+    experts, config.json in the dim / n_layers / n_routed_experts spelling)."""
+    from ..formats import safetensors_io
+    from . import mla_moe_gpu as mg
+    from .mla_moe import MlaMoeConfig
+    cfg = MlaMoeConfig.from_json(raw)
+    comm = make_comm(cfg.hidden_size) if make_comm else None
+    w = mg.MlaMoeGpuWeights(cfg, safetensors_io.read_checkpoint(directory), device, rank, world,
+                            dense_fp8=str(raw.get("dtype", "bf16")).lower() == "fp8")
+    if max_slots > 1:
+        return cfg, mg.MlaMoeBatchRuntime(cfg, w, max_slots=max_slots, max_context=max_context, num_blocks=num_blocks, comm=comm)
+    return cfg, _MlaSlotAdapter(mg.MlaMoeGpuRuntime(cfg, w, max_context=max_context, comm=comm))
+
+
+register_checkpoint(CheckpointSpec("mla_moe", "MLA + routed experts (DeepSeek inference layout)", _mla_matches, _mla_build,
+                                   chat_family="deepseek_v4"))
+
+
+def _rutulix_matches(raw) -> bool:
+    from .rutulix import RutulixConfig
+    return RutulixConfig.is_rutulix_json(raw)
+
+
+def _rutulix_build(raw, directory, device, rank=0, world=1, dtype=None, max_slots=1, max_context=4096, num_blocks=None,
+                   make_comm=None):
+    from ..formats import safetensors_io
+    from . import rutulix as rx
+    if world != 1:
+        raise ValueError("the scores of all heads are mixed: a Rutulix model runs on one rank")
+    cfg = rx.RutulixConfig.from_json(raw)
+    w = rx.RutulixWeights(cfg, safetensors_io.read_checkpoint(directory), device,
+                          _torch_dtype(dtype, ("bfloat16", "float32")))
+    return cfg, rx.RutulixRuntime(cfg, w, max_slots=max_slots, max_context=max_context, num_blocks=num_blocks)
+
+
+def _rutulix_sources() -> tuple[str, ...]:
+    from .rutulix import KERNEL_SOURCES
+    return KERNEL_SOURCES
+
+
+register_checkpoint(CheckpointSpec("rutulix", "Rutulix (head-mixed chunked attention, sandwich norms, looped layers)",
+                                   _rutulix_matches, _rutulix_build, dtypes=("bfloat16", "float32"),
+                                   kernel_sources=_rutulix_sources()))

@@ -61,6 +61,17 @@ def lib() -> ctypes.CDLL:
     return _lib
 
 
+def use_subset(name: str, sources) -> None:
+    """Let this process run on the kernels of one model family: when the full library has not been built, compile
+    ``sources`` (csrc/kernels files) into ``lib/libb200_<name>.so`` and load that.  No effect once the full library
+    exists or a library is loaded."""
+    global _LIB_PATH
+    if _lib is not None or _LIB_PATH.exists() or not sources:
+        return
+    from .. import build as _build
+    _LIB_PATH = _build.build_kernel_subset(name, sources)
+
+
 def stream() -> ctypes.c_void_p:
     return ctypes.c_void_p(torch.cuda.current_stream().cuda_stream)
 

@@ -89,6 +89,7 @@ def prefill(q, k_cache, v_cache, block_table, q_start, q_len, kv_len, max_q_len,
 
 
 _dec_ws: dict[int, torch.Tensor] = {}
+_outgrown: list[torch.Tensor] = []      # smaller workspaces stay alive: captured graphs hold their addresses
 
 
 def decode(q, k_cache, v_cache, block_table, kv_len, gate=None, scale=None, splits: int | None = None,
@@ -109,6 +110,8 @@ def decode(q, k_cache, v_cache, block_table, kv_len, gate=None, scale=None, spli
         dev = q.device.index or 0
         ws = _dec_ws.get(dev)
         if ws is None or ws.numel() < need:
+            if ws is not None:
+                _outgrown.append(ws)
             ws = torch.empty(max(need, 1 << 20), dtype=torch.float32, device=q.device)
             _dec_ws[dev] = ws
     rc = _lib.lib().b200_gqa_decode_ex(_lib.ptr(q), _lib.ptr(k_cache), _lib.ptr(v_cache), _lib.ptr(out), _lib.ptr(gate),
@@ -181,6 +184,8 @@ def decode_kv8(fmt: int, q, k8, v8, k_scale, v_scale, block_table, kv_len, gate=
         dev = q.device.index or 0
         ws = _dec_ws.get(dev)
         if ws is None or ws.numel() < need:
+            if ws is not None:
+                _outgrown.append(ws)
             ws = torch.empty(max(need, 1 << 20), dtype=torch.float32, device=q.device)
             _dec_ws[dev] = ws
     rc = _lib.lib().b200_gqa_decode_kv8(int(fmt), _lib.ptr(q), _lib.ptr(k8), _lib.ptr(v8), _lib.ptr(k_scale),

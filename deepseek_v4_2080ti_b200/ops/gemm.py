@@ -75,6 +75,7 @@ class PackedLinear:
 
 
 _workspaces: dict[int, tuple[torch.Tensor, torch.Tensor]] = {}
+_outgrown: list[torch.Tensor] = []      # smaller scratch buffers stay alive: captured graphs hold their addresses
 MAX_TILE_COUNTERS = 1 << 16
 
 
@@ -84,6 +85,8 @@ def _workspace(nfloats: int, device) -> tuple[torch.Tensor, torch.Tensor]:
     key = torch.device(device).index or 0
     ws = _workspaces.get(key)
     if ws is None or ws[0].numel() < nfloats:
+        if ws is not None:
+            _outgrown.append(ws[0])
         ws = (canary.empty(max(nfloats, 1 << 22), dtype=torch.float32, device=device, name="gemm split-K partials"),
               ws[1] if ws is not None else canary.zeros(MAX_TILE_COUNTERS, dtype=torch.int32, device=device,
                                                         name="gemm tile counters"))

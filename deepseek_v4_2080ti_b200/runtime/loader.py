@@ -3,7 +3,9 @@ for this rank, open the rank-0 -> workers command channel.
 
 Model strings:
   ``synthetic:qwen-tiny`` / ``synthetic:qwen-27b``  random-init models generated on the device
-  a directory with ``config.json`` + safetensors      Qwen-style hybrid FP8 checkpoints
+  ``synthetic:rutulix-tiny``                          likewise, the Rutulix decoder
+  a directory with ``config.json`` + safetensors      a family of ``models.registry`` (MLA + experts, Rutulix), else a
+                                                      Qwen-style hybrid FP8 checkpoint
   a ``.gguf`` file or bundle                          MoE families (routed by ``general.architecture``)
 """
 from __future__ import annotations
@@ -466,6 +468,26 @@ def _device(args) -> torch.device:
     return torch.device("cuda", int(os.environ.get("LOCAL_RANK", "0")))
 
 
+def checkpoint_family(directory: str, config_path: str | None = None):
+    """(parsed config.json or None, registered family or None) of a checkpoint folder."""
+    import json
+    from ..models import registry
+    try:
+        with open(config_path or os.path.join(directory, "config.json")) as f:
+            raw = json.load(f)
+    except (OSError, ValueError):
+        return None, None
+    return raw, registry.detect_checkpoint(raw)
+
+
+def build_family(spec, raw_config, directory: str, device, **kw):
+    """(config, runtime) of a registered checkpoint family on ``device``.  In a checkout without the full kernel library
+    only the kernels of the family are compiled."""
+    from ..ops import _lib
+    _lib.use_subset(spec.name, spec.kernel_sources)
+    return spec.build(raw_config, directory, device, **kw)
+
+
 def _load_host(args):
     """The Qwen-style hybrid on the host (``device="cpu"``): fp32 oracle, one rank, every drafter
     (``runtime/host_runtime.py``)."""
@@ -480,9 +502,13 @@ def _load_host(args):
         base = os.environ.get("POCKETLLM_NCCL_ID_PATH") or f"/tmp/pocketllm-{os.environ.get('MASTER_PORT', '0')}"
         channel = Channel(base, rank, world)
     model = args.model
+    if not model.startswith("synthetic:"):
+        spec = checkpoint_family(args.checkpoint_dir, args.config_path)[1]
+        if spec is not None:
+            raise ConfigurationError(f"the {spec.name} family needs a GPU")
     if model.startswith("synthetic:"):
-        if "tiny" not in model:
-            raise ConfigurationError("the host path generates only the tiny synthetic model")
+        if "tiny" not in model or "rutulix" in model:
+            raise ConfigurationError("the host path generates only the tiny synthetic hybrid model")
         cfg = qh.QwenHybridConfig.tiny()
         state = qh.synth_state(cfg, 0, "cpu", std=0.05)
     else:
@@ -566,31 +592,25 @@ def load_runtime(args):
         from pocketllm.backends.native_backend import NullChannel
         return CppRuntimeAdapter(args.checkpoint_dir, dev.index or 0, max_ctx, slots,
                                  args.prefill_chunk_tokens or 8192), None, NullChannel()
-    if not model.startswith("synthetic:"):
-        # MLA + routed-expert checkpoints (DeepSeek inference layout: FP8 block-128 or bf16 dense matrices, FP4 or
-        # bf16 experts, config.json in the dim / n_layers / n_routed_experts spelling) as safetensors shards
-        import json as _json
-        from ..models.mla_moe import MlaMoeConfig
-        cfg_path = args.config_path or os.path.join(args.checkpoint_dir, "config.json")
-        try:
-            with open(cfg_path) as f:
-                raw_cfg = _json.load(f)
-        except (OSError, ValueError):
-            raw_cfg = None
-        if MlaMoeConfig.is_mla_moe_json(raw_cfg):
-            from ..formats import safetensors_io
-            from ..models import mla_moe_gpu as mg
-            from ..models.registry import _MlaSlotAdapter
+    raw_cfg, family_spec = None, None
+    if model.startswith("synthetic:"):
+        if model.split(":", 1)[1] == "rutulix-tiny":
+            from ..models import rutulix as rx
             from pocketllm.backends.native_backend import NullChannel
-            mcfg = MlaMoeConfig.from_json(raw_cfg)
-            comm = make_comm(mcfg.hidden_size)
-            w = mg.MlaMoeGpuWeights(mcfg, safetensors_io.read_checkpoint(args.checkpoint_dir), dev, rank, world,
-                                    dense_fp8=str(raw_cfg.get("dtype", "bf16")).lower() == "fp8")
-            if slots > 1:
-                rt = mg.MlaMoeBatchRuntime(mcfg, w, max_slots=slots, max_context=max_ctx, comm=comm)
-            else:
-                rt = _MlaSlotAdapter(mg.MlaMoeGpuRuntime(mcfg, w, max_context=max_ctx, comm=comm))
-            return GgufRuntimeAdapter(rt, max_ctx, slots, dev), "deepseek_v4", channel or NullChannel()
+            rt = rx.build_synthetic(rx.RutulixConfig.tiny(), dev, max_slots=slots, max_context=max_ctx)
+            return GgufRuntimeAdapter(rt, max_ctx, slots, dev), None, channel or NullChannel()
+    else:
+        raw_cfg, family_spec = checkpoint_family(args.checkpoint_dir, args.config_path)
+    if family_spec is not None:
+        from pocketllm.api.errors import ConfigurationError
+        from pocketllm.backends.native_backend import NullChannel
+        try:
+            _, rt = build_family(family_spec, raw_cfg, args.checkpoint_dir, dev, rank=rank, world=world,
+                                 dtype=args.dtype if len(family_spec.dtypes) > 1 else None, max_slots=slots,
+                                 max_context=max_ctx, make_comm=make_comm)
+        except ValueError as exc:
+            raise ConfigurationError(str(exc)) from exc
+        return GgufRuntimeAdapter(rt, max_ctx, slots, dev), family_spec.chat_family, channel or NullChannel()
     if model.startswith("synthetic:"):
         name = model.split(":", 1)[1]
         cfg = qh.QwenHybridConfig.tiny() if name in ("qwen-tiny", "tiny") else qh.QwenHybridConfig.config2()
