@@ -3,6 +3,8 @@
     python -m torch.distributed.run --nproc-per-node 8 --master-addr 127.0.0.1 -m deepseek_v4_2080ti_b200.cli.generate_gguf \\
         --gguf model.gguf --token-ids 1,2,3 --max-new-tokens 64
 
+or from a folder (config.json + safetensors) of a family in ``models/registry.py``: ``--checkpoint DIR [--dtype float32]``.
+
 Prints the token ids and a ``RESULT prefill_tps=... decode_tps=...`` line (prompt tokens / prefill seconds, generated
 tokens after the first / decode seconds), the format of the reference's GGUF drivers
 (src/runtime/generation.py:168-276, src/cli/generate_gguf.py, generate_glm.py)."""
@@ -17,7 +19,10 @@ import torch
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="generate_gguf")
-    ap.add_argument("--gguf", required=True)
+    src = ap.add_mutually_exclusive_group(required=True)
+    src.add_argument("--gguf")
+    src.add_argument("--checkpoint", help="folder with config.json and safetensors of a registered family")
+    ap.add_argument("--dtype", help="activation dtype of a --checkpoint family that serves several")
     ap.add_argument("--token-ids", default="")
     ap.add_argument("--runtime-option", action="append", default=[], metavar="KEY=VALUE",
                     help="family-specific runtime option, repeatable (deepseek4: dspark=PATH|synthetic, dspark_block=N, "
@@ -37,11 +42,20 @@ def main(argv=None) -> int:
     dev = torch.device("cuda", local) if on_gpu else torch.device("cpu")     # host-only families run without a GPU
     if on_gpu:
         torch.cuda.set_device(dev)
-    b = read_bundle(a.gguf)
-    if a.prewarm:
-        from ..formats.gguf.prewarm import prewarm_bundle
-        prewarm_bundle(b)
-    spec = registry.detect(b)
+    b = raw = None
+    if a.checkpoint:
+        from ..runtime.loader import build_family, checkpoint_family
+        raw, spec = checkpoint_family(a.checkpoint)
+        if spec is None:
+            raise SystemExit(f"{a.checkpoint}: no registered model family claims this configuration")
+        if not on_gpu or not a.token_ids:
+            raise SystemExit("--checkpoint needs a GPU and --token-ids")
+    else:
+        b = read_bundle(a.gguf)
+        if a.prewarm:
+            from ..formats.gguf.prewarm import prewarm_bundle
+            prewarm_bundle(b)
+        spec = registry.detect(b)
     if a.token_ids:
         ids = [int(x) for x in a.token_ids.replace(" ", ",").split(",") if x]
     else:
@@ -57,7 +71,11 @@ def main(argv=None) -> int:
             raise SystemExit(f"--runtime-option {item!r}: expected KEY=VALUE")
         k, v = item.split("=", 1)
         extra[k.strip()] = v.strip()
-    cfg, rt = spec.build_runtime(b, dev, rank, world, comm, max_slots=1, max_context=a.max_context, **extra)
+    if a.checkpoint:
+        cfg, rt = build_family(spec, raw, a.checkpoint, dev, rank=rank, world=world, dtype=a.dtype, max_slots=1,
+                               max_context=a.max_context, make_comm=(lambda hidden: comm) if comm is not None else None)
+    else:
+        cfg, rt = spec.build_runtime(b, dev, rank, world, comm, max_slots=1, max_context=a.max_context, **extra)
     load_s = time.time() - t0
     vocab = int(getattr(cfg, "vocab_size", 0) or getattr(cfg, "vocab", 0) or 0)
     bad = [t for t in ids if t < 0 or (vocab and t >= vocab)]
@@ -82,7 +100,7 @@ def main(argv=None) -> int:
         print("tokens=" + ",".join(map(str, out)))
         if hasattr(rt, "stats"):
             print("runtime_stats " + " ".join(f"{k}={v}" for k, v in rt.stats().items()))
-        print(f"RESULT family={spec.architecture} world={world} load_seconds={load_s:.2f} prompt_tokens={len(ids)} "
+        print(f"RESULT family={spec.name if a.checkpoint else spec.architecture} world={world} load_seconds={load_s:.2f} prompt_tokens={len(ids)} "
               f"prefill_tps={len(ids) / max(t1 - t0, 1e-9):.2f} decode_tps={(len(out) - 1) / max(t2 - t1, 1e-9):.2f}", flush=True)
     if world > 1:
         torch.distributed.barrier()

@@ -1,6 +1,7 @@
 """Inspect a safetensors checkpoint directory without loading it: shards, tensors (dtype, shape, bytes), totals per
-dtype, an optional name filter, and for Qwen-style hybrid checkpoints the weight-map coverage audit (missing /
-unexpected tensors, shapes, dtypes, tensor-parallel divisibility; FP8 block-128 and mixed NVFP4 matrices).
+dtype, an optional name filter, and a coverage audit of the tensor inventory: registered families that list their
+tensors (``models/registry.py: CheckpointSpec``) by name and shape, Qwen-style hybrid checkpoints by the weight map
+(missing / unexpected tensors, shapes, dtypes, tensor-parallel divisibility; FP8 block-128 and mixed NVFP4 matrices).
 
     python -m deepseek_v4_2080ti_b200.cli.inspect_safetensors CKPT_DIR [--grep STR] [--audit] [--tp-world N] [--json]
 
@@ -41,7 +42,7 @@ def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="inspect_safetensors")
     ap.add_argument("checkpoint")
     ap.add_argument("--grep", default="", help="only tensors whose name contains this")
-    ap.add_argument("--audit", action="store_true", help="check the Qwen-style weight map (needs config.json)")
+    ap.add_argument("--audit", action="store_true", help="check the tensor inventory against config.json")
     ap.add_argument("--tp-world", type=int, default=1)
     ap.add_argument("--json", action="store_true")
     a = ap.parse_args(argv)
@@ -49,8 +50,13 @@ def main(argv=None) -> int:
     shown = [t for t in rep["tensors"] if a.grep in t["name"]]
     audit = None
     if a.audit:
-        from .. import pocketllm_cpp as core
-        audit = dict(core.qwen_audit(a.checkpoint, a.tp_world))
+        from ..runtime.loader import checkpoint_family
+        raw, spec = checkpoint_family(a.checkpoint)
+        if spec is not None and spec.tensor_shapes is not None:
+            audit = spec.audit(raw, {t["name"]: tuple(t["shape"]) for t in rep["tensors"]})
+        else:
+            from .. import pocketllm_cpp as core
+            audit = dict(core.qwen_audit(a.checkpoint, a.tp_world))
     if a.json:
         print(json.dumps({**{k: v for k, v in rep.items() if k != "tensors"}, "tensors": shown, "audit": audit}))
     else:
@@ -63,7 +69,7 @@ def main(argv=None) -> int:
                   f"wrong_shard={len(rep['index']['wrong_shard'])}")
         if audit is not None:
             for key in ("missing", "unexpected", "wrong_shape", "wrong_dtype", "not_divisible"):
-                for n in audit[key]:
+                for n in audit.get(key, ()):
                     print(f"audit_{key}={n}")
             print(f"audit ok={int(audit['ok'])} expected={audit['expected']} found={audit['found']} tp_world={a.tp_world}")
     return 0 if audit is None or audit["ok"] else 3

@@ -76,6 +76,16 @@ class PagedSequences:
     def blocks_needed(self, tokens: int) -> int:
         return (tokens + self.block_size - 1) // self.block_size
 
+    def history_span(self) -> int | None:
+        """Largest distance between a position and the first one it can look at (None: unbounded)."""
+        return None
+
+    def pages_held(self, tokens: int, portion: int) -> int:
+        """Upper bound on the pages a sequence of ``tokens`` tokens holds at any time when no step brings more than
+        ``portion`` of them: with a bounded history a step needs the pages from the history's start to its own end."""
+        total, span = self.blocks_needed(tokens), self.history_span()
+        return total if span is None else min(total, self.blocks_needed(span + portion) + 1)
+
     def _ensure_blocks(self, st: SeqState, new_len: int) -> None:
         """Pages for positions up to ``new_len`` of a sequence; pages no later token can see go back first."""
         need = self.blocks_needed(new_len)
@@ -142,6 +152,10 @@ class PagedRuntime(PagedSequences):
         from ..ops import basic
         return basic.argmax(logits)
 
+    def greedy(self, logits: torch.Tensor) -> list[int]:
+        """Arg-max tokens of ``step``'s logits."""
+        return [int(t) for t in self._next(logits.contiguous()).tolist()]
+
     # ---- one batch of portions and single tokens
     @torch.no_grad()
     def step(self, entries) -> torch.Tensor | None:
@@ -178,7 +192,8 @@ class PagedRuntime(PagedSequences):
         want = torch.tensor([first[i] + w for i, e in enumerate(entries) for w in e[2]], dtype=torch.int32)
         desc = torch.tensor([[first[i], lens[i], sts[i].length + lens[i], sts[i].slot] for i in tiles], dtype=torch.int32).reshape(-1)
         # one upload: [ids | positions | cache rows | table rows | tile descriptors | wanted rows]
-        up = cat([tok, pos, rows, seq, desc, want]).pin_memory().to(dev, non_blocking=True)
+        up = cat([tok, pos, rows, seq, desc, want])
+        up = up.pin_memory().to(dev, non_blocking=True) if dev.type == "cuda" else up
         ids, pos_d, slots_d, seq_d = (up[k * n_rows:(k + 1) * n_rows] for k in range(4))
         desc_d = up[4 * n_rows:4 * n_rows + desc.numel()].view(-1, 4)
         meta = {"mode": "mixed", "tile_rows": tile_rows, "row_seq": seq_d, "max_q_len": max([lens[i] for i in tiles], default=0),
@@ -236,7 +251,7 @@ class PagedRuntime(PagedSequences):
         buf["kv_len"].copy_(host[:, 1])
         buf["kv_slots"].copy_(host[:, 3])
         buf["bt"].copy_(self.block_table[host[:, 2].long()])
-        if not use_graph:
+        if not use_graph or dev.type != "cuda":
             l0 = _lib.LAUNCHES
             out = self._decode_body(buf, bucket)
             self.launches = _lib.LAUNCHES - l0

@@ -350,6 +350,16 @@ class CheckpointSpec:
     chat_family: str | None = None
     dtypes: tuple[str, ...] = ("bfloat16",)      # activation dtypes the runtime serves in
     kernel_sources: tuple[str, ...] = ()         # csrc/kernels files it needs (empty: the whole library)
+    tensor_shapes: Callable[[Any], dict[str, tuple[int, ...]]] | None = None     # parsed config.json -> every tensor
+
+    def audit(self, raw_config: Any, have: dict[str, tuple[int, ...]]) -> dict:
+        """Checkpoint inventory (name -> shape) against what the configuration asks for."""
+        want = self.tensor_shapes(raw_config)
+        rep = {"missing": sorted(set(want) - set(have)), "unexpected": sorted(set(have) - set(want)),
+               "wrong_shape": sorted(n for n in want if n in have and tuple(have[n]) != tuple(want[n])),
+               "expected": len(want), "found": sum(n in have for n in want)}
+        rep["ok"] = not (rep["missing"] or rep["unexpected"] or rep["wrong_shape"])
+        return rep
 
 
 _CHECKPOINTS: list[CheckpointSpec] = []
@@ -418,6 +428,11 @@ def _rutulix_build(raw, directory, device, rank=0, world=1, dtype=None, max_slot
     return cfg, rx.RutulixRuntime(cfg, w, max_slots=max_slots, max_context=max_context, num_blocks=num_blocks)
 
 
+def _rutulix_shapes(raw) -> dict[str, tuple[int, ...]]:
+    from .rutulix import RutulixConfig
+    return RutulixConfig.from_json(raw).tensor_shapes()
+
+
 def _rutulix_sources() -> tuple[str, ...]:
     from .rutulix import KERNEL_SOURCES
     return KERNEL_SOURCES
@@ -425,4 +440,4 @@ def _rutulix_sources() -> tuple[str, ...]:
 
 register_checkpoint(CheckpointSpec("rutulix", "Rutulix (head-mixed chunked attention, sandwich norms, looped layers)",
                                    _rutulix_matches, _rutulix_build, dtypes=("bfloat16", "float32"),
-                                   kernel_sources=_rutulix_sources()))
+                                   kernel_sources=_rutulix_sources(), tensor_shapes=_rutulix_shapes))

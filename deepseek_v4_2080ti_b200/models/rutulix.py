@@ -286,6 +286,9 @@ class RutulixRuntime(PagedRuntime):
     def history_floor(self, length: int) -> int:
         return min((length - length % c if c else 0) for c in self.chunks) if self.chunks else 0
 
+    def history_span(self) -> int | None:
+        return max(self.chunks) - 1 if self.chunks and all(self.chunks) else None
+
     def _attention(self, run: int, lw: RutulixLayer, y: torch.Tensor, positions, kv_slots, meta) -> torch.Tensor:
         m, k, v = lw.mix, self.k_cache[run], self.v_cache[run]
         t = y.shape[0]

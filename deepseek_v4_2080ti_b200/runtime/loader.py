@@ -321,14 +321,16 @@ class CppRuntimeAdapter:
 
 
 class GgufRuntimeAdapter:
-    """The same surface over a GGUF family runtime (``models.registry`` builds it: GQA-MoE with paged slots, or the
-    one-sequence MLA runtime): greedy decoding, sequences admitted up to the runtime's slot count."""
+    """The same surface over a registry family's runtime (``models.registry`` builds it: GQA-MoE and Rutulix with paged
+    slots and a mixed-batch step, or the MLA runtimes): sequences admitted up to the runtime's slot count; greedy, and
+    sampled where the runtime leaves its logits on the device."""
     supports_sampling = False
     supports_prefix_cache = False
     speculative_methods: tuple[str, ...] = ()
 
     def __init__(self, rt, max_context: int, max_slots: int, device, eos_token_ids=()):
         self.rt, self.max_context, self.device = rt, max_context, device
+        self.step_tokens = 4096                            # tokens of one mixed-batch pass
         self.max_slots = 1 if getattr(rt, "single_sequence", False) else max(1, int(max_slots))
         self.eos_token_ids = tuple(eos_token_ids)
         self.last_cached_tokens = 0
@@ -415,7 +417,16 @@ class GgufRuntimeAdapter:
         return out
 
     def generate_batch(self, prompts, max_new, eos_ids, max_batch):
+        """Greedy batch.  Runtimes with a mixed-batch step go through ``StepScheduler`` (prompt portions beside decoding
+        requests in one pass); the others prefill one request at a time and decode together."""
         import time
+        if hasattr(self.rt, "step") and getattr(self.rt.comm, "world", 1) == 1 and not self._active:
+            from .step_scheduler import StepScheduler
+            sched = StepScheduler(self.rt, eos_ids, min(int(max_batch), self.max_slots), self.step_tokens)
+            for i, (p, n) in enumerate(zip(prompts, max_new)):
+                sched.submit(i, p, min(int(n), self.max_context - len(p) + 1))
+            done = sched.run()
+            return [done[i] for i in range(len(prompts))]
         results: list[Any] = [None] * len(prompts)
         pending = list(range(len(prompts)))[::-1]
         active: dict[int, dict] = {}
