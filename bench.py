@@ -42,6 +42,10 @@ def parse():
                     help="config 2: also run greedy speculative decoding after the timed steps (mtp: a random-init "
                          "multi-token-prediction head is added to the synthetic checkpoint) and report acceptance")
     ap.add_argument("--spec-tokens", type=int, default=2)
+    ap.add_argument("--design", choices=["rutulix"], default=None,
+                    help="instead of the headline workload: one decoder design at model-like layer sizes beside the closest "
+                         "existing model, with the kernels' roofline fractions (utils/design_bench.py; one GPU)")
+    ap.add_argument("--design-size", choices=["small", "large"], default=None, help="--design: only this size")
     ap.add_argument("--config", type=int, default=2, choices=[2, 3, 4, 5],
                     help="benchmark configuration: 2 Qwen-shaped FP8 hybrid (the headline, default), 3 MiniMax-shaped "
                          "GGUF GQA-MoE, 4 DeepSeek-V4-Flash-shaped MLA + indexer + FP4 MoE, 5 GLM-shaped GGUF DSA-MoE")
@@ -125,6 +129,10 @@ def run_reference(args) -> None:
 
 def main() -> None:
     args = parse()
+    if args.design:
+        from deepseek_v4_2080ti_b200.utils import design_bench
+        print(json.dumps(design_bench.run(args)), flush=True)
+        return
     if args.config != 2:
         run_moe_config(args)
         return

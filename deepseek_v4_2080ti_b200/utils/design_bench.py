@@ -1,0 +1,207 @@
+"""Prefill and decode throughput of the Rutulix decoder at sizes of real models' layers (random weights), beside the
+framework's closest existing model at equal size, and the kernels of both beside their rooflines.
+
+    python bench.py --design rutulix [--design-size small|large] [--steps K] [--warmup W]
+
+Closest model: the Qwen-style decoder with full-attention layers only (per-head QK norm, grouped attention, SwiGLU with
+FP8 weights) of the same width, heads and feed-forward parameters.  Whole-model numbers: CUDA events around a prompt of
+``--prompt`` tokens and around replayed decode steps.  Kernel numbers: CUDA events around single launches, L2 flushed
+before each; fractions of the measured copy bandwidth / bf16 GEMM burst of MEASURED_PEAKS.json.
+"""
+from __future__ import annotations
+
+import json
+import os
+
+import torch
+
+PEAKS_FALLBACK = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
+# width, heads, kv heads, head dim, SwiGLU width of the closest model (the two-matrix feed-forward gets 3/2 of it), chunk
+SIZES = {"small": (2048, 16, 4, 128, 5632, 2048), "large": (4096, 32, 8, 128, 10752, 8192)}
+LAYERS, VOCAB = 4, 32768
+
+
+def _peaks() -> tuple[dict, str]:
+    path = os.path.join(os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__)))), "MEASURED_PEAKS.json")
+    try:
+        with open(path) as f:
+            return json.load(f), "of measured"
+    except OSError:
+        return PEAKS_FALLBACK, "of fallback"
+
+
+class _Timer:
+    def __init__(self, dev, steps: int, warmup: int):
+        self.steps, self.warmup = max(3, steps), max(3, warmup)
+        self.flush = torch.empty(96 << 20, dtype=torch.int32, device=dev)       # 384 MB, larger than L2
+
+    def __call__(self, fn, flush: bool = True) -> float:
+        """Median milliseconds of one call."""
+        ms = []
+        for i in range(self.warmup + self.steps):
+            if flush:
+                self.flush.fill_(i)
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            fn()
+            b.record()
+            torch.cuda.synchronize()
+            if i >= self.warmup:
+                ms.append(a.elapsed_time(b))
+        return sorted(ms)[len(ms) // 2]
+
+
+def _models(size: str, dev, prompt: int, slots: int):
+    from ..models import qwen_hybrid as qh
+    from ..models import rutulix as rx
+    width, heads, kv, dim, inter, chunk = SIZES[size]
+    cfg = rx.RutulixConfig.uniform(LAYERS, width, heads, kv, dim, inter * 3 // 2, VOCAB, chunk)
+    new = lambda: rx.build_synthetic(cfg, dev, max_slots=slots, max_context=prompt + 192)
+    qcfg = qh.QwenHybridConfig(vocab_size=VOCAB, hidden_size=width, intermediate_size=inter, num_hidden_layers=LAYERS,
+                               num_attention_heads=heads, num_key_value_heads=kv, attn_output_gate=False,
+                               layer_types=["full_attention"] * LAYERS)
+    old = lambda: qh.build_synthetic(qcfg, dev, max_slots=slots, max_context=prompt + 192)
+    return new, old
+
+
+def _throughput(make, dev, prompt: int, slots: int, timer: _Timer) -> dict:
+    rt = make()
+    gen = torch.Generator().manual_seed(1)
+    ids = torch.randint(0, VOCAB, (prompt,), generator=gen, dtype=torch.int32).to(dev)
+    slot = rt.allocate()
+
+    def prefill():
+        nonlocal slot
+        rt.free(slot)
+        slot = rt.allocate()
+        rt.prefill(slot, ids, prompt)
+    out = {"prefill_tok_s": round(prompt / timer(prefill) * 1e3, 0)}
+    slots_l = [slot]
+    while len(slots_l) < slots:
+        s = rt.allocate()
+        rt.prefill(s, ids, prompt)
+        slots_l.append(s)
+    for b in (1, slots):
+        tok = torch.ones(b, dtype=torch.int32, device=dev)
+        ms = timer(lambda: rt.decode(slots_l[:b], tok))
+        out[f"decode_b{b}_tok_s"] = round(b / ms * 1e3, 1)
+        out[f"decode_b{b}_ms"] = round(ms, 4)
+    return out
+
+
+def _kernels(size: str, dev, timer: _Timer, ctx: int) -> list[dict]:
+    """One row per kernel pair: (what, shape, new ms and fraction, like kernel ms and fraction)."""
+    from ..ops import attention, basic, gemm, mixattn
+    from ..models import rutulix as rx
+    width, H, G, D, inter, chunk = SIZES[size]
+    ff = inter * 3 // 2
+    peaks, _ = _peaks()
+    bw, fl = peaks["hbm_gbs"] * 1e6, peaks["bf16_tflops"] * 1e9            # bytes, flops per ms
+    rnd = lambda *s, dt=torch.bfloat16: torch.randn(*s, device=dev, dtype=torch.float32).to(dt)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    cfg = rx.RutulixConfig.uniform(1, width, H, G, D, ff, 64, chunk)
+    m = rx.RutulixWeights(cfg, rx.synth_state(cfg, 0, dev), dev).layers[0].mix
+    rows_out = []
+
+    def pair(what, shape, new, old):
+        rec = {"kernel": what, "shape": shape}
+        for tag, spec in (("new", new), ("like", old)):
+            if spec is None:
+                continue
+            fn, need_bytes, need_flops = spec
+            ms = timer(fn)
+            roof = max(need_bytes / bw, need_flops / fl)
+            rec[tag] = {"ms": round(ms, 4), "fraction": round(roof / ms, 3), "bound": "memory" if need_bytes / bw >= need_flops / fl else "tensor"}
+        if "like" in rec:
+            rec["distance_ratio"] = round(rec["like"]["fraction"] / rec["new"]["fraction"], 2)
+        rows_out.append(rec)
+
+    bs, pages = 64, (ctx + 63) // 64
+    for t in (8192, 32):
+        x32, x16, d16 = rnd(t, width, dt=torch.float32), rnd(t, width), rnd(t, width)
+        g32, g16 = torch.ones(width, device=dev), torch.ones(width, device=dev, dtype=torch.bfloat16)
+        # fp32 residual read + written, delta read, output written against a bf16 residual
+        pair("residual + norms", f"{t} x {width}",
+             (lambda: mixattn.residual_norm(x32, width, 1e-5, delta=d16, bias=g32, post_w=g32, pre_w=g32), t * width * 12, 0),
+             (lambda: basic.add_rmsnorm(x16, d16, g16, 1e-5), t * width * 8, 0))
+        z, gu = rnd(t, ff), rnd(t, 2 * inter)
+        bias = torch.ones(ff, device=dev)
+        pair("activation", f"{t} x {ff}", (lambda: mixattn.bias_xielu(z, bias, 0.7, 1.2), t * ff * 4, 0),
+             (lambda: basic.silu_mul(gu), t * inter * 6, 0))
+        # attention prologue
+        proj, qkv = rnd(t, (H + G) * D), rnd(t, (H + 2 * G) * D)
+        kc, vc = (torch.zeros(max(t, 64) // bs + 1, bs, G * D, dtype=torch.bfloat16, device=dev) for _ in range(2))
+        k4, v4 = (torch.zeros(max(t, 64) // bs + 1, G, bs, D, dtype=torch.bfloat16, device=dev) for _ in range(2))
+        pos, qn = torch.arange(t, dtype=torch.int32, device=dev), torch.ones(D, device=dev, dtype=torch.bfloat16)
+        inv = attention.rope_inv_freq(m.rot, 5e5, dev)
+        n_mix = t if t > 32 else 0
+        qout = t * H * (G * D * 2 if n_mix else D * 4)
+        pair("attention prologue", f"{t} tokens", (lambda: mixattn.qk_row_prep(proj, m, pos, pos, kc, vc, n_mix),
+                                                   t * (H + G) * D * 2 + t * 2 * G * D * 2 + qout, 0),
+             (lambda: attention.qk_norm_rope_append(qkv, 0, D, False, qkv, H * D, qkv, (H + G) * D, qn, qn, True, 1e-5, inv, m.rot,
+                                                    pos, pos, k4, v4, H, G), t * (H + 2 * G) * D * 2 * 2, 0))
+    # prompt attention: one chunk-aligned prompt
+    t = 8192
+    table = (torch.arange(t // bs, dtype=torch.int32, device=dev) + 1)[None]
+    q_mix, q = rnd(t, H, G * D), rnd(t, H, D)
+    kc, vc = (rnd(t // bs + 1, bs, G * D) for _ in range(2))
+    k4, v4 = kc.view(-1, G, bs, D), vc.view(-1, G, bs, D)
+    out = torch.empty(t, H * D, dtype=torch.bfloat16, device=dev)
+    pairs_n = sum((p % chunk + 1) for p in range(t))
+    full_n = t * (t + 1) // 2
+    args = (i32([0]), i32([t]), i32([t]), t)
+    new_fn = lambda: mixattn.prefill(q_mix, m, kc, vc, table, *args, out)
+    old_fn = lambda: attention.prefill(q, k4, v4, table, *args)
+    pair("prompt attention (multiplications executed)", f"{t} tokens, chunk {chunk}",
+         (new_fn, 0, 2 * pairs_n * H * (G * D + D)), (old_fn, 0, 2 * full_n * H * 2 * D))
+    pair("prompt attention (mixing counted as H x H per pair)", f"{t} tokens, chunk {chunk}",
+         (new_fn, 0, 2 * pairs_n * H * (2 * D + H)), (old_fn, 0, 2 * full_n * H * 2 * D))
+    # decode attention
+    for b in (1, 32):
+        keys = min(ctx, chunk)
+        tb = (torch.arange(b * pages, dtype=torch.int32, device=dev) + 1).view(b, pages)
+        kc, vc = (rnd(b * pages + 1, bs, G * D) for _ in range(2))
+        k4, v4 = kc.view(-1, G, bs, D), vc.view(-1, G, bs, D)
+        qr, q = rnd(b, H, D, dt=torch.float32), rnd(b, H, D)
+        ob = torch.empty(b, H * D, dtype=torch.bfloat16, device=dev)
+        pos, kvl = i32([keys - 1] * b), i32([keys] * b)
+        nbytes = b * keys * G * D * 2 * 2
+        pair("decode attention", f"batch {b}, {keys} keys", (lambda: mixattn.rows(qr, m, kc, vc, tb, pos, keys, ob), nbytes, 0),
+             (lambda: attention.decode(q, k4, v4, tb, kvl, max_kv_len=keys), nbytes, 0))
+    # projections (the same GEMM; listed for the share)
+    for t, n, k, what in ((8192, ff, width, "up projection"), (8192, (H + G) * D, width, "q | k projection"), (32, ff, width, "up projection"),
+                          (32, (H + G) * D, width, "q | k projection")):
+        w = gemm.PackedLinear.from_bf16(rnd(n, k))
+        x = rnd(t, k)
+        pair(what, f"{t} x {n} x {k}", (lambda: gemm.linear(x, w), (n * k + t * k + t * n) * 2, 2 * t * n * k), None)
+    return rows_out
+
+
+def run(args) -> dict:
+    from ..ops import _lib
+    from .clocks import ClockSampler
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    timer = _Timer(dev, args.steps, args.warmup)
+    prompt = args.prompt
+    out: dict = {"metric": "rutulix design: prefill and decode throughput", "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True,
+                 "steps": timer.steps, "warmup": timer.warmup, "dtype": "bf16", "data": "synthetic", "designs": {}}
+    slots = 32
+    with torch.no_grad(), ClockSampler(0) as clk:
+        for size in ([args.design_size] if args.design_size else list(SIZES)):
+            width, heads, kv, dim, inter, chunk = SIZES[size]
+            new, old = _models(size, dev, prompt, slots)
+            rec = {"layers": LAYERS, "width": width, "heads": heads, "kv_heads": kv, "dim": dim, "ff": inter * 3 // 2, "chunk": chunk,
+                   "prompt": prompt, "rutulix": _throughput(new, dev, prompt, slots, timer)}
+            torch.cuda.empty_cache()
+            rec["closest (full-attention decoder, fp8 weights)"] = _throughput(old, dev, prompt, slots, timer)
+            torch.cuda.empty_cache()
+            rec["kernels"] = _kernels(size, dev, timer, prompt)
+            torch.cuda.empty_cache()
+            out["designs"][size] = rec
+            _lib.check_status()
+    first = next(iter(out["designs"].values()))
+    out["value"] = first["rutulix"]["prefill_tok_s"]
+    out["clocks"] = clk.summary()
+    out["config"] = {"l2": "flushed before every timed call", "roofline": _peaks()[1], "prompt": prompt, "decode_batch": slots}
+    return out
