@@ -6,13 +6,15 @@
 // scores, no H x H arithmetic per key.
 //
 // One CTA = one 128-row query tile of one head.  Warp roles:
-//   warp 4  : TMA producer - the key tile of 128 tokens in slabs of 64 columns through a ring (with the query slab of the
-//             same columns beside it when the query tile does not fit in shared memory as a whole), and the value tile
-//             of the head's key/value group, page by page through the sequence's block table;
+//   warp 4  : TMA producer of the key tile of 128 tokens, in slabs of 64 columns through a ring (with the query slab of the
+//             same columns beside it when the query tile does not fit in shared memory as a whole), page by page through
+//             the sequence's block table;
+//   warp 6  : TMA producer of the value tile of the head's key/value group, on its own so that neither kind of tile waits
+//             for the other's buffers;
 //   warp 5  : tcgen05.mma issuer - S(j+1) into the other of two TMEM score buffers before P(j) V(j), so that the softmax
 //             of one tile overlaps the score GEMM of the next; O accumulates in TMEM, V consumed MN-major;
-//   warps 0-3: softmax - one query row per thread, online maximum / sum in the exp2 domain, P as bf16 into the swizzled
-//             K-major operand layout, lazy rescale of O.
+//   warps 0-3: softmax - one query row per thread, online maximum / sum in the exp2 domain, P as bf16 back into the tensor
+//             memory its scores came from (the P V product reads it there), lazy rescale of O.
 // Masks: causal, and (chunk > 0) only keys of the query's own chunk of `chunk` positions; key tiles below the first
 // row's chunk are skipped.  All mbarrier waits are bounded and unwind through the common exit.
 #include <cuda_bf16.h>
@@ -27,7 +29,7 @@ namespace mixattn {
 constexpr int BQ = 128;         // query rows per CTA
 constexpr int BKV = 128;        // keys per tile
 constexpr int ATOM = 16384;     // bytes of one [128 x 64] bf16 swizzled atom
-constexpr int NTHREADS = 192;
+constexpr int NTHREADS = 224;
 constexpr int MAX_STAGES = 8;
 constexpr int BUDGET = 232448 - 1024 /* alignment */ - 512 /* barriers */;
 
@@ -68,8 +70,7 @@ mix_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
   constexpr int STAGE = QRES ? ATOM : 2 * ATOM;
   extern __shared__ uint8_t smem_base[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_base) + 1023) & ~uintptr_t(1023));
-  uint8_t* sP = smem;                                   // 2 atoms
-  uint8_t* sV = sP + 2 * ATOM;                          // VA atoms
+  uint8_t* sV = smem;                                   // VA atoms
   uint8_t* sQ = sV + VA * ATOM;                         // slabs atoms when resident
   uint8_t* sR = sQ + (QRES ? p.slabs * ATOM : 0);       // ring: K slab (+ Q slab)
   uint64_t* bars = reinterpret_cast<uint64_t*>(sR + p.stages * STAGE);
@@ -153,12 +154,18 @@ mix_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         }
         return true;
       };
-      // keys run one tile ahead of values: S(j + 1) is issued before P(j) V(j)
-      ok = load_k(0);
+      for (int j = 0; ok && j < n_tiles && !*abort_flag; ++j) ok = load_k(j);
+      if (!ok) { atomicExch(p.status, ERR_WAIT_STAGE); *abort_flag = 1; }
+    }
+  } else if (warp == 6) {
+    if (lane == 0) {
+      const int* bt = p.block_table + (size_t)(p.seq ? p.seq[b] : b) * p.max_blocks;
+      const int bs = p.block_size;
+      const uint32_t sub_bytes = bs * 128;
+      bool ok = true;
       for (int j = 0; ok && j < n_tiles && !*abort_flag; ++j) {
-        if (j + 1 < n_tiles && !load_k(j + 1)) { ok = false; break; }
+        const int key0 = (tile0 + j) * BKV, page0 = key0 / bs, nblk = (min(BKV, kv_len - key0) + bs - 1) / bs;
         if (!mbar_wait(v_empty, (j & 1) ^ 1)) { ok = false; break; }
-        const int page0 = (tile0 + j) * BKV / bs, nblk = pages(j);
         mbar_expect_tx(v_full, nblk * sub_bytes * VA);
         for (int i = 0; i < nblk; ++i) {
           const int row = bt[page0 + i] * bs;
@@ -198,9 +205,8 @@ mix_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         tc_fence_after();
 #pragma unroll
         for (int kk = 0; kk < 8; ++kk) {
-          const uint64_t da = umma_desc_sw128(sP + (kk >> 2) * ATOM) + 2 * (kk & 3);
           const uint64_t db = desc_mn_sw128(sV + kk * 2048, ATOM, 1024);
-          umma_bf16_ss(tO, da, db, idesc_pv, (j | kk) ? 1u : 0u);
+          umma_bf16_ts(tO, tmem + (j & 1) * 128 + kk * 8, db, idesc_pv, (j | kk) ? 1u : 0u);
         }
         umma_commit(v_empty);
         umma_commit(pv_done);
@@ -242,19 +248,17 @@ mix_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
 #pragma unroll
         for (int i = 0; i < 128; ++i) m_tile = fmaxf(m_tile, s[i]);
       }
-      // P(j) overwrites what P(j-1) V(j-1) reads, and O may be rescaled: wait for that product
-      if (j > 0) {
-        bool ok2 = mbar_wait(pv_done, (j - 1) & 1);
-        ok2 = __all_sync(0xffffffffu, ok2);
-        if (!ok2) { alive = false; break; }
-        tc_fence_after();
-      }
       // a row whose keys were all masked so far has m_run = -inf, l_run = 0 and an O of zeros
       const float m_new = fmaxf(m_run, m_tile);
       const bool grow = m_new > m_run + 8.f || (m_run == -INFINITY && m_new > -INFINITY);
       if (j == 0) {
         m_run = m_new;
       } else if (__any_sync(0xffffffffu, grow)) {
+        // O is about to be rescaled: the product that last added to it must have finished
+        bool ok2 = mbar_wait(pv_done, (j - 1) & 1);
+        ok2 = __all_sync(0xffffffffu, ok2);
+        if (!ok2) { alive = false; break; }
+        tc_fence_after();
         const float m_next = grow ? m_new : m_run;
         const float alpha = (m_run == -INFINITY) ? 0.f : exp2f(m_run - m_next);
         l_run *= alpha;
@@ -272,29 +276,27 @@ mix_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       }
       const float m_use = m_run == -INFINITY ? 0.f : m_run;
       float lsum = 0.f;
-      uint8_t* prow = sP + (r >> 3) * 1024 + (r & 7) * 128;
-      const int sw = r & 7;
 #pragma unroll
-      for (int c8 = 0; c8 < 16; ++c8) {
-        float e[8];
+      for (int half = 0; half < 2; ++half) {
+        uint32_t w[32];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-          e[i] = exp2f(s[c8 * 8 + i] - m_use);
-          lsum += e[i];
+        for (int i = 0; i < 32; ++i) {
+          const float e0 = exp2f(s[half * 64 + 2 * i] - m_use), e1 = exp2f(s[half * 64 + 2 * i + 1] - m_use);
+          lsum += e0 + e1;
+          __nv_bfloat162 t = __floats2bfloat162_rn(e0, e1);
+          w[i] = *reinterpret_cast<uint32_t*>(&t);
         }
-        uint4 u;
-        __nv_bfloat162 t0 = __floats2bfloat162_rn(e[0], e[1]);
-        __nv_bfloat162 t1 = __floats2bfloat162_rn(e[2], e[3]);
-        __nv_bfloat162 t2 = __floats2bfloat162_rn(e[4], e[5]);
-        __nv_bfloat162 t3 = __floats2bfloat162_rn(e[6], e[7]);
-        u.x = *reinterpret_cast<uint32_t*>(&t0);
-        u.y = *reinterpret_cast<uint32_t*>(&t1);
-        u.z = *reinterpret_cast<uint32_t*>(&t2);
-        u.w = *reinterpret_cast<uint32_t*>(&t3);
-        *reinterpret_cast<uint4*>(prow + (c8 >> 3) * ATOM + (((c8 & 7) ^ sw) << 4)) = u;
+        // 64 keys = 32 columns of packed pairs over this tile's own scores, which are all in registers by now
+        tmem_st_32x32(tmem + sb * 128 + lane_off + half * 32, w);
       }
+      tmem_st_wait();
       l_run += lsum;
-      fence_proxy_async_smem();
+      // the issuer handles one P at a time: hand this one over only after the previous product is through
+      if (j > 0) {
+        bool ok2 = mbar_wait(pv_done, (j - 1) & 1);
+        ok2 = __all_sync(0xffffffffu, ok2);
+        if (!ok2) { alive = false; break; }
+      }
       tc_fence_before();
       mbar_arrive(p_full);
     }
@@ -388,7 +390,7 @@ extern "C" int b200_attn_mix_prefill(const void* q_mix, const void* k_cache, con
   const int KW = G * D, VA = (D + 63) / 64;
   Params p;
   p.slabs = (KW + 63) / 64;
-  const int fixed = (2 + VA) * ATOM;
+  const int fixed = VA * ATOM;
   const bool qres = fixed + p.slabs * ATOM + 3 * ATOM <= BUDGET;
   const int stage = qres ? ATOM : 2 * ATOM;
   p.stages = (BUDGET - fixed - (qres ? p.slabs * ATOM : 0)) / stage;

@@ -1,9 +1,11 @@
 // y = xIELU(z + bias) over rows: for z > 0  ap z^2 + z / 2,  otherwise  an (exp(z) - 1 - z) + z / 2, with the two
 // positive coefficients given as numbers.  bf16 or fp32 data, fp32 arithmetic; `ld` (a multiple of 8) columns per row,
-// columns whose input and bias are zero stay zero.
+// columns whose input and bias are zero stay zero.  (bf16 projections take the activation in the GEMM's epilogue instead,
+// b200_gemm_bf16_bias_xielu.)
 #include "launch.h"
 #include "ops.h"
 #include "vec8.cuh"
+#include "xielu.cuh"
 
 namespace {
 using namespace b200;
@@ -23,10 +25,7 @@ __global__ void bias_xielu_kernel(const T* __restrict__ in, const float* __restr
       for (int j = 0; j < 8; ++j) z[j] += b[j];
     }
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      const float v = z[j];
-      z[j] = (v > 0.f ? ap * v * v : an * (expm1f(v) - v)) + 0.5f * v;
-    }
+    for (int j = 0; j < 8; ++j) z[j] = xielu(z[j], ap, an);
     store8(out + i * 8, z);
   }
 }

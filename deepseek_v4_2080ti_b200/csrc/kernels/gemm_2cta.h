@@ -3,6 +3,7 @@
 #include <cuda_runtime.h>
 
 #include "../comm/comm.h"
+#include "xielu.cuh"
 
 #ifdef __cplusplus
 extern "C" {
@@ -22,4 +23,7 @@ int b200_gemm_bf16_2cta(const void* W, const void* X, void* out_bf16, int T, int
 
 #ifdef __cplusplus
 }
+// out[T, N] = xIELU(X W^T + bias) for the same shapes.
+int b200_gemm_bf16_2cta_xielu(const void* W, const void* X, void* out_bf16, int T, int N, int K,
+                              const b200::XieluEpilogue& act, int* status, cudaStream_t stream);
 #endif

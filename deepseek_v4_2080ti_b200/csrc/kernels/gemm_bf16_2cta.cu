@@ -117,6 +117,8 @@ struct Params {
   int* status;
   int mode;               // 0: store to out; 3: reduce-scatter push (see gemm_wdec_kernel.cuh ar_mode 3);
                           // 4: W rows interleaved [gate tile | up tile]: out[T, N/2] = silu(gate) * up
+                          // 5: out = xIELU(acc + bias)
+  XieluEpilogue act;      // mode 5
   int n_rot, sp_rows;
   int ag_wait, ag_flag_rows;
   unsigned long long budget_ns;
@@ -377,6 +379,32 @@ gemm_bf16_2cta_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_cons
             *reinterpret_cast<uint4*>(orow + c0 + q4 * 8) = o;
           }
         }
+      } else if (p.mode == 5) {
+        const float* bias = p.act.bias + (size_t)m2 * BN;
+#pragma unroll 1
+        for (int c0 = 0; c0 < BN; c0 += 32) {
+          uint32_t v[32];
+          tmem_ld_32x32(taddr + c0, v);
+          tmem_ld_wait();
+          if (c0 + 32 >= BN) {
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) remote_arrive(lead_acc_empty0 + buf * 8);
+          }
+#pragma unroll
+          for (int q4 = 0; q4 < 4; ++q4) {
+            const float4 b0 = __ldg(reinterpret_cast<const float4*>(bias + c0 + q4 * 8));
+            const float4 b1 = __ldg(reinterpret_cast<const float4*>(bias + c0 + q4 * 8 + 4));
+            const float bb[8] = {b0.x, b0.y, b0.z, b0.w, b1.x, b1.y, b1.z, b1.w};
+            uint4 o;
+            __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+              oh[e] = __floats2bfloat162_rn(xielu(__uint_as_float(v[q4 * 8 + 2 * e]) + bb[2 * e], p.act.ap, p.act.an),
+                                            xielu(__uint_as_float(v[q4 * 8 + 2 * e + 1]) + bb[2 * e + 1], p.act.ap, p.act.an));
+            *reinterpret_cast<uint4*>(drow + c0 + q4 * 8) = o;
+          }
+        }
       } else if (p.mode != 3) {
         // two TMEM reads in flight per wait: the read latency, not the store count, paces this loop
 #pragma unroll 1
@@ -595,10 +623,25 @@ static bool push_maps(const B200Comm& c, int ldo, g2::OutMaps* out) {
 // X [T, K] bf16, W [N, K] bf16 -> out [T, N] bf16 (mode 0), or the reduce-scatter push of the sequence-parallel path
 // (mode 3: out unused; comm, sp_rows and n_rot as in gemm_wdec_kernel.cuh), or out [T, N / 2] = silu(gate) * up for a
 // W whose rows are interleaved in 128-row tiles [gate | up] (mode 4).  ag_wait: X is the gathered buffer.
+static int launch_2cta(const void* W, const void* X, void* out_bf16, int T, int N, int K, int mode, const B200Comm* comm,
+                       int sp_rows, int n_rot, int ag_wait, int ag_flag_rows, unsigned long long budget_ns, int* status,
+                       const XieluEpilogue* act, cudaStream_t stream);
 extern "C" int b200_gemm_bf16_2cta(const void* W, const void* X, void* out_bf16, int T, int N, int K, int mode,
                                    const B200Comm* comm, int sp_rows, int n_rot, int ag_wait, int ag_flag_rows,
                                    unsigned long long budget_ns, int* status, cudaStream_t stream) {
-  if (!b200_gemm_2cta_supported(T, N, K) || (mode != 0 && mode != 3 && mode != 4) || (mode != 3 && !out_bf16))
+  if (mode != 0 && mode != 3 && mode != 4) return -ERR_BAD_ARG;
+  return launch_2cta(W, X, out_bf16, T, N, K, mode, comm, sp_rows, n_rot, ag_wait, ag_flag_rows, budget_ns, status, nullptr,
+                     stream);
+}
+// out [T, N] = xIELU(X W^T + bias), the activation taken on the fp32 accumulators (mode 5).
+int b200_gemm_bf16_2cta_xielu(const void* W, const void* X, void* out_bf16, int T, int N, int K, const XieluEpilogue& act,
+                              int* status, cudaStream_t stream) {
+  return launch_2cta(W, X, out_bf16, T, N, K, 5, nullptr, 0, 0, 0, 0, 0, status, &act, stream);
+}
+static int launch_2cta(const void* W, const void* X, void* out_bf16, int T, int N, int K, int mode, const B200Comm* comm,
+                       int sp_rows, int n_rot, int ag_wait, int ag_flag_rows, unsigned long long budget_ns, int* status,
+                       const XieluEpilogue* act, cudaStream_t stream) {
+  if (!b200_gemm_2cta_supported(T, N, K) || (mode != 3 && !out_bf16) || (mode == 5 && (!act || !act->bias)))
     return -ERR_BAD_ARG;
   if ((mode == 3 || ag_wait) && (!comm || sp_rows <= 0 || sp_rows % (2 * g2::BM))) return -ERR_BAD_ARG;
   if (ag_wait && (ag_flag_rows <= 0 || g2::BM % ag_flag_rows)) return -ERR_BAD_ARG;
@@ -612,6 +655,7 @@ extern "C" int b200_gemm_bf16_2cta(const void* W, const void* X, void* out_bf16,
   p.out = reinterpret_cast<__nv_bfloat16*>(out_bf16);
   p.status = status;
   p.mode = mode;
+  if (act) p.act = *act;
   p.n_rot = n_rot;
   p.sp_rows = sp_rows;
   p.ag_wait = ag_wait;

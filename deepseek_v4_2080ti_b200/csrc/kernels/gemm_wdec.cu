@@ -13,6 +13,7 @@ struct FusedOpts {
   unsigned long long budget_ns = 0;
   int sp_rows = 0;                 // rows per owner shard (reduce-scatter push, all-gather wait)
   int ag_wait = 0, ag_flag_rows = 0;
+  XieluEpilogue act = {nullptr, 0.f, 0.f, 0};   // activation of the finished sums (bf16 weights, no residual)
   int bn = 0;                      // token tile forced by the collective's layout (0: by T)
   int n_rot = 0;
 };
@@ -65,7 +66,9 @@ static int gemm_wdec_launch(int wfmt, const void* W, const float* scales, const 
     // prefill-sized bf16 problems that tile evenly go to the CTA-pair kernel (256 x 256 tiles, gemm_bf16_2cta.cu)
     const int mode = fo ? fo->ar_mode : 0;
     const bool sp_ok = !fo || !fo->comm || (!fo->sp_rows && !fo->ag_wait) || (fo->sp_rows % 256 == 0);
-    if (wfmt == WF_BF16 && BN == 256 && splits == 1 && !residual && !out_f32 && (mode == 0 || mode == 3) &&
+    if (fo && fo->act.on && fo->act.bias && wfmt == WF_BF16 && BN == 256 && out_bf16 && b200_gemm_2cta_supported(T, N, K))
+      return b200_gemm_bf16_2cta_xielu(W, X, out_bf16, T, N, K, fo->act, status, stream);
+    if ((!fo || !fo->act.on) && wfmt == WF_BF16 && BN == 256 && splits == 1 && !residual && !out_f32 && (mode == 0 || mode == 3) &&
         (out_bf16 || mode == 3) && sp_ok && b200_gemm_2cta_supported(T, N, K)) {
       // the rotation was computed in units of this launcher's token tile, which is also 256 here
       return b200_gemm_bf16_2cta(W, X, out_bf16, T, N, K, mode, fo ? fo->comm : nullptr, fo ? fo->sp_rows : 0,
@@ -93,6 +96,7 @@ static int gemm_wdec_launch(int wfmt, const void* W, const float* scales, const 
   p.ldo = N;
   p.status = status;
   p.tile_counters = tile_counters;
+  p.act = fo ? fo->act : XieluEpilogue{nullptr, 0.f, 0.f, 0};
   p.work_table = nullptr;
   p.num_work = nullptr;
   p.w_group_stride = 0;
@@ -154,6 +158,17 @@ static int gemm_wdec_launch(int wfmt, const void* W, const float* scales, const 
   }
 #undef B200_DISPATCH
   return -ERR_BAD_ARG;
+}
+
+// out[T, N] bf16 = xIELU(X W^T + bias) with bf16 weights: the bias and the activation are applied to the fp32 sums in the
+// epilogue (for splits > 1 by the CTA that reduces the partials; out_f32 and tile_counters as in b200_gemm_wdec_ex).
+extern "C" int b200_gemm_bf16_bias_xielu(const void* W, const void* X, const float* bias, float ap, float an, void* out_bf16,
+                                         float* out_f32, int T, int N, int K, int splits, int* tile_counters, int* status,
+                                         cudaStream_t stream) {
+  if (!out_bf16) return -ERR_BAD_ARG;
+  FusedOpts fo;
+  fo.act = XieluEpilogue{bias, ap, an, 1};
+  return gemm_wdec_launch(WF_BF16, W, nullptr, X, out_bf16, out_f32, nullptr, T, N, K, splits, tile_counters, status, stream, &fo);
 }
 
 // Grouped GEMM over ragged row segments (routed experts): out[r, :] = X[r, :] * W_g^T for every row r of the

@@ -32,6 +32,7 @@
 #include "../ptx/sm100.cuh"
 #include "tma_host.h"
 #include "ops.h"
+#include "xielu.cuh"
 #include "../comm/comm.h"
 
 namespace b200 {
@@ -97,6 +98,7 @@ struct GemmParams {
   float* out_f32;            // [splits, T, ldo] partials (splits > 1) or fp32 result
   const __nv_bfloat16* residual;  // optional [T, ldo], added in the epilogue (splits == 1)
   int ldo;
+  XieluEpilogue act;         // bf16 weights, bf16 output: bias + activation on the finished sums (off unless .on)
   int* status;
   // In-kernel split-K fix-up (splits > 1 with `out` set): every split writes its fp32 partial to
   // out_f32, then bumps tile_counters[tile]; the CTA that arrives last sums the partials in split
@@ -951,6 +953,12 @@ gemm_wdec_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
               if (c0 + j < wk.rows)
                 o[(size_t)j * p.ldo] =
                     __float2bfloat16(__uint_as_float(v[j]) + __bfloat162float(r[(size_t)j * p.ldo]));
+          } else if (WFMT == WF_BF16 && p.act.on) {
+            __nv_bfloat16* o = p.out + (size_t)t0 * p.ldo + f;
+            const float b = p.act.bias ? __ldg(p.act.bias + f) : 0.f;
+#pragma unroll
+            for (int j = 0; j < CH; ++j)
+              if (c0 + j < wk.rows) o[(size_t)j * p.ldo] = __float2bfloat16(xielu(__uint_as_float(v[j]) + b, p.act.ap, p.act.an));
           } else {
             __nv_bfloat16* o = p.out + (size_t)t0 * p.ldo + f;
 #pragma unroll
@@ -981,6 +989,8 @@ gemm_wdec_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
             float acc = p.residual ? __bfloat162float(p.residual[off]) : 0.f;
             for (int sp = 0; sp < p.splits; ++sp)
               acc += __ldcg(p.out_f32 + (size_t)sp * p.T * p.ldo + off);
+            if (WFMT == WF_BF16 && p.act.on)
+              acc = xielu(acc + (p.act.bias ? __ldg(p.act.bias + f) : 0.f), p.act.ap, p.act.an);
             p.out[off] = __float2bfloat16(acc);
           }
         }

@@ -175,6 +175,9 @@ int b200_kv8_dequantize(const void* k8, const void* v8, const float* k_scale, co
 int b200_residual_norm(float* x, const int* ids, const void* table, int vocab, const void* delta, const float* bias,
                        const float* post_w, const float* step, const float* pre_w, void* out, const int* rows, int n, int ld,
                        int cols, float eps, int rms, int unit_offset, int write_x, int f32, cudaStream_t stream);
+int b200_gemm_bf16_bias_xielu(const void* W, const void* X, const float* bias, float ap, float an, void* out_bf16,
+                              float* out_f32, int T, int N, int K, int splits, int* tile_counters, int* status,
+                              cudaStream_t stream);
 int b200_bias_xielu(const void* in, const float* bias, void* out, long long rows, int ld, float ap, float an, int f32,
                     cudaStream_t stream);
 int b200_qk_row_prep(const void* proj, int ld, int q_off, int k_off, int v_off, const float* q_w, const float* k_w,

@@ -308,7 +308,7 @@ class RutulixRuntime(PagedRuntime):
         return lw.o(out)
 
     def _mlp(self, lw: RutulixLayer, y: torch.Tensor) -> torch.Tensor:
-        return lw.down(mixattn.bias_xielu(lw.up(y), lw.up_b, *lw.act))
+        return lw.down(lw.up.bias_xielu(y, lw.up_b, *lw.act))
 
     def _forward(self, ids, positions, kv_slots, meta, rows):
         cfg, w = self.cfg, self.w

@@ -394,6 +394,28 @@ def linear(x: torch.Tensor, w: PackedLinear, residual: torch.Tensor | None = Non
     return out
 
 
+def linear_bias_xielu(x: torch.Tensor, w: PackedLinear, bias: torch.Tensor, ap: float, an: float) -> torch.Tensor:
+    """``xIELU(x @ w^T + bias)`` in one kernel for bf16 weights: bias (fp32 [N]) and activation are applied to the fp32
+    sums in the GEMM epilogue."""
+    assert x.dtype == torch.bfloat16 and x.is_cuda and x.dim() == 2 and x.is_contiguous() and w.wfmt == WF_BF16
+    t, k = x.shape
+    n = w.n
+    assert k == w.k and bias.dtype == torch.float32 and bias.numel() == n and bias.is_contiguous()
+    out = torch.empty(t, n, dtype=torch.bfloat16, device=x.device)
+    kb = (k + 63) // 64
+    splits = max(1, min(pick_splits(t, n, k), kb))
+    per = (kb + splits - 1) // splits
+    splits = (kb + per - 1) // per
+    if ((n + 127) // 128) * ((t + _bn(t) - 1) // _bn(t)) > MAX_TILE_COUNTERS:
+        splits = 1
+    ws, counters = _workspace(splits * t * n, x.device) if splits > 1 else (None, None)
+    rc = _lib.lib().b200_gemm_bf16_bias_xielu(_lib.ptr(w.weight), _lib.ptr(x), _lib.ptr(bias), ctypes.c_float(ap), ctypes.c_float(an),
+                                              _lib.ptr(out), _lib.ptr(ws), t, n, k, splits, _lib.ptr(counters),
+                                              _lib.ptr(_lib.status_word(x.device)), _lib.stream())
+    _lib.check(rc, "gemm_bf16_bias_xielu")
+    return out
+
+
 def linear_ref(x: torch.Tensor, w_fp32: torch.Tensor, residual: torch.Tensor | None = None) -> torch.Tensor:
     """fp32 oracle: x @ w^T (+ residual)."""
     y = x.float() @ w_fp32.float().t()

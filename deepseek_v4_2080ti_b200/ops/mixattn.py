@@ -59,6 +59,13 @@ class Projection:
             return gemm.linear(x, self.packed, out_f32=out_f32)
         return gemm_f32(x, self.w32)
 
+    def bias_xielu(self, x: torch.Tensor, bias: torch.Tensor, ap: float, an: float) -> torch.Tensor:
+        """xIELU(projection + bias): in the GEMM's epilogue, or as a second kernel in fp32."""
+        if self.w32 is None:
+            from . import gemm
+            return gemm.linear_bias_xielu(x, self.packed, bias, ap, an)
+        return bias_xielu(gemm_f32(x, self.w32), bias, ap, an)
+
     def nbytes(self) -> int:
         return self.n * self.k * (4 if self.packed is None else 2)
 
@@ -191,7 +198,7 @@ _outgrown: list[torch.Tensor] = []      # smaller workspaces stay alive: capture
 
 def pick_splits(rows: int, keys: int) -> int:
     """Slices of one row's keys: enough blocks for two per SM, at least 64 keys each."""
-    return max(1, min(64, (2 * NUM_SMS) // max(1, rows), (keys + 63) // 64))
+    return max(1, min(NUM_SMS, (2 * NUM_SMS) // max(1, rows), (keys + 63) // 64))
 
 
 def rows(q: torch.Tensor, m: HeadMix, k_cache, v_cache, block_table, positions, max_keys: int, out: torch.Tensor,

@@ -286,3 +286,19 @@ def test_workspace_growth_keeps_captured_addresses_alive():
     _run_rows(mx, m, talk, kc, vc, table, seqs, [(0, p) for p in range(60)], torch.bfloat16, 64)
     now = mx._ws[0]
     assert before is None or now is before or any(t is before for t in mx._outgrown)
+
+
+@pytest.mark.parametrize("t,n,k", [(3, 320, 192), (5, 96, 4096), (40, 256, 2048), (128, 128, 512), (300, 144, 80), (256, 512, 128), (512, 256, 1024)])
+def test_projection_with_activation_in_the_epilogue(t, n, k):
+    """Every route of the bf16 GEMM: one pass, split K with the reducing CTA, token tiles of all sizes, CTA pairs."""
+    lib, _ = _mods()
+    from deepseek_v4_2080ti_b200.ops import gemm
+    x, w = _rand(t, k, seed=1).bfloat16(), (_rand(n, k, seed=2) * 2 / k ** 0.5).bfloat16()
+    bias, act = _rand(n, seed=3), torch.tensor([0.2, -0.4]).double()
+    sp = torch.nn.functional.softplus(act)
+    got = gemm.linear_bias_xielu(x.cuda(), gemm.PackedLinear.from_bf16(w.cuda()), bias.cuda(), float(sp[0]), float(0.5 + sp[1]))
+    lib.check_status()
+    z = x.double() @ w.double().t() + bias.double()
+    assert _rel(got, ref.xielu(z, act)) < 4e-3
+    # a following plain product is not affected by the activation of this one
+    assert _rel(gemm.linear(x.cuda(), gemm.PackedLinear.from_bf16(w.cuda())), x.double() @ w.double().t()) < 4e-3
