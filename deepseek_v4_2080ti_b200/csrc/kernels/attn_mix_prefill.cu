@@ -139,18 +139,23 @@ mix_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       const int* bt = p.block_table + (size_t)(p.seq ? p.seq[b] : b) * p.max_blocks;
       const int bs = p.block_size;
       const uint32_t sub_bytes = bs * 128;   // 64 columns of one page
-      int it = 0;
       bool ok = true;
-      auto pages = [&](int j) { return (min(BKV, kv_len - (tile0 + j) * BKV) + bs - 1) / bs; };
+      int st = 0;
+      uint32_t ph = 1;
       auto load_k = [&](int j) {
-        const int page0 = (tile0 + j) * BKV / bs, nblk = pages(j);
-        for (int s = 0; s < p.slabs; ++s, ++it) {
-          const int st = it % p.stages;
-          if (!mbar_wait(&r_empty[st], ((it / p.stages) & 1) ^ 1)) return false;
+        const int key0 = (tile0 + j) * BKV, page0 = key0 / bs, nblk = (min(BKV, kv_len - key0) + bs - 1) / bs;
+        // pages of 64 tokens and more: the table is read once per tile, and a slab is two copies at most (this thread's
+        // instruction count per slab is what paces the whole pipeline)
+        const int row0 = bt[page0] * bs, row1 = nblk > 1 ? bt[page0 + 1] * bs : 0;
+        for (int s = 0; s < p.slabs; ++s) {
+          if (!mbar_wait(&r_empty[st], ph)) return false;
           uint8_t* dst = sR + st * STAGE;
           mbar_expect_tx(&r_full[st], nblk * sub_bytes + (QRES ? 0 : ATOM));
           if (!QRES) tma_load_2d(dst + ATOM, &tmQ, &r_full[st], qx + s * 64, q_row0);
-          for (int i = 0; i < nblk; ++i) tma_load_2d(dst + i * sub_bytes, &tmK, &r_full[st], s * 64, bt[page0 + i] * bs);
+          tma_load_2d(dst, &tmK, &r_full[st], s * 64, row0);
+          if (nblk > 1) tma_load_2d(dst + sub_bytes, &tmK, &r_full[st], s * 64, row1);
+          for (int i = 2; i < nblk; ++i) tma_load_2d(dst + i * sub_bytes, &tmK, &r_full[st], s * 64, bt[page0 + i] * bs);
+          if (++st == p.stages) { st = 0; ph ^= 1; }
         }
         return true;
       };
@@ -178,12 +183,12 @@ mix_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
   } else if (warp == 5) {
     if (lane == 0) {
       bool ok = !QRES || mbar_wait(q_full, 0);
-      int it = 0;
+      int st = 0;
+      uint32_t ph = 0;
       auto issue_s = [&](int j) -> bool {
         const uint32_t tS = tmem + (j & 1) * 128;
-        for (int s = 0; s < p.slabs; ++s, ++it) {
-          const int st = it % p.stages;
-          if (!mbar_wait(&r_full[st], (it / p.stages) & 1)) return false;
+        for (int s = 0; s < p.slabs; ++s) {
+          if (!mbar_wait(&r_full[st], ph)) return false;
           tc_fence_after();
           const uint8_t* k = sR + st * STAGE;
           const uint8_t* q = QRES ? sQ + s * ATOM : k + ATOM;
@@ -191,6 +196,7 @@ mix_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
           for (int kk = 0; kk < 4; ++kk)
             umma_bf16_ss(tS, umma_desc_sw128(q) + 2 * kk, umma_desc_sw128(k) + 2 * kk, idesc_qk, (s | kk) ? 1u : 0u);
           umma_commit(&r_empty[st]);
+          if (++st == p.stages) { st = 0; ph ^= 1; }
         }
         umma_commit(&s_full[j & 1]);
         return true;
