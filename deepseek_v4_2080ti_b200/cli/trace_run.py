@@ -4,15 +4,15 @@
 
 One JSON object per line on standard input:
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}
+    {"step": 7, "entries": [{"id": "q1", "tokens": [12, 40], "want": [1]}, {"id": "q2", "tokens": [9], "want": []}], "end": ["q2"]}
 
-``entries``: the next tokens of each request and the places among them whose logits are wanted; ``end``: requests that are
-finished after the step.  All entries of a step run as one batch on the runtime the loader builds for serving.  A step
-with wanted places writes OUT/<step>.f32 (little-endian fp32 [wanted, vocab], in the order of the entries and places);
-every step is acknowledged with a line ``done <step>``.
+An entry appends its tokens to its request (a new name takes a slot) and lists the rows whose logits are to be written; a
+request in ``end`` gives its slot and pages back once the step has run.  The entries of a step form one batch of the
+runtime that the loader builds for serving.  Logits go to OUT/<step>.f32 as little-endian fp32 rows of vocabulary length,
+entry by entry; each step is acknowledged with ``done <step>``, whether or not it wrote a file.
 
-The cache pool holds N tokens (rounded up to whole pages) shared by at most ``--slots`` live requests.  Exit codes: 0 at
-the end of input, 2 for a bad trace or model, 3 when the model's family does not run in the asked dtype.
+The page pool has room for N tokens, shared by up to ``--slots`` requests.  Exit codes: 0 when the input ends, 2 for a model
+that cannot be replayed, 3 when its family does not serve the asked dtype.
 """
 from __future__ import annotations
 
@@ -68,8 +68,8 @@ def main(argv: list[str] | None = None) -> int:
     ap.add_argument("--model", required=True, help="folder with config.json and model.safetensors")
     ap.add_argument("--dtype", choices=("bfloat16", "float32"), default="bfloat16")
     ap.add_argument("--out", required=True)
-    ap.add_argument("--max-tokens", type=int, required=True, help="most tokens that live requests hold at any time")
-    ap.add_argument("--slots", type=int, default=4, help="most requests that are live at any time")
+    ap.add_argument("--max-tokens", type=int, required=True, help="size of the page pool in tokens")
+    ap.add_argument("--slots", type=int, default=4, help="requests that may be open together")
     a = ap.parse_args(argv)
     import torch
     from ..ops import _lib

@@ -25,7 +25,7 @@ __global__ void bias_xielu_kernel(const T* __restrict__ in, const float* __restr
       for (int j = 0; j < 8; ++j) z[j] += b[j];
     }
 #pragma unroll
-    for (int j = 0; j < 8; ++j) z[j] = xielu(z[j], ap, an);
+    for (int j = 0; j < 8; ++j) z[j] = sizeof(T) == 2 ? xielu_bf16(z[j], ap, an) : xielu(z[j], ap, an);
     store8(out + i * 8, z);
   }
 }

@@ -400,8 +400,8 @@ gemm_bf16_2cta_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_cons
             __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&o);
 #pragma unroll
             for (int e = 0; e < 4; ++e)
-              oh[e] = __floats2bfloat162_rn(xielu(__uint_as_float(v[q4 * 8 + 2 * e]) + bb[2 * e], p.act.ap, p.act.an),
-                                            xielu(__uint_as_float(v[q4 * 8 + 2 * e + 1]) + bb[2 * e + 1], p.act.ap, p.act.an));
+              oh[e] = __floats2bfloat162_rn(xielu_bf16(__uint_as_float(v[q4 * 8 + 2 * e]) + bb[2 * e], p.act.ap, p.act.an),
+                                            xielu_bf16(__uint_as_float(v[q4 * 8 + 2 * e + 1]) + bb[2 * e + 1], p.act.ap, p.act.an));
             *reinterpret_cast<uint4*>(drow + c0 + q4 * 8) = o;
           }
         }

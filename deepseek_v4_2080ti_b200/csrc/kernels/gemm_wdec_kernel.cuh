@@ -958,7 +958,7 @@ gemm_wdec_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
             const float b = p.act.bias ? __ldg(p.act.bias + f) : 0.f;
 #pragma unroll
             for (int j = 0; j < CH; ++j)
-              if (c0 + j < wk.rows) o[(size_t)j * p.ldo] = __float2bfloat16(xielu(__uint_as_float(v[j]) + b, p.act.ap, p.act.an));
+              if (c0 + j < wk.rows) o[(size_t)j * p.ldo] = __float2bfloat16(xielu_bf16(__uint_as_float(v[j]) + b, p.act.ap, p.act.an));
           } else {
             __nv_bfloat16* o = p.out + (size_t)t0 * p.ldo + f;
 #pragma unroll
@@ -990,7 +990,7 @@ gemm_wdec_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
             for (int sp = 0; sp < p.splits; ++sp)
               acc += __ldcg(p.out_f32 + (size_t)sp * p.T * p.ldo + off);
             if (WFMT == WF_BF16 && p.act.on)
-              acc = xielu(acc + (p.act.bias ? __ldg(p.act.bias + f) : 0.f), p.act.ap, p.act.an);
+              acc = xielu_bf16(acc + (p.act.bias ? __ldg(p.act.bias + f) : 0.f), p.act.ap, p.act.an);
             p.out[off] = __float2bfloat16(acc);
           }
         }

@@ -126,7 +126,7 @@ def _kernels(size: str, dev, timer: _Timer, ctx: int) -> list[dict]:
              (lambda: basic.add_rmsnorm(x16, d16, g16, 1e-5), t * width * 8, 0))
         z, gu = rnd(t, ff), rnd(t, 2 * inter)
         bias = torch.ones(ff, device=dev)
-        pair("activation", f"{t} x {ff}", (lambda: mixattn.bias_xielu(z, bias, 0.7, 1.2), t * ff * 4, 0),
+        pair("activation on its own", f"{t} x {ff}", (lambda: mixattn.bias_xielu(z, bias, 0.7, 1.2), t * ff * 4, 0),
              (lambda: basic.silu_mul(gu), t * inter * 6, 0))
         # attention prologue
         proj, qkv = rnd(t, (H + G) * D), rnd(t, (H + 2 * G) * D)
@@ -168,12 +168,16 @@ def _kernels(size: str, dev, timer: _Timer, ctx: int) -> list[dict]:
         nbytes = b * keys * G * D * 2 * 2
         pair("decode attention", f"batch {b}, {keys} keys", (lambda: mixattn.rows(qr, m, kc, vc, tb, pos, keys, ob), nbytes, 0),
              (lambda: attention.decode(q, k4, v4, tb, kvl, max_kv_len=keys), nbytes, 0))
-    # projections (the same GEMM; listed for the share)
-    for t, n, k, what in ((8192, ff, width, "up projection"), (8192, (H + G) * D, width, "q | k projection"), (32, ff, width, "up projection"),
-                          (32, (H + G) * D, width, "q | k projection")):
-        w = gemm.PackedLinear.from_bf16(rnd(n, k))
-        x = rnd(t, k)
-        pair(what, f"{t} x {n} x {k}", (lambda: gemm.linear(x, w), (n * k + t * k + t * n) * 2, 2 * t * n * k), None)
+    # projections: the up projection with bias + activation in its epilogue beside the plain product of the same GEMM
+    for t in (8192, 32):
+        w, x, bias = gemm.PackedLinear.from_bf16(rnd(ff, width)), rnd(t, width), torch.ones(ff, device=dev)
+        need = ((ff * width + t * width + t * ff) * 2, 2 * t * ff * width)
+        pair("up projection + bias + activation (like: plain product)", f"{t} x {ff} x {width}",
+             (lambda: gemm.linear_bias_xielu(x, w, bias, 0.7, 1.2), *need), (lambda: gemm.linear(x, w), *need))
+        n = (H + G) * D
+        wq = gemm.PackedLinear.from_bf16(rnd(n, width))
+        pair("q | k projection", f"{t} x {n} x {width}",
+             (lambda: gemm.linear(x, wq), (n * width + t * width + t * n) * 2, 2 * t * n * width), None)
     return rows_out
 
 
