@@ -205,9 +205,8 @@ class RutulixWeights:
         shapes = cfg.tensor_shapes()
         missing = [n for n in shapes if n not in t]
         wrong = [f"{n} {tuple(t[n].shape)} != {s}" for n, s in shapes.items() if n in t and tuple(t[n].shape) != s]
-        extra = [n for n in t if n not in shapes]
-        if missing or wrong or extra:
-            raise ValueError(f"checkpoint does not fit the configuration: missing {missing[:4]}, shapes {wrong[:4]}, unknown {extra[:4]}")
+        if missing or wrong:                       # tensors the configuration does not mention are left unread
+            raise ValueError(f"checkpoint does not fit the configuration: missing {missing[:4]}, shapes {wrong[:4]}")
         dev, self.ld = self.device, pad16(cfg.width)
         proj = lambda w, pad_n=True: Projection.make(w, dtype, dev, pad_n)
 
