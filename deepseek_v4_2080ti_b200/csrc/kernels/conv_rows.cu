@@ -1,0 +1,99 @@
+// Causal depthwise convolution over a batch of rows that belong to several sequences, with optional bias and SiLU.
+//
+//   y[r, c] = act(bias[c] + sum_j w[j, c] x_{back(j)}[c]),   back(j) = taps - 1 - j rows before r in r's own sequence
+//
+// Rows of one sequence are neighbours; row_first[r] is the sequence's first row of this batch, row_slot[r] its state slot,
+// positions[r] its position.  Inputs from before the batch come from the slot's tail (the last taps - 1 inputs, oldest
+// first); inputs from before position 0 are zero, so a slot needs no clearing.  The tail is read here and replaced by the
+// kernel that runs the recurrence behind the convolution (selective_scan.cu).  One thread: 8 channels, `strip` rows.
+#include "launch.h"
+#include "ops.h"
+#include "vec8.cuh"
+
+namespace {
+using namespace b200;
+
+template <typename T>
+struct ConvRowsParams {
+  const T* x;              // [rows, ldx]
+  const float* w;          // [taps, C]
+  const float* bias;       // [C] or null
+  const T* tail;           // [slots, taps - 1, C]
+  const int *row_first, *row_slot, *positions;
+  T* y;                    // [rows, ldy]
+  int ldx, ldy, rows, C, taps, silu, strip;
+};
+
+template <typename T, int K>
+__global__ void __launch_bounds__(128) conv_rows_kernel(ConvRowsParams<T> p) {
+  pdl_grid_trigger();
+  const int taps = K ? K : p.taps;
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+  const bool on = c < p.C;
+  float w[K ? K : 1][8], b[8] = {};
+  if (on) {
+    if (p.bias) load8(p.bias + c, b);
+    if (K) {
+#pragma unroll
+      for (int j = 0; j < K; ++j) load8(p.w + (size_t)j * p.C + c, w[j]);
+    }
+  }
+  pdl_grid_wait();
+  if (!on) return;
+  const int r1 = min(p.rows, ((int)blockIdx.y + 1) * p.strip);
+  for (int r = blockIdx.y * p.strip; r < r1; ++r) {
+    const int off = r - p.row_first[r], pos = p.positions[r];
+    const T* tail = p.tail + ((size_t)p.row_slot[r] * (taps - 1)) * p.C + c;
+    float acc[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) acc[i] = b[i];
+#pragma unroll
+    for (int j = 0; j < taps; ++j) {
+      const int back = taps - 1 - j;
+      if (back > pos) continue;
+      float f[8];
+      load8(back <= off ? p.x + (size_t)(r - back) * p.ldx + c : tail + (size_t)(taps - 1 - (back - off)) * p.C, f);
+      if (!K) load8(p.w + (size_t)j * p.C + c, w[0]);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) acc[i] = fmaf(w[K ? j : 0][i], f[i], acc[i]);
+    }
+    if (p.silu) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        acc[i] = sizeof(T) == 2 ? __fdividef(acc[i], 1.f + __expf(-acc[i])) : acc[i] / (1.f + expf(-acc[i]));
+    }
+    store8(p.y + (size_t)r * p.ldy + c, acc);
+  }
+}
+
+template <typename T>
+int run_conv_rows(const void* x, int ldx, const float* w, const float* bias, const void* tail, const int* row_first,
+                  const int* row_slot, const int* positions, void* y, int ldy, int rows, int C, int taps, int silu,
+                  cudaStream_t stream) {
+  ConvRowsParams<T> p;
+  p.x = reinterpret_cast<const T*>(x); p.w = w; p.bias = bias; p.tail = reinterpret_cast<const T*>(tail);
+  p.row_first = row_first; p.row_slot = row_slot; p.positions = positions; p.y = reinterpret_cast<T*>(y);
+  p.ldx = ldx; p.ldy = ldy; p.rows = rows; p.C = C; p.taps = taps; p.silu = silu;
+  p.strip = 1;
+  while (p.strip < 8 && (long long)rows * C / 8 / p.strip > 148LL * 4096) p.strip *= 2;
+  const dim3 grid((C / 8 + 127) / 128, (rows + p.strip - 1) / p.strip);
+  if (grid.y > 65535) return -6;
+  switch (taps) {
+    case 2: return (int)launch_pdl(conv_rows_kernel<T, 2>, grid, dim3(128), 0, stream, p);
+    case 3: return (int)launch_pdl(conv_rows_kernel<T, 3>, grid, dim3(128), 0, stream, p);
+    case 4: return (int)launch_pdl(conv_rows_kernel<T, 4>, grid, dim3(128), 0, stream, p);
+    default: return (int)launch_pdl(conv_rows_kernel<T, 0>, grid, dim3(128), 0, stream, p);
+  }
+}
+
+}  // namespace
+
+// x rows of C channels (C, ldx, ldy multiples of 8); f32 != 0: x, tail, y are fp32, otherwise bf16.
+extern "C" int b200_conv_rows(const void* x, int ldx, const float* w, const float* bias, const void* tail, const int* row_first,
+                              const int* row_slot, const int* positions, void* y, int ldy, int rows, int C, int taps, int silu,
+                              int f32, cudaStream_t stream) {
+  if (rows <= 0 || C <= 0 || (C & 7) || (ldx & 7) || (ldy & 7) || ldx < C || ldy < C || taps < 1 || taps > 64) return -6;
+  return f32 ? run_conv_rows<float>(x, ldx, w, bias, tail, row_first, row_slot, positions, y, ldy, rows, C, taps, silu, stream)
+             : run_conv_rows<__nv_bfloat16>(x, ldx, w, bias, tail, row_first, row_slot, positions, y, ldy, rows, C, taps, silu,
+                                            stream);
+}

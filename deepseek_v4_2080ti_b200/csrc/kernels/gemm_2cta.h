@@ -3,6 +3,7 @@
 #include <cuda_runtime.h>
 
 #include "../comm/comm.h"
+#include "glu.cuh"
 #include "xielu.cuh"
 
 #ifdef __cplusplus
@@ -26,4 +27,7 @@ int b200_gemm_bf16_2cta(const void* W, const void* X, void* out_bf16, int T, int
 // out[T, N] = xIELU(X W^T + bias) for the same shapes.
 int b200_gemm_bf16_2cta_xielu(const void* W, const void* X, void* out_bf16, int T, int N, int K,
                               const b200::XieluEpilogue& act, int* status, cudaStream_t stream);
+// out[T, N / 2] = glu(gate, up) for W rows interleaved in 128-row tiles [gate | up].
+int b200_gemm_bf16_2cta_glu(const void* W, const void* X, void* out_bf16, int T, int N, int K, const b200::GluShape& glu_shape,
+                            int* status, cudaStream_t stream);
 #endif

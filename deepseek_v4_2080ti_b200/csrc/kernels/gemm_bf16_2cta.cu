@@ -116,9 +116,10 @@ struct Params {
   __nv_bfloat16* out;
   int* status;
   int mode;               // 0: store to out; 3: reduce-scatter push (see gemm_wdec_kernel.cuh ar_mode 3);
-                          // 4: W rows interleaved [gate tile | up tile]: out[T, N/2] = silu(gate) * up
+                          // 4: W rows interleaved [gate tile | up tile]: out[T, N/2] = glu(gate, up) (glu.cuh)
                           // 5: out = xIELU(acc + bias)
   XieluEpilogue act;      // mode 5
+  GluShape glu;           // mode 4
   int n_rot, sp_rows;
   int ag_wait, ag_flag_rows;
   unsigned long long budget_ns;
@@ -352,7 +353,7 @@ gemm_bf16_2cta_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_cons
       __nv_bfloat16* drow = dst + (size_t)(dst_row0 + row_in_tile) * p.ldo + (size_t)m2 * BN;
       const uint32_t taddr = tmem_base + (uint32_t(warp * 32) << 16) + buf * BN;
       if (p.mode == 4) {
-        // SwiGLU: accumulator columns [0, 128) are the gate and [128, 256) the up projection of the same 128
+        // gated unit: accumulator columns [0, 128) are the gate and [128, 256) the up projection of the same 128
         // features; the activation is taken on the fp32 accumulators and only the product is written
         __nv_bfloat16* orow = p.out + (size_t)(row0 + row_in_tile) * p.ldo + (size_t)m2 * (BN / 2);
 #pragma unroll 1
@@ -374,7 +375,7 @@ gemm_bf16_2cta_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_cons
             for (int e = 0; e < 4; ++e) {
               const float g0 = __uint_as_float(v[0][q4 * 8 + 2 * e]), g1 = __uint_as_float(v[0][q4 * 8 + 2 * e + 1]);
               const float u0 = __uint_as_float(v[1][q4 * 8 + 2 * e]), u1 = __uint_as_float(v[1][q4 * 8 + 2 * e + 1]);
-              oh[e] = __floats2bfloat162_rn(g0 / (1.f + __expf(-g0)) * u0, g1 / (1.f + __expf(-g1)) * u1);
+              oh[e] = __floats2bfloat162_rn(glu<true>(g0, u0, p.glu), glu<true>(g1, u1, p.glu));
             }
             *reinterpret_cast<uint4*>(orow + c0 + q4 * 8) = o;
           }
@@ -621,26 +622,31 @@ static bool push_maps(const B200Comm& c, int ldo, g2::OutMaps* out) {
 }
 
 // X [T, K] bf16, W [N, K] bf16 -> out [T, N] bf16 (mode 0), or the reduce-scatter push of the sequence-parallel path
-// (mode 3: out unused; comm, sp_rows and n_rot as in gemm_wdec_kernel.cuh), or out [T, N / 2] = silu(gate) * up for a
+// (mode 3: out unused; comm, sp_rows and n_rot as in gemm_wdec_kernel.cuh), or out [T, N / 2] = glu(gate, up) for a
 // W whose rows are interleaved in 128-row tiles [gate | up] (mode 4).  ag_wait: X is the gathered buffer.
 static int launch_2cta(const void* W, const void* X, void* out_bf16, int T, int N, int K, int mode, const B200Comm* comm,
                        int sp_rows, int n_rot, int ag_wait, int ag_flag_rows, unsigned long long budget_ns, int* status,
-                       const XieluEpilogue* act, cudaStream_t stream);
+                       const XieluEpilogue* act, const GluShape* glu_shape, cudaStream_t stream);
 extern "C" int b200_gemm_bf16_2cta(const void* W, const void* X, void* out_bf16, int T, int N, int K, int mode,
                                    const B200Comm* comm, int sp_rows, int n_rot, int ag_wait, int ag_flag_rows,
                                    unsigned long long budget_ns, int* status, cudaStream_t stream) {
   if (mode != 0 && mode != 3 && mode != 4) return -ERR_BAD_ARG;
   return launch_2cta(W, X, out_bf16, T, N, K, mode, comm, sp_rows, n_rot, ag_wait, ag_flag_rows, budget_ns, status, nullptr,
-                     stream);
+                     nullptr, stream);
 }
 // out [T, N] = xIELU(X W^T + bias), the activation taken on the fp32 accumulators (mode 5).
 int b200_gemm_bf16_2cta_xielu(const void* W, const void* X, void* out_bf16, int T, int N, int K, const XieluEpilogue& act,
                               int* status, cudaStream_t stream) {
-  return launch_2cta(W, X, out_bf16, T, N, K, 5, nullptr, 0, 0, 0, 0, 0, status, &act, stream);
+  return launch_2cta(W, X, out_bf16, T, N, K, 5, nullptr, 0, 0, 0, 0, 0, status, &act, nullptr, stream);
+}
+// out [T, N / 2] = glu(gate, up) for a W interleaved as in mode 4.
+int b200_gemm_bf16_2cta_glu(const void* W, const void* X, void* out_bf16, int T, int N, int K, const GluShape& glu_shape,
+                            int* status, cudaStream_t stream) {
+  return launch_2cta(W, X, out_bf16, T, N, K, 4, nullptr, 0, 0, 0, 0, 0, status, nullptr, &glu_shape, stream);
 }
 static int launch_2cta(const void* W, const void* X, void* out_bf16, int T, int N, int K, int mode, const B200Comm* comm,
                        int sp_rows, int n_rot, int ag_wait, int ag_flag_rows, unsigned long long budget_ns, int* status,
-                       const XieluEpilogue* act, cudaStream_t stream) {
+                       const XieluEpilogue* act, const GluShape* glu_shape, cudaStream_t stream) {
   if (!b200_gemm_2cta_supported(T, N, K) || (mode != 3 && !out_bf16) || (mode == 5 && (!act || !act->bias)))
     return -ERR_BAD_ARG;
   if ((mode == 3 || ag_wait) && (!comm || sp_rows <= 0 || sp_rows % (2 * g2::BM))) return -ERR_BAD_ARG;
@@ -656,6 +662,7 @@ static int launch_2cta(const void* W, const void* X, void* out_bf16, int T, int 
   p.status = status;
   p.mode = mode;
   if (act) p.act = *act;
+  if (glu_shape) p.glu = *glu_shape;      // zeros: the plain SwiGLU
   p.n_rot = n_rot;
   p.sp_rows = sp_rows;
   p.ag_wait = ag_wait;

@@ -342,6 +342,13 @@ extern "C" int b200_gemm_bf16_swiglu(const void* W, const void* X, void* out_bf1
                              budget_ns ? budget_ns : B200_WAIT_BUDGET_NS, status, stream);
 }
 
+// The same epilogue with the clamped one-plus unit of glu.cuh (limit > 0), one rank.
+extern "C" int b200_gemm_bf16_glu(const void* W, const void* X, void* out_bf16, int T, int N, int K, float limit, float slope,
+                                  int* status, cudaStream_t stream) {
+  if (!b200_gemm_2cta_supported(T, N, K) || !out_bf16) return -ERR_BAD_ARG;
+  return b200_gemm_bf16_2cta_glu(W, X, out_bf16, T, N, K, GluShape{limit, slope}, status, stream);
+}
+
 extern "C" int b200_splitk_reduce(const float* part, int splits, long long n, const void* residual,
                                   void* out_bf16, cudaStream_t stream) {
   const int threads = 256;

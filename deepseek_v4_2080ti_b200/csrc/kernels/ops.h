@@ -174,12 +174,16 @@ int b200_kv8_dequantize(const void* k8, const void* v8, const float* k_scale, co
 // bias_act.cu, qk_row_prep.cu, attn_mix_prefill.cu, attn_mix_rows.cu) and the fp32 projection GEMM (gemm_f32.cu)
 int b200_residual_norm(float* x, const int* ids, const void* table, int vocab, const void* delta, const float* bias,
                        const float* post_w, const float* step, const float* pre_w, void* out, const int* rows, int n, int ld,
-                       int cols, float eps, int rms, int unit_offset, int write_x, int f32, cudaStream_t stream);
+                       int cols, float eps, int rms, int unit_offset, int write_x, float table_scale, int f32, cudaStream_t stream);
 int b200_gemm_bf16_bias_xielu(const void* W, const void* X, const float* bias, float ap, float an, void* out_bf16,
                               float* out_f32, int T, int N, int K, int splits, int* tile_counters, int* status,
                               cudaStream_t stream);
 int b200_bias_xielu(const void* in, const float* bias, void* out, long long rows, int ld, float ap, float an, int f32,
                     cudaStream_t stream);
+int b200_glu(const void* in, void* out, long long rows, int inter, int tile, float limit, float slope, int f32,
+             cudaStream_t stream);
+int b200_gemm_bf16_glu(const void* W, const void* X, void* out_bf16, int T, int N, int K, float limit, float slope, int* status,
+                       cudaStream_t stream);
 int b200_qk_row_prep(const void* proj, int ld, int q_off, int k_off, int v_off, const float* q_w, const float* k_w,
                      int q_count, int k_count, float eps, const double* freq, int rot, float mscale, const float* talk_t,
                      const int* positions, const int* slots, void* q_mix, float* q_row, void* k_cache, void* v_cache, int T,
@@ -193,6 +197,32 @@ int b200_attn_mix_prefill(const void* q_mix, const void* k_cache, const void* v_
                           const int* seq, const int* q_start, const int* q_len, const int* kv_len, int batch, int max_q_len,
                           int q_rows, int max_blocks, int num_blocks, int block_size, int H, int G, int D, int chunk, int ldo,
                           float scale, int* status, cudaStream_t stream);
+// Differential attention (qk_head_prep.cu, attn_diff_prefill.cu, attn_diff_rows.cu) and the recurrent mixer (conv_rows.cu,
+// selective_scan.cu)
+int b200_qk_head_prep(const void* proj, int ld, int q_off, int k_off, int v_off, int n_q, int n_k, int v_width, int D, int dim,
+                      const float* q_w, const float* k_w, float eps, float coef, double every, const int* positions,
+                      const int* slots, void* q, void* k_cache, void* v_cache, int rows, int f32, cudaStream_t stream);
+int b200_attn_diff_rows(const void* q, const void* k_cache, const void* v_cache, void* out, const void* gate, int ld_gate,
+                        const int* block_table, const int* seq, const int* positions, float* partial, int rows, int max_blocks,
+                        int block_size, int H, int G, int D, int V, int vdim, int splits, int ldo, float scale, float lambda,
+                        float keep, float eps, int f32, cudaStream_t stream);
+int b200_attn_diff_finish(const float* diff, void* out, const void* gate, int ld_gate, int rows, int H, int V, int vdim, int ldo,
+                          float keep, float eps, cudaStream_t stream);
+int b200_attn_diff_prefill_slices(int H, int G, int D, int V, int block_size);
+int b200_attn_diff_prefill(const void* q, const void* k_cache, const void* v_cache, void* out, float* diff, const void* gate,
+                           int ld_gate, const int* block_table, const int* seq, const int* q_start, const int* q_len,
+                           const int* kv_len, int batch, int max_q_len, int q_rows, int max_blocks, int num_blocks, int block_size,
+                           int H, int G, int D, int V, int vdim, int ldo, float scale, float lambda, float keep, float eps,
+                           int* status, cudaStream_t stream);
+int b200_conv_rows(const void* x, int ldx, const float* w, const float* bias, const void* tail, const int* row_first,
+                   const int* row_slot, const int* positions, void* y, int ldy, int rows, int C, int taps, int silu, int f32,
+                   cudaStream_t stream);
+int b200_selective_scan_channels(int N);
+int b200_selective_scan(const void* x, int ldx, const float* dt, int ldd, const void* bc, int ldb, int b_off, int c_off,
+                        const void* z, int ldz, void* out, int ldo, const float* a, const float* dt_bias, const float* d_skip,
+                        float* state, const int* ent_first, const int* ent_len, const int* ent_slot, const int* positions,
+                        const void* xin, int ldin, void* tail, int taps, int C, int N, int entries, int slices, int per,
+                        float* ws_state, float* ws_sum, int f32, cudaStream_t stream);
 int b200_gemm_f32(const float* x, const float* w, float* y, int T, int N, int K, cudaStream_t stream);
 
 #ifdef __cplusplus

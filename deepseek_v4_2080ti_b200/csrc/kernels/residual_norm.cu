@@ -3,8 +3,9 @@
 //   x   (+)= norm(delta + bias) * post_w        the sublayer's output enters the fp32 residual through its own norm
 //   x    += step                                optional vector added between layers (start of a looped pass)
 //   out   = norm(x) * pre_w                     input of the next sublayer, or of the output head
+//   out   = x                                   without pre_w: the next sublayer reads the residual itself (rounded)
 //
-// Every part is optional.  The row may start from an embedding table instead of a stored residual (first layer), and
+// Every part is optional.  The row may start from a (scaled) embedding table instead of a stored residual (first layer), and
 // the launch may be restricted to a list of rows (output head of the wanted positions only).  The norm is a layer norm
 // (centred) or an RMS norm, with plain or one-plus weights.  The residual is fp32; delta and out are bf16 or fp32.
 // Rows are `ld` wide in memory (a multiple of 8); columns past `cols` are zero on input and written as zero.
@@ -29,7 +30,7 @@ struct ResidualNormParams {
   T* out;                    // [rows out, ld] or null
   const int* rows;           // not null: output row i works on stored row rows[i]
   int ld, cols, rms, unit_offset, write_x;
-  float eps;
+  float eps, table_scale;
 };
 
 template <typename T, int VEC>
@@ -89,7 +90,11 @@ __global__ void residual_norm_kernel(ResidualNormParams<T> p) {
     for (int j = 0; j < 8; ++j) x[it][j] = d[it][j] = 0.f;
     if (v < nvec) {
       if (!p.ids) load8(p.x + row * p.ld + v * 8, x[it]);
-      else if (src_row) load8(src_row + v * 8, x[it]);
+      else if (src_row) {
+        load8(src_row + v * 8, x[it]);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x[it][j] *= p.table_scale;
+      }
       if (p.delta) {
         load8(p.delta + row * p.ld + v * 8, d[it]);
         if (p.bias) {
@@ -122,7 +127,7 @@ __global__ void residual_norm_kernel(ResidualNormParams<T> p) {
     }
   }
   if (!p.out) return;
-  normalise(x, p.pre_w);
+  if (p.pre_w) normalise(x, p.pre_w);
 #pragma unroll
   for (int it = 0; it < VEC; ++it) {
     const int v = threadIdx.x + it * blockDim.x;
@@ -146,12 +151,12 @@ int launch_residual_norm(ResidualNormParams<T> p, int n, cudaStream_t stream) {
 template <typename T>
 int run_residual_norm(float* x, const int* ids, const void* table, int vocab, const void* delta, const float* bias,
                       const float* post_w, const float* step, const float* pre_w, void* out, const int* rows, int n, int ld,
-                      int cols, float eps, int rms, int unit_offset, int write_x, cudaStream_t stream) {
+                      int cols, float eps, int rms, int unit_offset, int write_x, float table_scale, cudaStream_t stream) {
   ResidualNormParams<T> p;
   p.x = x; p.ids = ids; p.table = reinterpret_cast<const T*>(table); p.vocab = vocab;
   p.delta = reinterpret_cast<const T*>(delta); p.bias = bias; p.post_w = post_w; p.step = step; p.pre_w = pre_w;
   p.out = reinterpret_cast<T*>(out); p.rows = rows; p.ld = ld; p.cols = cols; p.rms = rms; p.unit_offset = unit_offset;
-  p.write_x = write_x; p.eps = eps;
+  p.write_x = write_x; p.eps = eps; p.table_scale = table_scale;
   return launch_residual_norm(p, n, stream);
 }
 
@@ -161,11 +166,11 @@ int run_residual_norm(float* x, const int* ids, const void* table, int vocab, co
 extern "C" int b200_residual_norm(float* x, const int* ids, const void* table, int vocab, const void* delta,
                                   const float* bias, const float* post_w, const float* step, const float* pre_w, void* out,
                                   const int* rows, int n, int ld, int cols, float eps, int rms, int unit_offset, int write_x,
-                                  int f32, cudaStream_t stream) {
+                                  float table_scale, int f32, cudaStream_t stream) {
   if (n <= 0 || ld <= 0 || (ld & 7) || ld > 16384 || cols <= 0 || cols > ld) return -6;
-  if ((out && !pre_w) || (!ids && !x) || (write_x && !x) || (ids && !table)) return -6;
+  if ((pre_w && !out) || (!ids && !x) || (write_x && !x) || (ids && !table)) return -6;
   return f32 ? run_residual_norm<float>(x, ids, table, vocab, delta, bias, post_w, step, pre_w, out, rows, n, ld, cols, eps,
-                                        rms, unit_offset, write_x, stream)
+                                        rms, unit_offset, write_x, table_scale, stream)
              : run_residual_norm<__nv_bfloat16>(x, ids, table, vocab, delta, bias, post_w, step, pre_w, out, rows, n, ld,
-                                                cols, eps, rms, unit_offset, write_x, stream);
+                                                cols, eps, rms, unit_offset, write_x, table_scale, stream);
 }

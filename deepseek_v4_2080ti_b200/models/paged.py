@@ -15,6 +15,9 @@ from dataclasses import dataclass, field
 
 import torch
 
+from ..ops.scan import Segments
+from ..utils import canary
+
 
 @dataclass
 class SeqState:
@@ -127,7 +130,12 @@ class PagedRuntime(PagedSequences):
     ``meta["mode"]``: ``"decode"`` - one row per sequence, static buffers (``block_table`` row i belongs to row i,
     ``kv_len``, ``max_kv_len``); ``"mixed"`` - the first ``tile_rows`` rows are portions of several sequences
     (``tile_table``, ``q_start``, ``q_len``, ``kv_len``, ``max_q_len``; ``tile_seq`` / ``tile_pos_rows`` per row), the
-    rest single rows (``row_table``, ``row_kv_len``, ``max_kv_len``).
+    rest single rows (``row_seq``, ``max_kv_len``).  In both modes ``segments`` says which neighbouring rows form one
+    sequence's portion and which state slot it has, for mixers that carry a recurrent state.
+
+    Recurrent state is held per request slot in tensors from ``slot_state``; a slot's content is meaningless until its
+    sequence's first token, whose position 0 the kernels take as "start from zero".  The slot after the last one is scratch:
+    the pass that warms up a decode graph runs on it, because running a recurrent step twice would advance the state twice.
     """
     tile_min_rows = 2            # portions with fewer tokens run as single rows
 
@@ -137,6 +145,14 @@ class PagedRuntime(PagedSequences):
         self._graphs: dict[tuple, dict] = {}
         self.launches = 0
         self.last_logits: torch.Tensor | None = None
+
+    def slot_state(self, *shape: int, dtype: torch.dtype, name: str) -> torch.Tensor:
+        """[request slots + scratch, ...] of recurrent state."""
+        return canary.zeros(self.max_slots + 1, *shape, dtype=dtype, device=self.device, name=name)
+
+    @property
+    def scratch_slot(self) -> int:
+        return self.max_slots
 
     @property
     def max_blocks(self) -> int:
@@ -190,19 +206,21 @@ class PagedRuntime(PagedSequences):
         rows = cat([self.cache_rows(sts[i], sts[i].length, sts[i].length + lens[i]) for i in order])
         seq = cat([torch.full((lens[i],), sts[i].slot, dtype=torch.int32) for i in order])
         want = torch.tensor([first[i] + w for i, e in enumerate(entries) for w in e[2]], dtype=torch.int32)
-        desc = torch.tensor([[first[i], lens[i], sts[i].length + lens[i], sts[i].slot] for i in tiles], dtype=torch.int32).reshape(-1)
-        # one upload: [ids | positions | cache rows | table rows | tile descriptors | wanted rows]
-        up = cat([tok, pos, rows, seq, desc, want])
+        start = cat([torch.full((lens[i],), first[i], dtype=torch.int32) for i in order])
+        desc = torch.tensor([[first[i], lens[i], sts[i].length + lens[i], sts[i].slot] for i in order], dtype=torch.int32).t().reshape(-1)
+        # one upload: [ids | positions | cache rows | table rows | entry starts | entry descriptors | wanted rows]
+        up = cat([tok, pos, rows, seq, start, desc, want])
         up = up.pin_memory().to(dev, non_blocking=True) if dev.type == "cuda" else up
-        ids, pos_d, slots_d, seq_d = (up[k * n_rows:(k + 1) * n_rows] for k in range(4))
-        desc_d = up[4 * n_rows:4 * n_rows + desc.numel()].view(-1, 4)
+        ids, pos_d, slots_d, seq_d, start_d = (up[k * n_rows:(k + 1) * n_rows] for k in range(5))
+        e_first, e_len, e_kv, e_slot = up[5 * n_rows:5 * n_rows + desc.numel()].view(4, -1)
         meta = {"mode": "mixed", "tile_rows": tile_rows, "row_seq": seq_d, "max_q_len": max([lens[i] for i in tiles], default=0),
-                "max_kv_len": max(sts[i].length + lens[i] for i in range(len(entries)))}
+                "max_kv_len": max(sts[i].length + lens[i] for i in range(len(entries))),
+                "segments": Segments(start_d, seq_d, e_first, e_len, e_slot, max(lens))}
         if tiles:
-            meta.update(q_start=desc_d[:, 0].contiguous(), q_len=desc_d[:, 1].contiguous(), kv_len=desc_d[:, 2].contiguous(),
-                        tile_seq=desc_d[:, 3].contiguous())
+            n = len(tiles)
+            meta.update(q_start=e_first[:n], q_len=e_len[:n], kv_len=e_kv[:n], tile_seq=e_slot[:n])
         # a pass has to run even when no logits are asked for: it fills the cache
-        wanted = up[4 * n_rows + desc.numel():]
+        wanted = up[5 * n_rows + desc.numel():]
         logits = self._forward(ids, pos_d, slots_d, meta, wanted)
         for st, n in zip(sts, lens):
             st.length += n
@@ -226,7 +244,9 @@ class PagedRuntime(PagedSequences):
 
     # ---- one token for each of several requests
     def _decode_body(self, buf, bucket: int) -> torch.Tensor:
-        meta = {"mode": "decode", "block_table": buf["bt"], "kv_len": buf["kv_len"], "max_kv_len": bucket}
+        row = buf["row"]
+        meta = {"mode": "decode", "block_table": buf["bt"], "kv_len": buf["kv_len"], "max_kv_len": bucket,
+                "segments": Segments(row, buf["slots"], row, buf["one"], buf["slots"], 1)}
         buf["logits"] = self._forward(buf["ids"], buf["pos"], buf["kv_slots"], meta, None)
         return self._next(buf["logits"])
 
@@ -241,7 +261,9 @@ class PagedRuntime(PagedSequences):
         entry = self._graphs.setdefault((b, bucket), {"buf": None, "graph": None})
         if entry["buf"] is None:
             z = lambda *s: torch.zeros(*s, dtype=torch.int32, device=dev)
-            entry["buf"] = {"ids": z(b), "pos": z(b), "kv_slots": z(b), "kv_len": z(b) + 1, "bt": z(b, self.max_blocks)}
+            entry["buf"] = {"ids": z(b), "pos": z(b), "kv_slots": z(b), "kv_len": z(b) + 1, "bt": z(b, self.max_blocks),
+                            "slots": z(b) + self.scratch_slot, "one": z(b) + 1,
+                            "row": torch.arange(b, dtype=torch.int32, device=dev)}
         buf = entry["buf"]
         host = torch.tensor([[st.length, st.length + 1, st.slot,
                               st.blocks[st.length // self.block_size] * self.block_size + st.length % self.block_size]
@@ -251,19 +273,22 @@ class PagedRuntime(PagedSequences):
         buf["kv_len"].copy_(host[:, 1])
         buf["kv_slots"].copy_(host[:, 3])
         buf["bt"].copy_(self.block_table[host[:, 2].long()])
-        if not use_graph or dev.type != "cuda":
+        graphed = use_graph and dev.type == "cuda"
+        if graphed and entry["graph"] is None:
+            buf["slots"].fill_(self.scratch_slot)       # the K/V rows the warm-up writes are rewritten by the replay
+            self._decode_body(buf, bucket)
+            torch.cuda.synchronize()
+            g = torch.cuda.CUDAGraph()
+            l0 = _lib.LAUNCHES
+            with torch.cuda.graph(g):
+                entry["out"] = self._decode_body(buf, bucket)
+            entry["graph"], entry["launches"] = g, _lib.LAUNCHES - l0
+        buf["slots"].copy_(host[:, 2])
+        if not graphed:
             l0 = _lib.LAUNCHES
             out = self._decode_body(buf, bucket)
             self.launches = _lib.LAUNCHES - l0
         else:
-            if entry["graph"] is None:
-                self._decode_body(buf, bucket)          # warm-up: the K/V row written here is rewritten by the replay
-                torch.cuda.synchronize()
-                g = torch.cuda.CUDAGraph()
-                l0 = _lib.LAUNCHES
-                with torch.cuda.graph(g):
-                    entry["out"] = self._decode_body(buf, bucket)
-                entry["graph"], entry["launches"] = g, _lib.LAUNCHES - l0
             entry["graph"].replay()
             self.launches = entry["launches"]
             out = entry["out"]

@@ -441,3 +441,35 @@ def _rutulix_sources() -> tuple[str, ...]:
 register_checkpoint(CheckpointSpec("rutulix", "Rutulix (head-mixed chunked attention, sandwich norms, looped layers)",
                                    _rutulix_matches, _rutulix_build, dtypes=("bfloat16", "float32"),
                                    kernel_sources=_rutulix_sources(), tensor_shapes=_rutulix_shapes))
+
+
+def _zigasun_matches(raw) -> bool:
+    from .zigasun import ZigasunConfig
+    return ZigasunConfig.is_zigasun_json(raw)
+
+
+def _zigasun_build(raw, directory, device, rank=0, world=1, dtype=None, max_slots=1, max_context=4096, num_blocks=None,
+                   make_comm=None):
+    from ..formats import safetensors_io
+    from . import zigasun as zg
+    if world != 1:
+        raise ValueError("a Zigasun model runs on one rank")
+    cfg = zg.ZigasunConfig.from_json(raw)
+    w = zg.ZigasunWeights(cfg, safetensors_io.read_checkpoint(directory), device,
+                          _torch_dtype(dtype, ("bfloat16", "float32")))
+    return cfg, zg.ZigasunRuntime(cfg, w, max_slots=max_slots, max_context=max_context, num_blocks=num_blocks)
+
+
+def _zigasun_shapes(raw) -> dict[str, tuple[int, ...]]:
+    from .zigasun import ZigasunConfig
+    return ZigasunConfig.from_json(raw).tensor_shapes()
+
+
+def _zigasun_sources() -> tuple[str, ...]:
+    from .zigasun import KERNEL_SOURCES
+    return KERNEL_SOURCES
+
+
+register_checkpoint(CheckpointSpec("zigasun", "Zigasun (differential attention, selective scan, clamped gated feed-forward)",
+                                   _zigasun_matches, _zigasun_build, dtypes=("bfloat16", "float32"),
+                                   kernel_sources=_zigasun_sources(), tensor_shapes=_zigasun_shapes))

@@ -1,0 +1,154 @@
+"""Pieces shared by the decoders with an fp32 residual stream: padded projections, the boundary between sublayers
+(csrc/kernels/residual_norm.cu), activations (bias_act.cu) and the fp32 GEMM (gemm_f32.cu).
+
+All of them exist for bf16 and for fp32 activations; the tensors' dtype decides.  Row widths are padded to multiples of 16
+(``pad16``) with zero columns, so that every access is a full vector.
+"""
+from __future__ import annotations
+
+import ctypes
+from dataclasses import dataclass
+
+import torch
+
+from . import _lib
+
+_f = ctypes.c_float
+_ll = ctypes.c_longlong
+
+
+def pad16(n: int) -> int:
+    return (n + 15) // 16 * 16
+
+
+def pad8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+# ---------------------------------------------------------------------------------------------- projections
+@dataclass
+class Projection:
+    """[N, K] weight with both sides padded to multiples of 16 by zeros: bf16 for the tensor-core GEMM, fp32 for the
+    fp32 one."""
+    packed: object              # PackedLinear, or None
+    w32: torch.Tensor | None
+    n: int
+    k: int
+
+    @staticmethod
+    def make(w: torch.Tensor, dtype: torch.dtype, device, pad_n: bool = True, tile_n: bool = False) -> "Projection":
+        """``tile_n``: rows up to a multiple of 256 where that adds at most an eighth, so that prefill-sized batches tile
+        evenly on the CTA-pair GEMM."""
+        from .gemm import PackedLinear
+        n, k = w.shape
+        np_, kp = pad16(n) if pad_n else n, pad16(k)
+        if pad_n and tile_n and (n + 255) // 256 * 256 <= n + n // 8:
+            np_ = (n + 255) // 256 * 256
+        full = torch.zeros(np_, kp, dtype=dtype, device=device)
+        full[:n, :k] = w.to(device, dtype)
+        if dtype == torch.float32:
+            return Projection(None, full, np_, kp)
+        return Projection(PackedLinear.from_bf16(full), None, np_, kp)
+
+    def __call__(self, x: torch.Tensor, out_f32: bool = False) -> torch.Tensor:
+        if self.w32 is None:
+            from . import gemm
+            return gemm.linear(x, self.packed, out_f32=out_f32)
+        return gemm_f32(x, self.w32)
+
+    def glu(self, x: torch.Tensor, limit: float, slope: float = 1.702) -> torch.Tensor:
+        """Gated unit over this projection's [gate | up] features, which ``interleave_glu`` laid out in tiles: in the GEMM's
+        epilogue where the batch tiles evenly on the CTA-pair kernel, in a kernel of its own otherwise."""
+        if self.w32 is None:
+            from . import gemm
+            if gemm.glu_fusable(x.shape[0], self.packed):
+                return gemm.linear_glu(x, self.packed, limit, slope)
+        return glu(self(x), GLU_TILE, limit, slope)
+
+    def bias_xielu(self, x: torch.Tensor, bias: torch.Tensor, ap: float, an: float) -> torch.Tensor:
+        """xIELU(projection + bias): in the GEMM's epilogue, or as a second kernel in fp32."""
+        if self.w32 is None:
+            from . import gemm
+            return gemm.linear_bias_xielu(x, self.packed, bias, ap, an)
+        return bias_xielu(gemm_f32(x, self.w32), bias, ap, an)
+
+    def nbytes(self) -> int:
+        return self.n * self.k * (4 if self.packed is None else 2)
+
+
+GLU_TILE = 128          # features per gate / up tile of an interleaved projection
+
+
+def interleave_glu(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
+    """[I, K] gate and up weights -> [2 I', K] with their rows in alternating tiles, I' = I rounded up to whole tiles (the
+    zero rows give a unit of zero)."""
+    n, k = gate.shape
+    np_ = (n + GLU_TILE - 1) // GLU_TILE * GLU_TILE
+    out = torch.zeros(np_ // GLU_TILE, 2, GLU_TILE, k, dtype=gate.dtype, device=gate.device)
+    for i, w in enumerate((gate, up)):
+        full = torch.zeros(np_, k, dtype=w.dtype, device=w.device)
+        full[:n] = w
+        out[:, i] = full.view(-1, GLU_TILE, k)
+    return out.view(2 * np_, k)
+
+
+def gemm_f32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """fp32 [T, K] x [N, K]^T without any reduced-precision mode."""
+    t, k = x.shape
+    assert x.dtype == w.dtype == torch.float32 and x.is_contiguous() and w.is_contiguous() and w.shape[1] == k
+    y = torch.empty(t, w.shape[0], dtype=torch.float32, device=x.device)
+    _lib.check(_lib.lib().b200_gemm_f32(_lib.ptr(x), _lib.ptr(w), _lib.ptr(y), t, w.shape[0], k, _lib.stream()), "gemm_f32")
+    return y
+
+
+# ---------------------------------------------------------------------------------------------- residual stream
+def residual_norm(x: torch.Tensor, cols: int, eps: float, *, delta: torch.Tensor | None = None,
+                  bias: torch.Tensor | None = None, post_w: torch.Tensor | None = None, step: torch.Tensor | None = None,
+                  pre_w: torch.Tensor | None = None, ids: torch.Tensor | None = None, table: torch.Tensor | None = None,
+                  rows: torch.Tensor | None = None, dtype: torch.dtype | None = None, rms: bool = False,
+                  unit_offset: bool = False, write_x: bool = True, table_scale: float = 1.0,
+                  plain: bool = False) -> torch.Tensor | None:
+    """One boundary between sublayers of an fp32 residual ``x`` [T, ld] (updated in place):
+    ``x += norm(delta + bias) * post_w``, ``x += step``, and the return value ``norm(x) * pre_w`` in ``dtype`` (None
+    without ``pre_w``; with ``plain``: ``x`` itself).  ``ids`` / ``table``: the row starts as an embedding row times
+    ``table_scale`` instead of ``x``.  ``rows`` (int32): only these rows are processed, and ``x`` is left alone.  Layer norm,
+    or RMS norm with ``rms``."""
+    ld = x.shape[1]
+    n = rows.numel() if rows is not None else x.shape[0]
+    ref = delta if delta is not None else table
+    dtype = dtype or (ref.dtype if ref is not None else torch.bfloat16)
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    for t in (delta, table):
+        assert t is None or (t.dtype == dtype and t.shape[1] == ld and t.is_contiguous())
+    for t in (bias, post_w, step, pre_w):
+        assert t is None or (t.dtype == torch.float32 and t.numel() == ld)
+    if ids is not None:
+        _lib.check_indices(ids, 0, table.shape[0], 1)
+    if rows is not None:
+        _lib.check_indices(rows, 0, x.shape[0], 7)
+    out = torch.empty(n, ld, dtype=dtype, device=x.device) if pre_w is not None or plain else None
+    rc = _lib.lib().b200_residual_norm(
+        _lib.ptr(x), _lib.ptr(ids), _lib.ptr(table), 0 if table is None else table.shape[0], _lib.ptr(delta), _lib.ptr(bias),
+        _lib.ptr(post_w), _lib.ptr(step), _lib.ptr(pre_w), _lib.ptr(out), _lib.ptr(rows), n, ld, cols, _f(eps), int(rms),
+        int(unit_offset), int(write_x and rows is None), _f(table_scale), int(dtype == torch.float32), _lib.stream())
+    _lib.check(rc, "residual_norm")
+    return out
+
+
+def bias_xielu(z: torch.Tensor, bias: torch.Tensor | None, ap: float, an: float) -> torch.Tensor:
+    """xIELU(z + bias) with the positive-side and negative-side coefficients."""
+    out = torch.empty_like(z)
+    rc = _lib.lib().b200_bias_xielu(_lib.ptr(z), _lib.ptr(bias), _lib.ptr(out), _ll(z.shape[0]), z.shape[1], _f(ap), _f(an),
+                                    int(z.dtype == torch.float32), _lib.stream())
+    _lib.check(rc, "bias_xielu")
+    return out
+
+
+def glu(z: torch.Tensor, tile: int, limit: float, slope: float = 1.702) -> torch.Tensor:
+    """Gated unit over rows of gate and up features interleaved in tiles of ``tile`` columns: the clamped one-plus form
+    ``min(g, limit) sigmoid(slope min(g, limit)) (clamp(u, -limit, limit) + 1)``, or ``silu(g) u`` with ``limit`` 0."""
+    out = torch.empty(z.shape[0], z.shape[1] // 2, dtype=z.dtype, device=z.device)
+    rc = _lib.lib().b200_glu(_lib.ptr(z), _lib.ptr(out), _ll(z.shape[0]), out.shape[1], tile, _f(limit), _f(slope),
+                             int(z.dtype == torch.float32), _lib.stream())
+    _lib.check(rc, "glu")
+    return out

@@ -416,6 +416,23 @@ def linear_bias_xielu(x: torch.Tensor, w: PackedLinear, bias: torch.Tensor, ap: 
     return out
 
 
+def glu_fusable(t: int, w: PackedLinear) -> bool:
+    """Can ``linear_glu`` take bf16 matrix ``w`` for ``t`` tokens?  A prefill-sized batch that the CTA-pair kernel tiles
+    evenly."""
+    return w.wfmt == WF_BF16 and t > 128 and bool(_lib.lib().b200_gemm_2cta_supported(t, w.n, w.k))
+
+
+def linear_glu(x: torch.Tensor, w: PackedLinear, limit: float, slope: float) -> torch.Tensor:
+    """Gated unit of ``x @ w^T`` in one kernel for bf16 weights whose rows alternate in 128-row tiles [gate | up]: the clamped
+    one-plus form of csrc/kernels/glu.cuh on the fp32 sums in the GEMM epilogue."""
+    assert x.dtype == torch.bfloat16 and x.is_cuda and x.dim() == 2 and x.is_contiguous() and x.shape[1] == w.k
+    out = torch.empty(x.shape[0], w.n // 2, dtype=torch.bfloat16, device=x.device)
+    rc = _lib.lib().b200_gemm_bf16_glu(_lib.ptr(w.weight), _lib.ptr(x), _lib.ptr(out), x.shape[0], w.n, w.k, ctypes.c_float(limit),
+                                       ctypes.c_float(slope), _lib.ptr(_lib.status_word(x.device)), _lib.stream())
+    _lib.check(rc, "gemm_bf16_glu")
+    return out
+
+
 def linear_ref(x: torch.Tensor, w_fp32: torch.Tensor, residual: torch.Tensor | None = None) -> torch.Tensor:
     """fp32 oracle: x @ w^T (+ residual)."""
     y = x.float() @ w_fp32.float().t()
