@@ -221,8 +221,8 @@ int b200_selective_scan_channels(int N);
 int b200_selective_scan(const void* x, int ldx, const float* dt, int ldd, const void* bc, int ldb, int b_off, int c_off,
                         const void* z, int ldz, void* out, int ldo, const float* a, const float* dt_bias, const float* d_skip,
                         float* state, const int* ent_first, const int* ent_len, const int* ent_slot, const int* positions,
-                        const void* xin, int ldin, void* tail, int taps, int C, int N, int entries, int slices, int per,
-                        float* ws_state, float* ws_sum, int f32, cudaStream_t stream);
+                        const void* xin, int ldin, void* tail, int taps, int C, int N, int entries, int max_len, int singles,
+                        int slices, int per, float* ws_state, float* ws_sum, int f32, cudaStream_t stream);
 int b200_gemm_f32(const float* x, const float* w, float* y, int T, int N, int K, cudaStream_t stream);
 
 #ifdef __cplusplus

@@ -215,7 +215,7 @@ class PagedRuntime(PagedSequences):
         e_first, e_len, e_kv, e_slot = up[5 * n_rows:5 * n_rows + desc.numel()].view(4, -1)
         meta = {"mode": "mixed", "tile_rows": tile_rows, "row_seq": seq_d, "max_q_len": max([lens[i] for i in tiles], default=0),
                 "max_kv_len": max(sts[i].length + lens[i] for i in range(len(entries))),
-                "segments": Segments(start_d, seq_d, e_first, e_len, e_slot, max(lens))}
+                "segments": Segments(start_d, seq_d, e_first, e_len, e_slot, max(lens), min(lens))}
         if tiles:
             n = len(tiles)
             meta.update(q_start=e_first[:n], q_len=e_len[:n], kv_len=e_kv[:n], tile_seq=e_slot[:n])
@@ -246,7 +246,7 @@ class PagedRuntime(PagedSequences):
     def _decode_body(self, buf, bucket: int) -> torch.Tensor:
         row = buf["row"]
         meta = {"mode": "decode", "block_table": buf["bt"], "kv_len": buf["kv_len"], "max_kv_len": bucket,
-                "segments": Segments(row, buf["slots"], row, buf["one"], buf["slots"], 1)}
+                "segments": Segments(row, buf["slots"], row, buf["one"], buf["slots"], 1, 1)}
         buf["logits"] = self._forward(buf["ids"], buf["pos"], buf["kv_slots"], meta, None)
         return self._next(buf["logits"])
 

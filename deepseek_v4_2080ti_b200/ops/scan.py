@@ -28,6 +28,7 @@ class Segments:
     length: torch.Tensor
     slot: torch.Tensor
     max_length: int
+    min_length: int = 1
 
 
 def conv_rows(x: torch.Tensor, w_t: torch.Tensor, bias: torch.Tensor | None, tail: torch.Tensor, seg: Segments,
@@ -95,9 +96,9 @@ def selective_scan(x: torch.Tensor, dt: torch.Tensor, bc: torch.Tensor, b_off: i
         _lib.ptr(x), c, _lib.ptr(dt), dt.stride(0), _lib.ptr(bc), bc.stride(0), b_off, c_off, _lib.ptr(z), z.stride(0),
         _lib.ptr(out), c, _lib.ptr(a), _lib.ptr(dt_bias), _lib.ptr(d_skip), _lib.ptr(state), _lib.ptr(seg.first),
         _lib.ptr(seg.length), _lib.ptr(seg.slot), _lib.ptr(positions), _lib.ptr(x_in), 0 if x_in is None else x_in.stride(0),
-        _lib.ptr(tail), taps, c, n, entries, slices, per, _lib.ptr(ws_state), _lib.ptr(ws_sum), int(x.dtype == torch.float32),
+        _lib.ptr(tail), taps, c, n, entries, seg.max_length, int(seg.min_length == 1), slices, per, _lib.ptr(ws_state), _lib.ptr(ws_sum), int(x.dtype == torch.float32),
         _lib.stream())
-    _lib.check(rc, "selective_scan", 2 if slices > 1 else 1)
+    _lib.check(rc, "selective_scan", int(seg.min_length == 1) + (0 if seg.max_length == 1 else 2 if slices > 1 else 1))
     return out
 
 

@@ -1,10 +1,11 @@
-"""Prefill and decode throughput of the Rutulix decoder at sizes of real models' layers (random weights), beside the
+"""Prefill and decode throughput of one decoder design at sizes of real models' layers (random weights), beside the
 framework's closest existing model at equal size, and the kernels of both beside their rooflines.
 
-    python bench.py --design rutulix [--design-size small|large] [--steps K] [--warmup W]
+    python bench.py --design rutulix|zigasun [--design-size small|large] [--steps K] [--warmup W]
 
-Closest model: the Qwen-style decoder with full-attention layers only (per-head QK norm, grouped attention, SwiGLU with
-FP8 weights) of the same width, heads and feed-forward parameters.  Whole-model numbers: CUDA events around a prompt of
+Closest model of Rutulix: the Qwen-style decoder with full-attention layers only (per-head QK norm, grouped attention, SwiGLU
+with FP8 weights) of the same width, heads and feed-forward parameters.  Of Zigasun: the same decoder with Gated-DeltaNet and
+full-attention layers in turn (both recurrent states as wide as the scan's channels).  Whole-model numbers: CUDA events around a prompt of
 ``--prompt`` tokens and around replayed decode steps.  Kernel numbers: CUDA events around single launches, L2 flushed
 before each; fractions of the measured copy bandwidth / bf16 GEMM burst of MEASURED_PEAKS.json.
 """
@@ -16,8 +17,10 @@ import os
 import torch
 
 PEAKS_FALLBACK = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
-# width, heads, kv heads, head dim, SwiGLU width of the closest model (the two-matrix feed-forward gets 3/2 of it), chunk
+# Rutulix: width, heads, kv heads, head dim, SwiGLU width of the closest model (the two-matrix feed-forward gets 3/2 of it), chunk
 SIZES = {"small": (2048, 16, 4, 128, 5632, 2048), "large": (4096, 32, 8, 128, 10752, 8192)}
+# Zigasun: width, heads, kv heads, dim per map, value dim, feed-forward, scan channels, states, dt rank
+ZG_SIZES = {"small": (2048, 16, 4, 64, 128, 5632, 4096, 16, 128), "large": (4096, 32, 8, 64, 128, 10752, 8192, 16, 256)}
 LAYERS, VOCAB = 4, 32768
 
 
@@ -89,19 +92,12 @@ def _throughput(make, dev, prompt: int, slots: int, timer: _Timer) -> dict:
     return out
 
 
-def _kernels(size: str, dev, timer: _Timer, ctx: int) -> list[dict]:
-    """One row per kernel pair: (what, shape, new ms and fraction, like kernel ms and fraction)."""
-    from ..ops import attention, basic, gemm, mixattn
-    from ..models import rutulix as rx
-    width, H, G, D, inter, chunk = SIZES[size]
-    ff = inter * 3 // 2
+def _recorder(timer: _Timer):
+    """(rows, pair): ``pair(what, shape, new, like)`` times two (call, bytes, flops) and appends one row: ms and roofline
+    fraction of both and the distance ratio."""
     peaks, _ = _peaks()
     bw, fl = peaks["hbm_gbs"] * 1e6, peaks["bf16_tflops"] * 1e9            # bytes, flops per ms
-    rnd = lambda *s, dt=torch.bfloat16: torch.randn(*s, device=dev, dtype=torch.float32).to(dt)
-    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
-    cfg = rx.RutulixConfig.uniform(1, width, H, G, D, ff, 64, chunk)
-    m = rx.RutulixWeights(cfg, rx.synth_state(cfg, 0, dev), dev).layers[0].mix
-    rows_out = []
+    rows_out: list[dict] = []
 
     def pair(what, shape, new, old):
         rec = {"kernel": what, "shape": shape}
@@ -115,7 +111,20 @@ def _kernels(size: str, dev, timer: _Timer, ctx: int) -> list[dict]:
         if "like" in rec:
             rec["distance_ratio"] = round(rec["like"]["fraction"] / rec["new"]["fraction"], 2)
         rows_out.append(rec)
+    return rows_out, pair
 
+
+def _kernels(size: str, dev, timer: _Timer, ctx: int) -> list[dict]:
+    """One row per kernel pair: (what, shape, new ms and fraction, like kernel ms and fraction)."""
+    from ..ops import attention, basic, gemm, mixattn
+    from ..models import rutulix as rx
+    width, H, G, D, inter, chunk = SIZES[size]
+    ff = inter * 3 // 2
+    rnd = lambda *s, dt=torch.bfloat16: torch.randn(*s, device=dev, dtype=torch.float32).to(dt)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    cfg = rx.RutulixConfig.uniform(1, width, H, G, D, ff, 64, chunk)
+    m = rx.RutulixWeights(cfg, rx.synth_state(cfg, 0, dev), dev).layers[0].mix
+    rows_out, pair = _recorder(timer)
     bs, pages = 64, (ctx + 63) // 64
     for t in (8192, 32):
         x32, x16, d16 = rnd(t, width, dt=torch.float32), rnd(t, width), rnd(t, width)
@@ -181,31 +190,143 @@ def _kernels(size: str, dev, timer: _Timer, ctx: int) -> list[dict]:
     return rows_out
 
 
+def _zg_models(size: str, dev, prompt: int, slots: int):
+    from ..models import qwen_hybrid as qh
+    from ..models import zigasun as zg
+    width, heads, kv, dim, vdim, ff, inner, states, rank = ZG_SIZES[size]
+    cfg = zg.ZigasunConfig.alternating(LAYERS, width, heads, kv, dim, vdim, ff, inner, states, rank, VOCAB)
+    for L in cfg.layers:                       # the closest model has a feed-forward in every layer
+        L.ff, L.limit = ff, 7.0
+    new = lambda: zg.build_synthetic(cfg, dev, max_slots=slots, max_context=prompt + 192)
+    qcfg = qh.QwenHybridConfig(vocab_size=VOCAB, hidden_size=width, intermediate_size=ff, num_hidden_layers=LAYERS,
+                               num_attention_heads=heads, num_key_value_heads=kv, attn_output_gate=False,
+                               linear_num_key_heads=16, linear_num_value_heads=inner // 128,
+                               layer_types=["full_attention", "linear_attention"] * (LAYERS // 2))
+    old = lambda: qh.build_synthetic(qcfg, dev, max_slots=slots, max_context=prompt + 192)
+    return new, old
+
+
+def _zg_kernels(size: str, dev, timer: _Timer, ctx: int) -> list[dict]:
+    from ..models import zigasun as zg
+    from ..ops import attention, basic, decoder, diffattn, gdn, gemm, scan
+    width, H, G, D, V, ff, inner, N, rank = ZG_SIZES[size]
+    rnd = lambda *s, dt=torch.bfloat16: torch.randn(*s, device=dev, dtype=torch.float32).to(dt)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    cfg = zg.ZigasunConfig.alternating(2, width, H, G, D, V, ff, inner, N, rank, 64)
+    w = zg.ZigasunWeights(cfg, zg.synth_state(cfg, 0, dev), dev)
+    aw, sw = w.layers[0].mix, w.layers[1].mix
+    m = aw.m
+    rows_out, pair = _recorder(timer)
+    bs, pages = 64, (ctx + 63) // 64
+    hv, hk = inner // 128, 16
+    for t in (8192, 32):
+        x32, x16, d16 = rnd(t, width, dt=torch.float32), rnd(t, width), rnd(t, width)
+        g32, g16 = torch.ones(width, device=dev), torch.ones(width, device=dev, dtype=torch.bfloat16)
+        # fp32 residual read + written, delta read, output written against a bf16 residual
+        pair("residual + norm", f"{t} x {width}",
+             (lambda: decoder.residual_norm(x32, width, 1e-5, delta=d16, post_w=g32, rms=True, plain=True), t * width * 12, 0),
+             (lambda: basic.add_rmsnorm(x16, d16, g16, 1e-5), t * width * 8, 0))
+        gu = rnd(t, 2 * ff)
+        pair("gated unit on its own", f"{t} x {ff}", (lambda: decoder.glu(gu, decoder.GLU_TILE, 7.0), t * ff * 6, 0),
+             (lambda: basic.silu_mul(gu), t * ff * 6, 0))
+        proj, qkv = rnd(t, aw.proj.n), rnd(t, (H + 2 * G) * 128)
+        kc, vc = (torch.zeros(max(t, 64) // bs + 1, bs, n, dtype=torch.bfloat16, device=dev) for n in (m.k_width, m.v_width))
+        k4, v4 = (torch.zeros(max(t, 64) // bs + 1, G, bs, 128, dtype=torch.bfloat16, device=dev) for _ in range(2))
+        pos, qn = torch.arange(t, dtype=torch.int32, device=dev), torch.ones(128, device=dev, dtype=torch.bfloat16)
+        inv = attention.rope_inv_freq(64, 5e5, dev)
+        pair("attention prologue", f"{t} tokens",
+             (lambda: diffattn.head_prep(proj, m, pos, pos, kc, vc), t * (m.q_width + m.k_width + m.v_width) * 4, 0),
+             (lambda: attention.qk_norm_rope_append(qkv, 0, 128, False, qkv, H * 128, qkv, (H + G) * 128, qn, qn, True, 1e-5, inv, 64,
+                                                    pos, pos, k4, v4, H, G), t * (H + 2 * G) * 128 * 4, 0))
+        # up projection with the gated unit (epilogue of the pair GEMM, or a second kernel) beside the plain product
+        wu, xs = decoder.Projection.make(rnd(2 * ff, width), torch.bfloat16, dev), rnd(t, width)
+        need = ((2 * ff * width + t * width + t * ff) * 2, 2 * t * 2 * ff * width)
+        plain = ((2 * ff * width + t * width + 2 * t * ff) * 2, 2 * t * 2 * ff * width)
+        pair("gate | up projection + gated unit (like: plain product)", f"{t} x {2 * ff} x {width}",
+             (lambda: wu.glu(xs, 7.0), *need), (lambda: gemm.linear(xs, wu.packed), *plain))
+        for what, pr, o32 in (("q | k | v | g projection (like: none)", aw.proj, False), ("B | C | dt projection (like: none)", sw.x, False),
+                              ("step size projection (like: none)", sw.dt, True)):
+            xk = rnd(t, pr.k)
+            pair(what, f"{t} x {pr.n} x {pr.k}", (lambda: pr(xk, out_f32=o32), (pr.n * pr.k + t * pr.k) * 2 + t * pr.n * (4 if o32 else 2),
+                                                  2 * t * pr.n * pr.k), None)
+        # convolution
+        xin, cw = rnd(t, 2 * inner), rnd(inner, 4)
+        tails = torch.zeros(t if t <= 32 else 1, 3, inner, dtype=torch.bfloat16, device=dev)
+        ar, one, zero = torch.arange(t, dtype=torch.int32, device=dev), torch.ones(t, dtype=torch.int32, device=dev), torch.zeros(t, dtype=torch.int32, device=dev)
+        seg = scan.Segments(ar, ar, ar, one, ar, 1) if t <= 32 else scan.Segments(zero, zero, i32([0]), i32([t]), i32([0]), t)
+        pos1 = ar + 5
+        like_conv = (lambda: basic.conv_silu_step(xin[:, :inner], cw, tails, ar)) if t <= 32 else (lambda: basic.conv_silu(xin[:, :inner], cw, tails[0]))
+        cbytes = t * inner * 4 + (t * 3 * inner * 2 if t <= 32 else 0)
+        pair("convolution", f"{t} x {inner}", (lambda: scan.conv_rows(xin[:, :inner], sw.conv, sw.conv_b, tails, seg, pos1), cbytes, 0),
+             (like_conv, cbytes, 0))
+        # recurrence: rows in and out, state read and written once per sequence
+        xc, dt, bc = rnd(t, inner), rnd(t, inner, dt=torch.float32), rnd(t, sw.x.n)
+        n_seq = seg.first.numel()
+        st = torch.zeros(n_seq, inner, N, dtype=torch.float32, device=dev)
+        sbytes = t * inner * 10 + t * sw.x.n * 2 + n_seq * inner * N * 8
+        mixed, gg = rnd(t, (2 * hk + hv) * 128), -torch.rand(t, hv, device=dev)
+        beta = torch.rand(t, hv, device=dev)
+        gst = torch.zeros(n_seq, hv, 128, 128, dtype=torch.float32, device=dev)
+        gbytes = t * (2 * hk + 2 * hv) * 256 + t * hv * 8 + n_seq * hv * 128 * 128 * 8
+        like = (lambda: gdn.step(gst, ar, mixed, 0, hk * 128, 2 * hk * 128, gg, beta, hv, hk)) if t <= 32 else \
+            (lambda: gdn.chunked(mixed, 0, hk * 128, 2 * hk * 128, gg, beta, gst[0], hv, hk))
+        pair("recurrence", f"{t} tokens, {inner} channels x {N} states",
+             (lambda: scan.selective_scan(xc, dt, bc, sw.b_off, sw.c_off, xin[:, inner:], sw.a, sw.dt_b, sw.d, st, seg, pos1, xin[:, :inner], tails), sbytes, 0),
+             (like, gbytes, 0))
+    t = 8192
+    table = (torch.arange(t // bs, dtype=torch.int32, device=dev) + 1)[None]
+    q, q1 = rnd(t, H, 2, D), rnd(t, H, 128)
+    kc, vc = rnd(t // bs + 1, bs, m.k_width), rnd(t // bs + 1, bs, m.v_width)
+    k4, v4 = (rnd(t // bs + 1, G, bs, 128) for _ in range(2))
+    out, gate = torch.empty(t, H * V, dtype=torch.bfloat16, device=dev), rnd(t, H)
+    full_n = t * (t + 1) // 2
+    args = (i32([0]), i32([t]), i32([t]), t)
+    pair("prompt attention", f"{t} tokens", (lambda: diffattn.prefill(q, m, kc, vc, gate, table, *args, out), 0, 2 * full_n * H * 2 * (D + V)),
+         (lambda: attention.prefill(q1, k4, v4, table, *args), 0, 2 * full_n * H * 2 * 128))
+    for b in (1, 32):
+        tb = (torch.arange(b * pages, dtype=torch.int32, device=dev) + 1).view(b, pages)
+        kc, vc = rnd(b * pages + 1, bs, m.k_width), rnd(b * pages + 1, bs, m.v_width)
+        k4, v4 = (rnd(b * pages + 1, G, bs, 128) for _ in range(2))
+        q, q1, gate = rnd(b, H, 2, D), rnd(b, H, 128), rnd(b, H)
+        ob = torch.empty(b, H * V, dtype=torch.bfloat16, device=dev)
+        pos, kvl = i32([ctx - 1] * b), i32([ctx] * b)
+        pair("decode attention", f"batch {b}, {ctx} keys", (lambda: diffattn.rows(q, m, kc, vc, gate, tb, pos, ctx, ob), b * ctx * (m.k_width + m.v_width) * 2, 0),
+             (lambda: attention.decode(q1, k4, v4, tb, kvl, max_kv_len=ctx), b * ctx * G * 128 * 4, 0))
+    return rows_out
+
+
 def run(args) -> dict:
     from ..ops import _lib
     from .clocks import ClockSampler
     dev = torch.device("cuda", 0)
     torch.cuda.set_device(dev)
     timer = _Timer(dev, args.steps, args.warmup)
-    prompt = args.prompt
-    out: dict = {"metric": "rutulix design: prefill and decode throughput", "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True,
+    prompt, name = args.prompt, args.design
+    out: dict = {"metric": f"{name} design: prefill and decode throughput", "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True,
                  "steps": timer.steps, "warmup": timer.warmup, "dtype": "bf16", "data": "synthetic", "designs": {}}
     slots = 32
+    sizes = SIZES if name == "rutulix" else ZG_SIZES
+    models, kernels = (_models, _kernels) if name == "rutulix" else (_zg_models, _zg_kernels)
     with torch.no_grad(), ClockSampler(0) as clk:
-        for size in ([args.design_size] if args.design_size else list(SIZES)):
-            width, heads, kv, dim, inter, chunk = SIZES[size]
-            new, old = _models(size, dev, prompt, slots)
-            rec = {"layers": LAYERS, "width": width, "heads": heads, "kv_heads": kv, "dim": dim, "ff": inter * 3 // 2, "chunk": chunk,
-                   "prompt": prompt, "rutulix": _throughput(new, dev, prompt, slots, timer)}
+        for size in ([args.design_size] if args.design_size else list(sizes)):
+            new, old = models(size, dev, prompt, slots)
+            if name == "rutulix":
+                width, heads, kv, dim, inter, chunk = SIZES[size]
+                rec = {"layers": LAYERS, "width": width, "heads": heads, "kv_heads": kv, "dim": dim, "ff": inter * 3 // 2, "chunk": chunk}
+            else:
+                keys = ("width", "heads", "kv_heads", "dim", "vdim", "ff", "inner", "state", "dt_rank")
+                rec = {"layers": LAYERS, **dict(zip(keys, ZG_SIZES[size]))}
+            rec.update({"prompt": prompt, name: _throughput(new, dev, prompt, slots, timer)})
             torch.cuda.empty_cache()
-            rec["closest (full-attention decoder, fp8 weights)"] = _throughput(old, dev, prompt, slots, timer)
+            rec["closest (" + ("full-attention decoder" if name == "rutulix" else "Gated-DeltaNet / full-attention decoder") + ", fp8 weights)"] = \
+                _throughput(old, dev, prompt, slots, timer)
             torch.cuda.empty_cache()
-            rec["kernels"] = _kernels(size, dev, timer, prompt)
+            rec["kernels"] = kernels(size, dev, timer, prompt)
             torch.cuda.empty_cache()
             out["designs"][size] = rec
             _lib.check_status()
     first = next(iter(out["designs"].values()))
-    out["value"] = first["rutulix"]["prefill_tok_s"]
+    out["value"] = first[name]["prefill_tok_s"]
     out["clocks"] = clk.summary()
     out["config"] = {"l2": "flushed before every timed call", "roofline": _peaks()[1], "prompt": prompt, "decode_batch": slots}
     return out
