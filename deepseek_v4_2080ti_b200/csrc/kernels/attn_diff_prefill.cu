@@ -26,7 +26,7 @@ namespace diffattn {
 constexpr int BQ = 128;         // query rows per CTA
 constexpr int BKV = 128;        // keys per tile
 constexpr int ATOM = 16384;     // bytes of one [128 x 64] bf16 swizzled slab
-constexpr int NTHREADS = 320;
+constexpr int NTHREADS = 384;   // three warpgroups; the third has the two single-thread roles and gives its registers up
 constexpr int MAX_STAGES = 12;
 constexpr int BUDGET = 232448 - 1024 /* alignment */ - 512 /* barriers */ - 1024 /* row sums */;
 
@@ -118,8 +118,10 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   tc_fence_after();
   const uint32_t tmem = *tmem_slot;
 
-  if (warp == 8) {
-    if (lane == 0) {
+  // registers per thread at launch: 168 (3 x 168 = 2 x 216 + 72)
+  if (warp >= 8) {
+    asm volatile("setmaxnreg.dec.sync.aligned.u32 72;");
+    if (warp == 8 && lane == 0) {
       tma_prefetch_desc(&tmQ);
       tma_prefetch_desc(&tmK);
       tma_prefetch_desc(&tmV);
@@ -157,9 +159,7 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           if (ok) ok = slab(&tmV, g * p.V + v0 + s * 64);
       }
       if (!ok) { atomicExch(p.status, ERR_WAIT_STAGE); *abort_flag = 1; }
-    }
-  } else if (warp == 9) {
-    if (lane == 0) {
+    } else if (warp == 9 && lane == 0) {
       bool ok = mbar_wait(q_full, 0);
       // the ring's consumption order differs from its fill order only in that a tile's value slabs are held while the next
       // tile's first-map keys, which lie behind them, are consumed
@@ -207,6 +207,7 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       if (!ok) { atomicExch(p.status, ERR_WAIT_TMA); *abort_flag = 1; }
     }
   } else {
+    asm volatile("setmaxnreg.inc.sync.aligned.u32 216;");
     const int m = warp >> 2;                 // map
     const int r = (warp & 3) * 32 + lane;    // query row in the tile == TMEM lane
     const int limit = pos0 + r;              // last visible key of this row
@@ -219,28 +220,22 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       ok = __all_sync(0xffffffffu, ok) && !*abort_flag;
       if (!ok) { alive = false; break; }
       tc_fence_after();
-      float s[128];
+      uint32_t sv[4][32];                    // the row's 128 scores
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        uint32_t v[32];
-        tmem_ld_32x32(tS + c * 32, v);
-        tmem_ld_wait();
-#pragma unroll
-        for (int i = 0; i < 32; ++i) s[c * 32 + i] = __uint_as_float(v[i]);
-      }
+      for (int c = 0; c < 4; ++c) tmem_ld_32x32(tS + c * 32, sv[c]);
+      tmem_ld_wait();
       const int kmax = min(limit, kv_len - 1) - j * BKV;
-      float m_tile = -INFINITY;
       if (kmax < 127) {
 #pragma unroll
-        for (int i = 0; i < 128; ++i) {
-          if (i > kmax) s[i] = -INFINITY;
-          m_tile = fmaxf(m_tile, s[i]);
-        }
-      } else {
-#pragma unroll
-        for (int i = 0; i < 128; ++i) m_tile = fmaxf(m_tile, s[i]);
+        for (int i = 0; i < 128; ++i)
+          if (i > kmax) sv[i >> 5][i & 31] = 0xff800000u;      // -inf
       }
-      m_tile *= p.scale_log2;
+      float mx[8];                           // independent chains
+#pragma unroll
+      for (int i = 0; i < 8; ++i) mx[i] = __uint_as_float(sv[0][i]);
+#pragma unroll
+      for (int i = 8; i < 128; ++i) mx[i & 7] = fmaxf(mx[i & 7], __uint_as_float(sv[i >> 5][i & 31]));
+      const float m_tile = p.scale_log2 * fmaxf(fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])), fmaxf(fmaxf(mx[4], mx[5]), fmaxf(mx[6], mx[7])));
       // every row sees key 0, so the first tile gives a finite maximum
       const float m_new = fmaxf(m_run, m_tile);
       const bool grow = m_new > m_run + 8.f;
@@ -273,8 +268,9 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         uint32_t w[32];
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
-          const float e0 = exp2f(fmaf(s[half * 64 + 2 * i], p.scale_log2, -m_run));
-          const float e1 = exp2f(fmaf(s[half * 64 + 2 * i + 1], p.scale_log2, -m_run));
+          const int k = half * 64 + 2 * i;
+          const float e0 = exp2f(fmaf(__uint_as_float(sv[k >> 5][k & 31]), p.scale_log2, -m_run));
+          const float e1 = exp2f(fmaf(__uint_as_float(sv[k >> 5][(k & 31) + 1]), p.scale_log2, -m_run));
           lsum[i & 3] += e0 + e1;
           __nv_bfloat162 t = __floats2bfloat162_rn(e0, e1);
           w[i] = *reinterpret_cast<uint32_t*>(&t);

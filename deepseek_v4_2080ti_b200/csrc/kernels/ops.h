@@ -217,7 +217,7 @@ int b200_attn_diff_prefill(const void* q, const void* k_cache, const void* v_cac
 int b200_conv_rows(const void* x, int ldx, const float* w, const float* bias, const void* tail, const int* row_first,
                    const int* row_slot, const int* positions, void* y, int ldy, int rows, int C, int taps, int silu, int f32,
                    cudaStream_t stream);
-int b200_selective_scan_channels(int N);
+int b200_selective_scan_slices(int C, int N, int entries, int max_len);
 int b200_selective_scan(const void* x, int ldx, const float* dt, int ldd, const void* bc, int ldb, int b_off, int c_off,
                         const void* z, int ldz, void* out, int ldo, const float* a, const float* dt_bias, const float* d_skip,
                         float* state, const int* ent_first, const int* ent_len, const int* ent_slot, const int* positions,

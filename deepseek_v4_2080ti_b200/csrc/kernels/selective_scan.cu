@@ -8,10 +8,11 @@
 // The state lives in a slot per sequence and starts at zero when the sequence's first row of the batch has position 0.
 //
 // L lanes share a channel, NS states each; a block owns 128 / L channels of one sequence (or of one time slice of it) and
-// walks tiles of 32 rows: step sizes and inputs are converted once per (row, channel) into shared memory, the recurrence
-// runs out of it with the states in registers, and four steps' partial sums are reduced over the lanes together
-// (transposing butterfly).  The next tile's rows are in flight meanwhile.  Sequences that bring a single row (decoding) take
-// a kernel of their own without the tiles.
+// walks tiles of 32 rows: step sizes and inputs are converted once per (row, channel) into shared memory (as pairs, for the
+// two-wide fp32 instructions), the recurrence runs out of it with the states in registers, and four steps' partial sums are
+// reduced over the lanes together (transposing butterfly).  The next tile's rows are in flight meanwhile, unconverted: a
+// conversion would wait for them.  Narrow models take more lanes per channel.  Sequences that bring a single row (decoding)
+// take a kernel of their own without the tiles.
 //
 // A long sequence with few channels does not fill the device: its rows are then cut into slices.  A first pass runs every
 // slice but the last from a zero state (the first one from the slot's state) and keeps the end state and the sum of the
@@ -63,24 +64,37 @@ __device__ __forceinline__ float softplus(float v) {
   return fmaxf(v, 0.f) + (e < 0.0625f ? series : __logf(1.f + e));
 }
 
-__device__ __forceinline__ void load4(const __nv_bfloat16* p, float (&f)[4]) {
-  const uint2 u = *reinterpret_cast<const uint2*>(p);
-  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
-  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
-  f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+// Two neighbouring channels of a row as they lie in memory, converted when they are used.
+__device__ __forceinline__ float2 widen(uint32_t v) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v)); }
+__device__ __forceinline__ float2 widen(float2 v) { return v; }
+template <typename T> struct Pair;
+template <> struct Pair<__nv_bfloat16> { using type = uint32_t; };
+template <> struct Pair<float> { using type = float2; };
+__device__ __forceinline__ void store_pair(__nv_bfloat16* p, float a, float b) {
+  *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b);
 }
-__device__ __forceinline__ void load4(const float* p, float (&f)[4]) {
-  const float4 a = *reinterpret_cast<const float4*>(p);
-  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+__device__ __forceinline__ void store_pair(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+
+// fp32 pairs in 64-bit registers
+__device__ __forceinline__ uint64_t pair_of(float a, float b) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
 }
-__device__ __forceinline__ void store4(__nv_bfloat16* p, const float (&f)[4]) {
-  uint2 u;
-  *reinterpret_cast<__nv_bfloat162*>(&u.x) = __floats2bfloat162_rn(f[0], f[1]);
-  *reinterpret_cast<__nv_bfloat162*>(&u.y) = __floats2bfloat162_rn(f[2], f[3]);
-  *reinterpret_cast<uint2*>(p) = u;
+__device__ __forceinline__ float2 halves_of(uint64_t v) {
+  float2 f;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(v));
+  return f;
 }
-__device__ __forceinline__ void store4(float* p, const float (&f)[4]) {
-  *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
 }
 template <bool FAST>
 __device__ __forceinline__ float silu(float z) {
@@ -98,47 +112,90 @@ __device__ __forceinline__ void replace_tail(const ScanParams<T>& p, int slot, i
   }
 }
 
-template <int NS>
-__device__ __forceinline__ void load_ns(const float* p, float (&f)[NS]) {
-  if constexpr (NS % 4 == 0) {
+// States of one lane, in pairs where their number is even.
+template <int NS, bool FAST>
+struct Lane {
+  static constexpr int P = (NS + 1) / 2;
+  uint64_t s[P], a[P];
+
+  // S <- exp(delta a) S + dx b; returns this lane's part of sum_n S c.  dd: (delta, delta, dx, dx)
+  template <bool OUT>
+  __device__ __forceinline__ float step(const float4& dd, const float* b, const float* c) {
+    if constexpr (NS == 1) {
+      const float2 v = halves_of(s[0]);
+      const float t = fmaf(decay<FAST>(dd.x * halves_of(a[0]).x), v.x, dd.z * b[0]);
+      s[0] = pair_of(t, 0.f);
+      return OUT ? t * c[0] : 0.f;
+    } else {
+      const uint64_t d2 = pair_of(dd.x, dd.y), x2 = pair_of(dd.z, dd.w);
+      uint64_t bb[P], cc[P], y = 0;
+      load(b, bb);
+      if (OUT) load(c, cc);
 #pragma unroll
-    for (int i = 0; i < NS; i += 4) *reinterpret_cast<float4*>(f + i) = *reinterpret_cast<const float4*>(p + i);
-  } else if constexpr (NS % 2 == 0) {
-#pragma unroll
-    for (int i = 0; i < NS; i += 2) *reinterpret_cast<float2*>(f + i) = *reinterpret_cast<const float2*>(p + i);
-  } else {
-#pragma unroll
-    for (int i = 0; i < NS; ++i) f[i] = p[i];
+      for (int i = 0; i < P; ++i) {
+        const float2 e = halves_of(mul2(d2, a[i]));
+        s[i] = fma2(pair_of(decay<FAST>(e.x), decay<FAST>(e.y)), s[i], mul2(x2, bb[i]));
+        if (OUT) y = i ? fma2(s[i], cc[i], y) : mul2(s[i], cc[i]);
+      }
+      const float2 f = halves_of(y);
+      return f.x + f.y;
+    }
   }
-}
+  __device__ __forceinline__ static void load(const float* p, uint64_t (&v)[P]) {
+    if constexpr (NS % 4 == 0) {
+#pragma unroll
+      for (int i = 0; i < P; i += 2) {
+        const ulonglong2 t = *reinterpret_cast<const ulonglong2*>(p + 2 * i);
+        v[i] = t.x;
+        v[i + 1] = t.y;
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < P; ++i) v[i] = *reinterpret_cast<const uint64_t*>(p + 2 * i);
+    }
+  }
+  // f(n): value of the lane's n-th state
+  template <typename F>
+  __device__ __forceinline__ static void fill(uint64_t (&v)[P], F f) {
+#pragma unroll
+    for (int i = 0; i < P; ++i) v[i] = pair_of(f(2 * i), 2 * i + 1 < NS ? f(2 * i + 1) : 0.f);
+  }
+  template <typename F>
+  __device__ __forceinline__ void each(F f) const {
+#pragma unroll
+    for (int i = 0; i < P; ++i) {
+      const float2 v = halves_of(s[i]);
+      f(2 * i, v.x);
+      if (2 * i + 1 < NS) f(2 * i + 1, v.y);
+    }
+  }
+};
 
 // PASS 0: the whole sequence or (slices > 1) the outputs of one slice; PASS 1: end state of one slice.
 template <typename T, int L, int NS, int PASS>
 __global__ void __launch_bounds__(THREADS) scan_kernel(ScanParams<T> p) {
   constexpr bool FAST = sizeof(T) == 2;
-  constexpr int CB = THREADS / L, NP = L * NS;
-  constexpr int CV = CB / 4, UNITS = TT * CV, U = (UNITS + THREADS - 1) / THREADS, UR = THREADS / CV;   // units of 4 channels
+  constexpr int CB = THREADS / L, NP = L * NS, YP = CB + 8;
+  constexpr int CV = CB / 2, UR = THREADS / CV, U = (TT + UR - 1) / UR;         // units of two channels; rows UR apart
+  using pair_t = typename Pair<T>::type;
   extern __shared__ __align__(16) float sm[];
-  float2* sdt = reinterpret_cast<float2*>(sm);              // [TT][CB]: (delta, delta x)
-  float* sy = sm + TT * CB * 2;                             // [TT][CB]
-  float* sbc = sy + TT * CB;                                // [TT][2][NP]
+  float4* sdt = reinterpret_cast<float4*>(sm);              // [TT][CB]: (delta, delta, delta x, delta x)
+  float* sbc = sm + TT * CB * 4;                            // [TT][2][NP]
+  float* sy = sbc + TT * 2 * NP;                            // [TT][YP]
   pdl_grid_trigger();
   const int tid = threadIdx.x, ch = tid / L, lane = tid % L, c0 = blockIdx.x * CB, c = c0 + ch;
   const bool on = c < p.C;
-  float a[NS];
-#pragma unroll
-  for (int i = 0; i < NS; ++i) {
-    const int n = lane * NS + i;
-    a[i] = on && n < p.N ? p.a[(size_t)c * p.N + n] : 0.f;
-  }
+  using LaneT = Lane<NS, FAST>;
+  LaneT st;
+  LaneT::fill(st.a, [&](int i) { return on && lane * NS + i < p.N ? p.a[(size_t)c * p.N + lane * NS + i] : 0.f; });
   for (int i = tid; i < TT * 2 * NP; i += THREADS) sbc[i] = 0.f;        // states past N stay zero
-  // this thread's units of a tile: rows vt, vt + UR, .., channels vc..vc+3
-  const int vt = tid / CV, vl = (tid % CV) * 4, vc = c0 + vl;
-  const bool v_on = vc < p.C;
-  float bias4[4] = {}, d4[4] = {};
+  // this thread's units of a tile: rows vt, vt + UR, .., channels vc, vc + 1
+  const int vt = tid / CV, vl = (tid % CV) * 2, vc = c0 + vl;
+  const bool v_on = vc < p.C && vt < TT;
+  float2 bias = make_float2(0.f, 0.f), dskip = bias;
   if (v_on) {
-    load4(p.dt_bias + vc, bias4);
-    load4(p.d_skip + vc, d4);
+    bias = *reinterpret_cast<const float2*>(p.dt_bias + vc);
+    dskip = *reinterpret_cast<const float2*>(p.d_skip + vc);
   }
   pdl_grid_wait();
   const int e = blockIdx.z, slice = blockIdx.y;
@@ -147,40 +204,36 @@ __global__ void __launch_bounds__(THREADS) scan_kernel(ScanParams<T> p) {
   if (len == 1 || lo >= len || (PASS == 1 && (single || hi == len))) return;      // uniform per block
   const int first = p.ent_first[e], slot = p.ent_slot[e], pos = p.positions[first];
   const size_t cn = (size_t)p.C * p.N;
-  float* st = p.state + (size_t)slot * cn + (size_t)c * p.N;
+  float* state = p.state + (size_t)slot * cn + (size_t)c * p.N;
   float* ws = p.ws_state ? p.ws_state + (size_t)e * p.slices * cn + (size_t)c * p.N : nullptr;
 
-  float s[NS];
-#pragma unroll
-  for (int i = 0; i < NS; ++i) {
+  LaneT::fill(st.s, [&](int i) {
     const int n = lane * NS + i;
-    s[i] = 0.f;
-    if (on && n < p.N) {
-      if (slice == 0) {
-        if (PASS == 1 || single) s[i] = pos == 0 ? 0.f : st[n];
-        else s[i] = ws[(size_t)(p.slices - 1) * cn + n];
-        if (PASS == 1) ws[(size_t)(p.slices - 1) * cn + n] = s[i];
-      } else if (PASS == 0) {
-        s[i] = ws[n];
-        for (int k = 1; k < slice; ++k)
-          s[i] = decay<FAST>(p.ws_sum[((size_t)e * p.slices + k) * p.C + c] * a[i]) * s[i] + ws[k * cn + n];
-      }
+    if (!on || n >= p.N) return 0.f;
+    float v;
+    if (slice == 0) {
+      v = PASS == 1 || single ? (pos == 0 ? 0.f : state[n]) : ws[(size_t)(p.slices - 1) * cn + n];
+      if (PASS == 1) ws[(size_t)(p.slices - 1) * cn + n] = v;
+      return v;
     }
-  }
+    if (PASS == 1) return 0.f;
+    v = ws[n];
+    const float an = p.a[(size_t)c * p.N + n];
+    for (int k = 1; k < slice; ++k) v = fmaf(decay<FAST>(p.ws_sum[((size_t)e * p.slices + k) * p.C + c] * an), v, ws[k * cn + n]);
+    return v;
+  });
 
   const int nb8 = (p.c_off - p.b_off) / 8, nbc = 2 * nb8;               // vectors of B (and of C) per row
-  float x4[U][4], dt4[U][4], z4[U][4], bc8[8];
-  auto fetch_bc = [&](int i, int row0, float (&f)[8]) {
-    const int t = i / nbc, v = i % nbc;
-    if (row0 + t < hi) load8(p.bc + (size_t)(first + row0 + t) * p.ldb + p.b_off + v * 8, f);
-    else {
-#pragma unroll
-      for (int j = 0; j < 8; ++j) f[j] = 0.f;
-    }
-  };
-  auto put_bc = [&](int i, const float (&f)[8]) {
-    const int t = i / nbc, v = i % nbc, half = v / nb8, n0 = (v % nb8) * 8;
-    float* dst = sbc + (t * 2 + half) * NP + n0;
+  pair_t xr[U], zr[U];
+  float2 dtr[U];
+  constexpr int BW = 8 * (int)sizeof(T) / 16;                           // 16-byte words of eight values
+  uint4 bcr[BW];
+  const int bt = tid / nbc, bv = tid % nbc;                             // first B | C vector of this thread
+  float* const bdst = sbc + (bt * 2 + bv / nb8) * NP + (bv % nb8) * 8;
+  const int bn0 = (bv % nb8) * 8;
+  auto put_bc = [&](float* dst, int n0, const uint4 (&raw)[BW]) {
+    float f[8];
+    load8(reinterpret_cast<const T*>(raw), f);
     if constexpr (NP % 8 == 0) {
       if (n0 < NP) store8(dst, f);
     } else {
@@ -189,69 +242,65 @@ __global__ void __launch_bounds__(THREADS) scan_kernel(ScanParams<T> p) {
         if (n0 + j < NP) dst[j] = f[j];
     }
   };
+  auto fetch_bc = [&](int t, int v, int row0, uint4 (&raw)[BW]) {
+#pragma unroll
+    for (int j = 0; j < BW; ++j)
+      raw[j] = row0 + t < hi ? reinterpret_cast<const uint4*>(p.bc + (size_t)(first + row0 + t) * p.ldb + p.b_off + v * 8)[j]
+                             : make_uint4(0, 0, 0, 0);
+  };
   auto fetch = [&](int row0) {
 #pragma unroll
     for (int u = 0; u < U; ++u) {
-#pragma unroll
-      for (int j = 0; j < 4; ++j) x4[u][j] = dt4[u][j] = z4[u][j] = 0.f;
       const int t = vt + u * UR, row = first + row0 + t;
-      if (v_on && t < TT && row0 + t < hi) {
-        load4(p.x + (size_t)row * p.ldx + vc, x4[u]);
-        load4(p.dt + (size_t)row * p.ldd + vc, dt4[u]);
-        if (PASS == 0) load4(p.z + (size_t)row * p.ldz + vc, z4[u]);
+      if (v_on && row0 + t < hi) {
+        xr[u] = *reinterpret_cast<const pair_t*>(p.x + (size_t)row * p.ldx + vc);
+        dtr[u] = *reinterpret_cast<const float2*>(p.dt + (size_t)row * p.ldd + vc);
+        if (PASS == 0) zr[u] = *reinterpret_cast<const pair_t*>(p.z + (size_t)row * p.ldz + vc);
       }
     }
-    if (tid < TT * nbc) fetch_bc(tid, row0, bc8);
+    if (bt < TT) fetch_bc(bt, bv, row0, bcr);
   };
   fetch(lo);
   float sum = 0.f;
   for (int row0 = lo; row0 < hi; row0 += TT) {
-    float xc[U][4], zc[U][4];
+    pair_t xc[U], zc[U];
 #pragma unroll
     for (int u = 0; u < U; ++u) {
       const int t = vt + u * UR;
-      const bool have = v_on && row0 + t < hi;
-      float v[4];
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        xc[u][j] = x4[u][j];
-        zc[u][j] = z4[u][j];
-        v[j] = have ? softplus<FAST>(dt4[u][j] + bias4[j]) : 0.f;
+      if (U * UR > TT && t >= TT) continue;
+      float4 q0 = make_float4(0.f, 0.f, 0.f, 0.f), q1 = q0;
+      if (v_on && row0 + t < hi) {
+        const float2 x = widen(xr[u]);
+        const float d0 = softplus<FAST>(dtr[u].x + bias.x), d1 = softplus<FAST>(dtr[u].y + bias.y);
+        q0 = make_float4(d0, d0, d0 * x.x, d0 * x.x);
+        q1 = make_float4(d1, d1, d1 * x.y, d1 * x.y);
+        xc[u] = xr[u];
+        if (PASS == 0) zc[u] = zr[u];
       }
-      if (t < TT) {
-        float4* dst = reinterpret_cast<float4*>(sdt + t * CB + vl);
-        dst[0] = make_float4(v[0], v[0] * xc[u][0], v[1], v[1] * xc[u][1]);
-        dst[1] = make_float4(v[2], v[2] * xc[u][2], v[3], v[3] * xc[u][3]);
-      }
+      sdt[t * CB + vl] = q0;
+      sdt[t * CB + vl + 1] = q1;
     }
-    if (tid < TT * nbc) put_bc(tid, bc8);
+    if (bt < TT) put_bc(bdst, bn0, bcr);
     for (int i = tid + THREADS; i < TT * nbc; i += THREADS) {
-      float f[8];
-      fetch_bc(i, row0, f);
-      put_bc(i, f);
+      const int t = i / nbc, v = i % nbc, n0 = (v % nb8) * 8;
+      uint4 raw[BW];
+      fetch_bc(t, v, row0, raw);
+      put_bc(sbc + (t * 2 + v / nb8) * NP + n0, n0, raw);
     }
     __syncthreads();
     if (row0 + TT < hi) fetch(row0 + TT);
     const int n_rows = min(TT, hi - row0);
-    for (int t = 0; t < n_rows; t += 4) {
+    const float4* dp = sdt + ch;
+    const float* bp = sbc + lane * NS;
+    float* yp = sy + lane * YP + ch;
+#pragma unroll 2
+    for (int t = 0; t < n_rows; t += 4, dp += 4 * CB, bp += 8 * NP, yp += 4 * YP) {
       float y[4];
 #pragma unroll
       for (int u = 0; u < 4; ++u) {
-        const float2 dd = sdt[(t + u) * CB + ch];
-        const float* bcr = sbc + (t + u) * 2 * NP + lane * NS;
-        float b[NS];
-        load_ns(bcr, b);
-#pragma unroll
-        for (int i = 0; i < NS; ++i) s[i] = fmaf(decay<FAST>(dd.x * a[i]), s[i], dd.y * b[i]);
-        if (PASS == 0) {
-          float cc[NS];
-          load_ns(bcr + NP, cc);
-          y[u] = 0.f;
-#pragma unroll
-          for (int i = 0; i < NS; ++i) y[u] = fmaf(s[i], cc[i], y[u]);
-        } else {
-          sum += dd.x;
-        }
+        const float4 dd = dp[u * CB];
+        y[u] = st.template step<PASS == 0>(dd, bp + u * 2 * NP, bp + u * 2 * NP + NP);
+        if (PASS == 1) sum += dd.x;
       }
       if (PASS == 0) {
         // lane l (mod 4) ends up with the sum of step l
@@ -262,7 +311,7 @@ __global__ void __launch_bounds__(THREADS) scan_kernel(ScanParams<T> p) {
         float q = (up1 ? q1 : q0) + __shfl_xor_sync(0xffffffffu, up1 ? q0 : q1, 1);
 #pragma unroll
         for (int o = 4; o < L; o <<= 1) q += __shfl_xor_sync(0xffffffffu, q, o);
-        if (lane < 4) sy[(t + lane) * CB + ch] = q;
+        if (lane < 4) *yp = q;
       }
     }
     __syncthreads();
@@ -271,11 +320,9 @@ __global__ void __launch_bounds__(THREADS) scan_kernel(ScanParams<T> p) {
       for (int u = 0; u < U; ++u) {
         const int t = vt + u * UR;
         if (v_on && t < TT && row0 + t < hi) {
-          float o[4];
-          load4(sy + t * CB + vl, o);
-#pragma unroll
-          for (int j = 0; j < 4; ++j) o[j] = fmaf(d4[j], xc[u][j], o[j]) * silu<FAST>(zc[u][j]);
-          store4(p.out + (size_t)(first + row0 + t) * p.ldo + vc, o);
+          const float2 y = *reinterpret_cast<const float2*>(sy + t * YP + vl), x = widen(xc[u]), z = widen(zc[u]);
+          store_pair(p.out + (size_t)(first + row0 + t) * p.ldo + vc, fmaf(dskip.x, x.x, y.x) * silu<FAST>(z.x),
+                     fmaf(dskip.y, x.y, y.y) * silu<FAST>(z.y));
         }
       }
     }
@@ -283,90 +330,110 @@ __global__ void __launch_bounds__(THREADS) scan_kernel(ScanParams<T> p) {
 
   if (PASS == 1) {
     if (on) {
-#pragma unroll
-      for (int i = 0; i < NS; ++i) {
-        const int n = lane * NS + i;
-        if (n < p.N) ws[slice * cn + n] = s[i];
-      }
+      st.each([&](int i, float v) {
+        if (lane * NS + i < p.N) ws[slice * cn + lane * NS + i] = v;
+      });
       if (lane == 0) p.ws_sum[((size_t)e * p.slices + slice) * p.C + c] = sum;
     }
     return;
   }
   if (hi < len) return;
-  if (on) {
-#pragma unroll
-    for (int i = 0; i < NS; ++i) {
-      const int n = lane * NS + i;
-      if (n < p.N) st[n] = s[i];
-    }
-  }
+  if (on)
+    st.each([&](int i, float v) {
+      if (lane * NS + i < p.N) state[lane * NS + i] = v;
+    });
   if (p.xin && tid < CB && c0 + tid < p.C) replace_tail(p, slot, first, len, c0 + tid);
 }
 
-// Sequences with a single row: L lanes share a channel, NS states each, straight from and to memory.
-template <typename T, int L, int NS>
+// Sequences with a single row, straight from and to memory: L lanes share a channel, NS states each, KC channels per lane
+// group so that enough loads are in flight.
+template <typename T, int L, int NS, int KC>
 __global__ void __launch_bounds__(THREADS) scan_step_kernel(ScanParams<T> p) {
   constexpr bool FAST = sizeof(T) == 2;
   constexpr int CB = THREADS / L;
+  using LaneT = Lane<NS, FAST>;
   pdl_grid_trigger();
-  const int ch = threadIdx.x / L, lane = threadIdx.x % L, c = blockIdx.x * CB + ch, e = blockIdx.y;
-  const bool on = c < p.C;
+  const int lane = threadIdx.x % L, c0 = blockIdx.x * CB * KC + threadIdx.x / L, e = blockIdx.y;
   const bool vec = NS % 4 == 0 && p.N == L * NS;              // rows of whole 16-byte vectors
-  float a[NS], s[NS], b[NS], cc[NS];
+  LaneT st[KC];
+  float bias[KC], dskip[KC];
 #pragma unroll
-  for (int i = 0; i < NS; ++i) {
-    const int n = lane * NS + i;
-    a[i] = on && n < p.N ? p.a[(size_t)c * p.N + n] : 0.f;
+  for (int k = 0; k < KC; ++k) {
+    const int c = c0 + k * CB;
+    const float* a = p.a + (size_t)c * p.N + lane * NS;
+    if (vec && c < p.C) LaneT::load(a, st[k].a);
+    else LaneT::fill(st[k].a, [&](int i) { return c < p.C && lane * NS + i < p.N ? a[i] : 0.f; });
+    bias[k] = c < p.C ? p.dt_bias[c] : 0.f;
+    dskip[k] = c < p.C ? p.d_skip[c] : 0.f;
   }
-  const float bias = on ? p.dt_bias[c] : 0.f, dskip = on ? p.d_skip[c] : 0.f;
   pdl_grid_wait();
+  const int row = p.ent_first[e], slot = p.ent_slot[e];
   if (p.ent_len[e] != 1) return;                              // uniform per block
-  const int row = p.ent_first[e], slot = p.ent_slot[e], pos = p.positions[row];
-  float* st = p.state + ((size_t)slot * p.C + c) * p.N;
+  const int pos = p.positions[row];
+  float* state = p.state + (size_t)slot * p.C * p.N;
   const T* bcr = p.bc + (size_t)row * p.ldb;
-  if (vec && on) {
-    load_ns<NS>(st + lane * NS, s);
-  } else {
+  float dt[KC], x[KC], z[KC], b[NS], cc[NS];
 #pragma unroll
-    for (int i = 0; i < NS; ++i) s[i] = on && lane * NS + i < p.N ? st[lane * NS + i] : 0.f;
+  for (int k = 0; k < KC; ++k) {
+    const int c = c0 + k * CB;
+    const bool on = c < p.C;
+    const float* s = state + (size_t)c * p.N + lane * NS;
+    if (vec && on) LaneT::load(s, st[k].s);
+    else LaneT::fill(st[k].s, [&](int i) { return on && lane * NS + i < p.N ? s[i] : 0.f; });
+    dt[k] = on ? p.dt[(size_t)row * p.ldd + c] : 0.f;
+    x[k] = on ? (float)p.x[(size_t)row * p.ldx + c] : 0.f;
+    z[k] = on ? (float)p.z[(size_t)row * p.ldz + c] : 0.f;
   }
-  const float dt = on ? p.dt[(size_t)row * p.ldd + c] : 0.f;
-  const float x = on ? (float)p.x[(size_t)row * p.ldx + c] : 0.f, z = on ? (float)p.z[(size_t)row * p.ldz + c] : 0.f;
 #pragma unroll
   for (int i = 0; i < NS; ++i) {
     const int n = lane * NS + i;
     b[i] = n < p.N ? (float)bcr[p.b_off + n] : 0.f;
     cc[i] = n < p.N ? (float)bcr[p.c_off + n] : 0.f;
-    if (pos == 0) s[i] = 0.f;
-  }
-  const float delta = softplus<FAST>(dt + bias), dx = delta * x;
-  float y = 0.f;
-#pragma unroll
-  for (int i = 0; i < NS; ++i) {
-    s[i] = fmaf(decay<FAST>(delta * a[i]), s[i], dx * b[i]);
-    y = fmaf(s[i], cc[i], y);
   }
 #pragma unroll
-  for (int o = 1; o < L; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-  if (!on) return;
-  if (vec) {
+  for (int k = 0; k < KC; ++k) {
+    const int c = c0 + k * CB;
+    if (pos == 0) LaneT::fill(st[k].s, [](int) { return 0.f; });
+    const float delta = softplus<FAST>(dt[k] + bias[k]), dx = delta * x[k];
+    const float2 d2 = make_float2(delta, dx);
+    float y = 0.f;
 #pragma unroll
-    for (int i = 0; i < NS; i += 4) *reinterpret_cast<float4*>(st + lane * NS + i) = make_float4(s[i], s[i + 1 < NS ? i + 1 : 0], s[i + 2 < NS ? i + 2 : 0], s[i + 3 < NS ? i + 3 : 0]);
-  } else {
+    for (int i = 0; i < LaneT::P; ++i) {
+      const float2 a = halves_of(st[k].a[i]), s = halves_of(st[k].s[i]);
+      const float s0 = fmaf(decay<FAST>(d2.x * a.x), s.x, d2.y * b[2 * i]);
+      float s1 = 0.f;
+      y = fmaf(s0, cc[2 * i], y);
+      if (2 * i + 1 < NS) {
+        s1 = fmaf(decay<FAST>(d2.x * a.y), s.y, d2.y * b[2 * i + 1 < NS ? 2 * i + 1 : 0]);
+        y = fmaf(s1, cc[2 * i + 1 < NS ? 2 * i + 1 : 0], y);
+      }
+      st[k].s[i] = pair_of(s0, s1);
+    }
 #pragma unroll
-    for (int i = 0; i < NS; ++i)
-      if (lane * NS + i < p.N) st[lane * NS + i] = s[i];
-  }
-  if (lane == 0) {
-    p.out[(size_t)row * p.ldo + c] = (T)(fmaf(dskip, x, y) * silu<FAST>(z));
-    if (p.xin) replace_tail(p, slot, row, 1, c);
+    for (int o = 1; o < L; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+    if (c >= p.C) continue;
+    float* s = state + (size_t)c * p.N + lane * NS;
+    if (vec) {
+      if constexpr (NS % 4 == 0) {
+#pragma unroll
+        for (int i = 0; i < NS / 2; i += 2) *reinterpret_cast<ulonglong2*>(s + 2 * i) = make_ulonglong2(st[k].s[i], st[k].s[i + 1]);
+      }
+    } else {
+      st[k].each([&](int i, float v) {
+        if (lane * NS + i < p.N) s[i] = v;
+      });
+    }
+    if (lane == 0) {
+      p.out[(size_t)row * p.ldo + c] = (T)(fmaf(dskip[k], x[k], y) * silu<FAST>(z[k]));
+      if (p.xin) replace_tail(p, slot, row, 1, c);
+    }
   }
 }
 
 template <typename T, int L, int NS>
-int launch_scan(const ScanParams<T>& p, int entries, int max_len, int singles, cudaStream_t stream) {
+int launch_tiles(const ScanParams<T>& p, int entries, cudaStream_t stream) {
   constexpr int CB = THREADS / L;
-  const size_t smem = (size_t)(TT * CB * 3 + TT * 2 * L * NS) * 4;
+  const size_t smem = (size_t)(TT * CB * 4 + TT * 2 * L * NS + TT * (CB + 8)) * 4;
   static PerDeviceOnce once_;
   bool& configured = once_.slot();
   if (!configured) {
@@ -377,34 +444,68 @@ int launch_scan(const ScanParams<T>& p, int entries, int max_len, int singles, c
   }
   const int blocks = (p.C + CB - 1) / CB;
   cudaError_t e = cudaSuccess;
-  if (singles) e = launch_pdl(scan_step_kernel<T, L, NS>, dim3(blocks, entries), dim3(THREADS), 0, stream, p);
-  if (e == cudaSuccess && max_len > 1 && p.slices > 1)
-    e = launch_pdl(scan_kernel<T, L, NS, 1>, dim3(blocks, p.slices - 1, entries), dim3(THREADS), smem, stream, p);
-  if (e == cudaSuccess && max_len > 1)
+  if (p.slices > 1) e = launch_pdl(scan_kernel<T, L, NS, 1>, dim3(blocks, p.slices - 1, entries), dim3(THREADS), smem, stream, p);
+  if (e == cudaSuccess)
     e = launch_pdl(scan_kernel<T, L, NS, 0>, dim3(blocks, p.slices, entries), dim3(THREADS), smem, stream, p);
   return (int)e;
 }
 
+template <typename T, int L, int NS>
+int launch_step(const ScanParams<T>& p, int entries, cudaStream_t stream) {
+  constexpr int KC = NS <= 4 ? 4 : 2, PER = THREADS / L * KC;
+  return (int)launch_pdl(scan_step_kernel<T, L, NS, KC>, dim3((p.C + PER - 1) / PER, entries), dim3(THREADS), 0, stream, p);
+}
+
+// Lanes per channel of the tile kernel: as few as hold the states, more for batches whose channels alone would leave the
+// schedulers with less than three warps.
+int pick_lanes(int C, int N, int entries) {
+  int lanes = N <= 32 ? 4 : N <= 64 ? 8 : N <= 128 ? 16 : 32;
+  if (lanes == 4 && N > 8 && (N <= 16 || N > 24) && (long long)C * entries * 4 < 148LL * 12 * 32) lanes = 8;
+  return lanes;
+}
+
 template <typename T>
-int run_scan(ScanParams<T> p, int entries, int max_len, int singles, cudaStream_t stream) {
+int run_scan(const ScanParams<T>& p, int entries, int max_len, int singles, cudaStream_t stream) {
   const int per_lane = (p.N + 3) / 4;
-  if (per_lane <= 1) return launch_scan<T, 4, 1>(p, entries, max_len, singles, stream);
-  if (per_lane <= 2) return launch_scan<T, 4, 2>(p, entries, max_len, singles, stream);
-  if (per_lane <= 4) return launch_scan<T, 4, 4>(p, entries, max_len, singles, stream);
-  if (per_lane <= 6) return launch_scan<T, 4, 6>(p, entries, max_len, singles, stream);
-  if (per_lane <= 8) return launch_scan<T, 4, 8>(p, entries, max_len, singles, stream);
-  if (per_lane <= 16) return launch_scan<T, 8, 8>(p, entries, max_len, singles, stream);
-  if (per_lane <= 32) return launch_scan<T, 16, 8>(p, entries, max_len, singles, stream);
-  if (per_lane <= 64) return launch_scan<T, 32, 8>(p, entries, max_len, singles, stream);
-  return -6;
+  int e = 0;
+  if (singles) {
+    e = per_lane <= 1    ? launch_step<T, 4, 1>(p, entries, stream)
+        : per_lane <= 2  ? launch_step<T, 4, 2>(p, entries, stream)
+        : per_lane <= 4  ? launch_step<T, 4, 4>(p, entries, stream)
+        : per_lane <= 8  ? launch_step<T, 8, 4>(p, entries, stream)
+        : per_lane <= 16 ? launch_step<T, 16, 4>(p, entries, stream)
+        : per_lane <= 32 ? launch_step<T, 32, 4>(p, entries, stream)
+                         : launch_step<T, 32, 8>(p, entries, stream);
+    if (e || max_len == 1) return e;
+  }
+  const int lanes = pick_lanes(p.C, p.N, entries);
+  if (lanes == 4) {
+    if (per_lane <= 1) return launch_tiles<T, 4, 1>(p, entries, stream);
+    if (per_lane <= 2) return launch_tiles<T, 4, 2>(p, entries, stream);
+    if (per_lane <= 4) return launch_tiles<T, 4, 4>(p, entries, stream);
+    if (per_lane <= 6) return launch_tiles<T, 4, 6>(p, entries, stream);
+    return launch_tiles<T, 4, 8>(p, entries, stream);
+  }
+  if (lanes == 8) {
+    if (per_lane <= 4) return launch_tiles<T, 8, 2>(p, entries, stream);
+    if (per_lane <= 8) return launch_tiles<T, 8, 4>(p, entries, stream);
+    return launch_tiles<T, 8, 8>(p, entries, stream);
+  }
+  return lanes == 16 ? launch_tiles<T, 16, 8>(p, entries, stream) : launch_tiles<T, 32, 8>(p, entries, stream);
 }
 
 }  // namespace
 
-// Channels per block of the kernel that serves N states (the caller chooses the slices from it); 0: not supported.
-extern "C" int b200_selective_scan_channels(int N) {
-  if (N <= 0 || N > 256) return 0;
-  return THREADS / (N <= 32 ? 4 : N <= 64 ? 8 : N <= 128 ? 16 : 32);
+// Time slices per sequence of at most max_len rows: cutting doubles the recurrence's work, so only where whole sequences
+// occupy less than half of the SMs.  0: a state count the kernel does not serve.
+extern "C" int b200_selective_scan_slices(int C, int N, int entries, int max_len) {
+  if (C <= 0 || N <= 0 || N > 256 || entries <= 0) return 0;
+  const int cb = THREADS / pick_lanes(C, N, entries);
+  const long long blocks = (long long)((C + cb - 1) / cb) * entries;
+  if (blocks * 2 > 148) return 1;
+  long long s = 4 * 148 / blocks;
+  if (s > max_len / 256) s = max_len / 256;
+  return s < 1 ? 1 : (int)s;
 }
 
 // rows of `entries` sequences (ent_first / ent_len / ent_slot; positions per row), the longest with max_len rows; singles != 0:

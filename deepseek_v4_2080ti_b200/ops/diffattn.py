@@ -103,8 +103,8 @@ WS_LIMIT = 1 << 28                      # floats of partial results per launch; 
 
 
 def pick_splits(rows: int, blocks_per_row: int, keys: int) -> int:
-    """Slices of one row's keys: enough blocks for three per SM, at least 64 keys each."""
-    return max(1, min(NUM_SMS, (3 * NUM_SMS) // max(1, rows * blocks_per_row), (keys + 63) // 64))
+    """Slices of one row's keys: enough blocks for nearly two per SM, at least 192 keys each."""
+    return max(1, min(NUM_SMS, 256 // max(1, rows * blocks_per_row), (keys + 191) // 192))
 
 
 def rows(q: torch.Tensor, m: DiffAttention, k_cache, v_cache, gate: torch.Tensor, block_table, positions, max_keys: int,

@@ -14,9 +14,7 @@ import torch
 from ..utils import canary
 from . import _lib
 
-NUM_SMS = 148
 SLICE_ROWS = 32                 # a time slice is a multiple of this
-MIN_SLICE = 256
 
 
 @dataclass
@@ -60,15 +58,6 @@ def _workspace(need: int, device) -> torch.Tensor:
     return ws
 
 
-def pick_slices(rows: int, channels: int, states: int, entries: int) -> int:
-    """Time slices per entry: cutting doubles the recurrence's work, so only where whole sequences leave most of the device
-    idle (fewer than one block per SM)."""
-    blocks = (channels + (per := _lib.lib().b200_selective_scan_channels(states)) - 1) // max(per, 1) * entries
-    if blocks >= NUM_SMS:
-        return 1
-    return max(1, min((4 * NUM_SMS) // blocks, rows // MIN_SLICE))
-
-
 def selective_scan(x: torch.Tensor, dt: torch.Tensor, bc: torch.Tensor, b_off: int, c_off: int, z: torch.Tensor, a: torch.Tensor,
                    dt_bias: torch.Tensor, d_skip: torch.Tensor, state: torch.Tensor, seg: Segments, positions: torch.Tensor,
                    x_in: torch.Tensor | None = None, tail: torch.Tensor | None = None, slices: int | None = None) -> torch.Tensor:
@@ -82,7 +71,7 @@ def selective_scan(x: torch.Tensor, dt: torch.Tensor, bc: torch.Tensor, b_off: i
     _lib.check_indices(seg.slot, 0, state.shape[0], 4)
     entries = seg.first.numel()
     if slices is None:
-        slices = pick_slices(seg.max_length, c, n, entries)
+        slices = _lib.lib().b200_selective_scan_slices(c, n, entries, seg.max_length)
     per = max(SLICE_ROWS, (seg.max_length + slices - 1) // slices)
     per = (per + SLICE_ROWS - 1) // SLICE_ROWS * SLICE_ROWS
     slices = (seg.max_length + per - 1) // per
@@ -106,7 +95,3 @@ def scan_decay(a_log: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
     """-exp(A_log) in fp32, times log2(e) for the bf16 kernels (their exponential is a power of two)."""
     a = -torch.exp(a_log.double())
     return ((a / torch.log(torch.tensor(2.0, dtype=torch.float64, device=a.device))) if dtype == torch.bfloat16 else a).float().contiguous()
-
-
-def supported(states: int) -> bool:
-    return _lib.lib().b200_selective_scan_channels(states) > 0
