@@ -48,15 +48,33 @@ struct Params {
   int* status;
 };
 
-// MN-major operand, 128-byte swizzle: 64-element MN atoms LBO bytes apart, 8-row K groups SBO bytes apart.
-__device__ __forceinline__ uint64_t desc_mn_sw128(const void* p, uint32_t lbo, uint32_t sbo) {
-  uint64_t d = 0;
-  d |= (uint64_t)((smem_u32(p) & 0x3FFFF) >> 4);
-  d |= (uint64_t)(lbo >> 4) << 16;
-  d |= (uint64_t)(sbo >> 4) << 32;
-  d |= (uint64_t)1 << 46;
-  d |= (uint64_t)2 << 61;
-  return d;
+// Shared-memory descriptors (128-byte swizzle, 8-row groups 1024 bytes apart, sm_100 version) as two words: the low one holds
+// the start address, and for an MN-major operand (values) the distance of its 64-element atoms in the upper half.
+constexpr uint32_t DESC_K_HI = (1024 >> 4) | (1u << 14) | (2u << 29);
+__device__ __forceinline__ uint32_t desc_lo(const void* p) { return (smem_u32(p) & 0x3FFFF) >> 4; }
+
+// Products issued by the lanes with `on` (one of the warp) while the warp stays converged.
+__device__ __forceinline__ void umma_ss_if(uint32_t on, uint32_t d, uint32_t a_lo, uint32_t b_lo, uint32_t hi, uint32_t idesc,
+                                           uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\t.reg .b64 a, b;\n\t"
+      "setp.ne.b32 p, %6, 0;\n\tsetp.ne.b32 q, %0, 0;\n\t"
+      "mov.b64 a, {%2, %4};\n\tmov.b64 b, {%3, %4};\n\t"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%1], a, b, %5, p;\n\t}\n"
+      :
+      : "r"(on), "r"(d), "r"(a_lo), "r"(b_lo), "r"(hi), "r"(idesc), "r"(accumulate)
+      : "memory");
+}
+__device__ __forceinline__ void umma_ts_if(uint32_t on, uint32_t d, uint32_t a, uint32_t b_lo, uint32_t hi, uint32_t idesc,
+                                           uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\t.reg .b64 b;\n\t"
+      "setp.ne.b32 p, %6, 0;\n\tsetp.ne.b32 q, %0, 0;\n\t"
+      "mov.b64 b, {%3, %4};\n\t"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%1], [%2], b, %5, p;\n\t}\n"
+      :
+      : "r"(on), "r"(d), "r"(a), "r"(b_lo), "r"(hi), "r"(idesc), "r"(accumulate)
+      : "memory");
 }
 
 // VN: columns of a value slice rounded up to 32 (the accumulator's width in tensor memory and of the products).
@@ -159,52 +177,66 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           if (ok) ok = slab(&tmV, g * p.V + v0 + s * 64);
       }
       if (!ok) { atomicExch(p.status, ERR_WAIT_STAGE); *abort_flag = 1; }
-    } else if (warp == 9 && lane == 0) {
-      bool ok = mbar_wait(q_full, 0);
-      // the ring's consumption order differs from its fill order only in that a tile's value slabs are held while the next
-      // tile's first-map keys, which lie behind them, are consumed
-      const int per_tile = 2 * p.slabs + VS;
-      auto wait_slab = [&](int i) { return mbar_wait(&r_full[i % p.stages], (i / p.stages) & 1); };
-      auto issue_s = [&](int j, int m) -> bool {
-        for (int s = 0; s < p.slabs; ++s) {
-          const int i = j * per_tile + m * p.slabs + s;
-          if (!wait_slab(i)) return false;
-          tc_fence_after();
-          const uint64_t dk = umma_desc_sw128(sR + (i % p.stages) * ATOM), dq = umma_desc_sw128(sQ + (m * p.slabs + s) * ATOM);
-          const int steps = min(4, (p.D - s * 64) / 16);
-          for (int kk = 0; kk < steps; ++kk) umma_bf16_ss(tmem + m * 128, dq + 2 * kk, dk + 2 * kk, idesc_qk, (s | kk) ? 1u : 0u);
-          umma_commit(&r_empty[i % p.stages]);
-        }
-        umma_commit(&s_full[m]);
-        return true;
+    } else if (warp == 9) {
+      // The whole warp walks the loop so that addresses and descriptors stay warp-uniform; one lane's instructions count.
+      // (A single diverged lane took ten times as long between two products as the products themselves.)
+      const uint32_t lead = lane == 0;
+      bool ok = true;
+      auto wait = [&](uint64_t* bar, uint32_t parity) {
+        ok = __all_sync(0xffffffffu, mbar_wait(bar, parity));
+        return ok;
       };
-      ok = ok && issue_s(0, 0) && issue_s(0, 1);
+      wait(q_full, 0);
+      // slabs are waited for in the order they were filled; only a tile's value slabs are given back later (after the next
+      // tile's first-map keys, which lie behind them)
+      int st = 0;
+      uint32_t ph = 0;
+      const uint32_t ring = desc_lo(sR), dq0 = desc_lo(sQ);
+      const int stages = p.stages, slabs = p.slabs, last_steps = (p.D - (slabs - 1) * 64) / 16;
+      auto issue_s = [&](const int m) {
+        for (int s = 0; s < slabs; ++s) {
+          if (!wait(&r_full[st], ph)) return;
+          tc_fence_after();
+          const uint32_t dk = ring + st * (ATOM >> 4), dq = dq0 + (m * slabs + s) * (ATOM >> 4);
+          const int steps = s + 1 < slabs ? 4 : last_steps;
+#pragma unroll
+          for (int kk = 0; kk < 4; ++kk)
+            umma_ss_if(lead & (kk < steps), tmem + m * 128, dq + 2 * kk, dk + 2 * kk, DESC_K_HI, idesc_qk, (s | kk) ? 1u : 0u);
+          if (lead) umma_commit(&r_empty[st]);
+          if (++st == stages) { st = 0; ph ^= 1; }
+        }
+        if (lead) umma_commit(&s_full[m]);
+      };
+      if (ok) issue_s(0);
+      if (ok) issue_s(1);
       for (int j = 0; ok && j < n_tiles && !*abort_flag; ++j) {
-        const int iv = j * per_tile + 2 * p.slabs;
-        for (int m = 0; ok && m < 2; ++m) {
-          if (!mbar_wait(&p_full[m], j & 1)) { ok = false; break; }
+        int sv = 0;
+#pragma unroll
+        for (int m = 0; m < 2; ++m) {
+          if (!ok || !wait(&p_full[m], j & 1)) break;
           if (m == 0) {
+            // two slabs of a tile are neighbours: the ring has an even number of stages and a tile an even number of slabs
+            sv = st;
 #pragma unroll
             for (int s = 0; s < VS; ++s)
-              if (ok) ok = wait_slab(iv + s);
+              if (ok && wait(&r_full[st], ph) && ++st == stages) { st = 0; ph ^= 1; }
             if (!ok) break;
           }
           tc_fence_after();
-          // two slabs of a tile are neighbours: the ring has an even number of stages and a tile an even number of slabs
-          const uint8_t* sv = sR + (iv % p.stages) * ATOM;
+          const uint32_t dv = ring + sv * (ATOM >> 4);
 #pragma unroll
           for (int kk = 0; kk < 8; ++kk)
-            umma_bf16_ts(tmem + 256 + m * 128, tmem + m * 128 + kk * 8, desc_mn_sw128(sv + kk * 2048, ATOM, 1024), idesc_pv,
-                         (j | kk) ? 1u : 0u);
-          umma_commit(&pv_done[m]);
-          if (m == 1) {
+            umma_ts_if(lead, tmem + 256 + m * 128, tmem + m * 128 + kk * 8, (dv + kk * 128) | (uint32_t(ATOM >> 4) << 16), DESC_K_HI,
+                       idesc_pv, (j | kk) ? 1u : 0u);
+          if (lead) umma_commit(&pv_done[m]);
+          if (m == 1 && lead) {
 #pragma unroll
-            for (int s = 0; s < VS; ++s) umma_commit(&r_empty[(iv + s) % p.stages]);
+            for (int s = 0; s < VS; ++s) umma_commit(&r_empty[sv + s]);
           }
-          if (j + 1 < n_tiles) ok = issue_s(j + 1, m);
+          if (j + 1 < n_tiles) issue_s(m);
         }
       }
-      if (!ok) { atomicExch(p.status, ERR_WAIT_TMA); *abort_flag = 1; }
+      if (!ok && lead) { atomicExch(p.status, ERR_WAIT_TMA); *abort_flag = 1; }
     }
   } else {
     asm volatile("setmaxnreg.inc.sync.aligned.u32 216;");

@@ -4,8 +4,9 @@
 //
 // Rows of one sequence are neighbours; row_first[r] is the sequence's first row of this batch, row_slot[r] its state slot,
 // positions[r] its position.  Inputs from before the batch come from the slot's tail (the last taps - 1 inputs, oldest
-// first); inputs from before position 0 are zero, so a slot needs no clearing.  The tail is read here and replaced by the
-// kernel that runs the recurrence behind the convolution (selective_scan.cu).  One thread: 8 channels, `strip` rows.
+// first); inputs from before position 0 are zero, so a slot needs no clearing.  A sequence that brings a single row has its
+// tail replaced right here (one thread holds all of it); the tail of a longer portion, which several blocks read, is replaced
+// by the kernel that runs the recurrence behind the convolution (selective_scan.cu).  One thread: 8 channels, `strip` rows.
 #include "launch.h"
 #include "ops.h"
 #include "vec8.cuh"
@@ -18,7 +19,7 @@ struct ConvRowsParams {
   const T* x;              // [rows, ldx]
   const float* w;          // [taps, C]
   const float* bias;       // [C] or null
-  const T* tail;           // [slots, taps - 1, C]
+  T* tail;                 // [slots, taps - 1, C]
   const int *row_first, *row_slot, *positions;
   T* y;                    // [rows, ldy]
   int ldx, ldy, rows, C, taps, silu, strip;
@@ -43,19 +44,37 @@ __global__ void __launch_bounds__(128) conv_rows_kernel(ConvRowsParams<T> p) {
   const int r1 = min(p.rows, ((int)blockIdx.y + 1) * p.strip);
   for (int r = blockIdx.y * p.strip; r < r1; ++r) {
     const int off = r - p.row_first[r], pos = p.positions[r];
-    const T* tail = p.tail + ((size_t)p.row_slot[r] * (taps - 1)) * p.C + c;
-    float acc[8];
+    T* tail = p.tail + ((size_t)p.row_slot[r] * (taps - 1)) * p.C + c;
+    const bool solo = off == 0 && (r + 1 == p.rows || p.row_first[r + 1] == r + 1);
+    float acc[8], old[K ? K : 1][8];
 #pragma unroll
     for (int i = 0; i < 8; ++i) acc[i] = b[i];
 #pragma unroll
     for (int j = 0; j < taps; ++j) {
       const int back = taps - 1 - j;
-      if (back > pos) continue;
-      float f[8];
+      float (&f)[8] = old[K ? j : 0];
+      if (back > pos) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] = 0.f;
+        continue;
+      }
       load8(back <= off ? p.x + (size_t)(r - back) * p.ldx + c : tail + (size_t)(taps - 1 - (back - off)) * p.C, f);
       if (!K) load8(p.w + (size_t)j * p.C + c, w[0]);
 #pragma unroll
       for (int i = 0; i < 8; ++i) acc[i] = fmaf(w[K ? j : 0][i], f[i], acc[i]);
+    }
+    if (solo) {
+      // the inputs of the last taps - 1 positions, this row's included: exact copies, they were widened from T
+      if (K) {
+#pragma unroll
+        for (int j = 1; j < K; ++j) store8(tail + (size_t)(j - 1) * p.C, old[j]);
+      } else {
+        for (int j = 1; j < taps; ++j) {
+          float f[8];
+          load8(j + 1 < taps ? tail + (size_t)j * p.C : p.x + (size_t)r * p.ldx + c, f);
+          store8(tail + (size_t)(j - 1) * p.C, f);
+        }
+      }
     }
     if (p.silu) {
 #pragma unroll
@@ -67,11 +86,11 @@ __global__ void __launch_bounds__(128) conv_rows_kernel(ConvRowsParams<T> p) {
 }
 
 template <typename T>
-int run_conv_rows(const void* x, int ldx, const float* w, const float* bias, const void* tail, const int* row_first,
+int run_conv_rows(const void* x, int ldx, const float* w, const float* bias, void* tail, const int* row_first,
                   const int* row_slot, const int* positions, void* y, int ldy, int rows, int C, int taps, int silu,
                   cudaStream_t stream) {
   ConvRowsParams<T> p;
-  p.x = reinterpret_cast<const T*>(x); p.w = w; p.bias = bias; p.tail = reinterpret_cast<const T*>(tail);
+  p.x = reinterpret_cast<const T*>(x); p.w = w; p.bias = bias; p.tail = reinterpret_cast<T*>(tail);
   p.row_first = row_first; p.row_slot = row_slot; p.positions = positions; p.y = reinterpret_cast<T*>(y);
   p.ldx = ldx; p.ldy = ldy; p.rows = rows; p.C = C; p.taps = taps; p.silu = silu;
   p.strip = 1;
@@ -89,7 +108,7 @@ int run_conv_rows(const void* x, int ldx, const float* w, const float* bias, con
 }  // namespace
 
 // x rows of C channels (C, ldx, ldy multiples of 8); f32 != 0: x, tail, y are fp32, otherwise bf16.
-extern "C" int b200_conv_rows(const void* x, int ldx, const float* w, const float* bias, const void* tail, const int* row_first,
+extern "C" int b200_conv_rows(const void* x, int ldx, const float* w, const float* bias, void* tail, const int* row_first,
                               const int* row_slot, const int* positions, void* y, int ldy, int rows, int C, int taps, int silu,
                               int f32, cudaStream_t stream) {
   if (rows <= 0 || C <= 0 || (C & 7) || (ldx & 7) || (ldy & 7) || ldx < C || ldy < C || taps < 1 || taps > 64) return -6;

@@ -214,7 +214,7 @@ int b200_attn_diff_prefill(const void* q, const void* k_cache, const void* v_cac
                            const int* kv_len, int batch, int max_q_len, int q_rows, int max_blocks, int num_blocks, int block_size,
                            int H, int G, int D, int V, int vdim, int ldo, float scale, float lambda, float keep, float eps,
                            int* status, cudaStream_t stream);
-int b200_conv_rows(const void* x, int ldx, const float* w, const float* bias, const void* tail, const int* row_first,
+int b200_conv_rows(const void* x, int ldx, const float* w, const float* bias, void* tail, const int* row_first,
                    const int* row_slot, const int* positions, void* y, int ldy, int rows, int C, int taps, int silu, int f32,
                    cudaStream_t stream);
 int b200_selective_scan_slices(int C, int N, int entries, int max_len);

@@ -19,7 +19,8 @@
 // step sizes; since the decay over a slice is exp(A sum delta), the second pass composes the state at its own start from
 // those and produces the outputs.
 //
-// The last slice also replaces the slot's convolution tail (the inputs of the convolution in front, see conv_rows.cu).
+// The last slice also replaces the slot's convolution tail (the inputs of the convolution in front); for a single row the
+// convolution has done so already (conv_rows.cu).
 #include "launch.h"
 #include "ops.h"
 #include "per_device.h"
@@ -30,6 +31,7 @@ using namespace b200;
 
 constexpr int THREADS = 128;
 constexpr int TT = 32;                   // rows per tile
+constexpr int STEP_THREADS = 256, STEP_CHANNELS = 1;      // single-row kernel
 
 template <typename T>
 struct ScanParams {
@@ -74,6 +76,18 @@ __device__ __forceinline__ void store_pair(__nv_bfloat16* p, float a, float b) {
   *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b);
 }
 __device__ __forceinline__ void store_pair(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+
+template <int NS>
+__device__ __forceinline__ void load_quad(const __nv_bfloat16* p, float (&f)[NS]) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = widen(u.x), b = widen(u.y);
+  f[0] = a.x; f[1 % NS] = a.y; f[2 % NS] = b.x; f[3 % NS] = b.y;
+}
+template <int NS>
+__device__ __forceinline__ void load_quad(const float* p, float (&f)[NS]) {
+  const float4 a = *reinterpret_cast<const float4*>(p);
+  f[0] = a.x; f[1 % NS] = a.y; f[2 % NS] = a.z; f[3 % NS] = a.w;
+}
 
 // fp32 pairs in 64-bit registers
 __device__ __forceinline__ uint64_t pair_of(float a, float b) {
@@ -345,12 +359,11 @@ __global__ void __launch_bounds__(THREADS) scan_kernel(ScanParams<T> p) {
   if (p.xin && tid < CB && c0 + tid < p.C) replace_tail(p, slot, first, len, c0 + tid);
 }
 
-// Sequences with a single row, straight from and to memory: L lanes share a channel, NS states each, KC channels per lane
-// group so that enough loads are in flight.
+// Sequences with a single row, straight from and to memory: L lanes share a channel, NS states each, KC channels per thread.
 template <typename T, int L, int NS, int KC>
-__global__ void __launch_bounds__(THREADS) scan_step_kernel(ScanParams<T> p) {
+__global__ void __launch_bounds__(STEP_THREADS) scan_step_kernel(ScanParams<T> p) {
   constexpr bool FAST = sizeof(T) == 2;
-  constexpr int CB = THREADS / L;
+  constexpr int CB = STEP_THREADS / L;
   using LaneT = Lane<NS, FAST>;
   pdl_grid_trigger();
   const int lane = threadIdx.x % L, c0 = blockIdx.x * CB * KC + threadIdx.x / L, e = blockIdx.y;
@@ -360,59 +373,62 @@ __global__ void __launch_bounds__(THREADS) scan_step_kernel(ScanParams<T> p) {
 #pragma unroll
   for (int k = 0; k < KC; ++k) {
     const int c = c0 + k * CB;
-    const float* a = p.a + (size_t)c * p.N + lane * NS;
-    if (vec && c < p.C) LaneT::load(a, st[k].a);
-    else LaneT::fill(st[k].a, [&](int i) { return c < p.C && lane * NS + i < p.N ? a[i] : 0.f; });
+    const float* src = p.a + (size_t)c * p.N + lane * NS;
+    if (vec && c < p.C) LaneT::load(src, st[k].a);
+    else LaneT::fill(st[k].a, [&](int i) { return c < p.C && lane * NS + i < p.N ? src[i] : 0.f; });
     bias[k] = c < p.C ? p.dt_bias[c] : 0.f;
     dskip[k] = c < p.C ? p.d_skip[c] : 0.f;
   }
   pdl_grid_wait();
   const int row = p.ent_first[e], slot = p.ent_slot[e];
   if (p.ent_len[e] != 1) return;                              // uniform per block
-  const int pos = p.positions[row];
-  float* state = p.state + (size_t)slot * p.C * p.N;
-  const T* bcr = p.bc + (size_t)row * p.ldb;
   float dt[KC], x[KC], z[KC], b[NS], cc[NS];
 #pragma unroll
   for (int k = 0; k < KC; ++k) {
     const int c = c0 + k * CB;
     const bool on = c < p.C;
-    const float* s = state + (size_t)c * p.N + lane * NS;
+    const float* s = p.state + ((size_t)slot * p.C + c) * p.N + lane * NS;
     if (vec && on) LaneT::load(s, st[k].s);
     else LaneT::fill(st[k].s, [&](int i) { return on && lane * NS + i < p.N ? s[i] : 0.f; });
     dt[k] = on ? p.dt[(size_t)row * p.ldd + c] : 0.f;
     x[k] = on ? (float)p.x[(size_t)row * p.ldx + c] : 0.f;
     z[k] = on ? (float)p.z[(size_t)row * p.ldz + c] : 0.f;
   }
+  const T* bcr = p.bc + (size_t)row * p.ldb + lane * NS;
+  if (NS == 4 && lane * NS < p.N) {                           // B and C are padded to whole vectors of eight
+    load_quad(bcr + p.b_off, b);
+    load_quad(bcr + p.c_off, cc);
+  } else {
 #pragma unroll
-  for (int i = 0; i < NS; ++i) {
-    const int n = lane * NS + i;
-    b[i] = n < p.N ? (float)bcr[p.b_off + n] : 0.f;
-    cc[i] = n < p.N ? (float)bcr[p.c_off + n] : 0.f;
+    for (int i = 0; i < NS; ++i) {
+      b[i] = lane * NS + i < p.N ? (float)bcr[p.b_off + i] : 0.f;
+      cc[i] = lane * NS + i < p.N ? (float)bcr[p.c_off + i] : 0.f;
+    }
   }
+  const bool fresh = p.positions[row] == 0;
 #pragma unroll
   for (int k = 0; k < KC; ++k) {
     const int c = c0 + k * CB;
-    if (pos == 0) LaneT::fill(st[k].s, [](int) { return 0.f; });
     const float delta = softplus<FAST>(dt[k] + bias[k]), dx = delta * x[k];
-    const float2 d2 = make_float2(delta, dx);
+    if (fresh) LaneT::fill(st[k].s, [](int) { return 0.f; });
     float y = 0.f;
 #pragma unroll
     for (int i = 0; i < LaneT::P; ++i) {
-      const float2 a = halves_of(st[k].a[i]), s = halves_of(st[k].s[i]);
-      const float s0 = fmaf(decay<FAST>(d2.x * a.x), s.x, d2.y * b[2 * i]);
-      float s1 = 0.f;
-      y = fmaf(s0, cc[2 * i], y);
-      if (2 * i + 1 < NS) {
-        s1 = fmaf(decay<FAST>(d2.x * a.y), s.y, d2.y * b[2 * i + 1 < NS ? 2 * i + 1 : 0]);
-        y = fmaf(s1, cc[2 * i + 1 < NS ? 2 * i + 1 : 0], y);
+      const float2 av = halves_of(st[k].a[i]), sv = halves_of(st[k].s[i]);
+      float out[2] = {0.f, 0.f};
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        if (2 * i + h < NS) {
+          out[h] = fmaf(decay<FAST>(delta * (h ? av.y : av.x)), h ? sv.y : sv.x, dx * b[2 * i + h < NS ? 2 * i + h : 0]);
+          y = fmaf(out[h], cc[2 * i + h < NS ? 2 * i + h : 0], y);
+        }
       }
-      st[k].s[i] = pair_of(s0, s1);
+      st[k].s[i] = pair_of(out[0], out[1]);
     }
 #pragma unroll
     for (int o = 1; o < L; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
     if (c >= p.C) continue;
-    float* s = state + (size_t)c * p.N + lane * NS;
+    float* s = p.state + ((size_t)slot * p.C + c) * p.N + lane * NS;
     if (vec) {
       if constexpr (NS % 4 == 0) {
 #pragma unroll
@@ -423,10 +439,7 @@ __global__ void __launch_bounds__(THREADS) scan_step_kernel(ScanParams<T> p) {
         if (lane * NS + i < p.N) s[i] = v;
       });
     }
-    if (lane == 0) {
-      p.out[(size_t)row * p.ldo + c] = (T)(fmaf(dskip[k], x[k], y) * silu<FAST>(z[k]));
-      if (p.xin) replace_tail(p, slot, row, 1, c);
-    }
+    if (lane == 0) p.out[(size_t)row * p.ldo + c] = (T)(fmaf(dskip[k], x[k], y) * silu<FAST>(z[k]));
   }
 }
 
@@ -443,17 +456,18 @@ int launch_tiles(const ScanParams<T>& p, int entries, cudaStream_t stream) {
     configured = true;
   }
   const int blocks = (p.C + CB - 1) / CB;
-  cudaError_t e = cudaSuccess;
-  if (p.slices > 1) e = launch_pdl(scan_kernel<T, L, NS, 1>, dim3(blocks, p.slices - 1, entries), dim3(THREADS), smem, stream, p);
-  if (e == cudaSuccess)
-    e = launch_pdl(scan_kernel<T, L, NS, 0>, dim3(blocks, p.slices, entries), dim3(THREADS), smem, stream, p);
-  return (int)e;
+  // ordinary launches: a grid of one long wave that starts while its predecessor still holds some of the SMs is crowded
+  // onto the others for its whole run
+  if (p.slices > 1) scan_kernel<T, L, NS, 1><<<dim3(blocks, p.slices - 1, entries), THREADS, smem, stream>>>(p);
+  scan_kernel<T, L, NS, 0><<<dim3(blocks, p.slices, entries), THREADS, smem, stream>>>(p);
+  return (int)cudaGetLastError();
 }
 
 template <typename T, int L, int NS>
 int launch_step(const ScanParams<T>& p, int entries, cudaStream_t stream) {
-  constexpr int KC = NS <= 4 ? 4 : 2, PER = THREADS / L * KC;
-  return (int)launch_pdl(scan_step_kernel<T, L, NS, KC>, dim3((p.C + PER - 1) / PER, entries), dim3(THREADS), 0, stream, p);
+  constexpr int PER = STEP_THREADS / L * STEP_CHANNELS;
+  return (int)launch_pdl(scan_step_kernel<T, L, NS, STEP_CHANNELS>, dim3((p.C + PER - 1) / PER, entries), dim3(STEP_THREADS), 0,
+                         stream, p);
 }
 
 // Lanes per channel of the tile kernel: as few as hold the states, more for batches whose channels alone would leave the

@@ -31,7 +31,8 @@ class Segments:
 
 def conv_rows(x: torch.Tensor, w_t: torch.Tensor, bias: torch.Tensor | None, tail: torch.Tensor, seg: Segments,
               positions: torch.Tensor, silu: bool = True) -> torch.Tensor:
-    """x [T, >= C] (row stride allowed), w_t fp32 [taps, C], tail [slots, taps - 1, C] (read only) -> [T, C]."""
+    """x [T, >= C] (row stride allowed), w_t fp32 [taps, C], tail [slots, taps - 1, C] -> [T, C].  The tails of sequences with a
+    single row are replaced here, those of longer portions by ``selective_scan``."""
     taps, c = w_t.shape
     t = x.shape[0]
     assert x.stride(1) == 1 and tail.dtype == x.dtype and tail.shape[1:] == (max(taps - 1, 1), c)
@@ -63,7 +64,8 @@ def selective_scan(x: torch.Tensor, dt: torch.Tensor, bc: torch.Tensor, b_off: i
                    x_in: torch.Tensor | None = None, tail: torch.Tensor | None = None, slices: int | None = None) -> torch.Tensor:
     """x [T, C] (after the convolution), dt fp32 [T, C] (before bias and softplus), bc rows with B and C at the given columns,
     z [T, >= C]; ``a`` fp32 [C, N] as ``scan_decay`` prepares it; state fp32 [slots, C, N], updated in place.  Returns
-    ``y silu(z)`` [T, C].  ``x_in`` / ``tail``: inputs of the convolution in front, whose last rows replace the slots' tails."""
+    ``y silu(z)`` [T, C].  ``x_in`` / ``tail``: inputs of the convolution in front, whose last rows replace the tails of the
+    sequences that bring more than one row."""
     t, c = x.shape
     n = a.shape[1]
     assert dt.dtype == state.dtype == torch.float32 and state.shape[1:] == (c, n) and state.is_contiguous() and a.is_contiguous()
