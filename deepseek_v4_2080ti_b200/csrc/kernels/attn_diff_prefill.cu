@@ -48,33 +48,15 @@ struct Params {
   int* status;
 };
 
-// Shared-memory descriptors (128-byte swizzle, 8-row groups 1024 bytes apart, sm_100 version) as two words: the low one holds
-// the start address, and for an MN-major operand (values) the distance of its 64-element atoms in the upper half.
-constexpr uint32_t DESC_K_HI = (1024 >> 4) | (1u << 14) | (2u << 29);
-__device__ __forceinline__ uint32_t desc_lo(const void* p) { return (smem_u32(p) & 0x3FFFF) >> 4; }
-
-// Products issued by the lanes with `on` (one of the warp) while the warp stays converged.
-__device__ __forceinline__ void umma_ss_if(uint32_t on, uint32_t d, uint32_t a_lo, uint32_t b_lo, uint32_t hi, uint32_t idesc,
-                                           uint32_t accumulate) {
-  asm volatile(
-      "{\n\t.reg .pred p, q;\n\t.reg .b64 a, b;\n\t"
-      "setp.ne.b32 p, %6, 0;\n\tsetp.ne.b32 q, %0, 0;\n\t"
-      "mov.b64 a, {%2, %4};\n\tmov.b64 b, {%3, %4};\n\t"
-      "@q tcgen05.mma.cta_group::1.kind::f16 [%1], a, b, %5, p;\n\t}\n"
-      :
-      : "r"(on), "r"(d), "r"(a_lo), "r"(b_lo), "r"(hi), "r"(idesc), "r"(accumulate)
-      : "memory");
-}
-__device__ __forceinline__ void umma_ts_if(uint32_t on, uint32_t d, uint32_t a, uint32_t b_lo, uint32_t hi, uint32_t idesc,
-                                           uint32_t accumulate) {
-  asm volatile(
-      "{\n\t.reg .pred p, q;\n\t.reg .b64 b;\n\t"
-      "setp.ne.b32 p, %6, 0;\n\tsetp.ne.b32 q, %0, 0;\n\t"
-      "mov.b64 b, {%3, %4};\n\t"
-      "@q tcgen05.mma.cta_group::1.kind::f16 [%1], [%2], b, %5, p;\n\t}\n"
-      :
-      : "r"(on), "r"(d), "r"(a), "r"(b_lo), "r"(hi), "r"(idesc), "r"(accumulate)
-      : "memory");
+// MN-major operand, 128-byte swizzle: 64-element MN atoms LBO bytes apart, 8-row K groups SBO bytes apart.
+__device__ __forceinline__ uint64_t desc_mn_sw128(const void* p, uint32_t lbo, uint32_t sbo) {
+  uint64_t d = 0;
+  d |= (uint64_t)((smem_u32(p) & 0x3FFFF) >> 4);
+  d |= (uint64_t)(lbo >> 4) << 16;
+  d |= (uint64_t)(sbo >> 4) << 32;
+  d |= (uint64_t)1 << 46;
+  d |= (uint64_t)2 << 61;
+  return d;
 }
 
 // VN: columns of a value slice rounded up to 32 (the accumulator's width in tensor memory and of the products).
@@ -101,7 +83,7 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(q_full + 8);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0), lane = threadIdx.x & 31;   // uniform: the issuer depends on it
   const int b = blockIdx.z, qt = (int)gridDim.x - 1 - (int)blockIdx.x;   // long tiles first
   const int h = blockIdx.y / p.v_slices, v0 = (blockIdx.y % p.v_slices) * 128;
   const int q_len = p.q_len[b], kv_len = p.kv_len[b];
@@ -178,9 +160,7 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       }
       if (!ok) { atomicExch(p.status, ERR_WAIT_STAGE); *abort_flag = 1; }
     } else if (warp == 9) {
-      // The whole warp walks the loop so that addresses and descriptors stay warp-uniform; one lane's instructions count.
-      // (A single diverged lane took ten times as long between two products as the products themselves.)
-      const uint32_t lead = lane == 0;
+      // The whole warp walks the loop, so that addresses and descriptors stay warp-uniform, and one elected lane issues.
       bool ok = true;
       auto wait = [&](uint64_t* bar, uint32_t parity) {
         ok = __all_sync(0xffffffffu, mbar_wait(bar, parity));
@@ -191,21 +171,24 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       // tile's first-map keys, which lie behind them)
       int st = 0;
       uint32_t ph = 0;
-      const uint32_t ring = desc_lo(sR), dq0 = desc_lo(sQ);
+      const uint64_t ring = umma_desc_sw128(sR), dq0 = umma_desc_sw128(sQ);
       const int stages = p.stages, slabs = p.slabs, last_steps = (p.D - (slabs - 1) * 64) / 16;
       auto issue_s = [&](const int m) {
         for (int s = 0; s < slabs; ++s) {
           if (!wait(&r_full[st], ph)) return;
           tc_fence_after();
-          const uint32_t dk = ring + st * (ATOM >> 4), dq = dq0 + (m * slabs + s) * (ATOM >> 4);
+          const uint64_t dk = ring + st * (ATOM >> 4), dq = dq0 + (m * slabs + s) * (ATOM >> 4);
           const int steps = s + 1 < slabs ? 4 : last_steps;
+          if (elect_one()) {
+            umma_bf16_ss(tmem + m * 128, dq, dk, idesc_qk, s ? 1u : 0u);
 #pragma unroll
-          for (int kk = 0; kk < 4; ++kk)
-            umma_ss_if(lead & (kk < steps), tmem + m * 128, dq + 2 * kk, dk + 2 * kk, DESC_K_HI, idesc_qk, (s | kk) ? 1u : 0u);
-          if (lead) umma_commit(&r_empty[st]);
+            for (int kk = 1; kk < 4; ++kk)
+              if (kk < steps) umma_bf16_ss(tmem + m * 128, dq + 2 * kk, dk + 2 * kk, idesc_qk, 1u);
+            umma_commit(&r_empty[st]);
+            if (s + 1 == slabs) umma_commit(&s_full[m]);
+          }
           if (++st == stages) { st = 0; ph ^= 1; }
         }
-        if (lead) umma_commit(&s_full[m]);
       };
       if (ok) issue_s(0);
       if (ok) issue_s(1);
@@ -223,20 +206,21 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
             if (!ok) break;
           }
           tc_fence_after();
-          const uint32_t dv = ring + sv * (ATOM >> 4);
+          const uint64_t dv = desc_mn_sw128(sR, ATOM, 1024) + sv * (ATOM >> 4);
+          if (elect_one()) {
+            umma_bf16_ts(tmem + 256 + m * 128, tmem + m * 128, dv, idesc_pv, j ? 1u : 0u);
 #pragma unroll
-          for (int kk = 0; kk < 8; ++kk)
-            umma_ts_if(lead, tmem + 256 + m * 128, tmem + m * 128 + kk * 8, (dv + kk * 128) | (uint32_t(ATOM >> 4) << 16), DESC_K_HI,
-                       idesc_pv, (j | kk) ? 1u : 0u);
-          if (lead) umma_commit(&pv_done[m]);
-          if (m == 1 && lead) {
+            for (int kk = 1; kk < 8; ++kk) umma_bf16_ts(tmem + 256 + m * 128, tmem + m * 128 + kk * 8, dv + kk * 128, idesc_pv, 1u);
+            umma_commit(&pv_done[m]);
+            if (m == 1) {
 #pragma unroll
-            for (int s = 0; s < VS; ++s) umma_commit(&r_empty[sv + s]);
+              for (int s = 0; s < VS; ++s) umma_commit(&r_empty[sv + s]);
+            }
           }
           if (j + 1 < n_tiles) issue_s(m);
         }
       }
-      if (!ok && lead) { atomicExch(p.status, ERR_WAIT_TMA); *abort_flag = 1; }
+      if (!ok && lane == 0) { atomicExch(p.status, ERR_WAIT_TMA); *abort_flag = 1; }
     }
   } else {
     asm volatile("setmaxnreg.inc.sync.aligned.u32 216;");

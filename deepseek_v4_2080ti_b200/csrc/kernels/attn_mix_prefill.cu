@@ -85,7 +85,7 @@ mix_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(q_full + 7);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0), lane = threadIdx.x & 31;   // uniform: the issuer depends on it
   const int b = blockIdx.z, h = blockIdx.y, qt = (int)gridDim.x - 1 - (int)blockIdx.x;   // long tiles first
   const int q_len = p.q_len[b], kv_len = p.kv_len[b];
   const int q0 = qt * BQ;

@@ -41,33 +41,66 @@ __global__ void __launch_bounds__(128) conv_rows_kernel(ConvRowsParams<T> p) {
   }
   pdl_grid_wait();
   if (!on) return;
-  const int r1 = min(p.rows, ((int)blockIdx.y + 1) * p.strip);
-  for (int r = blockIdx.y * p.strip; r < r1; ++r) {
+  const int r0 = blockIdx.y * p.strip, r1 = min(p.rows, r0 + p.strip);
+  auto finish = [&](int r, float (&acc)[8]) {
+    if (p.silu) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        acc[i] = sizeof(T) == 2 ? __fdividef(acc[i], 1.f + __expf(-acc[i])) : acc[i] / (1.f + expf(-acc[i]));
+    }
+    store8(p.y + (size_t)r * p.ldy + c, acc);
+  };
+  if (K > 1 && p.strip > 1) {
+    const int first = p.row_first[r0];
+    if (r0 - first >= K - 1 && p.row_first[r1 - 1] == first) {
+      // a strip inside one sequence's portion: every row is read once and stays in a window of registers
+      float win[K ? K : 1][8];
+#pragma unroll
+      for (int j = 1; j < K; ++j) load8(p.x + (size_t)(r0 - K + j) * p.ldx + c, win[j]);
+#pragma unroll 4
+      for (int r = r0; r < r1; ++r) {
+        float acc[8];
+#pragma unroll
+        for (int j = 0; j + 1 < K; ++j)
+#pragma unroll
+          for (int i = 0; i < 8; ++i) win[j][i] = win[j + 1][i];
+        load8(p.x + (size_t)r * p.ldx + c, win[K ? K - 1 : 0]);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) acc[i] = b[i];
+#pragma unroll
+        for (int j = 0; j < K; ++j)
+#pragma unroll
+          for (int i = 0; i < 8; ++i) acc[i] = fmaf(w[j][i], win[j][i], acc[i]);
+        finish(r, acc);
+      }
+      return;
+    }
+  }
+  for (int r = r0; r < r1; ++r) {
     const int off = r - p.row_first[r], pos = p.positions[r];
     T* tail = p.tail + ((size_t)p.row_slot[r] * (taps - 1)) * p.C + c;
     const bool solo = off == 0 && (r + 1 == p.rows || p.row_first[r + 1] == r + 1);
-    float acc[8], old[K ? K : 1][8];
+    float acc[8];
 #pragma unroll
     for (int i = 0; i < 8; ++i) acc[i] = b[i];
 #pragma unroll
     for (int j = 0; j < taps; ++j) {
       const int back = taps - 1 - j;
-      float (&f)[8] = old[K ? j : 0];
-      if (back > pos) {
-#pragma unroll
-        for (int i = 0; i < 8; ++i) f[i] = 0.f;
-        continue;
-      }
+      if (back > pos) continue;
+      float f[8];
       load8(back <= off ? p.x + (size_t)(r - back) * p.ldx + c : tail + (size_t)(taps - 1 - (back - off)) * p.C, f);
       if (!K) load8(p.w + (size_t)j * p.C + c, w[0]);
 #pragma unroll
       for (int i = 0; i < 8; ++i) acc[i] = fmaf(w[K ? j : 0][i], f[i], acc[i]);
     }
     if (solo) {
-      // the inputs of the last taps - 1 positions, this row's included: exact copies, they were widened from T
+      // the inputs of the last taps - 1 positions, this row's included (loaded again: exact copies of what lies there)
       if (K) {
+        float keep[K ? K : 1][8];
 #pragma unroll
-        for (int j = 1; j < K; ++j) store8(tail + (size_t)(j - 1) * p.C, old[j]);
+        for (int j = 1; j < K; ++j) load8(j + 1 < K ? tail + (size_t)j * p.C : p.x + (size_t)r * p.ldx + c, keep[j]);
+#pragma unroll
+        for (int j = 1; j < K; ++j) store8(tail + (size_t)(j - 1) * p.C, keep[j]);
       } else {
         for (int j = 1; j < taps; ++j) {
           float f[8];
@@ -76,12 +109,7 @@ __global__ void __launch_bounds__(128) conv_rows_kernel(ConvRowsParams<T> p) {
         }
       }
     }
-    if (p.silu) {
-#pragma unroll
-      for (int i = 0; i < 8; ++i)
-        acc[i] = sizeof(T) == 2 ? __fdividef(acc[i], 1.f + __expf(-acc[i])) : acc[i] / (1.f + expf(-acc[i]));
-    }
-    store8(p.y + (size_t)r * p.ldy + c, acc);
+    finish(r, acc);
   }
 }
 
@@ -94,7 +122,7 @@ int run_conv_rows(const void* x, int ldx, const float* w, const float* bias, voi
   p.row_first = row_first; p.row_slot = row_slot; p.positions = positions; p.y = reinterpret_cast<T*>(y);
   p.ldx = ldx; p.ldy = ldy; p.rows = rows; p.C = C; p.taps = taps; p.silu = silu;
   p.strip = 1;
-  while (p.strip < 8 && (long long)rows * C / 8 / p.strip > 148LL * 4096) p.strip *= 2;
+  while (p.strip < 16 && (long long)rows * C / 8 / p.strip > 148LL * 4096) p.strip *= 2;
   const dim3 grid((C / 8 + 127) / 128, (rows + p.strip - 1) / p.strip);
   if (grid.y > 65535) return -6;
   switch (taps) {

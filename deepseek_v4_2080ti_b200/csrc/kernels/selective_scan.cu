@@ -31,7 +31,7 @@ using namespace b200;
 
 constexpr int THREADS = 128;
 constexpr int TT = 32;                   // rows per tile
-constexpr int STEP_THREADS = 256, STEP_CHANNELS = 1;      // single-row kernel
+constexpr int STEP_THREADS = 128, STEP_CHANNELS = 1;      // single-row kernel
 
 template <typename T>
 struct ScanParams {
