@@ -273,6 +273,18 @@ def _zg_kernels(size: str, dev, timer: _Timer, ctx: int) -> list[dict]:
         pair("recurrence", f"{t} tokens, {inner} channels x {N} states",
              (lambda: scan.selective_scan(xc, dt, bc, sw.b_off, sw.c_off, xin[:, inner:], sw.a, sw.dt_b, sw.d, st, seg, pos1, xin[:, :inner], tails), sbytes, 0),
              (like, gbytes, 0))
+    # decoding step with as much state as the like kernel holds for 32 sequences
+    t = 32 * 128 // N
+    xc, dt, bc, xin = rnd(t, inner), rnd(t, inner, dt=torch.float32), rnd(t, sw.x.n), rnd(t, 2 * inner)
+    ar, one = torch.arange(t, dtype=torch.int32, device=dev), torch.ones(t, dtype=torch.int32, device=dev)
+    seg, pos1, st = scan.Segments(ar, ar, ar, one, ar, 1), ar + 5, torch.zeros(t, inner, N, dtype=torch.float32, device=dev)
+    mixed, gg, beta = rnd(32, (2 * hk + hv) * 128), -torch.rand(32, hv, device=dev), torch.rand(32, hv, device=dev)
+    gst = torch.zeros(32, hv, 128, 128, dtype=torch.float32, device=dev)
+    pair("recurrence, equal state bytes", f"{t} sequences (like: 32), {inner} channels x {N} states",
+         (lambda: scan.selective_scan(xc, dt, bc, sw.b_off, sw.c_off, xin[:, inner:], sw.a, sw.dt_b, sw.d, st, seg, pos1),
+          t * inner * 10 + t * sw.x.n * 2 + t * inner * N * 8, 0),
+         (lambda: gdn.step(gst, ar[:32], mixed, 0, hk * 128, 2 * hk * 128, gg, beta, hv, hk),
+          32 * (2 * hk + 2 * hv) * 256 + 32 * hv * 8 + 32 * hv * 128 * 128 * 8, 0))
     t = 8192
     table = (torch.arange(t // bs, dtype=torch.int32, device=dev) + 1)[None]
     q, q1 = rnd(t, H, 2, D), rnd(t, H, 128)
