@@ -1,0 +1,234 @@
+// Gated linear attention: per head a state S [D, V] in fp32 with a decay per key channel,
+//
+//   S_t = diag(alpha_t) S_(t-1) + k_t v_t^T,     o_t = S_t^T q_t,     alpha = sigmoid(z)^(1 / tau)
+//
+// over a batch of rows of several sequences (entries of neighbouring rows, one state slot each; a portion that begins at
+// position 0 starts from zero).  Head widths are padded to multiples of 16 with zero channels.
+//
+//   gla_decay    log alpha from the low-rank logits z = W2 a + b, fp32
+//   gla_scan     one token after the other; the state's columns are independent, so a block takes 32 of them, a lane per
+//                column, and the warps share the rows.  fp32 results, and bf16 portions too short for chunk_scan
+//   gla_step     one token of many sequences: a block per head and sequence reads, updates and writes the state once and
+//                finishes the row (norm, gate) itself
+//   gla_finish   per head o / rms(o) * weight * silu(g)
+#include "launch.h"
+#include "ops.h"
+#include "per_device.h"
+#include "vec8.cuh"
+
+namespace {
+using namespace b200;
+
+__device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+
+constexpr int DR = 8;           // rows per block of gla_decay
+
+// a: [rows, >= rank] (row stride ld); w2 [channels, rank]; la [rows, channels].  rank a multiple of 8.
+template <typename T>
+__global__ void gla_decay_kernel(const T* __restrict__ a, int ld, const T* __restrict__ w2, const float* __restrict__ bias,
+                                 float inv_tau, float* __restrict__ la, int rows, int channels, int rank) {
+  extern __shared__ float sa[];            // [DR][rank]
+  pdl_grid_trigger();
+  pdl_grid_wait();
+  const int r0 = blockIdx.x * DR, n = min(DR, rows - r0);
+  for (int i = threadIdx.x; i < DR * rank; i += blockDim.x)
+    sa[i] = i / rank < n ? (float)a[(size_t)(r0 + i / rank) * ld + i % rank] : 0.f;
+  __syncthreads();
+  for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < channels; c += gridDim.y * blockDim.x) {
+    float z[DR];
+#pragma unroll
+    for (int r = 0; r < DR; ++r) z[r] = bias[c];
+    for (int k = 0; k < rank; k += 8) {
+      float w[8];
+      load8(w2 + (size_t)c * rank + k, w);
+#pragma unroll
+      for (int r = 0; r < DR; ++r)
+#pragma unroll
+        for (int j = 0; j < 8; ++j) z[r] = fmaf(w[j], sa[r * rank + k + j], z[r]);
+    }
+#pragma unroll
+    for (int r = 0; r < DR; ++r)
+      if (r < n) la[(size_t)(r0 + r) * channels + c] = log_sigmoid(z[r]) * inv_tau;
+  }
+}
+
+template <typename T>
+struct GlaParams {
+  const T *q, *k, *v;        // head h of row t at ptr + t * ld + h * D (V)
+  const float* la;           // [rows, H * D]
+  float* state;              // [slots, H, D, V]
+  float* o;                  // [rows, H * V]
+  const int *first, *length, *slot, *positions;
+  int ld, H, D, V;
+  float scale;
+};
+
+constexpr int CT = 16;          // rows staged together
+constexpr int SW = 8;           // warps
+
+// grid (ceil(V / 32), H, entries).  RD: state rows per warp (and per thread).
+template <typename T, int RD>
+__global__ void __launch_bounds__(SW * 32) gla_scan_kernel(GlaParams<T> p) {
+  extern __shared__ float sm[];
+  pdl_grid_trigger();
+  const int D = p.D, V = p.V, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  float* sq = sm;                          // [CT][D]
+  float* sk = sq + CT * D;
+  float* sg = sk + CT * D;
+  float* sv = sg + CT * D;                 // [CT][32]
+  float* red = sv + CT * 32;               // [CT][SW][32]
+  const int h = blockIdx.y, e = blockIdx.z, c = blockIdx.x * 32 + lane;
+  pdl_grid_wait();
+  const int t0 = p.first[e], n = p.length[e];
+  float* st = p.state + ((size_t)p.slot[e] * p.H + h) * D * V;
+  const bool fresh = p.positions[t0] == 0;
+  float s[RD];
+#pragma unroll
+  for (int i = 0; i < RD; ++i) {
+    const int d = i * SW + warp;
+    s[i] = !fresh && d < D && c < V ? st[(size_t)d * V + c] : 0.f;
+  }
+  for (int r0 = 0; r0 < n; r0 += CT) {
+    const int m = min(CT, n - r0);
+    __syncthreads();
+    for (int i = tid; i < m * D; i += SW * 32) {
+      const int r = i / D, d = i - r * D;
+      const size_t row = (size_t)(t0 + r0 + r);
+      sq[i] = (float)p.q[row * p.ld + h * D + d] * p.scale;
+      sk[i] = (float)p.k[row * p.ld + h * D + d];
+      sg[i] = expf(p.la[(row * p.H + h) * D + d]);
+    }
+    for (int i = tid; i < m * 32; i += SW * 32)
+      sv[i] = blockIdx.x * 32 + (i & 31) < V ? (float)p.v[(size_t)(t0 + r0 + (i >> 5)) * p.ld + h * V + blockIdx.x * 32 + (i & 31)] : 0.f;
+    __syncthreads();
+    for (int r = 0; r < m; ++r) {
+      const float v = sv[r * 32 + lane];
+      float acc = 0.f;
+#pragma unroll
+      for (int i = 0; i < RD; ++i) {
+        const int d = i * SW + warp;
+        if (d < D) {
+          s[i] = fmaf(sg[r * D + d], s[i], sk[r * D + d] * v);
+          acc = fmaf(s[i], sq[r * D + d], acc);
+        }
+      }
+      red[(r * SW + warp) * 32 + lane] = acc;
+    }
+    __syncthreads();
+    for (int i = tid; i < m * 32; i += SW * 32) {
+      const int r = i >> 5, col = blockIdx.x * 32 + (i & 31);
+      float a = 0.f;
+#pragma unroll
+      for (int w = 0; w < SW; ++w) a += red[(r * SW + w) * 32 + (i & 31)];
+      if (col < V) p.o[((size_t)(t0 + r0 + r) * p.H + h) * V + col] = a;
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < RD; ++i) {
+    const int d = i * SW + warp;
+    if (d < D && c < V) st[(size_t)d * V + c] = s[i];
+  }
+}
+
+// grid rows: out[row, h * V + c] = o / rms over the head's vdim values * weight * silu(gate).
+template <typename T>
+__global__ void gla_finish_kernel(const float* __restrict__ o, const T* __restrict__ gate, int ld_gate, const float* __restrict__ w,
+                                  T* __restrict__ out, int ldo, int H, int V, int vdim, float eps) {
+  pdl_grid_trigger();
+  pdl_grid_wait();
+  const size_t row = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int h = warp; h < H; h += blockDim.x >> 5) {
+    const float* src = o + (row * H + h) * V;
+    float ss = 0.f;
+    for (int c = lane * 4; c < V; c += 128) {
+      const float4 f = *reinterpret_cast<const float4*>(src + c);
+      ss += f.x * f.x + f.y * f.y + f.z * f.z + f.w * f.w;               // padded columns are zero
+    }
+    const float inv = 1.f / sqrtf(warp_sum_all(ss) / (float)vdim + eps);
+    for (int c = lane * 8; c < V; c += 256) {
+      float f[8], g[8], ww[8];
+      load8(src + c, f);
+      load8(gate + row * ld_gate + h * V + c, g);
+      load8(w + c, ww);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) f[j] = f[j] * inv * ww[j] * (g[j] / (1.f + expf(-g[j])));
+      store8(out + row * ldo + h * V + c, f);
+    }
+  }
+  for (int c = H * V + threadIdx.x; c < ldo; c += blockDim.x) out[row * ldo + c] = (T)0.f;
+}
+
+template <typename T, int RD>
+int launch_scan(const GlaParams<T>& p, int entries, cudaStream_t stream) {
+  const size_t smem = (size_t)(3 * CT * p.D + CT * 32 + CT * SW * 32) * 4;
+  static PerDeviceOnce once_;
+  bool& configured = once_.slot();
+  if (!configured) {
+    const cudaError_t e = cudaFuncSetAttribute(gla_scan_kernel<T, RD>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    if (e != cudaSuccess) return (int)e;
+    configured = true;
+  }
+  return (int)launch_pdl(gla_scan_kernel<T, RD>, dim3((p.V + 31) / 32, p.H, entries), dim3(SW * 32), smem, stream, p);
+}
+
+template <typename T>
+int run_scan(const void* q, const void* k, const void* v, int ld, const float* la, float* state, float* o, const int* first,
+             const int* length, const int* slot, const int* positions, int entries, int H, int D, int V, float scale,
+             cudaStream_t stream) {
+  GlaParams<T> p;
+  p.q = reinterpret_cast<const T*>(q); p.k = reinterpret_cast<const T*>(k); p.v = reinterpret_cast<const T*>(v); p.la = la;
+  p.state = state; p.o = o; p.first = first; p.length = length; p.slot = slot; p.positions = positions; p.ld = ld; p.H = H; p.D = D;
+  p.V = V; p.scale = scale;
+  if (D <= 4 * SW) return launch_scan<T, 4>(p, entries, stream);
+  if (D <= 8 * SW) return launch_scan<T, 8>(p, entries, stream);
+  if (D <= 16 * SW) return launch_scan<T, 16>(p, entries, stream);
+  if (D <= 32 * SW) return launch_scan<T, 32>(p, entries, stream);
+  if (D <= 64 * SW) return launch_scan<T, 64>(p, entries, stream);
+  return -6;
+}
+
+template <typename T>
+int run_decay(const void* a, int ld, const void* w2, const float* bias, float inv_tau, float* la, int rows, int channels, int rank,
+              cudaStream_t stream) {
+  const int threads = channels >= 256 ? 256 : (channels + 31) / 32 * 32;
+  int cols = (channels + threads - 1) / threads;
+  const dim3 grid((rows + DR - 1) / DR, cols);
+  return (int)launch_pdl(gla_decay_kernel<T>, grid, dim3(threads), (size_t)DR * rank * 4, stream, reinterpret_cast<const T*>(a), ld,
+                         reinterpret_cast<const T*>(w2), bias, inv_tau, la, rows, channels, rank);
+}
+
+template <typename T>
+int run_finish(const float* o, const void* gate, int ld_gate, const float* w, void* out, int ldo, int rows, int H, int V, int vdim,
+               float eps, cudaStream_t stream) {
+  const int warps = H < 8 ? H : 8;
+  return (int)launch_pdl(gla_finish_kernel<T>, dim3(rows), dim3(warps * 32), 0, stream, o, reinterpret_cast<const T*>(gate), ld_gate, w,
+                         reinterpret_cast<T*>(out), ldo, H, V, vdim, eps);
+}
+
+}  // namespace
+
+// a rows `ld` apart, w2 [channels, rank] in the activations' type, la fp32 [rows, channels]; rank % 8 == 0, at most 1024.
+extern "C" int b200_gla_decay(const void* a, int ld, const void* w2, const float* bias, float inv_tau, float* la, int rows,
+                              int channels, int rank, int f32, cudaStream_t stream) {
+  if (rows <= 0 || channels <= 0 || rank <= 0 || (rank & 7) || rank > 1024) return -6;
+  return f32 ? run_decay<float>(a, ld, w2, bias, inv_tau, la, rows, channels, rank, stream)
+             : run_decay<__nv_bfloat16>(a, ld, w2, bias, inv_tau, la, rows, channels, rank, stream);
+}
+
+// D at most 512; state [slots, H, D, V] fp32 in place; o fp32 [rows, H * V].
+extern "C" int b200_gla_scan(const void* q, const void* k, const void* v, int ld, const float* la, float* state, float* o,
+                             const int* first, const int* length, const int* slot, const int* positions, int entries, int H, int D,
+                             int V, float scale, int f32, cudaStream_t stream) {
+  if (entries <= 0 || entries > 65535 || H <= 0 || H > 65535 || D <= 0 || V <= 0) return -6;
+  return f32 ? run_scan<float>(q, k, v, ld, la, state, o, first, length, slot, positions, entries, H, D, V, scale, stream)
+             : run_scan<__nv_bfloat16>(q, k, v, ld, la, state, o, first, length, slot, positions, entries, H, D, V, scale, stream);
+}
+
+// V % 16 == 0; out [rows, ldo] (columns behind the heads are zeroed).
+extern "C" int b200_gla_finish(const float* o, const void* gate, int ld_gate, const float* w, void* out, int ldo, int rows, int H,
+                               int V, int vdim, float eps, int f32, cudaStream_t stream) {
+  if (rows <= 0 || H <= 0 || V <= 0 || (V & 15) || vdim <= 0 || vdim > V || ldo < H * V || (ldo & 7) || (ld_gate & 7)) return -6;
+  return f32 ? run_finish<float>(o, gate, ld_gate, w, out, ldo, rows, H, V, vdim, eps, stream)
+             : run_finish<__nv_bfloat16>(o, gate, ld_gate, w, out, ldo, rows, H, V, vdim, eps, stream);
+}

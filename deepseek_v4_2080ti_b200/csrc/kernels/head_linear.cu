@@ -1,0 +1,89 @@
+// A small matrix per head on the rows of a short batch: y[t, h, :N] = x[t, h, :K] W[h]^T in bf16 with fp32 sums (the up
+// projections of latent attention around its absorbed form).  The weights are streamed once per 64 rows; operands go from
+// global memory straight into tensor-core fragments: the order of the dimensions inside a dot product is free, so a lane takes
+// 16 contiguous bytes of a row as its share of two k-steps.  Prompt-sized batches use the big GEMMs instead.
+#include <cuda_bf16.h>
+#include <stdint.h>
+#include "launch.h"
+#include "ops.h"
+
+namespace {
+using namespace b200;
+
+__device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+constexpr int WARPS = 4, NW = 16;          // features per warp
+
+// grid (features / 64, heads, rows / (16 MT)), 128 threads; K % 16 == 0 (32-wide chunks, the last may be half).
+template <int MT>
+__global__ void __launch_bounds__(WARPS * 32)
+head_linear_kernel(const __nv_bfloat16* __restrict__ x, int ldx, int x_head, const __nv_bfloat16* __restrict__ w,
+                   __nv_bfloat16* __restrict__ y, int ldy, int y_head, int T, int N, int K) {
+  pdl_grid_trigger();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gr = lane >> 2, kk = lane & 3;
+  const int h = blockIdx.y, n0 = blockIdx.x * WARPS * NW + warp * NW, t0 = blockIdx.z * 16 * MT;
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  const __nv_bfloat16* wh = w + (size_t)h * N * K;
+  float acc[MT][2][4] = {};
+  pdl_grid_wait();
+  if (n0 >= N) return;
+  auto load_w = [&](int k0, uint4 (&b)[2]) {
+    const int k = k0 + kk * 8;
+#pragma unroll
+    for (int nb = 0; nb < 2; ++nb) {
+      const int n = n0 + nb * 8 + gr;
+      b[nb] = n < N && k < K ? *reinterpret_cast<const uint4*>(wh + (size_t)n * K + k) : zero;
+    }
+  };
+  uint4 b[2], bn[2];
+  load_w(0, b);
+  for (int k0 = 0; k0 < K; k0 += 32) {
+    if (k0 + 32 < K) load_w(k0 + 32, bn);
+    const int k = k0 + kk * 8;
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt) {
+      const int ta = t0 + mt * 16 + gr, tb = ta + 8;
+      const uint4 a0 = ta < T && k < K ? *reinterpret_cast<const uint4*>(x + (size_t)ta * ldx + h * x_head + k) : zero;
+      const uint4 a1 = tb < T && k < K ? *reinterpret_cast<const uint4*>(x + (size_t)tb * ldx + h * x_head + k) : zero;
+#pragma unroll
+      for (int nb = 0; nb < 2; ++nb) {
+        mma_bf16(acc[mt][nb], a0.x, a1.x, a0.y, a1.y, b[nb].x, b[nb].y);
+        mma_bf16(acc[mt][nb], a0.z, a1.z, a0.w, a1.w, b[nb].z, b[nb].w);
+      }
+    }
+    b[0] = bn[0];
+    b[1] = bn[1];
+  }
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int nb = 0; nb < 2; ++nb)
+#pragma unroll
+      for (int hf = 0; hf < 2; ++hf) {
+        const int t = t0 + mt * 16 + gr + hf * 8, n = n0 + nb * 8 + kk * 2;
+        if (t < T && n < N)
+          *reinterpret_cast<__nv_bfloat162*>(y + (size_t)t * ldy + h * y_head + n) =
+              __floats2bfloat162_rn(acc[mt][nb][hf * 2], acc[mt][nb][hf * 2 + 1]);
+      }
+}
+
+}  // namespace
+
+// Rows `ldx` / `ldy` elements apart, heads `x_head` / `y_head` apart (multiples of 8), W [H, N, K]; N even, K % 16 == 0.
+extern "C" int b200_head_linear(const void* x, int ldx, int x_head, const void* w, void* y, int ldy, int y_head, int T, int H, int N,
+                                int K, cudaStream_t stream) {
+  if (T <= 0 || H <= 0 || H > 65535 || N <= 0 || (N & 1) || K <= 0 || (K & 15) || ((ldx | x_head | ldy | y_head) & 7)) return -6;
+  const int mt = T <= 16 ? 1 : T <= 32 ? 2 : 4;
+  if ((T + 16 * mt - 1) / (16 * mt) > 65535) return -6;
+  const dim3 grid((N + WARPS * NW - 1) / (WARPS * NW), H, (T + 16 * mt - 1) / (16 * mt)), block(WARPS * 32);
+  auto xp = reinterpret_cast<const __nv_bfloat16*>(x);
+  auto wp = reinterpret_cast<const __nv_bfloat16*>(w);
+  auto yp = reinterpret_cast<__nv_bfloat16*>(y);
+  if (mt == 1) return (int)launch_pdl(head_linear_kernel<1>, grid, block, 0, stream, xp, ldx, x_head, wp, yp, ldy, y_head, T, N, K);
+  if (mt == 2) return (int)launch_pdl(head_linear_kernel<2>, grid, block, 0, stream, xp, ldx, x_head, wp, yp, ldy, y_head, T, N, K);
+  return (int)launch_pdl(head_linear_kernel<4>, grid, block, 0, stream, xp, ldx, x_head, wp, yp, ldy, y_head, T, N, K);
+}

@@ -4,7 +4,7 @@
 //                      route in expert-sorted order, and the (expert, m_tile, row0, rows) work table of both grouped
 //                      GEMMs, all on the device (nothing is read back by the host);
 //   moe_gather       - token rows -> expert-sorted rows;
-//   moe_swiglu       - silu(gate) * up on the sorted rows (with the DeepSeek clamp);
+//   moe_glu          - gated unit on the sorted rows: silu(gate) * up (with the DeepSeek clamp) or the one-plus form;
 //   moe_combine      - out[t] = (shared[t]) + sum_k w[t,k] * y[row(t,k)], k ascending (deterministic).
 // Routes whose expert lives on another rank are dropped locally (expert-range sharding) or carried by the
 // dispatch kernels of csrc/comm.
@@ -13,43 +13,45 @@
 // moe_finalize_reduce (:4917).
 #include <cuda_bf16.h>
 #include <stdint.h>
+#include "glu.cuh"
 #include "ops.h"
+#include "vec8.cuh"
 
 namespace {
 
-constexpr int MAX_TOPK = 16;
 constexpr int MAX_EXPERTS = 1024;
 
 __device__ __forceinline__ float score_fn(float x, int fn) {
-  if (fn == 1) return 1.f / (1.f + __expf(-x));                       // sigmoid
-  if (fn == 2) return sqrtf(x > 20.f ? x : log1pf(__expf(x)));        // sqrt(softplus)
+  if (fn == 1) return 1.f / (1.f + expf(-x));                         // sigmoid
+  if (fn == 2) return sqrtf(x > 20.f ? x : log1pf(expf(x)));          // sqrt(softplus)
   return x;                                                           // softmax handled by the caller
 }
 
-// One warp per token. logits fp32 [T, E]; bias fp32 [E] or null.
-__global__ void moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int T, int E, int K,
+// One warp per token. logits fp32 [T, ld], the first E of a row; bias fp32 [E] or null; E <= 32 J.
+template <int J>
+__global__ void moe_route_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ bias, int T, int E, int K,
                                  int fn, int norm_topk, float route_scale, int* __restrict__ idx,
                                  float* __restrict__ wts) {
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
   if (t >= T) return;
-  const float* row = logits + (size_t)t * E;
+  const float* row = logits + (size_t)t * ld;
   // softmax statistics
   float mx = -INFINITY, den = 1.f;
   if (fn == 0) {
     for (int e = lane; e < E; e += 32) mx = fmaxf(mx, row[e]);
     for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
     den = 0.f;
-    for (int e = lane; e < E; e += 32) den += __expf(row[e] - mx);
+    for (int e = lane; e < E; e += 32) den += expf(row[e] - mx);
     for (int o = 16; o > 0; o >>= 1) den += __shfl_xor_sync(0xffffffffu, den, o);
   }
-  // each lane keeps the scores of experts lane, lane+32, ... (E <= 1024 -> 32 per lane)
-  float sc[MAX_EXPERTS / 32], sel[MAX_EXPERTS / 32];
+  // each lane keeps the scores of experts lane, lane + 32, ...
+  float sc[J], sel[J];
 #pragma unroll
-  for (int j = 0; j < MAX_EXPERTS / 32; ++j) {
+  for (int j = 0; j < J; ++j) {
     const int e = j * 32 + lane;
     if (e < E) {
-      sc[j] = fn == 0 ? __expf(row[e] - mx) / den : score_fn(row[e], fn);
+      sc[j] = fn == 0 ? expf(row[e] - mx) / den : score_fn(row[e], fn);
       sel[j] = sc[j] + (bias ? bias[e] : 0.f);
     } else {
       sc[j] = 0.f;
@@ -57,13 +59,11 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
     }
   }
   float wsum = 0.f;
-  float my_w = 0.f;
-  int my_i = 0;
   for (int k = 0; k < K; ++k) {
     float best = -INFINITY;
     int be = 0x7fffffff;
 #pragma unroll
-    for (int j = 0; j < MAX_EXPERTS / 32; ++j) {
+    for (int j = 0; j < J; ++j) {
       const int e = j * 32 + lane;
       if (sel[j] > best || (sel[j] == best && e < be)) { best = sel[j]; be = e; }
     }
@@ -75,86 +75,99 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
     // the owning lane reports the unbiased score and retires the expert
     float w = 0.f;
 #pragma unroll
-    for (int j = 0; j < MAX_EXPERTS / 32; ++j)
+    for (int j = 0; j < J; ++j)
       if (j * 32 + lane == be) { w = sc[j]; sel[j] = -INFINITY; }
     for (int o = 16; o > 0; o >>= 1) w += __shfl_xor_sync(0xffffffffu, w, o);
     wsum += w;
-    if (lane == k) { my_w = w; my_i = be; }
+    if (lane == (k & 31)) {
+      idx[(size_t)t * K + k] = be;
+      wts[(size_t)t * K + k] = w * route_scale;
+    }
   }
-  if (lane < K) {
-    float w = my_w;
-    if (fn != 0 && norm_topk) w /= wsum;
-    idx[(size_t)t * K + lane] = my_i;
-    wts[(size_t)t * K + lane] = w * route_scale;
-  }
+  if (fn != 0 && norm_topk)
+    for (int k = lane; k < K; k += 32) wts[(size_t)t * K + k] /= wsum;     // lane k & 31 wrote entry k
 }
 
-// Single block.  idx [R] global expert ids (R = T*K); experts [lo, hi) are local.
+__device__ __forceinline__ int warp_scan(int v, int lane) {                // inclusive
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const int u = __shfl_up_sync(0xffffffffu, v, o);
+    if (lane >= o) v += u;
+  }
+  return v;
+}
+// Exclusive prefix sum over a block of 1024 threads; `ws` holds 32 ints; total: the block's sum.
+__device__ __forceinline__ int block_scan(int v, int* ws, int& total) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int inc = warp_scan(v, lane);
+  if (lane == 31) ws[warp] = inc;
+  __syncthreads();
+  if (warp == 0) ws[lane] = warp_scan(ws[lane], lane);
+  __syncthreads();
+  const int base = warp ? ws[warp - 1] : 0;
+  total = ws[31];
+  __syncthreads();
+  return base + inc - v;
+}
+
+// One block of 1024 threads per local expert.  idx [R] global expert ids (R = T*K); experts [lo, hi) are local.
 // Outputs: offsets [EL+1], route_row [R] (row in sorted order or -1), row_token [rows] (source token of a sorted row),
-// work tables for token tiles of bn13 / bn2 rows, counts.
+// work tables for token tiles of bn13 / bn2 rows, counts.  Every block counts all routes, so that it knows where its expert's
+// rows and work entries begin, and places its own expert's routes in their order (stable: results are run-to-run identical).
 __global__ void __launch_bounds__(1024)
 moe_plan_kernel(const int* __restrict__ idx, int R, int K, int lo, int hi, int* __restrict__ offsets,
                 int* __restrict__ route_row, int* __restrict__ row_token, int4* __restrict__ work13, int* __restrict__ n13,
                 int m_tiles13, int bn13, int4* __restrict__ work2, int* __restrict__ n2, int m_tiles2, int bn2,
                 int max_work) {
-  __shared__ int cnt[MAX_EXPERTS], off[MAX_EXPERTS + 1], cur[MAX_EXPERTS], wbase13[MAX_EXPERTS + 1], wbase2[MAX_EXPERTS + 1];
-  const int EL = hi - lo;
-  for (int e = threadIdx.x; e < EL; e += blockDim.x) cnt[e] = 0;
+  __shared__ int cnt[MAX_EXPERTS], ws[32], mine[4];
+  const int EL = hi - lo, e = blockIdx.x, tid = threadIdx.x;
+  cnt[tid] = 0;
   __syncthreads();
-  for (int r = threadIdx.x; r < R; r += blockDim.x) {
-    const int e = idx[r] - lo;
-    if (e >= 0 && e < EL) atomicAdd(&cnt[e], 1);
+  for (int r = tid; r < R; r += 1024) {
+    const int x = idx[r] - lo;
+    if (x >= 0 && x < EL) atomicAdd(&cnt[x], 1);
+    else if (e == 0) route_row[r] = -1;
   }
   __syncthreads();
-  if (threadIdx.x == 0) {
-    int a = 0, w13 = 0, w2 = 0;
-    for (int e = 0; e < EL; ++e) {
-      off[e] = a;
-      wbase13[e] = w13;
-      wbase2[e] = w2;
-      a += cnt[e];
-      w13 += m_tiles13 * ((cnt[e] + bn13 - 1) / bn13);
-      w2 += m_tiles2 * ((cnt[e] + bn2 - 1) / bn2);
+  const int c_t = tid < EL ? cnt[tid] : 0;                                 // thread t stands for expert t here
+  int total, total13, total2;
+  const int off_t = block_scan(c_t, ws, total);
+  const int w13_t = block_scan(m_tiles13 * ((c_t + bn13 - 1) / bn13), ws, total13);
+  const int w2_t = block_scan(m_tiles2 * ((c_t + bn2 - 1) / bn2), ws, total2);
+  if (e == 0) {
+    if (tid < EL) offsets[tid] = off_t;
+    if (tid == 0) {
+      offsets[EL] = total;
+      *n13 = min(total13, max_work);
+      *n2 = min(total2, max_work);
     }
-    off[EL] = a;
-    wbase13[EL] = w13;
-    wbase2[EL] = w2;
-    *n13 = min(w13, max_work);
-    *n2 = min(w2, max_work);
   }
+  if (tid == e) { mine[0] = c_t; mine[1] = off_t; mine[2] = w13_t; mine[3] = w2_t; }
   __syncthreads();
-  for (int e = threadIdx.x; e <= EL; e += blockDim.x) {
-    offsets[e] = off[e];
-    if (e < EL) cur[e] = 0;
-  }
-  __syncthreads();
-  // stable placement: routes are scanned in order by one thread per expert to keep results run-to-run identical
-  for (int e = threadIdx.x; e < EL; e += blockDim.x) {
-    if (cnt[e] == 0) continue;
-    int c = 0;
-    for (int r = 0; r < R; ++r)
-      if (idx[r] - lo == e) {
-        route_row[r] = off[e] + c;
-        row_token[off[e] + c] = r / K;
-        ++c;
-      }
-  }
-  for (int r = threadIdx.x; r < R; r += blockDim.x) {
-    const int e = idx[r] - lo;
-    if (e < 0 || e >= EL) route_row[r] = -1;
+  const int c = mine[0], off = mine[1];
+  if (c == 0) return;
+  int placed = 0;
+  for (int r0 = 0; r0 < R && placed < c; r0 += 1024) {
+    const int r = r0 + tid;
+    const int hit = r < R && idx[r] - lo == e;
+    int n;
+    const int at = off + placed + block_scan(hit, ws, n);
+    if (hit) {
+      route_row[r] = at;
+      row_token[at] = r / K;
+    }
+    placed += n;
   }
   // work tables: m-tile fastest inside a token tile so one expert's weight tiles are swept once per token tile
-  for (int e = threadIdx.x; e < EL; e += blockDim.x) {
-    const int c = cnt[e];
-    int w = wbase13[e];
-    for (int nt = 0; nt * bn13 < c; ++nt)
-      for (int m = 0; m < m_tiles13; ++m, ++w)
-        if (w < max_work) work13[w] = make_int4(e, m, off[e] + nt * bn13, min(bn13, c - nt * bn13));
-    w = wbase2[e];
-    for (int nt = 0; nt * bn2 < c; ++nt)
-      for (int m = 0; m < m_tiles2; ++m, ++w)
-        if (w < max_work) work2[w] = make_int4(e, m, off[e] + nt * bn2, min(bn2, c - nt * bn2));
-  }
+  auto emit = [&](int4* work, int base, int m_tiles, int bn) {
+    const int n = m_tiles * ((c + bn - 1) / bn);
+    for (int i = tid; i < n; i += 1024) {
+      const int nt = i / m_tiles;
+      if (base + i < max_work) work[base + i] = make_int4(e, i - nt * m_tiles, off + nt * bn, min(bn, c - nt * bn));
+    }
+  };
+  emit(work13, mine[2], m_tiles13, bn13);
+  emit(work2, mine[3], m_tiles2, bn2);
 }
 
 // xs[row, :] = x[row_token[row], :]; one block per sorted row; H % 8 == 0.
@@ -167,19 +180,31 @@ __global__ void moe_gather_kernel(const __nv_bfloat16* __restrict__ x, const int
   for (int i = threadIdx.x; i < H / 8; i += blockDim.x) dst[i] = src[i];
 }
 
-__global__ void moe_swiglu_kernel(const __nv_bfloat16* __restrict__ gu, const int* __restrict__ offsets, int EL,
-                                  __nv_bfloat16* __restrict__ act, int I, float limit) {
+// rows [gate | up] of 2 I columns -> gated unit (glu.cuh); slope 0: silu(min(g, limit)) clamp(u), the limit optional.
+template <typename T>
+__global__ void moe_glu_kernel(const T* __restrict__ gu, const int* __restrict__ offsets, int EL, T* __restrict__ act, int I,
+                               float limit, float slope) {
   const int row = blockIdx.x;
   if (row >= offsets[EL]) return;
-  const __nv_bfloat16* g = gu + (size_t)row * 2 * I;
-  const __nv_bfloat16* u = g + I;
-  for (int i = threadIdx.x; i < I; i += blockDim.x) {
-    float gv = __bfloat162float(g[i]), uv = __bfloat162float(u[i]);
-    if (limit > 0.f) {
-      uv = fminf(fmaxf(uv, -limit), limit);
-      gv = fminf(gv, limit);
+  const T* g = gu + (size_t)row * 2 * I;
+  const b200::GluShape shape = {limit, slope};
+  for (int i = threadIdx.x * 8; i < I; i += blockDim.x * 8) {
+    float gv[8], uv[8];
+    b200::load8(g + i, gv);
+    b200::load8(g + I + i, uv);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      if (slope > 0.f) {
+        gv[j] = b200::glu<sizeof(T) == 2>(gv[j], uv[j], shape);
+        continue;
+      }
+      if (limit > 0.f) {
+        uv[j] = fminf(fmaxf(uv[j], -limit), limit);
+        gv[j] = fminf(gv[j], limit);
+      }
+      gv[j] = __fdividef(gv[j], 1.f + __expf(-gv[j])) * uv[j];
     }
-    act[(size_t)row * I + i] = __float2bfloat16(gv / (1.f + __expf(-gv)) * uv);
+    b200::store8(act + (size_t)row * I + i, gv);
   }
 }
 
@@ -202,14 +227,20 @@ __global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ y, const in
 
 extern "C" {
 
-// score_fn: 0 softmax, 1 sigmoid, 2 sqrt(softplus). idx int32 [T, K], wts fp32 [T, K].
-int b200_moe_route(const float* logits, const float* bias, int T, int E, int K, int score_fn, int norm_topk,
+// score_fn: 0 softmax, 1 sigmoid, 2 sqrt(softplus). logits rows of `ld` floats; idx int32 [T, K], wts fp32 [T, K].
+int b200_moe_route(const float* logits, int ld, const float* bias, int T, int E, int K, int score_fn, int norm_topk,
                    float route_scale, int* idx, float* wts, cudaStream_t stream) {
-  if (T <= 0 || E <= 0 || E > MAX_EXPERTS || K <= 0 || K > MAX_TOPK || K > 32 || K > E) return -6;
+  if (T <= 0 || E <= 0 || E > MAX_EXPERTS || K <= 0 || K > E || ld < E) return -6;
   const int wpb = 4;
-  moe_route_kernel<<<(T + wpb - 1) / wpb, wpb * 32, 0, stream>>>(logits, bias, T, E, K, score_fn, norm_topk, route_scale,
-                                                               idx, wts);
-  return (int)cudaGetLastError();
+  const dim3 grid((T + wpb - 1) / wpb), block(wpb * 32);
+#define B200_ROUTE(J)                                                                                                 \
+  if (E <= 32 * J) {                                                                                                  \
+    moe_route_kernel<J><<<grid, block, 0, stream>>>(logits, ld, bias, T, E, K, score_fn, norm_topk, route_scale, idx, wts); \
+    return (int)cudaGetLastError();                                                                                   \
+  }
+  B200_ROUTE(1) B200_ROUTE(2) B200_ROUTE(4) B200_ROUTE(8) B200_ROUTE(16) B200_ROUTE(32)
+#undef B200_ROUTE
+  return -6;
 }
 
 // Plans the grouped GEMMs of this rank's experts [expert_lo, expert_hi).  All outputs are device buffers:
@@ -219,7 +250,7 @@ int b200_moe_plan(const int* idx, int T, int K, int expert_lo, int expert_hi, in
                   int bn2, int max_work, cudaStream_t stream) {
   const int EL = expert_hi - expert_lo;
   if (T <= 0 || K <= 0 || EL <= 0 || EL > MAX_EXPERTS || max_work <= 0) return -6;
-  moe_plan_kernel<<<1, 1024, 0, stream>>>(idx, T * K, K, expert_lo, expert_hi, offsets, route_row, row_token,
+  moe_plan_kernel<<<EL, 1024, 0, stream>>>(idx, T * K, K, expert_lo, expert_hi, offsets, route_row, row_token,
                                           reinterpret_cast<int4*>(work13), n13, m_tiles13, bn13,
                                           reinterpret_cast<int4*>(work2), n2, m_tiles2, bn2, max_work);
   return (int)cudaGetLastError();
@@ -233,11 +264,17 @@ int b200_moe_gather(const void* x, const int* row_token, const int* offsets, int
   return (int)cudaGetLastError();
 }
 
-int b200_moe_swiglu(const void* gu, const int* offsets, int EL, void* act, int max_rows, int I, float limit,
-                    cudaStream_t stream) {
-  if (max_rows <= 0 || I <= 0) return -6;
-  moe_swiglu_kernel<<<max_rows, 256, 0, stream>>>(reinterpret_cast<const __nv_bfloat16*>(gu), offsets, EL,
-                                                  reinterpret_cast<__nv_bfloat16*>(act), I, limit);
+// slope > 0: the clamped one-plus unit of glu.cuh, else SwiGLU with the optional clamp.  I % 8 == 0.
+int b200_moe_glu(const void* gu, const int* offsets, int EL, void* act, int max_rows, int I, float limit, float slope, int f32,
+                 cudaStream_t stream) {
+  if (max_rows <= 0 || I <= 0 || (I & 7)) return -6;
+  const int threads = I >= 2048 ? 256 : I >= 1024 ? 128 : I >= 512 ? 64 : 32;
+  if (f32)
+    moe_glu_kernel<float><<<max_rows, threads, 0, stream>>>(reinterpret_cast<const float*>(gu), offsets, EL,
+                                                            reinterpret_cast<float*>(act), I, limit, slope);
+  else
+    moe_glu_kernel<__nv_bfloat16><<<max_rows, threads, 0, stream>>>(reinterpret_cast<const __nv_bfloat16*>(gu), offsets, EL,
+                                                                    reinterpret_cast<__nv_bfloat16*>(act), I, limit, slope);
   return (int)cudaGetLastError();
 }
 

@@ -45,15 +45,15 @@ int b200_silu_mul_split(const void* gu, void* xq, float* inv_c, int T, int inter
 int b200_gemm_wdec_grouped(int wfmt, const void* W, const float* scales, const void* X, void* out_bf16, int rows_total,
                            int N, int K, int groups, const void* work_table, const int* num_work, int bn, int* status,
                            cudaStream_t stream);
-int b200_moe_route(const float* logits, const float* bias, int T, int E, int K, int score_fn, int norm_topk,
+int b200_moe_route(const float* logits, int ld, const float* bias, int T, int E, int K, int score_fn, int norm_topk,
                    float route_scale, int* idx, float* wts, cudaStream_t stream);
 int b200_moe_plan(const int* idx, int T, int K, int expert_lo, int expert_hi, int* offsets, int* route_row,
                   int* row_token, void* work13, int* n13, int m_tiles13, int bn13, void* work2, int* n2, int m_tiles2,
                   int bn2, int max_work, cudaStream_t stream);
 int b200_moe_gather(const void* x, const int* row_token, const int* offsets, int EL, void* xs, int max_rows, int H,
                     cudaStream_t stream);
-int b200_moe_swiglu(const void* gu, const int* offsets, int EL, void* act, int max_rows, int I, float limit,
-                    cudaStream_t stream);
+int b200_moe_glu(const void* gu, const int* offsets, int EL, void* act, int max_rows, int I, float limit, float slope, int f32,
+                 cudaStream_t stream);
 int b200_moe_combine(const void* y, const int* route_row, const float* wts, const void* base, void* out, int T, int K,
                      int H, cudaStream_t stream);
 

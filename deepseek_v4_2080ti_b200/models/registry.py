@@ -350,13 +350,14 @@ class CheckpointSpec:
     chat_family: str | None = None
     dtypes: tuple[str, ...] = ("bfloat16",)      # activation dtypes the runtime serves in
     kernel_sources: tuple[str, ...] = ()         # csrc/kernels files it needs (empty: the whole library)
-    tensor_shapes: Callable[[Any], dict[str, tuple[int, ...]]] | None = None     # parsed config.json -> every tensor
+    tensor_shapes: Callable[[Any], dict[str, tuple[int | None, ...]]] | None = None     # parsed config.json -> every tensor
 
     def audit(self, raw_config: Any, have: dict[str, tuple[int, ...]]) -> dict:
         """Checkpoint inventory (name -> shape) against what the configuration asks for."""
         want = self.tensor_shapes(raw_config)
+        fits = lambda h, w: len(h) == len(w) and all(b is None or a == b for a, b in zip(h, w))      # None: any size
         rep = {"missing": sorted(set(want) - set(have)), "unexpected": sorted(set(have) - set(want)),
-               "wrong_shape": sorted(n for n in want if n in have and tuple(have[n]) != tuple(want[n])),
+               "wrong_shape": sorted(n for n in want if n in have and not fits(tuple(have[n]), tuple(want[n]))),
                "expected": len(want), "found": sum(n in have for n in want)}
         rep["ok"] = not (rep["missing"] or rep["unexpected"] or rep["wrong_shape"])
         return rep
@@ -473,3 +474,35 @@ def _zigasun_sources() -> tuple[str, ...]:
 register_checkpoint(CheckpointSpec("zigasun", "Zigasun (differential attention, selective scan, clamped gated feed-forward)",
                                    _zigasun_matches, _zigasun_build, dtypes=("bfloat16", "float32"),
                                    kernel_sources=_zigasun_sources(), tensor_shapes=_zigasun_shapes))
+
+
+def _kemirax_matches(raw) -> bool:
+    from .kemirax import KemiraxConfig
+    return KemiraxConfig.is_kemirax_json(raw)
+
+
+def _kemirax_build(raw, directory, device, rank=0, world=1, dtype=None, max_slots=1, max_context=4096, num_blocks=None,
+                   make_comm=None):
+    from ..formats import safetensors_io
+    from . import kemirax as kx
+    if world != 1:
+        raise ValueError("a Kemirax model runs on one rank")
+    cfg = kx.KemiraxConfig.from_json(raw)
+    w = kx.KemiraxWeights(cfg, safetensors_io.read_checkpoint(directory), device,
+                          _torch_dtype(dtype, ("bfloat16", "float32")))
+    return cfg, kx.KemiraxRuntime(cfg, w, max_slots=max_slots, max_context=max_context, num_blocks=num_blocks)
+
+
+def _kemirax_shapes(raw) -> dict[str, tuple[int | None, ...]]:
+    from .kemirax import KemiraxConfig
+    return KemiraxConfig.from_json(raw).tensor_shapes()
+
+
+def _kemirax_sources() -> tuple[str, ...]:
+    from .kemirax import KERNEL_SOURCES
+    return KERNEL_SOURCES
+
+
+register_checkpoint(CheckpointSpec("kemirax", "Kemirax (latent attention, gated linear attention, side-by-side sublayers, routed experts)",
+                                   _kemirax_matches, _kemirax_build, dtypes=("bfloat16", "float32"),
+                                   kernel_sources=_kemirax_sources(), tensor_shapes=_kemirax_shapes))

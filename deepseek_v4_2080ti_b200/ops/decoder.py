@@ -135,6 +135,61 @@ def residual_norm(x: torch.Tensor, cols: int, eps: float, *, delta: torch.Tensor
     return out
 
 
+@dataclass
+class Routed:
+    """Routed experts' outputs of a batch, not yet summed: rows in expert order, where each (token, choice) went, its expert
+    (numbers from ``experts`` on are identity experts) and its weight."""
+    y: torch.Tensor             # [routes, >= ld]
+    row: torch.Tensor           # int32 [T, top]
+    idx: torch.Tensor           # int32 [T, top]
+    weights: torch.Tensor       # fp32 [T, top]
+    experts: int
+
+
+def parallel_step(x: torch.Tensor | None, cols: int, weight: float, eps: float, *, ld: int, n: int, dtype: torch.dtype,
+                  x_out: torch.Tensor | None = None, ids: torch.Tensor | None = None, table: torch.Tensor | None = None,
+                  mix: torch.Tensor | None = None, gates: torch.Tensor | None = None, gate_b: torch.Tensor | None = None,
+                  h: torch.Tensor | None = None, routed: Routed | None = None, shared: torch.Tensor | None = None,
+                  shared_gate: torch.Tensor | None = None, shift: torch.Tensor | None = None, tail: torch.Tensor | None = None,
+                  seg=None, positions: torch.Tensor | None = None, rows: torch.Tensor | None = None,
+                  norm: bool = True) -> tuple[torch.Tensor | None, torch.Tensor | None]:
+    """Step between layers whose sublayers run side by side (csrc/kernels/parallel_step.cu):
+    ``x + mix sigmoid(gates[:, :ld] + b) + ff sigmoid(gates[:, ld:] + b)`` goes to ``x_out`` (another buffer than ``x``),
+    with ``ff`` the sum of the routed experts, of identity experts (``h``) and of ``shared`` behind its gate (a column of
+    logits).  Returns (RMS norm of it times ``weight``, that norm moved towards the row before it by ``shift``): the second
+    only with ``shift``, which also keeps the sequences' ``tail`` [slots, ld].  ``rows``: only these rows, norm only."""
+    dev = (x if x is not None else ids).device
+    assert x is None or (x.dtype == torch.float32 and x.shape[1] == ld and x.is_contiguous())
+    for t in (mix, h, shared, table):
+        assert t is None or (t.dtype == dtype and t.shape[1] == ld and t.is_contiguous())
+    assert gates is None or (gates.dtype == dtype and gates.stride(1) == 1 and gates.shape[1] >= ld)
+    if ids is not None:
+        _lib.check_indices(ids, 0, table.shape[0], 1)
+    if rows is not None:
+        _lib.check_indices(rows, 0, x.shape[0], 7)
+    if seg is not None and tail is not None:
+        _lib.check_indices(seg.row_slot, 0, tail.shape[0], 4)
+    count = rows.numel() if rows is not None else n
+    out = torch.empty(count, ld, dtype=dtype, device=dev) if norm else None
+    m = torch.empty(n, ld, dtype=dtype, device=dev) if shift is not None else None
+    r = routed
+    rc = _lib.lib().b200_parallel_step(
+        _lib.ptr(x), _lib.ptr(x_out), _lib.ptr(ids), _lib.ptr(table), 0 if table is None else table.shape[0], _lib.ptr(mix),
+        _lib.ptr(gates), 0 if gates is None else gates.stride(0), _lib.ptr(gate_b), _lib.ptr(h), _lib.ptr(r.y if r else None),
+        r.y.stride(0) if r else 0, _lib.ptr(r.row if r else None), _lib.ptr(r.idx if r else None),
+        _lib.ptr(r.weights if r else None), r.idx.shape[1] if r else 0, r.experts if r else 0, _lib.ptr(shared),
+        _lib.ptr(shared_gate), 0 if shared_gate is None else shared_gate.stride(0), _f(weight), _f(eps), _lib.ptr(out), _lib.ptr(m),
+        _lib.ptr(shift), _lib.ptr(tail), _lib.ptr(seg.row_first if m is not None else None),
+        _lib.ptr(seg.row_slot if m is not None else None), _lib.ptr(positions), _lib.ptr(rows), count, ld, cols,
+        int(dtype == torch.float32), _lib.stream())
+    _lib.check(rc, "parallel_step")
+    if m is not None and seg.max_length > 1:       # single rows replaced their tail in the kernel
+        rc = _lib.lib().b200_shift_tails(_lib.ptr(out), _lib.ptr(tail), _lib.ptr(seg.first), _lib.ptr(seg.length),
+                                         _lib.ptr(seg.slot), seg.first.numel(), ld, int(dtype == torch.float32), _lib.stream())
+        _lib.check(rc, "shift_tails")
+    return out, m
+
+
 def bias_xielu(z: torch.Tensor, bias: torch.Tensor | None, ap: float, an: float) -> torch.Tensor:
     """xIELU(z + bias) with the positive-side and negative-side coefficients."""
     out = torch.empty_like(z)

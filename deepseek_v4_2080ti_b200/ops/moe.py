@@ -12,6 +12,7 @@ from . import _lib, gemm
 from .gemm import WF_BF16, WF_FP8_B128
 
 WF_FP4 = 2
+WF_F32 = 100                   # not a GEMM format: plain fp32 matrices on the CUDA cores (gemm_f32.cu)
 SCORE_FN = {"softmax": 0, "sigmoid": 1, "sqrtsoftplus": 2}
 
 
@@ -62,6 +63,11 @@ class ExpertWeights:
         return ExpertWeights(gguf_gemm.WF[gguf_gemm.GGMLType(ggml_type)], w, lut, n, k, len(raws))
 
     @staticmethod
+    def from_f32(ws: list[torch.Tensor]) -> "ExpertWeights":
+        n, k = ws[0].shape
+        return ExpertWeights(WF_F32, torch.cat([x.float() for x in ws]).contiguous(), None, n, k, len(ws))
+
+    @staticmethod
     def from_bf16(ws: list[torch.Tensor]) -> "ExpertWeights":
         n, k = ws[0].shape
         assert n % 128 == 0, "bf16 expert matrices need a multiple of 128 output features"
@@ -70,14 +76,74 @@ class ExpertWeights:
 
 def route(logits: torch.Tensor, bias: torch.Tensor | None, k: int, score_func: str, norm_topk: bool,
           route_scale: float) -> tuple[torch.Tensor, torch.Tensor]:
-    """fp32 logits [T, E] -> (idx int32 [T, k], weights fp32 [T, k])."""
+    """fp32 logits [T, E] (row stride allowed) -> (idx int32 [T, k], weights fp32 [T, k])."""
     t, e = logits.shape
+    assert logits.dtype == torch.float32 and logits.stride(1) == 1
     idx = torch.empty(t, k, dtype=torch.int32, device=logits.device)
     wts = torch.empty(t, k, dtype=torch.float32, device=logits.device)
-    rc = _lib.lib().b200_moe_route(_lib.ptr(logits), _lib.ptr(bias), t, e, k, SCORE_FN[score_func], int(norm_topk),
-                                   ctypes.c_float(route_scale), _lib.ptr(idx), _lib.ptr(wts), _lib.stream())
+    rc = _lib.lib().b200_moe_route(_lib.ptr(logits), logits.stride(0), _lib.ptr(bias), t, e, k, SCORE_FN[score_func],
+                                   int(norm_topk), ctypes.c_float(route_scale), _lib.ptr(idx), _lib.ptr(wts), _lib.stream())
     _lib.check(rc, "moe_route")
     return idx, wts
+
+
+F32_TILE = 64                   # rows and features of a tile of the fp32 grouped GEMM
+
+
+def experts_rows(x: torch.Tensor, idx: torch.Tensor, w13: ExpertWeights, w2: ExpertWeights, expert_lo: int = 0,
+                 limit: float = 0.0, slope: float = 0.0) -> tuple[torch.Tensor, torch.Tensor]:
+    """Outputs of the experts [expert_lo, expert_lo + E) held here for their tokens, in expert order (y [T k, w2.n]), and the
+    row of every route (int32 [T, k], -1: not held here).  x [T, H] bf16 (fp32 for fp32 weights); w13: [E] x [2I, H] (gate
+    rows then up rows); w2: [E] x [H', I].  The unit is SwiGLU with the optional clamp ``limit``, or with ``slope`` the
+    clamped one-plus form of csrc/kernels/glu.cuh."""
+    L = _lib.lib()
+    t, h = x.shape
+    k = idx.shape[1]
+    el = w13.experts
+    inter = w13.n // 2
+    r = t * k
+    dev = x.device
+    f32 = w13.wfmt == WF_F32
+    assert x.dtype == (torch.float32 if f32 else torch.bfloat16) and x.is_contiguous() and h == w13.k
+    bn = F32_TILE if f32 else gemm._bn(min(256, max(16, (r + el - 1) // el)))      # token tile sized for the average rows per expert
+    if 3 <= w13.wfmt < WF_F32:
+        bn = min(bn, int(L.b200_gguf_max_bn(w13.wfmt)), int(L.b200_gguf_max_bn(w2.wfmt)))
+    bm = F32_TILE if f32 else 128
+    mt13, mt2 = (w13.n + bm - 1) // bm, (w2.n + bm - 1) // bm
+    max_work = (mt13 + mt2) * ((r + bn - 1) // bn + el)
+    i32 = lambda *s: torch.empty(*s, dtype=torch.int32, device=dev)
+    offsets, route_row, row_token = i32(el + 1), i32(t, k), i32(r)
+    work13, work2 = i32(max_work, 4), i32(max_work, 4)
+    n13, n2 = i32(1), i32(1)
+    s = _lib.stream()
+    rc = L.b200_moe_plan(_lib.ptr(idx), t, k, expert_lo, expert_lo + el, _lib.ptr(offsets), _lib.ptr(route_row),
+                         _lib.ptr(row_token), _lib.ptr(work13), _lib.ptr(n13), mt13, bn, _lib.ptr(work2), _lib.ptr(n2),
+                         mt2, bn, max_work, s)
+    _lib.check(rc, "moe_plan")
+    # rows past the real count are never read: sized for the worst case (every route local)
+    xs = torch.empty(r, h, dtype=x.dtype, device=dev)
+    # 16-bit columns: an fp32 row counts twice
+    rc = L.b200_moe_gather(_lib.ptr(x), _lib.ptr(row_token), _lib.ptr(offsets), el, _lib.ptr(xs), r, 2 * h if f32 else h, s)
+    _lib.check(rc, "moe_gather")
+
+    def product(w: ExpertWeights, a: torch.Tensor, work, num, what: str) -> torch.Tensor:
+        out = torch.empty(r, w.n, dtype=x.dtype, device=dev)
+        if f32:
+            rc = L.b200_gemm_f32_grouped(_lib.ptr(a), _lib.ptr(w.weight), _lib.ptr(out), w.n, w.k, _lib.ptr(work), _lib.ptr(num),
+                                         max_work, s)
+        else:
+            grouped = L.b200_gemm_wdec_grouped if w.wfmt < 3 else L.b200_gemm_wdec_gguf_grouped
+            rc = grouped(w.wfmt, _lib.ptr(w.weight), _lib.ptr(w.scales), _lib.ptr(a), _lib.ptr(out), r, w.n, w.k, el,
+                         _lib.ptr(work), _lib.ptr(num), bn, _lib.ptr(_lib.status_word(dev)), s)
+        _lib.check(rc, what)
+        return out
+
+    gu = product(w13, xs, work13, n13, "grouped gemm w13")
+    act = torch.empty(r, inter, dtype=x.dtype, device=dev)
+    rc = L.b200_moe_glu(_lib.ptr(gu), _lib.ptr(offsets), el, _lib.ptr(act), r, inter, ctypes.c_float(limit), ctypes.c_float(slope),
+                        int(f32), s)
+    _lib.check(rc, "moe_glu")
+    return product(w2, act, work2, n2, "grouped gemm w2"), route_row
 
 
 def experts_forward(x: torch.Tensor, idx: torch.Tensor, wts: torch.Tensor, w13: ExpertWeights, w2: ExpertWeights,
@@ -89,54 +155,16 @@ def experts_forward(x: torch.Tensor, idx: torch.Tensor, wts: torch.Tensor, w13: 
     With ``comm`` (a peer-memory communicator of an expert-parallel group) the weighted combine, the sum over ranks
     and the residual add run as one kernel over NVLink (``PeerComm.moe_combine``): every rank gets
     ``residual + sum_ranks(base_r + local routes)``."""
-    L0 = _lib.lib()
     t, h = x.shape
     k = idx.shape[1]
-    el = w13.experts
-    inter = w13.n // 2
-    r = t * k
-    dev = x.device
-    bn = gemm._bn(min(256, max(16, (r + el - 1) // el)))      # token tile sized for the average rows per expert
-    if w13.wfmt >= 3:
-        bn = min(bn, int(L0.b200_gguf_max_bn(w13.wfmt)), int(L0.b200_gguf_max_bn(w2.wfmt)))
-    mt13, mt2 = (w13.n + 127) // 128, (w2.n + 127) // 128
-    max_work = (mt13 + mt2) * ((r + bn - 1) // bn + el)
-    i32 = lambda *s: torch.empty(*s, dtype=torch.int32, device=dev)
-    offsets, route_row, row_token = i32(el + 1), i32(r), i32(r)
-    work13, work2 = i32(max_work, 4), i32(max_work, 4)
-    n13, n2 = i32(1), i32(1)
-    L = _lib.lib()
-    s = _lib.stream()
-    rc = L.b200_moe_plan(_lib.ptr(idx), t, k, expert_lo, expert_lo + el, _lib.ptr(offsets), _lib.ptr(route_row),
-                         _lib.ptr(row_token), _lib.ptr(work13), _lib.ptr(n13), mt13, bn, _lib.ptr(work2), _lib.ptr(n2),
-                         mt2, bn, max_work, s)
-    _lib.check(rc, "moe_plan")
-    # rows past the real count are never read: sized for the worst case (every route local)
-    xs = torch.empty(r, h, dtype=torch.bfloat16, device=dev)
-    rc = L.b200_moe_gather(_lib.ptr(x), _lib.ptr(row_token), _lib.ptr(offsets), el, _lib.ptr(xs), r, h, s)
-    _lib.check(rc, "moe_gather")
-    st = _lib.status_word(dev)
-    gu = torch.empty(r, w13.n, dtype=torch.bfloat16, device=dev)
-    rc = L.b200_gemm_wdec_grouped(w13.wfmt, _lib.ptr(w13.weight), _lib.ptr(w13.scales), _lib.ptr(xs), _lib.ptr(gu), r,
-                                  w13.n, w13.k, el, _lib.ptr(work13), _lib.ptr(n13), bn, _lib.ptr(st), s) if w13.wfmt < 3 else \
-        L.b200_gemm_wdec_gguf_grouped(w13.wfmt, _lib.ptr(w13.weight), _lib.ptr(w13.scales), _lib.ptr(xs), _lib.ptr(gu), r,
-                                      w13.n, w13.k, el, _lib.ptr(work13), _lib.ptr(n13), bn, _lib.ptr(st), s)
-    _lib.check(rc, "grouped gemm w13")
-    act = torch.empty(r, inter, dtype=torch.bfloat16, device=dev)
-    rc = L.b200_moe_swiglu(_lib.ptr(gu), _lib.ptr(offsets), el, _lib.ptr(act), r, inter, ctypes.c_float(swiglu_limit), s)
-    _lib.check(rc, "moe_swiglu")
-    y = torch.empty(r, h, dtype=torch.bfloat16, device=dev)
-    rc = L.b200_gemm_wdec_grouped(w2.wfmt, _lib.ptr(w2.weight), _lib.ptr(w2.scales), _lib.ptr(act), _lib.ptr(y), r, w2.n,
-                                  w2.k, el, _lib.ptr(work2), _lib.ptr(n2), bn, _lib.ptr(st), s) if w2.wfmt < 3 else \
-        L.b200_gemm_wdec_gguf_grouped(w2.wfmt, _lib.ptr(w2.weight), _lib.ptr(w2.scales), _lib.ptr(act), _lib.ptr(y), r,
-                                      w2.n, w2.k, el, _lib.ptr(work2), _lib.ptr(n2), bn, _lib.ptr(st), s)
-    _lib.check(rc, "grouped gemm w2")
+    y, route_row = experts_rows(x, idx, w13, w2, expert_lo, swiglu_limit)
     if comm is not None and getattr(comm, "world", 1) > 1:
         return comm.moe_combine(y, route_row, wts, base, residual, t, k, h, comm_mode)
     if residual is not None:
         base = residual if base is None else base + residual
-    out = torch.empty(t, h, dtype=torch.bfloat16, device=dev)
-    rc = L.b200_moe_combine(_lib.ptr(y), _lib.ptr(route_row), _lib.ptr(wts), _lib.ptr(base), _lib.ptr(out), t, k, h, s)
+    out = torch.empty(t, h, dtype=torch.bfloat16, device=x.device)
+    rc = _lib.lib().b200_moe_combine(_lib.ptr(y), _lib.ptr(route_row), _lib.ptr(wts), _lib.ptr(base), _lib.ptr(out), t, k, h,
+                                     _lib.stream())
     _lib.check(rc, "moe_combine")
     return out
 
