@@ -19,6 +19,7 @@ import torch
 
 from ..ops import decoder, gla, latent, moe
 from ..ops.decoder import Projection, Routed, pad16
+from ..ops.gemm import PackedLinear
 from ..ops.gla import GatedLinear
 from ..ops.latent import LatentAttention
 from ..ops.mixattn import yarn_freqs
@@ -28,7 +29,8 @@ from .paged import PagedRuntime
 ARCH = "Kemirax"
 UNIT_SLOPE = 1.702
 # kernel sources the runtime launches (a partial build compiles only these)
-KERNEL_SOURCES = ("parallel_step.cu", "latent_prep.cu", "attn_latent_rows.cu", "head_linear.cu", "gated_linear.cu", "moe.cu",
+KERNEL_SOURCES = ("parallel_step.cu", "latent_prep.cu", "attn_latent_rows.cu", "attn_heads_prefill.cu",
+                  "head_linear.cu", "gated_linear.cu", "moe.cu",
                   "bias_act.cu", "gemm_f32.cu", "gemm_wdec.cu", "gemm_bf16_2cta.cu", "elementwise.cu", "sampling.cu", "bounds.cu")
 
 
@@ -252,6 +254,7 @@ class LatentWeights:
     uq: Projection                    # rows per head [d | r]
     uk: torch.Tensor                  # [heads, c, d]: query -> latent
     uv: torch.Tensor                  # [heads, v, c]
+    ukv: Any                          # PackedLinear with rows per head [d | v]: latent -> key, value (bf16)
     o: Projection
 
 
@@ -363,10 +366,11 @@ class KemiraxWeights:
         uk = _cat_rows([(_heads(t["uk"], a.heads, ((a.dim, d),)).t(), c)])                         # [c, heads * d]
         uv = torch.zeros(a.heads * v, c, dtype=t["uv"].dtype, device=t["uv"].device)
         uv[:, :a.kv_rank] = _heads(t["uv"], a.heads, ((a.vdim, v),))
+        both = torch.cat([uk.t().reshape(a.heads, d, c), uv.view(a.heads, v, c)], 1).reshape(-1, c)
+        ukv = PackedLinear.from_bf16(both.to(self.device)) if self.dtype == torch.bfloat16 else None
         return LatentWeights(m, self._proj(_cat_rows(parts), tile_n=True),
                              self._proj(_heads(t["uq"], a.heads, ((a.dim, d), (a.rot_dim, r))), tile_n=True),
-                             dev(uk.view(c, a.heads, d).permute(1, 0, 2)), dev(uv.view(a.heads, v, c)),
-                             self._proj(_heads(t["o"].t().contiguous(), a.heads, ((a.vdim, v),)).t()))
+                             dev(uk.view(c, a.heads, d).permute(1, 0, 2)), dev(uv.view(a.heads, v, c)), ukv, self._proj(_heads(t["o"].t().contiguous(), a.heads, ((a.vdim, v),)).t()))
 
     def _linear(self, s: LinearSpec, t: dict[str, torch.Tensor]) -> LinearWeights:
         rank = t["a1"].shape[0]
@@ -415,6 +419,7 @@ class KemiraxWeights:
             n += L.gates.nbytes()
             n += sum(p.nbytes() for p in ((m.down, m.uq, m.o) if isinstance(m, LatentWeights) else (m.proj, m.o)))
             n += sum(size(x) for x in ((m.uk, m.uv) if isinstance(m, LatentWeights) else (m.m.w2,)))
+            n += m.ukv.nbytes() if isinstance(m, LatentWeights) and m.ukv is not None else 0
             if L.ff:
                 n += sum(p.nbytes() for p in (L.ff.router, L.ff.up, L.ff.down) if p is not None)
                 n += size(L.ff.w13.weight) + size(L.ff.w2.weight)
@@ -424,6 +429,7 @@ class KemiraxWeights:
 # ---------------------------------------------------------------------------------------------- runtime
 class KemiraxRuntime(PagedRuntime):
     exposes_logits = True
+    tile_min_rows = latent.TILE_MIN_ROWS
 
     def __init__(self, cfg: KemiraxConfig, weights: KemiraxWeights, max_slots: int = 1, max_context: int = 4096,
                  block_size: int = 64, num_blocks: int | None = None, comm=None):
@@ -431,7 +437,10 @@ class KemiraxRuntime(PagedRuntime):
         if self.comm.world != 1:
             raise ValueError("a Kemirax model runs on one rank")
         self.cfg, self.w = cfg, weights
-        self.tile_min_rows = 1 << 30
+        tiles = weights.dtype == torch.bfloat16 and all(latent.tiles_supported(lw.mix.m) for lw in weights.layers
+                                                        if isinstance(lw.mix, LatentWeights))
+        if not tiles:
+            self.tile_min_rows = 1 << 30             # every row on the row kernel (fp32, or heads wider than the tile kernel takes)
         self.cache: list[torch.Tensor | None] = []
         self.state: list[torch.Tensor | None] = []
         self.tails: list[torch.Tensor] = []          # the previous token's norm output, one per layer
@@ -453,14 +462,26 @@ class KemiraxRuntime(PagedRuntime):
         m, cache, t = lw.m, self.cache[i], y.shape[0]
         q = lw.uq(latent.prep(lw.down(y), m, positions, kv_slots, cache))
         out = torch.empty(t, lw.o.k, dtype=y.dtype, device=y.device)
-        qa = torch.empty(t, m.heads, m.cache_width, dtype=y.dtype, device=y.device)
-        latent.rotate_heads(q, m, positions, qa, m.c)
-        latent.head_linear(q, q.stride(0), m.head_width, lw.uk, qa, qa.stride(0), qa.stride(1), t)
-        if meta["mode"] == "decode":
-            o = latent.attend_rows(qa, m, cache, meta["block_table"], positions, meta["max_kv_len"])
-        else:
-            o = latent.attend_rows(qa, m, cache, self.block_table, positions, meta["max_kv_len"], seq=meta["row_seq"])
-        latent.head_linear(o, o.stride(0), m.c, lw.uv, out, out.stride(0), m.v, t)
+        n = meta["tile_rows"] if meta["mode"] == "mixed" else 0
+        if n:                                        # portions of prompts: keys and values are expanded from the latents
+            src = self.cfg.layers[i].mixer.kv_from
+            src = i if src is None else src
+            contexts = meta.setdefault("contexts", {})
+            if src not in contexts:                  # layers that share a cache share its contiguous copy
+                contexts[src] = latent.gather(cache, m, self.block_table, meta["tile_seq"], meta["kv_len"], meta["kv_start"], meta["kv_total"])
+            latent.rotate_heads(q[:n], m, positions)
+            latent.attend_tiles(q[:n], m, *contexts[src], lw.ukv, meta["q_start"], meta["q_len"], meta["kv_len"], meta["kv_start"],
+                                meta["max_q_len"], out[:n])
+        if n < t:                                    # single rows: queries are brought to the latents
+            qr = q[n:]
+            qa = torch.empty(t - n, m.heads, m.cache_width, dtype=y.dtype, device=y.device)
+            latent.rotate_heads(qr, m, positions[n:], qa, m.c)
+            latent.head_linear(qr, qr.stride(0), m.head_width, lw.uk, qa, qa.stride(0), qa.stride(1), t - n)
+            if meta["mode"] == "decode":
+                o = latent.attend_rows(qa, m, cache, meta["block_table"], positions, meta["max_kv_len"])
+            else:
+                o = latent.attend_rows(qa, m, cache, self.block_table, positions[n:], meta["max_kv_len"], seq=meta["row_seq"][n:])
+            latent.head_linear(o, o.stride(0), m.c, lw.uv, out[n:], out.stride(0), m.v, t - n)
         return lw.o(out)
 
     def _linear(self, i: int, lw: LinearWeights, y: torch.Tensor, positions, meta) -> torch.Tensor:

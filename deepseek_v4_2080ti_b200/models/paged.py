@@ -129,8 +129,8 @@ class PagedRuntime(PagedSequences):
 
     ``meta["mode"]``: ``"decode"`` - one row per sequence, static buffers (``block_table`` row i belongs to row i,
     ``kv_len``, ``max_kv_len``); ``"mixed"`` - the first ``tile_rows`` rows are portions of several sequences
-    (``tile_table``, ``q_start``, ``q_len``, ``kv_len``, ``max_q_len``; ``tile_seq`` / ``tile_pos_rows`` per row), the
-    rest single rows (``row_seq``, ``max_kv_len``).  In both modes ``segments`` says which neighbouring rows form one
+    (``q_start``, ``q_len``, ``kv_len``, ``max_q_len``, ``tile_seq``; ``kv_start`` / ``kv_total``: where their contexts begin
+    when they are laid out one after the other), the rest single rows (``row_seq``, ``max_kv_len``).  In both modes ``segments`` says which neighbouring rows form one
     sequence's portion and which state slot it has, for mixers that carry a recurrent state.
 
     Recurrent state is held per request slot in tensors from ``slot_state``; a slot's content is meaningless until its
@@ -207,18 +207,23 @@ class PagedRuntime(PagedSequences):
         seq = cat([torch.full((lens[i],), sts[i].slot, dtype=torch.int32) for i in order])
         want = torch.tensor([first[i] + w for i, e in enumerate(entries) for w in e[2]], dtype=torch.int32)
         start = cat([torch.full((lens[i],), first[i], dtype=torch.int32) for i in order])
-        desc = torch.tensor([[first[i], lens[i], sts[i].length + lens[i], sts[i].slot] for i in order], dtype=torch.int32).t().reshape(-1)
+        kv_start, kv_total = [], 0                       # the contexts of the tile entries, laid out one after the other
+        for i in order:
+            kv_start.append(kv_total)
+            kv_total += sts[i].length + lens[i] if i in tiles else 0
+        desc = torch.tensor([[first[i], lens[i], sts[i].length + lens[i], sts[i].slot, k] for i, k in zip(order, kv_start)],
+                            dtype=torch.int32).t().reshape(-1)
         # one upload: [ids | positions | cache rows | table rows | entry starts | entry descriptors | wanted rows]
         up = cat([tok, pos, rows, seq, start, desc, want])
         up = up.pin_memory().to(dev, non_blocking=True) if dev.type == "cuda" else up
         ids, pos_d, slots_d, seq_d, start_d = (up[k * n_rows:(k + 1) * n_rows] for k in range(5))
-        e_first, e_len, e_kv, e_slot = up[5 * n_rows:5 * n_rows + desc.numel()].view(4, -1)
+        e_first, e_len, e_kv, e_slot, e_start = up[5 * n_rows:5 * n_rows + desc.numel()].view(5, -1)
         meta = {"mode": "mixed", "tile_rows": tile_rows, "row_seq": seq_d, "max_q_len": max([lens[i] for i in tiles], default=0),
                 "max_kv_len": max(sts[i].length + lens[i] for i in range(len(entries))),
                 "segments": Segments(start_d, seq_d, e_first, e_len, e_slot, max(lens), min(lens))}
         if tiles:
             n = len(tiles)
-            meta.update(q_start=e_first[:n], q_len=e_len[:n], kv_len=e_kv[:n], tile_seq=e_slot[:n])
+            meta.update(q_start=e_first[:n], q_len=e_len[:n], kv_len=e_kv[:n], tile_seq=e_slot[:n], kv_start=e_start[:n], kv_total=kv_total)
         # a pass has to run even when no logits are asked for: it fills the cache
         wanted = up[5 * n_rows + desc.numel():]
         logits = self._forward(ids, pos_d, slots_d, meta, wanted)

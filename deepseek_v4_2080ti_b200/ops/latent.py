@@ -1,5 +1,6 @@
 """Front-ends of latent attention over a paged cache of one row per token, [latent | rotated key part], shared by all heads:
-prologue (csrc/kernels/latent_prep.cu), single rows in the absorbed form (attn_latent_rows.cu, head_linear.cu).
+prologue (csrc/kernels/latent_prep.cu), single rows in the absorbed form (attn_latent_rows.cu, head_linear.cu), prompt tiles on
+the tensor cores over keys and values expanded from the latents (attn_heads_prefill.cu).
 
 All of it exists for bf16 and for fp32 activations; the tensors' dtype decides.  Widths are padded to multiples of 16 with
 zero columns.
@@ -16,6 +17,10 @@ from . import _lib
 
 _f = ctypes.c_float
 NUM_SMS = 148
+# Entries with fewer new rows than this take the row kernel: expanding a context of C-wide latents costs each of its rows
+# 2 C (d + v) products per head, once per entry, and saves 2 (2 C + r) - 2 (d + r + v) per head and query row, on faster units.
+TILE_MIN_ROWS = 32
+EXPANDED_LIMIT = 1 << 29                # values of expanded keys and values held at a time; more heads go in several rounds
 
 
 @dataclass
@@ -132,4 +137,43 @@ def attend_rows(q: torch.Tensor, m: LatentAttention, cache: torch.Tensor, block_
             _lib.ptr(None if seq is None else seq[lo:hi]), _lib.ptr(positions[lo:hi]), _lib.ptr(ws), hi - lo, block_table.shape[1], bs,
             m.heads, m.c, m.cache_width, int(splits), _f(m.scale), f32, _lib.stream())
         _lib.check(rc, "attn_latent_rows", 2 if splits > 1 else 1)
+    return out
+
+
+def tiles_supported(m: LatentAttention) -> bool:
+    return bool(_lib.lib().b200_attn_heads_prefill_supported(m.heads, m.d, m.r, m.v))
+
+
+def gather(cache: torch.Tensor, m: LatentAttention, block_table, seq, kv_len, kv_start, total: int) -> tuple[torch.Tensor, torch.Tensor]:
+    """Contexts of several sequences, one after the other: latents [rows, c] and rotated key parts [rows, 64-column slabs].
+    Rows are rounded up to 256 with zero rows, so that the expansion tiles evenly."""
+    nb, bs, _ = cache.shape
+    _lib.check_indices(block_table, 0, nb, 3)
+    rows, key_ld = (total + 255) // 256 * 256, max(64, (m.r + 63) // 64 * 64)
+    lat = torch.empty(rows, m.c, dtype=cache.dtype, device=cache.device)
+    key = torch.empty(rows, key_ld, dtype=cache.dtype, device=cache.device)
+    rc = _lib.lib().b200_latent_gather(_lib.ptr(cache), _lib.ptr(block_table), _lib.ptr(seq), _lib.ptr(kv_len), _lib.ptr(kv_start),
+                                       kv_len.numel(), block_table.shape[1], bs, m.c, m.r, key_ld, _lib.ptr(lat), _lib.ptr(key), rows,
+                                       _lib.stream())
+    _lib.check(rc, "latent_gather")
+    return lat, key
+
+
+def attend_tiles(q: torch.Tensor, m: LatentAttention, lat: torch.Tensor, key: torch.Tensor, w_kv, q_start, q_len, kv_len, kv_start,
+                 max_q_len: int, out: torch.Tensor) -> torch.Tensor:
+    """Rows of several sequences' portions.  q [rows, >= heads (d + r)], rotated; ``lat`` / ``key`` from ``gather``; ``w_kv``
+    (``PackedLinear``): rows per head [d | v] that expand a latent; ``out`` [rows, >= heads v] in place."""
+    from . import gemm
+    rows, per = lat.shape[0], m.d + m.v
+    group = max(1, min(m.heads, EXPANDED_LIMIT // (rows * per)))
+    L = _lib.lib()
+    for h0 in range(0, m.heads, group):
+        n = min(group, m.heads - h0)
+        part = gemm.PackedLinear(w_kv.wfmt, w_kv.weight[h0 * per:(h0 + n) * per], None, n * per, m.c)
+        kv = gemm.linear(lat, part)
+        rc = L.b200_attn_heads_prefill(
+            _lib.ptr(q), q.stride(0), _lib.ptr(kv), _lib.ptr(key), key.shape[1], _lib.ptr(out), out.stride(0), _lib.ptr(q_start),
+            _lib.ptr(q_len), _lib.ptr(kv_len), _lib.ptr(kv_start), q_len.numel(), int(max_q_len), q.shape[0], rows, h0, n, m.d, m.r, m.v,
+            _f(m.scale), _lib.ptr(_lib.status_word(out.device)), _lib.stream())
+        _lib.check(rc, "attn_heads_prefill")
     return out
