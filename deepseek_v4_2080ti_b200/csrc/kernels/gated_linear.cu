@@ -7,7 +7,7 @@
 //
 //   gla_decay    log alpha from the low-rank logits z = W2 a + b, fp32
 //   gla_scan     one token after the other; the state's columns are independent, so a block takes 32 of them, a lane per
-//                column, and the warps share the rows.  fp32 results, and bf16 portions too short for chunk_scan
+//                column, and the warps share the rows.  For fp32, and for bf16 portions too short for gla_chunk.cu
 //   gla_step     one token of many sequences: a block per head and sequence reads, updates and writes the state once and
 //                finishes the row (norm, gate) itself
 //   gla_finish   per head o / rms(o) * weight * silu(g)
@@ -60,6 +60,7 @@ struct GlaParams {
   float* o;                  // [rows, H * V]
   const int *first, *length, *slot, *positions;
   int ld, H, D, V;
+  int max_len;               // longer entries are left alone (0: none)
   float scale;
 };
 
@@ -80,6 +81,7 @@ __global__ void __launch_bounds__(SW * 32) gla_scan_kernel(GlaParams<T> p) {
   const int h = blockIdx.y, e = blockIdx.z, c = blockIdx.x * 32 + lane;
   pdl_grid_wait();
   const int t0 = p.first[e], n = p.length[e];
+  if (p.max_len && n > p.max_len) return;
   float* st = p.state + ((size_t)p.slot[e] * p.H + h) * D * V;
   const bool fresh = p.positions[t0] == 0;
   float s[RD];
@@ -130,6 +132,107 @@ __global__ void __launch_bounds__(SW * 32) gla_scan_kernel(GlaParams<T> p) {
   }
 }
 
+template <typename T>
+struct GlaStepParams {
+  GlaParams<T> b;
+  const T *a, *gate;         // decay latent and gate columns of the projection
+  const T* w2;               // [H * D, rank]
+  const float *bias, *norm_w;
+  T* out;                    // [rows, ldo]
+  int rank, vdim, ldo;
+  float inv_tau, eps;
+};
+
+constexpr int STEP_THREADS = 256;
+
+// grid (H, entries): one row per entry.  A thread owns four value columns and every (threads / (V / 4))-th channel.
+template <typename T>
+__global__ void __launch_bounds__(STEP_THREADS) gla_step_kernel(GlaStepParams<T> p) {
+  extern __shared__ float sm[];
+  __shared__ float red[32];
+  pdl_grid_trigger();
+  const int D = p.b.D, V = p.b.V, nq = V / 4, groups = STEP_THREADS / nq, tid = threadIdx.x;
+  float* sq = sm;                          // [D] query, key, decay
+  float* sk = sq + D;
+  float* sg = sk + D;
+  float* sa = sg + D;                      // [rank]
+  float* so = sa + p.rank;                 // [groups][V]
+  const int h = blockIdx.x, e = blockIdx.y;
+  pdl_grid_wait();
+  const size_t row = p.b.first[e];
+  float* st = p.b.state + ((size_t)p.b.slot[e] * p.b.H + h) * D * V;
+  const bool fresh = p.b.positions[row] == 0;
+  for (int i = tid; i < p.rank; i += STEP_THREADS) sa[i] = (float)p.a[row * p.b.ld + i];
+  for (int d = tid; d < D; d += STEP_THREADS) {
+    sq[d] = (float)p.b.q[row * p.b.ld + h * D + d] * p.b.scale;
+    sk[d] = (float)p.b.k[row * p.b.ld + h * D + d];
+  }
+  const int col = tid % nq, grp = tid / nq;
+  const bool on = grp < groups;
+  float v[4] = {0.f, 0.f, 0.f, 0.f};
+  if (on)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) v[j] = (float)p.b.v[row * p.b.ld + h * V + col * 4 + j];
+  __syncthreads();
+  for (int d = tid; d < D; d += STEP_THREADS) {
+    float z = p.bias[h * D + d];
+    for (int k = 0; k < p.rank; k += 8) {
+      float w[8];
+      load8(p.w2 + (size_t)(h * D + d) * p.rank + k, w);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) z = fmaf(w[j], sa[k + j], z);
+    }
+    sg[d] = expf(log_sigmoid(z) * p.inv_tau);
+  }
+  __syncthreads();
+  float acc[4] = {0.f, 0.f, 0.f, 0.f};
+  if (on) {
+    constexpr int U = 8;                   // channels in flight
+    for (int d0 = grp; d0 < D; d0 += groups * U) {
+      float4 s[U];
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int d = d0 + u * groups;
+        s[u] = !fresh && d < D ? *reinterpret_cast<const float4*>(st + (size_t)d * V + col * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int d = d0 + u * groups;
+        if (d < D) {
+          const float a = sg[d], k = sk[d], q = sq[d];
+          s[u].x = fmaf(a, s[u].x, k * v[0]); s[u].y = fmaf(a, s[u].y, k * v[1]);
+          s[u].z = fmaf(a, s[u].z, k * v[2]); s[u].w = fmaf(a, s[u].w, k * v[3]);
+          acc[0] = fmaf(s[u].x, q, acc[0]); acc[1] = fmaf(s[u].y, q, acc[1]);
+          acc[2] = fmaf(s[u].z, q, acc[2]); acc[3] = fmaf(s[u].w, q, acc[3]);
+          *reinterpret_cast<float4*>(st + (size_t)d * V + col * 4) = s[u];
+        }
+      }
+    }
+    *reinterpret_cast<float4*>(so + grp * V + col * 4) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+  }
+  __syncthreads();
+  float o[4], ss = 0.f;                    // V <= 4 * STEP_THREADS
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const int c = tid + j * STEP_THREADS;
+    o[j] = 0.f;
+    if (c < V)
+      for (int w = 0; w < groups; ++w) o[j] += so[w * V + c];
+    ss += o[j] * o[j];
+  }
+  const float inv = 1.f / sqrtf(block_sum_all(ss, red) / (float)p.vdim + p.eps);
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const int c = tid + j * STEP_THREADS;
+    if (c < V) {
+      const float g = (float)p.gate[row * p.b.ld + h * V + c];
+      p.out[row * p.ldo + h * V + c] = (T)(o[j] * inv * p.norm_w[c] * (g / (1.f + expf(-g))));
+    }
+  }
+  if (h == 0)
+    for (int c = p.b.H * V + tid; c < p.ldo; c += STEP_THREADS) p.out[row * p.ldo + c] = (T)0.f;
+}
+
 // grid rows: out[row, h * V + c] = o / rms over the head's vdim values * weight * silu(gate).
 template <typename T>
 __global__ void gla_finish_kernel(const float* __restrict__ o, const T* __restrict__ gate, int ld_gate, const float* __restrict__ w,
@@ -174,9 +277,10 @@ int launch_scan(const GlaParams<T>& p, int entries, cudaStream_t stream) {
 
 template <typename T>
 int run_scan(const void* q, const void* k, const void* v, int ld, const float* la, float* state, float* o, const int* first,
-             const int* length, const int* slot, const int* positions, int entries, int H, int D, int V, float scale,
+             const int* length, const int* slot, const int* positions, int entries, int max_len, int H, int D, int V, float scale,
              cudaStream_t stream) {
   GlaParams<T> p;
+  p.max_len = max_len;
   p.q = reinterpret_cast<const T*>(q); p.k = reinterpret_cast<const T*>(k); p.v = reinterpret_cast<const T*>(v); p.la = la;
   p.state = state; p.o = o; p.first = first; p.length = length; p.slot = slot; p.positions = positions; p.ld = ld; p.H = H; p.D = D;
   p.V = V; p.scale = scale;
@@ -206,6 +310,20 @@ int run_finish(const float* o, const void* gate, int ld_gate, const float* w, vo
                          reinterpret_cast<T*>(out), ldo, H, V, vdim, eps);
 }
 
+template <typename T>
+int run_step(const void* q, const void* k, const void* v, const void* gate, const void* a, int ld, const void* w2, const float* bias,
+             float inv_tau, int rank, float* state, const int* first, const int* slot, const int* positions, int entries, int H, int D,
+             int V, int vdim, float scale, const float* norm_w, float eps, void* out, int ldo, cudaStream_t stream) {
+  GlaStepParams<T> p;
+  p.b.q = reinterpret_cast<const T*>(q); p.b.k = reinterpret_cast<const T*>(k); p.b.v = reinterpret_cast<const T*>(v); p.b.la = nullptr;
+  p.b.state = state; p.b.o = nullptr; p.b.first = first; p.b.length = nullptr; p.b.slot = slot; p.b.positions = positions; p.b.ld = ld;
+  p.b.H = H; p.b.D = D; p.b.V = V; p.b.max_len = 0; p.b.scale = scale;
+  p.a = reinterpret_cast<const T*>(a); p.gate = reinterpret_cast<const T*>(gate); p.w2 = reinterpret_cast<const T*>(w2); p.bias = bias;
+  p.norm_w = norm_w; p.out = reinterpret_cast<T*>(out); p.rank = rank; p.vdim = vdim; p.ldo = ldo; p.inv_tau = inv_tau; p.eps = eps;
+  const size_t smem = (size_t)(3 * D + rank + STEP_THREADS / (V / 4) * V) * 4;
+  return (int)launch_pdl(gla_step_kernel<T>, dim3(H, entries), dim3(STEP_THREADS), smem, stream, p);
+}
+
 }  // namespace
 
 // a rows `ld` apart, w2 [channels, rank] in the activations' type, la fp32 [rows, channels]; rank % 8 == 0, at most 1024.
@@ -216,13 +334,13 @@ extern "C" int b200_gla_decay(const void* a, int ld, const void* w2, const float
              : run_decay<__nv_bfloat16>(a, ld, w2, bias, inv_tau, la, rows, channels, rank, stream);
 }
 
-// D at most 512; state [slots, H, D, V] fp32 in place; o fp32 [rows, H * V].
+// D at most 512; entries of at most max_len rows (0: all); state [slots, H, D, V] fp32 in place; o fp32 [rows, H * V].
 extern "C" int b200_gla_scan(const void* q, const void* k, const void* v, int ld, const float* la, float* state, float* o,
-                             const int* first, const int* length, const int* slot, const int* positions, int entries, int H, int D,
-                             int V, float scale, int f32, cudaStream_t stream) {
+                             const int* first, const int* length, const int* slot, const int* positions, int entries, int max_len,
+                             int H, int D, int V, float scale, int f32, cudaStream_t stream) {
   if (entries <= 0 || entries > 65535 || H <= 0 || H > 65535 || D <= 0 || V <= 0) return -6;
-  return f32 ? run_scan<float>(q, k, v, ld, la, state, o, first, length, slot, positions, entries, H, D, V, scale, stream)
-             : run_scan<__nv_bfloat16>(q, k, v, ld, la, state, o, first, length, slot, positions, entries, H, D, V, scale, stream);
+  return f32 ? run_scan<float>(q, k, v, ld, la, state, o, first, length, slot, positions, entries, max_len, H, D, V, scale, stream)
+             : run_scan<__nv_bfloat16>(q, k, v, ld, la, state, o, first, length, slot, positions, entries, max_len, H, D, V, scale, stream);
 }
 
 // V % 16 == 0; out [rows, ldo] (columns behind the heads are zeroed).
@@ -231,4 +349,18 @@ extern "C" int b200_gla_finish(const float* o, const void* gate, int ld_gate, co
   if (rows <= 0 || H <= 0 || V <= 0 || (V & 15) || vdim <= 0 || vdim > V || ldo < H * V || (ldo & 7) || (ld_gate & 7)) return -6;
   return f32 ? run_finish<float>(o, gate, ld_gate, w, out, ldo, rows, H, V, vdim, eps, stream)
              : run_finish<__nv_bfloat16>(o, gate, ld_gate, w, out, ldo, rows, H, V, vdim, eps, stream);
+}
+
+// One row per entry (row first[e]): decay, state update, norm and gate in one launch.  V % 16 == 0, at most 1024; D at most 2048.
+extern "C" int b200_gla_step(const void* q, const void* k, const void* v, const void* gate, const void* a, int ld, const void* w2,
+                             const float* bias, float inv_tau, int rank, float* state, const int* first, const int* slot,
+                             const int* positions, int entries, int H, int D, int V, int vdim, float scale, const float* norm_w,
+                             float eps, void* out, int ldo, int f32, cudaStream_t stream) {
+  if (entries <= 0 || entries > 65535 || H <= 0 || D <= 0 || D > 2048 || V <= 0 || (V & 15) || V > 4 * STEP_THREADS || vdim <= 0 ||
+      vdim > V || rank <= 0 || (rank & 7) || rank > 1024 || ldo < H * V)
+    return -6;
+  return f32 ? run_step<float>(q, k, v, gate, a, ld, w2, bias, inv_tau, rank, state, first, slot, positions, entries, H, D, V, vdim, scale,
+                               norm_w, eps, out, ldo, stream)
+             : run_step<__nv_bfloat16>(q, k, v, gate, a, ld, w2, bias, inv_tau, rank, state, first, slot, positions, entries, H, D, V,
+                                       vdim, scale, norm_w, eps, out, ldo, stream);
 }

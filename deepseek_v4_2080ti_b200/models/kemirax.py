@@ -30,7 +30,7 @@ ARCH = "Kemirax"
 UNIT_SLOPE = 1.702
 # kernel sources the runtime launches (a partial build compiles only these)
 KERNEL_SOURCES = ("parallel_step.cu", "latent_prep.cu", "attn_latent_rows.cu", "attn_heads_prefill.cu",
-                  "head_linear.cu", "gated_linear.cu", "moe.cu",
+                  "head_linear.cu", "gated_linear.cu", "gla_chunk.cu", "moe.cu",
                   "bias_act.cu", "gemm_f32.cu", "gemm_wdec.cu", "gemm_bf16_2cta.cu", "elementwise.cu", "sampling.cu", "bounds.cu")
 
 

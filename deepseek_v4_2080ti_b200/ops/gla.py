@@ -1,5 +1,6 @@
-"""Front-ends of gated linear attention (csrc/kernels/gated_linear.cu): decay per key channel from low-rank logits, recurrence
-over a batch of rows of several sequences (``ops.scan.Segments``), per-head norm and gate."""
+"""Front-ends of gated linear attention (csrc/kernels/gated_linear.cu, gla_chunk.cu): decay per key channel from low-rank
+logits, recurrence over a batch of rows of several sequences (``ops.scan.Segments``), per-head norm and gate.  Batches of
+single rows are one launch; bf16 portions run in chunks on the tensor cores, fp32 and very short portions token by token."""
 from __future__ import annotations
 
 import ctypes
@@ -10,6 +11,8 @@ import torch
 from . import _lib
 
 _f = ctypes.c_float
+CHUNK_MIN_ROWS = 16             # bf16 portions with fewer rows run token by token
+STEP_MAX_V = 1024               # widest value head of the single-row kernel
 
 
 @dataclass
@@ -44,15 +47,35 @@ def recurrence(proj: torch.Tensor, m: GatedLinear, state: torch.Tensor, seg, pos
     L, dev = _lib.lib(), proj.device
     q, k, v, g, a = (proj[:, o:] for o in m.offsets)
     ld = proj.stride(0)
+    scale, entries = m.dim ** -0.5, seg.first.numel()
+    if seg.max_length == 1 and m.v <= STEP_MAX_V:
+        out = torch.empty(t, ldo, dtype=proj.dtype, device=dev)
+        rc = L.b200_gla_step(_lib.ptr(q), _lib.ptr(k), _lib.ptr(v), _lib.ptr(g), _lib.ptr(a), ld, _lib.ptr(m.w2), _lib.ptr(m.b2),
+                             _f(1.0 / m.tau), m.rank, _lib.ptr(state), _lib.ptr(seg.first), _lib.ptr(seg.slot), _lib.ptr(positions),
+                             entries, m.heads, m.d, m.v, m.vdim, _f(scale), _lib.ptr(m.norm_w), _f(m.eps), _lib.ptr(out), ldo, f32,
+                             _lib.stream())
+        _lib.check(rc, "gla_step")
+        return out
     la = torch.empty(t, m.heads * m.d, dtype=torch.float32, device=dev)
     rc = L.b200_gla_decay(_lib.ptr(a), ld, _lib.ptr(m.w2), _lib.ptr(m.b2), _f(1.0 / m.tau), _lib.ptr(la), t, m.heads * m.d, m.rank, f32,
                           _lib.stream())
     _lib.check(rc, "gla_decay")
     o = torch.empty(t, m.heads * m.v, dtype=torch.float32, device=dev)
-    rc = L.b200_gla_scan(_lib.ptr(q), _lib.ptr(k), _lib.ptr(v), ld, _lib.ptr(la), _lib.ptr(state), _lib.ptr(o), _lib.ptr(seg.first),
-                         _lib.ptr(seg.length), _lib.ptr(seg.slot), _lib.ptr(positions), seg.first.numel(), m.heads, m.d, m.v,
-                         _f(m.dim ** -0.5), f32, _lib.stream())
-    _lib.check(rc, "gla_scan")
+    rows = 0 if f32 else L.b200_gla_chunk_rows(m.d)
+    chunked = rows > 0 and seg.max_length >= CHUNK_MIN_ROWS
+    if chunked:
+        chunks = t // rows + entries
+        ws = torch.empty(chunks * m.heads * L.b200_gla_chunk_ws(m.d), dtype=torch.bfloat16, device=dev)
+        end = torch.empty(chunks * m.heads * L.b200_gla_chunk_end(m.d), dtype=torch.float32, device=dev)
+        rc = L.b200_gla_chunk(_lib.ptr(q), _lib.ptr(k), _lib.ptr(v), ld, _lib.ptr(la), _lib.ptr(state), _lib.ptr(o),
+                              _lib.ptr(seg.first), _lib.ptr(seg.length), _lib.ptr(seg.slot), _lib.ptr(positions), entries,
+                              CHUNK_MIN_ROWS, chunks, _lib.ptr(ws), _lib.ptr(end), m.heads, m.d, m.v, _f(scale), _lib.stream())
+        _lib.check(rc, "gla_chunk", 2)
+    if not chunked or seg.min_length < CHUNK_MIN_ROWS:
+        rc = L.b200_gla_scan(_lib.ptr(q), _lib.ptr(k), _lib.ptr(v), ld, _lib.ptr(la), _lib.ptr(state), _lib.ptr(o),
+                             _lib.ptr(seg.first), _lib.ptr(seg.length), _lib.ptr(seg.slot), _lib.ptr(positions), entries,
+                             CHUNK_MIN_ROWS - 1 if chunked else 0, m.heads, m.d, m.v, _f(scale), f32, _lib.stream())
+        _lib.check(rc, "gla_scan")
     out = torch.empty(t, ldo, dtype=proj.dtype, device=dev)
     rc = L.b200_gla_finish(_lib.ptr(o), _lib.ptr(g), ld, _lib.ptr(m.norm_w), _lib.ptr(out), ldo, t, m.heads, m.v, m.vdim, _f(m.eps), f32,
                            _lib.stream())
