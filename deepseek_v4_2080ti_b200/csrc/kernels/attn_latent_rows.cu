@@ -11,7 +11,7 @@
 // probabilities travel through shared memory, and each sums its 16-column blocks of the latent.
 // fp32 and wider latents (latent_rows_kernel): CUDA cores, four heads per block, a warp per key for the dot products.
 //
-// Slices leave (unnormalised sum, maximum, sum of weights) per head; latent_rows_merge_kernel combines them.
+// Slices leave their unnormalised sums, then (maximum, sum of weights) per head; latent_rows_merge_kernel combines them.
 #include <cuda_bf16.h>
 #include <stdint.h>
 #include "launch.h"
@@ -30,7 +30,8 @@ struct Rows {
   const int* positions;       // [rows]
   int max_blocks, bs, H, C, D, splits;      // C: latent columns, D: columns of a cache row
   float scale_log2;
-  float* partial;             // [rows, H, splits, C + 2], or null: one slice
+  float* partial;             // [rows, H, splits, C], or null: one slice
+  float* stats;               // [rows, H, splits, 2] maximum, sum
 };
 
 __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
@@ -205,7 +206,8 @@ latent_rows_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
   for (int hf = 0; hf < 2; ++hf) {
     const int h = h0 + 16 * mt + g + 8 * hf;
     if (h >= p.H) continue;
-    float* part = p.partial ? p.partial + (((size_t)b * p.H + h) * p.splits + split) * (C + 2) : nullptr;
+    const size_t at = ((size_t)b * p.H + h) * p.splits + split;
+    float* part = p.partial ? p.partial + at * C : nullptr;
     const float inv = part ? 1.f : 1.f / l_run[hf];
     __nv_bfloat16* dst = out + ((size_t)b * p.H + h) * C;
 #pragma unroll
@@ -218,7 +220,7 @@ latent_rows_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
         if (part) *reinterpret_cast<float2*>(part + col) = make_float2(v0, v1);
         else *reinterpret_cast<uint32_t*>(dst + col) = pack_bf16(v0, v1);
       }
-    if (part && warp == 0 && tig == 0) { part[C] = m_run[hf]; part[C + 1] = l_run[hf]; }
+    if (part && warp == 0 && tig == 0) { p.stats[2 * at] = m_run[hf]; p.stats[2 * at + 1] = l_run[hf]; }
   }
 }
 
@@ -311,7 +313,8 @@ __global__ void __launch_bounds__(ST) latent_rows_kernel(const T* __restrict__ q
   for (int h = 0; h < SH; ++h) {
     if (h0 + h >= p.H) continue;
     const float m = sml[h], l = sml[SH + h];
-    float* part = p.partial ? p.partial + (((size_t)b * p.H + h0 + h) * p.splits + split) * (C + 2) : nullptr;
+    const size_t at = ((size_t)b * p.H + h0 + h) * p.splits + split;
+    float* part = p.partial ? p.partial + at * C : nullptr;
 #pragma unroll
     for (int i = 0; i < CI; ++i) {
       const int c = tid + i * ST;
@@ -319,38 +322,57 @@ __global__ void __launch_bounds__(ST) latent_rows_kernel(const T* __restrict__ q
       if (part) part[c] = acc[h][i];
       else out[((size_t)b * p.H + h0 + h) * C + c] = (T)(acc[h][i] / l);
     }
-    if (part && tid == 0) { part[C] = m; part[C + 1] = l; }
+    if (part && tid == 0) { p.stats[2 * at] = m; p.stats[2 * at + 1] = l; }
   }
 }
 
-// grid (H, rows): combine the slices of one head and row.
+constexpr int MW = 8;         // warps of the merge kernel: each takes every eighth slice
+
+// grid (H, rows, ceil(C / 128)): combine the slices of one head and row, 128 columns per block.
 template <typename T>
-__global__ void latent_rows_merge_kernel(const float* __restrict__ partial, T* __restrict__ out, int H, int C, int splits) {
-  extern __shared__ float s_w[];                           // [splits]
+__global__ void __launch_bounds__(MW * 32)
+latent_rows_merge_kernel(const float* __restrict__ partial, const float* __restrict__ stats, T* __restrict__ out, int H, int C, int splits) {
+  extern __shared__ float s_w[];                           // [splits] weights, then [MW][128]
   pdl_grid_trigger();
   pdl_grid_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const size_t hr = (size_t)blockIdx.y * H + blockIdx.x;
-  const float* base = partial + hr * splits * (C + 2);
-  if (threadIdx.x < 32) {
-    const int lane = threadIdx.x;
+  const float* st = stats + hr * splits * 2;
+  float* s_o = s_w + (splits + 3) / 4 * 4;
+  if (warp == 0) {
     float M = -INFINITY, L = 0.f;
-    for (int s = lane; s < splits; s += 32) M = fmaxf(M, base[(size_t)s * (C + 2) + C]);
+    for (int s = lane; s < splits; s += 32) M = fmaxf(M, st[2 * s]);
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, o));
     for (int s = lane; s < splits; s += 32) {
-      const float m = base[(size_t)s * (C + 2) + C], w = m == -INFINITY ? 0.f : exp2f(m - M);    // an empty slice has no maximum
-      L += w * base[(size_t)s * (C + 2) + C + 1];
+      const float m = st[2 * s], w = m == -INFINITY ? 0.f : exp2f(m - M);            // an empty slice has no maximum
+      L += w * st[2 * s + 1];
       s_w[s] = w;
     }
     L = warp_sum_all(L);
+    __syncwarp();
     for (int s = lane; s < splits; s += 32) s_w[s] /= L;
   }
   __syncthreads();
-  for (int c = threadIdx.x; c < C; c += blockDim.x) {
-    float v = 0.f;
+  const int c = blockIdx.z * 128 + lane * 4;
+  float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (c < C) {
+    const float* base = partial + hr * splits * C + c;
 #pragma unroll 4
-    for (int s = 0; s < splits; ++s) v = s_w[s] != 0.f ? fmaf(s_w[s], base[(size_t)s * (C + 2) + c], v) : v;
-    out[hr * C + c] = (T)v;
+    for (int s = warp; s < splits; s += MW) {
+      const float4 f = *reinterpret_cast<const float4*>(base + (size_t)s * C);       // an empty slice left zeros
+      const float w = s_w[s];
+      v.x = fmaf(w, f.x, v.x); v.y = fmaf(w, f.y, v.y); v.z = fmaf(w, f.z, v.z); v.w = fmaf(w, f.w, v.w);
+    }
+  }
+  *reinterpret_cast<float4*>(s_o + warp * 128 + lane * 4) = v;
+  __syncthreads();
+  const int col = blockIdx.z * 128 + threadIdx.x;
+  if (threadIdx.x < 128 && col < C) {
+    float a = 0.f;
+#pragma unroll
+    for (int w = 0; w < MW; ++w) a += s_o[w * 128 + threadIdx.x];
+    out[hr * C + col] = (T)a;
   }
 }
 
@@ -402,8 +424,9 @@ int run_simt(const void* q, const void* cache, void* out, const Rows& p, int row
 
 template <typename T>
 int merge(const Rows& p, void* out, int rows, cudaStream_t stream) {
-  return (int)launch_pdl(latent_rows_merge_kernel<T>, dim3(p.H, rows), dim3(p.C <= 128 ? 128 : 256), (size_t)p.splits * 4, stream,
-                         (const float*)p.partial, reinterpret_cast<T*>(out), p.H, p.C, p.splits);
+  return (int)launch_pdl(latent_rows_merge_kernel<T>, dim3(p.H, rows, (p.C + 127) / 128), dim3(MW * 32),
+                         (size_t)((p.splits + 3) / 4 * 4 + MW * 128) * 4, stream, (const float*)p.partial, (const float*)p.stats,
+                         reinterpret_cast<T*>(out), p.H, p.C, p.splits);
 }
 
 }  // namespace
@@ -417,7 +440,7 @@ extern "C" int b200_attn_latent_rows_heads(int H, int C, int D, int rows, int f3
 }
 
 // q [rows, H, D], cache [pages * bs, D], out [rows, H, C]; C, D multiples of 16, C <= 2048; partial: fp32
-// [rows, H, splits, C + 2] when splits > 1.
+// [rows * H * splits * (C + 2)] when splits > 1.
 extern "C" int b200_attn_latent_rows(const void* q, const void* cache, void* out, const int* block_table, const int* seq,
                                      const int* positions, float* partial, int rows, int max_blocks, int bs, int H, int C, int D,
                                      int splits, float scale, int f32, cudaStream_t stream) {
@@ -426,6 +449,7 @@ extern "C" int b200_attn_latent_rows(const void* q, const void* cache, void* out
   Rows p;
   p.block_table = block_table; p.seq = seq; p.positions = positions; p.max_blocks = max_blocks; p.bs = bs; p.H = H; p.C = C; p.D = D;
   p.splits = splits; p.scale_log2 = scale * 1.4426950408889634f; p.partial = splits > 1 ? partial : nullptr;
+  p.stats = partial + (size_t)rows * H * splits * C;
   int rc;
   const int heads = b200_attn_latent_rows_heads(H, C, D, rows, f32);
   if (f32) rc = run_simt<float>(q, cache, out, p, rows, stream);

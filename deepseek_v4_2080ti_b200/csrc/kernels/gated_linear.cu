@@ -27,7 +27,7 @@ constexpr int DR = 8;           // rows per block of gla_decay
 template <typename T>
 __global__ void gla_decay_kernel(const T* __restrict__ a, int ld, const T* __restrict__ w2, const float* __restrict__ bias,
                                  float inv_tau, float* __restrict__ la, int rows, int channels, int rank) {
-  extern __shared__ float sa[];            // [DR][rank]
+  extern __shared__ __align__(16) float sa[];   // [DR][rank]
   pdl_grid_trigger();
   pdl_grid_wait();
   const int r0 = blockIdx.x * DR, n = min(DR, rows - r0);
@@ -42,9 +42,12 @@ __global__ void gla_decay_kernel(const T* __restrict__ a, int ld, const T* __res
       float w[8];
       load8(w2 + (size_t)c * rank + k, w);
 #pragma unroll
-      for (int r = 0; r < DR; ++r)
+      for (int r = 0; r < DR; ++r) {
+        float a8[8];
+        load8(sa + r * rank + k, a8);
 #pragma unroll
-        for (int j = 0; j < 8; ++j) z[r] = fmaf(w[j], sa[r * rank + k + j], z[r]);
+        for (int j = 0; j < 8; ++j) z[r] = fmaf(w[j], a8[j], z[r]);
+      }
     }
 #pragma unroll
     for (int r = 0; r < DR; ++r)
@@ -233,33 +236,58 @@ __global__ void __launch_bounds__(STEP_THREADS) gla_step_kernel(GlaStepParams<T>
     for (int c = p.b.H * V + tid; c < p.ldo; c += STEP_THREADS) p.out[row * p.ldo + c] = (T)0.f;
 }
 
-// grid rows: out[row, h * V + c] = o / rms over the head's vdim values * weight * silu(gate).
-template <typename T>
+__device__ __forceinline__ float silu_of(float z, __nv_bfloat16) { return __fdividef(z, 1.f + __expf(-z)); }
+__device__ __forceinline__ float silu_of(float z, float) { return z / (1.f + expf(-z)); }
+
+// A warp per (row, head): out[row, h * V + c] = o / rms over the head's vdim values * weight * silu(gate).
+template <typename T, int KEEP>             // KEEP: 256-column rounds held in registers
 __global__ void gla_finish_kernel(const float* __restrict__ o, const T* __restrict__ gate, int ld_gate, const float* __restrict__ w,
-                                  T* __restrict__ out, int ldo, int H, int V, int vdim, float eps) {
+                                  T* __restrict__ out, int ldo, int rows, int H, int V, int vdim, float eps) {
   pdl_grid_trigger();
   pdl_grid_wait();
-  const size_t row = blockIdx.x;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int h = warp; h < H; h += blockDim.x >> 5) {
-    const float* src = o + (row * H + h) * V;
-    float ss = 0.f;
-    for (int c = lane * 4; c < V; c += 128) {
-      const float4 f = *reinterpret_cast<const float4*>(src + c);
-      ss += f.x * f.x + f.y * f.y + f.z * f.z + f.w * f.w;               // padded columns are zero
-    }
-    const float inv = 1.f / sqrtf(warp_sum_all(ss) / (float)vdim + eps);
-    for (int c = lane * 8; c < V; c += 256) {
-      float f[8], g[8], ww[8];
-      load8(src + c, f);
-      load8(gate + row * ld_gate + h * V + c, g);
-      load8(w + c, ww);
+  const int lane = threadIdx.x & 31;
+  const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const size_t row = item / H;
+  const int h = (int)(item - (long long)row * H);
+  if (row >= (size_t)rows) return;
+  const float* src = o + item * V;
+  const T* gsrc = gate + row * ld_gate + h * V;
+  float f[KEEP][8], g[KEEP][8], ss = 0.f;
 #pragma unroll
-      for (int j = 0; j < 8; ++j) f[j] = f[j] * inv * ww[j] * (g[j] / (1.f + expf(-g[j])));
-      store8(out + row * ldo + h * V + c, f);
+  for (int i = 0; i < KEEP; ++i) {
+    const int c = i * 256 + lane * 8;
+    if (c < V) {
+      load8(src + c, f[i]);
+      load8(gsrc + c, g[i]);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss += f[i][j] * f[i][j];               // padded columns are zero
     }
   }
-  for (int c = H * V + threadIdx.x; c < ldo; c += blockDim.x) out[row * ldo + c] = (T)0.f;
+  for (int c = KEEP * 256 + lane * 8; c < V; c += 256) {
+    float t[8];
+    load8(src + c, t);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss += t[j] * t[j];
+  }
+  const float inv = 1.f / sqrtf(warp_sum_all(ss) / (float)vdim + eps);
+  auto finish = [&](int c, float (&v)[8], const float (&gv)[8]) {
+    float ww[8];
+    load8(w + c, ww);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = v[j] * inv * ww[j] * silu_of(gv[j], T());
+    store8(out + row * ldo + h * V + c, v);
+  };
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i)
+    if (i * 256 + lane * 8 < V) finish(i * 256 + lane * 8, f[i], g[i]);
+  for (int c = KEEP * 256 + lane * 8; c < V; c += 256) {
+    float v[8], gv[8];
+    load8(src + c, v);
+    load8(gsrc + c, gv);
+    finish(c, v, gv);
+  }
+  if (h == H - 1)
+    for (int c = H * V + lane; c < ldo; c += 32) out[row * ldo + c] = (T)0.f;
 }
 
 template <typename T, int RD>
@@ -305,9 +333,12 @@ int run_decay(const void* a, int ld, const void* w2, const float* bias, float in
 template <typename T>
 int run_finish(const float* o, const void* gate, int ld_gate, const float* w, void* out, int ldo, int rows, int H, int V, int vdim,
                float eps, cudaStream_t stream) {
-  const int warps = H < 8 ? H : 8;
-  return (int)launch_pdl(gla_finish_kernel<T>, dim3(rows), dim3(warps * 32), 0, stream, o, reinterpret_cast<const T*>(gate), ld_gate, w,
-                         reinterpret_cast<T*>(out), ldo, H, V, vdim, eps);
+  const long long items = (long long)rows * H;
+  const dim3 grid((unsigned)((items + 7) / 8)), block(256);
+  auto gp = reinterpret_cast<const T*>(gate);
+  auto op = reinterpret_cast<T*>(out);
+  if (V <= 256) return (int)launch_pdl(gla_finish_kernel<T, 1>, grid, block, 0, stream, o, gp, ld_gate, w, op, ldo, rows, H, V, vdim, eps);
+  return (int)launch_pdl(gla_finish_kernel<T, 2>, grid, block, 0, stream, o, gp, ld_gate, w, op, ldo, rows, H, V, vdim, eps);
 }
 
 template <typename T>

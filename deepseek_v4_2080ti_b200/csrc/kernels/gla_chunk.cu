@@ -10,8 +10,9 @@
 // Hardware-Efficient Training").
 //
 //   gla_chunk_prep   one block per chunk and head: decayed q and k, A, e^{b_end} -> workspace
-//   gla_chunk_scan   one warp per 16 value columns walks the chunks.  It keeps S^T of its columns in registers: the
-//                    accumulator fragments of S^T are the operand fragments of q S, so the state never leaves them
+//   gla_chunk_scan   four or eight warps per 16 value columns walk the chunks.  Each keeps its share of the channels of
+//                    S^T in registers and updates it; for q S, of which each takes 16 rows and 8 columns (or 16), the
+//                    shares are exchanged through shared memory once per chunk
 //
 // Decayed operands, A and the state enter the products as two bf16 terms (16 significant bits); sums are fp32.
 #include <cuda_bf16.h>
@@ -82,9 +83,11 @@ __device__ __forceinline__ int chunks_of(const ChunkParams& p, int e, int CL) {
 template <int DT, int CL>
 constexpr size_t ws_elems() { return (size_t)4 * CL * DT + 2 * CL * CL; }
 
-// grid (chunks, H), 128 threads.
+constexpr int PT = 256;
+
+// grid (chunks, H).  Warps 0 .. CL / 16 - 1 take the diagonal blocks of A, the next ones the blocks to the left.
 template <int DT, int CL>
-__global__ void __launch_bounds__(128) gla_chunk_prep_kernel(ChunkParams p) {
+__global__ void __launch_bounds__(PT) gla_chunk_prep_kernel(ChunkParams p) {
   constexpr int LB = DT + 4, LQ = DT + 8, X = DT / 32;
   extern __shared__ __align__(16) uint8_t smem[];
   float* sb = reinterpret_cast<float*>(smem);                       // [CL][LB] summed log2 decays
@@ -104,7 +107,7 @@ __global__ void __launch_bounds__(128) gla_chunk_prep_kernel(ChunkParams p) {
   const size_t at = (size_t)blockIdx.x * p.H + h;
   __nv_bfloat16* ws = p.ws + at * ws_elems<DT, CL>();
   const uint4 zero = make_uint4(0, 0, 0, 0);
-  for (int i = tid; i < CL * (DT / 8); i += 128) {
+  for (int i = tid; i < CL * (DT / 8); i += PT) {
     const int t = i / (DT / 8), d = i % (DT / 8) * 8;
     const bool ok = t < n && d < p.D;                               // D is a multiple of 16
     const size_t row = (size_t)(t0 + t);
@@ -119,7 +122,7 @@ __global__ void __launch_bounds__(128) gla_chunk_prep_kernel(ChunkParams p) {
     }
   }
   __syncthreads();
-  for (int d = tid; d < DT; d += 128) {
+  for (int d = tid; d < DT; d += PT) {
     float acc = 0.f;
     for (int t = 0; t < CL; t += 16) {
       float f[16];
@@ -132,7 +135,7 @@ __global__ void __launch_bounds__(128) gla_chunk_prep_kernel(ChunkParams p) {
   }
   __syncthreads();
   // decayed queries and keys
-  for (int i = tid; i < CL * (DT / 8); i += 128) {
+  for (int i = tid; i < CL * (DT / 8); i += PT) {
     const int t = i / (DT / 8), d = i % (DT / 8) * 8;
     uint4 hi[2], lo[2];
     uint32_t* H[2] = {reinterpret_cast<uint32_t*>(&hi[0]), reinterpret_cast<uint32_t*>(&hi[1])};
@@ -152,36 +155,38 @@ __global__ void __launch_bounds__(128) gla_chunk_prep_kernel(ChunkParams p) {
       *reinterpret_cast<uint4*>(ws + (size_t)(2 * u + 1) * CL * DT + t * DT + d) = lo[u];
     }
   }
-  if (warp >= CL / 16) return;
   __nv_bfloat16 *a_hi = ws + (size_t)4 * CL * DT, *a_lo = a_hi + CL * CL;
-  const int i0 = warp * 16;
+  const int i0 = warp % (CL / 16) * 16;
   // diagonal block: a lane owns channels lane, lane + 32, ...
+  if (warp < CL / 16) {
 #pragma unroll 1
-  for (int t = 0; t < 16; ++t) {
-    float q[X], b[X], mine = 0.f;
+    for (int t = 0; t < 16; ++t) {
+      float q[X], b[X], mine = 0.f;
 #pragma unroll
-    for (int x = 0; x < X; ++x) {
-      q[x] = __bfloat162float(sq[(i0 + t) * LQ + lane + 32 * x]) * p.scale;
-      b[x] = sb[(i0 + t) * LB + lane + 32 * x];
-    }
+      for (int x = 0; x < X; ++x) {
+        q[x] = __bfloat162float(sq[(i0 + t) * LQ + lane + 32 * x]) * p.scale;
+        b[x] = sb[(i0 + t) * LB + lane + 32 * x];
+      }
 #pragma unroll 4
-    for (int s = 0; s <= t; ++s) {
-      float a = 0.f;
+      for (int s = 0; s <= t; ++s) {
+        float a = 0.f;
 #pragma unroll
-      for (int x = 0; x < X; ++x)
-        a = fmaf(q[x] * __bfloat162float(sk[(i0 + s) * LQ + lane + 32 * x]), pow2(b[x] - sb[(i0 + s) * LB + lane + 32 * x]), a);
+        for (int x = 0; x < X; ++x)
+          a = fmaf(q[x] * __bfloat162float(sk[(i0 + s) * LQ + lane + 32 * x]), pow2(b[x] - sb[(i0 + s) * LB + lane + 32 * x]), a);
 #pragma unroll
-      for (int o = 16; o > 0; o >>= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
-      if (lane == s) mine = a;
+        for (int o = 16; o > 0; o >>= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
+        if (lane == s) mine = a;
+      }
+      if (lane < 16) {
+        const __nv_bfloat16 hi = __float2bfloat16(mine);
+        a_hi[(i0 + t) * CL + i0 + lane] = hi;
+        a_lo[(i0 + t) * CL + i0 + lane] = __float2bfloat16(mine - __bfloat162float(hi));
+      }
     }
-    if (lane < 16) {
-      const __nv_bfloat16 hi = __float2bfloat16(mine);
-      a_hi[(i0 + t) * CL + i0 + lane] = hi;
-      a_lo[(i0 + t) * CL + i0 + lane] = __float2bfloat16(mine - __bfloat162float(hi));
-    }
+    return;
   }
   // blocks to the left, 8 columns at a time, against the last row before this block
-  if (i0 == 0) return;
+  if (i0 == 0 || warp >= CL / 8) return;
   constexpr int NT = (CL / 16 - 1) * 2;
   float acc[NT][4];
 #pragma unroll
@@ -237,15 +242,23 @@ template <int DT, int CL>
 __host__ __device__ constexpr size_t stage_bytes(int VB) {
   return ((size_t)4 * CL * (DT + 8) + 2 * CL * (CL + 8) + CL * (VB + 8)) * 2 + DT * 4;
 }
-
-// grid (ceil(V / (16 warps)), H, entries); a warp owns 16 value columns.
 template <int DT, int CL>
-__global__ void __launch_bounds__(128) gla_chunk_scan_kernel(ChunkParams p) {
-  constexpr int LQ = DT + 8, LA = CL + 8, MT = CL / 16;
+constexpr size_t scan_smem(int VB) { return 2 * stage_bytes<DT, CL>(VB) + (size_t)2 * VB * (DT + 8) * 2; }
+
+template <int DT>
+constexpr int SUBS = DT >= 128 ? 8 : 4;                 // warps per 16 value columns
+
+// grid (ceil(V / VB), H, entries), SUBS VB / 16 warps: SUBS of them own value columns 16 i .. 16 i + 15.
+template <int DT, int CL>
+__global__ void __launch_bounds__(512) gla_chunk_scan_kernel(ChunkParams p) {
+  constexpr int LQ = DT + 8, LA = CL + 8, MT = CL / 16, W = SUBS<DT>, ND = DT / W, NS = ND / 8, NJ = W == 8 ? 1 : 2;
+  // channels, fragments of S^T and 8-column tiles of the output of a warp
   extern __shared__ __align__(16) uint8_t smem[];
-  const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tig = lane & 3;
-  const int VB = nthr / 2, LV = VB + 8, h = blockIdx.y, e = blockIdx.z, v0 = blockIdx.x * VB;
+  const int tid = threadIdx.x, nthr = blockDim.x, lane = tid & 31, g = lane >> 2, tig = lane & 3;
+  const int vg = tid / (32 * W), sub = (tid >> 5) % W;
+  const int VB = nthr / (2 * W), LV = VB + 8, h = blockIdx.y, e = blockIdx.z, v0 = blockIdx.x * VB;
   const size_t stage = stage_bytes<DT, CL>(VB);
+  __nv_bfloat16* ss = reinterpret_cast<__nv_bfloat16*>(smem + 2 * stage) + (size_t)vg * 2 * 16 * LQ;     // [hi, lo][16][LQ]
   pdl_grid_trigger();
   pdl_grid_wait();
   const int chunks = chunks_of(p, e, CL);
@@ -278,112 +291,127 @@ __global__ void __launch_bounds__(128) gla_chunk_scan_kernel(ChunkParams p) {
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   fetch(0, 0);
-  const int vw = v0 + warp * 16;
+  const int vw = v0 + vg * 16, d_own = sub * ND;
   const bool live = vw < p.V;
   float* st = p.state + ((size_t)p.slot[e] * p.H + h) * p.D * p.V;
   const bool fresh = p.positions[r0] == 0;
-  float S[DT / 8][4];                                   // S^T: value columns g, g + 8; channels 8 i + 2 tig, + 1
+  float S[NS][4];                                       // S^T: value columns g, g + 8; channels d_own + 8 i + 2 tig, + 1
 #pragma unroll
-  for (int i = 0; i < DT / 8; ++i)
+  for (int i = 0; i < NS; ++i)
 #pragma unroll
     for (int x = 0; x < 4; ++x) {
-      const int d = i * 8 + 2 * tig + (x & 1), v = vw + g + 8 * (x >> 1);
+      const int d = d_own + i * 8 + 2 * tig + (x & 1), v = vw + g + 8 * (x >> 1);
       S[i][x] = live && !fresh && d < p.D ? st[(size_t)d * p.V + v] : 0.f;
     }
-  const int row16 = lane & 15, col8 = (lane >> 4) * 8;                       // non-transposed 16 x 16 tiles
-  const int trow = (lane & 7) + ((lane >> 3) & 1) * 8;                       // transposed, right operand
-  const int arow = (lane & 7) + (lane >> 4) * 8, acol = ((lane >> 3) & 1) * 8;   // transposed, left operand
+  auto publish = [&]() {
+#pragma unroll
+    for (int i = 0; i < NS; ++i)
+#pragma unroll
+      for (int w = 0; w < 2; ++w) {
+        uint32_t hi, lo;
+        split2(S[i][2 * w], S[i][2 * w + 1], hi, lo);
+        __nv_bfloat16* dst = ss + (g + 8 * w) * LQ + d_own + i * 8 + 2 * tig;
+        *reinterpret_cast<uint32_t*>(dst) = hi;
+        *reinterpret_cast<uint32_t*>(dst + 16 * LQ) = lo;
+      }
+  };
+  publish();
+  const int row16 = lane & 15, col8 = (lane >> 4) * 8;                       // non-transposed 16 x 16 tiles, left operand
+  const int brow = (lane & 7) + (lane >> 4) * 8, bcol = ((lane >> 3) & 1) * 8;   // right operand stored by column; left, transposed
+  const int trow = (lane & 7) + ((lane >> 3) & 1) * 8;                       // right operand, transposed
   for (int c = 0; c < chunks; ++c) {
     asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();                                    // chunk landed; the other buffer's readers are done
+    __syncthreads();                                    // chunk and state landed; the other buffer's readers are done
     if (c + 1 < chunks) fetch(c + 1, (c + 1) & 1);
-    if (!live) continue;
     const __nv_bfloat16* sq = reinterpret_cast<const __nv_bfloat16*>(smem + (c & 1) * stage);
     const __nv_bfloat16* sk = sq + 2 * CL * LQ;
     const __nv_bfloat16* sa = sk + 2 * CL * LQ;
     const __nv_bfloat16* sv = sa + 2 * CL * LA;
     const float* end = reinterpret_cast<const float*>(sv + CL * LV);
-    float o[MT][2][4];
+    if (live && sub < MT * 2 / NJ) {
+      const int m = NJ == 2 ? sub : sub >> 1, j0 = NJ == 2 ? 0 : sub & 1;
+      float o[NJ][4] = {}, ol[NJ][4] = {};              // sums of the leading and of the correcting products
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
+      for (int k2 = 0; k2 < DT / 32; ++k2) {
+        uint32_t bh[NJ][4], bl[NJ][4];                  // two k-steps of 8 columns
 #pragma unroll
-      for (int j = 0; j < 2; ++j) o[m][j][0] = o[m][j][1] = o[m][j][2] = o[m][j][3] = 0.f;
+        for (int j = 0; j < NJ; ++j) {
+          const __nv_bfloat16* b = ss + ((j0 + j) * 8 + (lane & 7)) * LQ + k2 * 32 + (lane >> 3) * 8;
+          ldmatrix_x4(bh[j], b);
+          ldmatrix_x4(bl[j], b + 16 * LQ);
+        }
 #pragma unroll
-    for (int kk = 0; kk < DT / 16; ++kk) {
-      uint32_t bh[2][2], bl[2][2];                      // [value half][channel half]
+        for (int u = 0; u < 2; ++u) {
+          uint32_t ah[4], al[4];
+          ldmatrix_x4(ah, sq + (m * 16 + row16) * LQ + k2 * 32 + u * 16 + col8);
+          ldmatrix_x4(al, sq + (CL + m * 16 + row16) * LQ + k2 * 32 + u * 16 + col8);
 #pragma unroll
-      for (int j = 0; j < 2; ++j)
-#pragma unroll
-        for (int u = 0; u < 2; ++u) split2(S[2 * kk + u][2 * j], S[2 * kk + u][2 * j + 1], bh[j][u], bl[j][u]);
-#pragma unroll
-      for (int m = 0; m < MT; ++m) {
-        uint32_t ah[4], al[4];
-        ldmatrix_x4(ah, sq + (m * 16 + row16) * LQ + kk * 16 + col8);
-        ldmatrix_x4(al, sq + (CL + m * 16 + row16) * LQ + kk * 16 + col8);
-#pragma unroll
-        for (int j = 0; j < 2; ++j) {
-          mma(o[m][j], ah, bh[j][0], bh[j][1]);
-          mma(o[m][j], ah, bl[j][0], bl[j][1]);
-          mma(o[m][j], al, bh[j][0], bh[j][1]);
+          for (int j = 0; j < NJ; ++j) {
+            mma(o[j], ah, bh[j][2 * u], bh[j][2 * u + 1]);
+            mma(ol[j], ah, bl[j][2 * u], bl[j][2 * u + 1]);
+            mma(ol[j], al, bh[j][2 * u], bh[j][2 * u + 1]);
+          }
         }
       }
-    }
 #pragma unroll
-    for (int ks = 0; ks < MT; ++ks) {
-      uint32_t b[4];
-      ldmatrix_x4_trans(b, sv + (ks * 16 + trow) * LV + warp * 16 + col8);
-#pragma unroll
-      for (int m = ks; m < MT; ++m) {
-        uint32_t ah[4], al[4];
+      for (int ks = 0; ks < MT; ++ks) {
+        if (ks > m) break;
+        uint32_t b[4], ah[4], al[4];
+        ldmatrix_x4_trans(b, sv + (ks * 16 + trow) * LV + vg * 16 + col8);
         ldmatrix_x4(ah, sa + (m * 16 + row16) * LA + ks * 16 + col8);
         ldmatrix_x4(al, sa + (CL + m * 16 + row16) * LA + ks * 16 + col8);
 #pragma unroll
-        for (int j = 0; j < 2; ++j) {
-          mma(o[m][j], ah, b[2 * j], b[2 * j + 1]);
-          mma(o[m][j], al, b[2 * j], b[2 * j + 1]);
+        for (int j = 0; j < NJ; ++j) {
+          const uint32_t b0 = j0 + j ? b[2] : b[0], b1 = j0 + j ? b[3] : b[1];
+          mma(o[j], ah, b0, b1);
+          mma(ol[j], al, b0, b1);
         }
       }
-    }
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
 #pragma unroll
       for (int w = 0; w < 2; ++w) {
         const int t = c * CL + m * 16 + g + 8 * w;
         if (t < len) {
-          float* dst = p.o + ((size_t)(r0 + t) * p.H + h) * p.V + vw + 2 * tig;
+          float* dst = p.o + ((size_t)(r0 + t) * p.H + h) * p.V + vw + j0 * 8 + 2 * tig;
 #pragma unroll
-          for (int j = 0; j < 2; ++j) *reinterpret_cast<float2*>(dst + j * 8) = make_float2(o[m][j][2 * w], o[m][j][2 * w + 1]);
-        }
-      }
-#pragma unroll
-    for (int i = 0; i < DT / 8; ++i) {
-      const float2 f = *reinterpret_cast<const float2*>(end + i * 8 + 2 * tig);
-      S[i][0] *= f.x; S[i][1] *= f.y;
-      S[i][2] *= f.x; S[i][3] *= f.y;
-    }
-#pragma unroll
-    for (int ks = 0; ks < MT; ++ks) {
-      uint32_t a[4];
-      ldmatrix_x4_trans(a, sv + (ks * 16 + arow) * LV + warp * 16 + acol);
-#pragma unroll
-      for (int i = 0; i < DT / 16; ++i) {
-        uint32_t bh[4], bl[4];
-        ldmatrix_x4_trans(bh, sk + (ks * 16 + trow) * LQ + i * 16 + col8);
-        ldmatrix_x4_trans(bl, sk + (CL + ks * 16 + trow) * LQ + i * 16 + col8);
-#pragma unroll
-        for (int u = 0; u < 2; ++u) {
-          mma(S[2 * i + u], a, bh[2 * u], bh[2 * u + 1]);
-          mma(S[2 * i + u], a, bl[2 * u], bl[2 * u + 1]);
+          for (int j = 0; j < NJ; ++j)
+            *reinterpret_cast<float2*>(dst + j * 8) = make_float2(o[j][2 * w] + ol[j][2 * w], o[j][2 * w + 1] + ol[j][2 * w + 1]);
         }
       }
     }
+    if (live) {
+#pragma unroll
+      for (int i = 0; i < NS; ++i) {
+        const float2 f = *reinterpret_cast<const float2*>(end + d_own + i * 8 + 2 * tig);
+        S[i][0] *= f.x; S[i][1] *= f.y;
+        S[i][2] *= f.x; S[i][3] *= f.y;
+      }
+#pragma unroll
+      for (int ks = 0; ks < MT; ++ks) {
+        uint32_t a[4];
+        ldmatrix_x4_trans(a, sv + (ks * 16 + brow) * LV + vg * 16 + bcol);
+#pragma unroll
+        for (int i = 0; i < NS / 2; ++i) {
+          uint32_t bh[4], bl[4];
+          ldmatrix_x4_trans(bh, sk + (ks * 16 + trow) * LQ + d_own + i * 16 + col8);
+          ldmatrix_x4_trans(bl, sk + (CL + ks * 16 + trow) * LQ + d_own + i * 16 + col8);
+#pragma unroll
+          for (int u = 0; u < 2; ++u) {
+            mma(S[2 * i + u], a, bh[2 * u], bh[2 * u + 1]);
+            mma(S[2 * i + u], a, bl[2 * u], bl[2 * u + 1]);
+          }
+        }
+      }
+    }
+    __syncthreads();                                    // everyone has read the state of before the chunk
+    publish();
   }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
   if (!live) return;
 #pragma unroll
-  for (int i = 0; i < DT / 8; ++i)
+  for (int i = 0; i < NS; ++i)
 #pragma unroll
     for (int x = 0; x < 4; ++x) {
-      const int d = i * 8 + 2 * tig + (x & 1), v = vw + g + 8 * (x >> 1);
+      const int d = d_own + i * 8 + 2 * tig + (x & 1), v = vw + g + 8 * (x >> 1);
       if (d < p.D) st[(size_t)d * p.V + v] = S[i][x];
     }
 }
@@ -400,14 +428,16 @@ int launch(ChunkParams p, int chunks, cudaStream_t stream) {
     configured = true;
   }
   const size_t prep = (size_t)CL * (DT + 4) * 4 + (size_t)2 * CL * (DT + 8) * 2;
-  cudaError_t e = launch_pdl(gla_chunk_prep_kernel<DT, CL>, dim3(chunks, p.H), dim3(128), prep, stream, p);
+  cudaError_t e = launch_pdl(gla_chunk_prep_kernel<DT, CL>, dim3(chunks, p.H), dim3(PT), prep, stream, p);
   if (e != cudaSuccess) return (int)e;
-  // fewer columns per block while that leaves SMs idle
-  int warps = 4;
-  while (warps > 1 && (long long)p.entries * p.H * ((p.V + 16 * warps - 1) / (16 * warps)) < 74) warps >>= 1;
-  while (warps > 1 && 16 * (warps / 2) >= p.V) warps >>= 1;
-  return (int)launch_pdl(gla_chunk_scan_kernel<DT, CL>, dim3((p.V + 16 * warps - 1) / (16 * warps), p.H, p.entries), dim3(warps * 32),
-                         2 * stage_bytes<DT, CL>(16 * warps), stream, p);
+  // 16 columns per block where one wave of blocks takes them, more otherwise
+  constexpr int W = SUBS<DT>;
+  int groups = 1;
+  while (groups * W < 16 && (long long)p.entries * p.H * ((p.V + 16 * groups - 1) / (16 * groups)) > 148 && 16 * groups < p.V &&
+         scan_smem<DT, CL>(32 * groups) <= 227 * 1024)
+    groups <<= 1;
+  return (int)launch_pdl(gla_chunk_scan_kernel<DT, CL>, dim3((p.V + 16 * groups - 1) / (16 * groups), p.H, p.entries), dim3(groups * W * 32),
+                         scan_smem<DT, CL>(16 * groups), stream, p);
 }
 
 }  // namespace
@@ -417,9 +447,9 @@ extern "C" int b200_gla_chunk_rows(int D) { return D <= 0 || D % 16 || D > 256 ?
 
 // bf16 elements of workspace per chunk and head, and fp32 ones.
 extern "C" int b200_gla_chunk_ws(int D) {
-  return D <= 32 ? ws_elems<32, 64>() : D <= 64 ? ws_elems<64, 64>() : D <= 128 ? ws_elems<128, 64>() : ws_elems<256, 32>();
+  return D <= 64 ? ws_elems<64, 64>() : D <= 128 ? ws_elems<128, 64>() : ws_elems<256, 32>();
 }
-extern "C" int b200_gla_chunk_end(int D) { return D <= 32 ? 32 : D <= 64 ? 64 : D <= 128 ? 128 : 256; }
+extern "C" int b200_gla_chunk_end(int D) { return D <= 64 ? 64 : D <= 128 ? 128 : 256; }
 
 // Entries with at least min_len rows; chunks: upper bound on their number (rows / chunk rows + entries).  D, V multiples of 16,
 // D <= 256; state [slots, H, D, V] fp32 in place; o fp32 [rows, H * V].
@@ -433,7 +463,6 @@ extern "C" int b200_gla_chunk(const void* q, const void* k, const void* v, int l
   p.v = reinterpret_cast<const __nv_bfloat16*>(v); p.la = la; p.state = state; p.o = o; p.first = first; p.length = length; p.slot = slot;
   p.positions = positions; p.ws = reinterpret_cast<__nv_bfloat16*>(ws); p.end = end; p.ld = ld; p.H = H; p.D = D; p.V = V;
   p.entries = entries; p.min_len = min_len; p.scale = scale;
-  if (D <= 32) return launch<32, 64>(p, chunks, stream);
   if (D <= 64) return launch<64, 64>(p, chunks, stream);
   if (D <= 128) return launch<128, 64>(p, chunks, stream);
   return launch<256, 32>(p, chunks, stream);

@@ -16,34 +16,31 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1
                : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
-constexpr int WARPS = 4, NW = 16;          // features per warp
+constexpr int WARPS = 4, NW = 16;          // features per block; the warps share K
 
-// grid (features / 64, heads, rows / (16 MT)), 128 threads; K % 16 == 0 (32-wide chunks, the last may be half).
+// grid (features / 16, heads, rows / (16 MT)), 128 threads; K % 16 == 0 (32-wide chunks, the last may be half).  The warps'
+// sums are added up through shared memory.
 template <int MT>
 __global__ void __launch_bounds__(WARPS * 32)
 head_linear_kernel(const __nv_bfloat16* __restrict__ x, int ldx, int x_head, const __nv_bfloat16* __restrict__ w,
                    __nv_bfloat16* __restrict__ y, int ldy, int y_head, int T, int N, int K) {
+  __shared__ float red[WARPS][MT][2][4][32];
   pdl_grid_trigger();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gr = lane >> 2, kk = lane & 3;
-  const int h = blockIdx.y, n0 = blockIdx.x * WARPS * NW + warp * NW, t0 = blockIdx.z * 16 * MT;
+  const int h = blockIdx.y, n0 = blockIdx.x * NW, t0 = blockIdx.z * 16 * MT;
   const uint4 zero = make_uint4(0, 0, 0, 0);
   const __nv_bfloat16* wh = w + (size_t)h * N * K;
   float acc[MT][2][4] = {};
   pdl_grid_wait();
-  if (n0 >= N) return;
-  auto load_w = [&](int k0, uint4 (&b)[2]) {
+#pragma unroll 4
+  for (int k0 = warp * 32; k0 < K; k0 += 32 * WARPS) {
     const int k = k0 + kk * 8;
+    uint4 b[2];
 #pragma unroll
     for (int nb = 0; nb < 2; ++nb) {
       const int n = n0 + nb * 8 + gr;
       b[nb] = n < N && k < K ? *reinterpret_cast<const uint4*>(wh + (size_t)n * K + k) : zero;
     }
-  };
-  uint4 b[2], bn[2];
-  load_w(0, b);
-  for (int k0 = 0; k0 < K; k0 += 32) {
-    if (k0 + 32 < K) load_w(k0 + 32, bn);
-    const int k = k0 + kk * 8;
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt) {
       const int ta = t0 + mt * 16 + gr, tb = ta + 8;
@@ -55,20 +52,26 @@ head_linear_kernel(const __nv_bfloat16* __restrict__ x, int ldx, int x_head, con
         mma_bf16(acc[mt][nb], a0.z, a1.z, a0.w, a1.w, b[nb].z, b[nb].w);
       }
     }
-    b[0] = bn[0];
-    b[1] = bn[1];
   }
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
     for (int nb = 0; nb < 2; ++nb)
 #pragma unroll
-      for (int hf = 0; hf < 2; ++hf) {
-        const int t = t0 + mt * 16 + gr + hf * 8, n = n0 + nb * 8 + kk * 2;
-        if (t < T && n < N)
-          *reinterpret_cast<__nv_bfloat162*>(y + (size_t)t * ldy + h * y_head + n) =
-              __floats2bfloat162_rn(acc[mt][nb][hf * 2], acc[mt][nb][hf * 2 + 1]);
-      }
+      for (int i = 0; i < 4; ++i) red[warp][mt][nb][i][lane] = acc[mt][nb][i];
+  __syncthreads();
+  // item: (row tile, feature half, row half), a pair of features per lane
+  for (int item = warp; item < MT * 4; item += WARPS) {
+    const int mt = item >> 2, nb = (item >> 1) & 1, hf = item & 1;
+    float v0 = 0.f, v1 = 0.f;
+#pragma unroll
+    for (int u = 0; u < WARPS; ++u) {
+      v0 += red[u][mt][nb][hf * 2][lane];
+      v1 += red[u][mt][nb][hf * 2 + 1][lane];
+    }
+    const int t = t0 + mt * 16 + gr + hf * 8, n = n0 + nb * 8 + kk * 2;
+    if (t < T && n < N) *reinterpret_cast<__nv_bfloat162*>(y + (size_t)t * ldy + h * y_head + n) = __floats2bfloat162_rn(v0, v1);
+  }
 }
 
 }  // namespace
@@ -79,7 +82,7 @@ extern "C" int b200_head_linear(const void* x, int ldx, int x_head, const void* 
   if (T <= 0 || H <= 0 || H > 65535 || N <= 0 || (N & 1) || K <= 0 || (K & 15) || ((ldx | x_head | ldy | y_head) & 7)) return -6;
   const int mt = T <= 16 ? 1 : T <= 32 ? 2 : 4;
   if ((T + 16 * mt - 1) / (16 * mt) > 65535) return -6;
-  const dim3 grid((N + WARPS * NW - 1) / (WARPS * NW), H, (T + 16 * mt - 1) / (16 * mt)), block(WARPS * 32);
+  const dim3 grid((N + NW - 1) / NW, H, (T + 16 * mt - 1) / (16 * mt)), block(WARPS * 32);
   auto xp = reinterpret_cast<const __nv_bfloat16*>(x);
   auto wp = reinterpret_cast<const __nv_bfloat16*>(w);
   auto yp = reinterpret_cast<__nv_bfloat16*>(y);

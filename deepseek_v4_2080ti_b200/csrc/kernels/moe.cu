@@ -1,4 +1,5 @@
 // Routed-expert plumbing around the grouped GEMM (gemm_wdec.cu, grouped mode):
+//   moe_router_rows  - router logits of a short batch;
 //   moe_route        - scores (softmax | sigmoid | sqrt-softplus) + selection bias + top-k + weight normalisation;
 //   moe_plan         - counting sort of the (token, k) routes by local expert: per-expert offsets, the row of every
 //                      route in expert-sorted order, and the (expert, m_tile, row0, rows) work table of both grouped
@@ -14,6 +15,7 @@
 #include <cuda_bf16.h>
 #include <stdint.h>
 #include "glu.cuh"
+#include "launch.h"
 #include "ops.h"
 #include "vec8.cuh"
 
@@ -88,6 +90,37 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int ld, const
     for (int k = lane; k < K; k += 32) wts[(size_t)t * K + k] /= wsum;     // lane k & 31 wrote entry k
 }
 
+// z[t, n] = x[t] . w[n] in fp32 for a handful of rows: a warp per output feature, its weights read once for RT rows.
+constexpr int RT = 8;
+
+__global__ void __launch_bounds__(128) moe_router_rows_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w,
+                                                              float* __restrict__ z, int T, int N, int K) {
+  b200::pdl_grid_trigger();
+  b200::pdl_grid_wait();
+  const int n = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31, t0 = blockIdx.y * RT;
+  if (n >= N) return;
+  float acc[RT] = {};
+#pragma unroll 2
+  for (int k = lane * 8; k < K; k += 256) {
+    float f[8];
+    b200::load8(w + (size_t)n * K + k, f);
+#pragma unroll
+    for (int t = 0; t < RT; ++t) {
+      if (t0 + t < T) {
+        float a[8];
+        b200::load8(x + (size_t)(t0 + t) * K + k, a);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) acc[t] = fmaf(f[j], a[j], acc[t]);
+      }
+    }
+  }
+#pragma unroll
+  for (int t = 0; t < RT; ++t) {
+    const float v = b200::warp_sum_all(acc[t]);
+    if (lane == 0 && t0 + t < T) z[(size_t)(t0 + t) * N + n] = v;
+  }
+}
+
 __device__ __forceinline__ int warp_scan(int v, int lane) {                // inclusive
 #pragma unroll
   for (int o = 1; o < 32; o <<= 1) {
@@ -123,10 +156,31 @@ moe_plan_kernel(const int* __restrict__ idx, int R, int K, int lo, int hi, int* 
   const int EL = hi - lo, e = blockIdx.x, tid = threadIdx.x;
   cnt[tid] = 0;
   __syncthreads();
-  for (int r = tid; r < R; r += 1024) {
-    const int x = idx[r] - lo;
-    if (x >= 0 && x < EL) atomicAdd(&cnt[x], 1);
-    else if (e == 0) route_row[r] = -1;
+  constexpr int U = 8;                     // neighbouring routes per thread and round, two 16-byte loads
+  auto load = [&](int r, int (&x)[U]) {    // local expert of routes r .. r + 7; -1: none
+#pragma unroll
+    for (int u = 0; u < U; u += 4) {
+      int4 v = make_int4(-1, -1, -1, -1);
+      if (r + u + 4 <= R) {
+        v = *reinterpret_cast<const int4*>(idx + r + u);
+      } else {
+        if (r + u < R) v.x = idx[r + u];
+        if (r + u + 1 < R) v.y = idx[r + u + 1];
+        if (r + u + 2 < R) v.z = idx[r + u + 2];
+      }
+      x[u] = v.x - lo; x[u + 1] = v.y - lo; x[u + 2] = v.z - lo; x[u + 3] = v.w - lo;
+    }
+  };
+#pragma unroll 2
+  for (int r = tid * U; r < R; r += 1024 * U) {
+    int x[U];
+    load(r, x);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      if (r + u >= R) break;
+      if (x[u] >= 0 && x[u] < EL) atomicAdd(&cnt[x[u]], 1);
+      else if (e == 0) route_row[r + u] = -1;
+    }
   }
   __syncthreads();
   const int c_t = tid < EL ? cnt[tid] : 0;                                 // thread t stands for expert t here
@@ -147,15 +201,19 @@ moe_plan_kernel(const int* __restrict__ idx, int R, int K, int lo, int hi, int* 
   const int c = mine[0], off = mine[1];
   if (c == 0) return;
   int placed = 0;
-  for (int r0 = 0; r0 < R && placed < c; r0 += 1024) {
-    const int r = r0 + tid;
-    const int hit = r < R && idx[r] - lo == e;
-    int n;
-    const int at = off + placed + block_scan(hit, ws, n);
-    if (hit) {
-      route_row[r] = at;
-      row_token[at] = r / K;
-    }
+  for (int r0 = 0; r0 < R && placed < c; r0 += 1024 * U) {
+    const int r = r0 + tid * U;
+    int x[U], hits = 0, n;
+    load(r, x);
+#pragma unroll
+    for (int u = 0; u < U; ++u) hits |= (r + u < R && x[u] == e) << u;
+    int at = off + placed + block_scan(__popc(hits), ws, n);
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+      if (hits >> u & 1) {
+        route_row[r + u] = at;
+        row_token[at++] = (r + u) / K;
+      }
     placed += n;
   }
   // work tables: m-tile fastest inside a token tile so one expert's weight tiles are swept once per token tile
@@ -241,6 +299,13 @@ int b200_moe_route(const float* logits, int ld, const float* bias, int T, int E,
   B200_ROUTE(1) B200_ROUTE(2) B200_ROUTE(4) B200_ROUTE(8) B200_ROUTE(16) B200_ROUTE(32)
 #undef B200_ROUTE
   return -6;
+}
+
+// fp32 logits z [T, N] of bf16 rows x [T, K] and router w [N, K] for short batches; K % 8 == 0.
+int b200_moe_router_rows(const void* x, const void* w, float* z, int T, int N, int K, cudaStream_t stream) {
+  if (T <= 0 || N <= 0 || K <= 0 || (K & 7)) return -6;
+  return (int)b200::launch_pdl(moe_router_rows_kernel, dim3((N + 3) / 4, (T + RT - 1) / RT), dim3(128), 0, stream,
+                               reinterpret_cast<const __nv_bfloat16*>(x), reinterpret_cast<const __nv_bfloat16*>(w), z, T, N, K);
 }
 
 // Plans the grouped GEMMs of this rank's experts [expert_lo, expert_hi).  All outputs are device buffers:

@@ -490,7 +490,7 @@ class KemiraxRuntime(PagedRuntime):
     def _experts(self, ew: ExpertsWeights, h: torch.Tensor) -> dict:
         f = ew.spec
         total = f.experts + f.identity
-        z = ew.router(h, out_f32=True)
+        z = moe.router_logits(h, ew.router)
         idx, weights = moe.route(z[:, :total], ew.correction, f.top, "softmax", False, 1.0)
         y, row = moe.experts_rows(h, idx, ew.w13, ew.w2, 0, f.limit, UNIT_SLOPE)
         out = {"h": h, "routed": Routed(y, row, idx, weights, f.experts)}
@@ -500,31 +500,27 @@ class KemiraxRuntime(PagedRuntime):
 
     def _forward(self, ids, positions, kv_slots, meta, rows):
         cfg, w, n = self.cfg, self.w, ids.numel()
-        # two buffers in turn: a block that needs its neighbour's row reads what the layer started from
-        x = [torch.empty(n, w.ld, dtype=torch.float32, device=self.device) for _ in range(2)]
+        x = torch.empty(n, w.ld, dtype=torch.float32, device=self.device)
         common = {"ld": w.ld, "n": n, "dtype": w.dtype}
         pending: dict = {"ids": ids, "table": w.embed}       # the residual starts from it
-        at = 0
 
         def boundary(weight: float, **kw):
             """What is pending enters the residual; the next layer's inputs."""
-            nonlocal pending, at
-            src = None if "ids" in pending else x[at]
-            out = decoder.parallel_step(src, cfg.width, weight, cfg.eps, **common, **pending, **kw)
-            if kw.get("x_out") is not None:
-                pending, at = {}, 1 - at
+            nonlocal pending
+            out = decoder.parallel_step(None if "ids" in pending else x, cfg.width, weight, cfg.eps, **common, **pending, **kw)
+            pending = {}
             return out
 
         for i, lw in enumerate(w.layers):
-            h, m = boundary(lw.norm, x_out=x[1 - at], shift=lw.shift, tail=self.tails[i], seg=meta["segments"], positions=positions)
+            h, m = boundary(lw.norm, x_out=x, shift=lw.shift, tail=self.tails[i], seg=meta["segments"], positions=positions)
             pending = {"gates": lw.gates(h), "gate_b": lw.gate_b}
             pending["mix"] = (self._latent(i, lw.mix, m, positions, kv_slots, meta) if isinstance(lw.mix, LatentWeights)
                               else self._linear(i, lw.mix, m, positions, meta))
             if lw.ff is not None:
                 pending.update(self._experts(lw.ff, h))
             if self.residual_tap is not None:
-                boundary(1.0, x_out=x[1 - at], norm=False)
-                self.residual_tap(i, x[at][:, :cfg.width].clone())
+                boundary(1.0, x_out=x, norm=False)
+                self.residual_tap(i, x[:, :cfg.width].clone())
         if rows is not None and rows.numel() == 0:
             return None
         return w.head(boundary(w.final_norm, rows=rows)[0], out_f32=True)

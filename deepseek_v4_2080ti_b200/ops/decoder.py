@@ -154,8 +154,7 @@ def parallel_step(x: torch.Tensor | None, cols: int, weight: float, eps: float, 
                   seg=None, positions: torch.Tensor | None = None, rows: torch.Tensor | None = None,
                   norm: bool = True) -> tuple[torch.Tensor | None, torch.Tensor | None]:
     """Step between layers whose sublayers run side by side (csrc/kernels/parallel_step.cu):
-    ``x + mix sigmoid(gates[:, :ld] + b) + ff sigmoid(gates[:, ld:] + b)`` goes to ``x_out`` (another buffer than ``x``),
-    with ``ff`` the sum of the routed experts, of identity experts (``h``) and of ``shared`` behind its gate (a column of
+    ``x + mix sigmoid(gates[:, :ld] + b) + ff sigmoid(gates[:, ld:] + b)`` goes to ``x_out`` (which may be ``x``), with ``ff`` the sum of the routed experts, of identity experts (``h``) and of ``shared`` behind its gate (a column of
     logits).  Returns (RMS norm of it times ``weight``, that norm moved towards the row before it by ``shift``): the second
     only with ``shift``, which also keeps the sequences' ``tail`` [slots, ld].  ``rows``: only these rows, norm only."""
     dev = (x if x is not None else ids).device
@@ -172,21 +171,22 @@ def parallel_step(x: torch.Tensor | None, cols: int, weight: float, eps: float, 
     count = rows.numel() if rows is not None else n
     out = torch.empty(count, ld, dtype=dtype, device=dev) if norm else None
     m = torch.empty(n, ld, dtype=dtype, device=dev) if shift is not None else None
-    r = routed
+    single = m is not None and seg.max_length == 1      # no row needs its neighbour: shift and tails in the same launch
+    f32, r = int(dtype == torch.float32), routed
     rc = _lib.lib().b200_parallel_step(
         _lib.ptr(x), _lib.ptr(x_out), _lib.ptr(ids), _lib.ptr(table), 0 if table is None else table.shape[0], _lib.ptr(mix),
         _lib.ptr(gates), 0 if gates is None else gates.stride(0), _lib.ptr(gate_b), _lib.ptr(h), _lib.ptr(r.y if r else None),
         r.y.stride(0) if r else 0, _lib.ptr(r.row if r else None), _lib.ptr(r.idx if r else None),
         _lib.ptr(r.weights if r else None), r.idx.shape[1] if r else 0, r.experts if r else 0, _lib.ptr(shared),
-        _lib.ptr(shared_gate), 0 if shared_gate is None else shared_gate.stride(0), _f(weight), _f(eps), _lib.ptr(out), _lib.ptr(m),
-        _lib.ptr(shift), _lib.ptr(tail), _lib.ptr(seg.row_first if m is not None else None),
-        _lib.ptr(seg.row_slot if m is not None else None), _lib.ptr(positions), _lib.ptr(rows), count, ld, cols,
-        int(dtype == torch.float32), _lib.stream())
+        _lib.ptr(shared_gate), 0 if shared_gate is None else shared_gate.stride(0), _f(weight), _f(eps), _lib.ptr(out),
+        _lib.ptr(m if single else None), _lib.ptr(shift), _lib.ptr(tail), _lib.ptr(seg.row_slot if single else None),
+        _lib.ptr(positions), _lib.ptr(rows), count, ld, cols, f32, _lib.stream())
     _lib.check(rc, "parallel_step")
-    if m is not None and seg.max_length > 1:       # single rows replaced their tail in the kernel
-        rc = _lib.lib().b200_shift_tails(_lib.ptr(out), _lib.ptr(tail), _lib.ptr(seg.first), _lib.ptr(seg.length),
-                                         _lib.ptr(seg.slot), seg.first.numel(), ld, int(dtype == torch.float32), _lib.stream())
-        _lib.check(rc, "shift_tails")
+    if m is not None and not single:
+        rc = _lib.lib().b200_shift_rows(_lib.ptr(out), _lib.ptr(m), _lib.ptr(shift), _lib.ptr(tail), _lib.ptr(seg.row_first),
+                                        _lib.ptr(seg.row_slot), _lib.ptr(positions), _lib.ptr(seg.first), _lib.ptr(seg.length),
+                                        _lib.ptr(seg.slot), seg.first.numel(), n, ld, f32, _lib.stream())
+        _lib.check(rc, "shift_rows", 2)
     return out, m
 
 

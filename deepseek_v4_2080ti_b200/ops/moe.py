@@ -74,6 +74,21 @@ class ExpertWeights:
         return ExpertWeights(WF_BF16, torch.cat([x.to(torch.bfloat16) for x in ws]).contiguous(), None, n, k, len(ws))
 
 
+ROUTER_MAX_ROWS = 64            # batches up to this take the row kernel: a tensor-core tile would leave all but one SM idle
+
+
+def router_logits(x: torch.Tensor, w) -> torch.Tensor:
+    """fp32 logits [T, w.n] of a router (``ops.decoder.Projection``)."""
+    if x.dtype != torch.bfloat16 or x.shape[0] > ROUTER_MAX_ROWS:
+        return w(x, out_f32=True)
+    t, k = x.shape
+    assert x.is_contiguous() and k == w.k
+    z = torch.empty(t, w.n, dtype=torch.float32, device=x.device)
+    rc = _lib.lib().b200_moe_router_rows(_lib.ptr(x), _lib.ptr(w.packed.weight), _lib.ptr(z), t, w.n, k, _lib.stream())
+    _lib.check(rc, "moe_router_rows")
+    return z
+
+
 def route(logits: torch.Tensor, bias: torch.Tensor | None, k: int, score_func: str, norm_topk: bool,
           route_scale: float) -> tuple[torch.Tensor, torch.Tensor]:
     """fp32 logits [T, E] (row stride allowed) -> (idx int32 [T, k], weights fp32 [T, k])."""

@@ -1,11 +1,12 @@
 """Prefill and decode throughput of one decoder design at sizes of real models' layers (random weights), beside the
 framework's closest existing model at equal size, and the kernels of both beside their rooflines.
 
-    python bench.py --design rutulix|zigasun [--design-size small|large] [--steps K] [--warmup W]
+    python bench.py --design rutulix|zigasun|kemirax [--design-size small|large] [--steps K] [--warmup W]
 
 Closest model of Rutulix: the Qwen-style decoder with full-attention layers only (per-head QK norm, grouped attention, SwiGLU
 with FP8 weights) of the same width, heads and feed-forward parameters.  Of Zigasun: the same decoder with Gated-DeltaNet and
-full-attention layers in turn (both recurrent states as wide as the scan's channels).  Whole-model numbers: CUDA events around a prompt of
+full-attention layers in turn (both recurrent states as wide as the scan's channels).  Of Kemirax: the latent-attention
+decoder with routed experts, equal width, heads, latents and experts; its recurrence stands beside Gated DeltaNet.  Whole-model numbers: CUDA events around a prompt of
 ``--prompt`` tokens and around replayed decode steps.  Kernel numbers: CUDA events around single launches, L2 flushed
 before each; fractions of the measured copy bandwidth / bf16 GEMM burst of MEASURED_PEAKS.json.
 """
@@ -21,6 +22,10 @@ PEAKS_FALLBACK = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
 SIZES = {"small": (2048, 16, 4, 128, 5632, 2048), "large": (4096, 32, 8, 128, 10752, 8192)}
 # Zigasun: width, heads, kv heads, dim per map, value dim, feed-forward, scan channels, states, dt rank
 ZG_SIZES = {"small": (2048, 16, 4, 64, 128, 5632, 4096, 16, 128), "large": (4096, 32, 8, 64, 128, 10752, 8192, 16, 256)}
+# Kemirax: width, heads, dim, rotated dim, value dim, query latent, latent, linear-attention heads (128 x 128), expert and shared
+# width, experts, identity experts, experts per token
+KX_SIZES = {"small": (2048, 16, 128, 64, 128, 768, 512, 16, 1024, 64, 8, 6), "large": (4096, 32, 128, 64, 128, 1536, 512, 32, 1536, 128, 16, 8)}
+KX_LAYERS = "gaba"
 LAYERS, VOCAB = 4, 32768
 
 
@@ -100,16 +105,17 @@ def _recorder(timer: _Timer):
     rows_out: list[dict] = []
 
     def pair(what, shape, new, old):
-        rec = {"kernel": what, "shape": shape}
+        rec, frac = {"kernel": what, "shape": shape}, {}
         for tag, spec in (("new", new), ("like", old)):
             if spec is None:
                 continue
             fn, need_bytes, need_flops = spec
             ms = timer(fn)
             roof = max(need_bytes / bw, need_flops / fl)
+            frac[tag] = roof / ms
             rec[tag] = {"ms": round(ms, 4), "fraction": round(roof / ms, 3), "bound": "memory" if need_bytes / bw >= need_flops / fl else "tensor"}
         if "like" in rec:
-            rec["distance_ratio"] = round(rec["like"]["fraction"] / rec["new"]["fraction"], 2)
+            rec["distance_ratio"] = round(frac["like"] / frac["new"], 2)
         rows_out.append(rec)
     return rows_out, pair
 
@@ -307,6 +313,127 @@ def _zg_kernels(size: str, dev, timer: _Timer, ctx: int) -> list[dict]:
     return rows_out
 
 
+def _kx_models(size: str, dev, prompt: int, slots: int):
+    from ..models import kemirax as kx
+    from ..models import mla_moe as mm
+    from ..models import mla_moe_gpu as mg
+    width, H, d, r, v, qr, c, gh, ff, E, ident, top = KX_SIZES[size]
+    cfg = kx.KemiraxConfig.pattern(KX_LAYERS, width, H, d, r, v, qr, c, gh, 128, 128, ff, E, ident, top, ff, VOCAB)
+    new = lambda: kx.build_synthetic(cfg, dev, max_slots=slots, max_context=prompt + 192)
+    mcfg = mm.MlaMoeConfig(vocab_size=VOCAB, hidden_size=width, num_layers=len(KX_LAYERS), first_dense_layers=0, q_lora_rank=qr,
+                           kv_lora_rank=c, num_heads=H, qk_nope_dim=d, qk_rope_dim=r, v_head_dim=v, index_heads=0, index_dim=0,
+                           index_topk=0, num_experts=E, experts_per_token=top, num_shared_experts=1, expert_intermediate=ff,
+                           score_func="softmax", route_scale=1.0, norm_topk=False, expert_format="bf16")
+    old = lambda: mg.MlaMoeBatchRuntime(mcfg, mg.MlaMoeGpuWeights(mcfg, mm.synth_state(mcfg, 0, dev), dev), max_slots=slots,
+                                        max_context=prompt + 192)
+    return new, old
+
+
+def _kx_kernels(size: str, dev, timer: _Timer, ctx: int) -> list[dict]:
+    from ..models import kemirax as kx
+    from ..ops import basic, decoder, gdn, gemm, gla, latent, mla, moe, scan
+    width, H, d, r, v, qr, c, gh, ff, E, ident, top = KX_SIZES[size]
+    rnd = lambda *s, dt=torch.bfloat16: torch.randn(*s, device=dev, dtype=torch.float32).to(dt)
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    cfg = kx.KemiraxConfig.pattern("ag", width, H, d, r, v, qr, c, gh, 128, 128, ff, E, ident, top, ff, 64)
+    w = kx.KemiraxWeights(cfg, kx.synth_state(cfg, 0, dev), dev)
+    lay, aw, gw, ew = w.layers[0], w.layers[0].mix, w.layers[1].mix, w.layers[0].ff
+    m, gm = aw.m, gw.m
+    rows_out, pair = _recorder(timer)
+    bs, pages, cw = 64, (ctx + 63) // 64, c + r
+    for t in (8192, 32):
+        ar, one, zero = torch.arange(t, dtype=torch.int32, device=dev), torch.ones(t, dtype=torch.int32, device=dev), torch.zeros(t, dtype=torch.int32, device=dev)
+        seg = scan.Segments(ar, ar, ar, one, ar, 1) if t <= 32 else scan.Segments(zero, zero, i32([0]), i32([t]), i32([0]), t)
+        n_seq, pos1 = seg.first.numel(), ar + 5
+        # ---- step between the layers: everything the residual takes, beside the plain residual add + norm
+        x32, x16, h16, d16 = rnd(t, width, dt=torch.float32), rnd(t, width), rnd(t, width), rnd(t, width)
+        xo, g16 = torch.empty_like(x32), torch.ones(width, device=dev, dtype=torch.bfloat16)
+        z = moe.router_logits(h16, ew.router)
+        idx, wts = moe.route(z[:, :E + ident], ew.correction, top, "softmax", False, 1.0)
+        y, row = moe.experts_rows(h16, idx, ew.w13, ew.w2, 0, 7.0, kx.UNIT_SLOPE)
+        gates, tails = lay.gates(h16), torch.zeros(max(n_seq, 1), width, dtype=torch.bfloat16, device=dev)
+        local = int((idx < E).sum())
+        args = dict(ld=width, n=t, dtype=torch.bfloat16, x_out=xo, mix=d16, gates=gates, gate_b=lay.gate_b, h=h16,
+                    routed=decoder.Routed(y, row, idx, wts, E), shared=x16, shared_gate=z[:, E + ident:], shift=lay.shift, tail=tails,
+                    seg=seg, positions=pos1)
+        pair("step between layers (gates, experts' sum, residual, norm, shift; like: residual + norm)", f"{t} x {width}",
+             (lambda: decoder.parallel_step(x32, width, 1.0, 1e-5, **args), t * width * (8 + 2 + 4 + 2 + 2 + 2 + 2) + local * width * 2, 0),
+             (lambda: basic.add_rmsnorm(x16, d16, g16, 1e-5), t * width * 8, 0))
+        # ---- experts: routing, plan, gather, both products, unit; beside the same with SwiGLU and the combine
+        ebytes = min(E, t * top) * 3 * width * ff * 2
+        need = (ebytes + t * width * 2 + local * width * 2, 2 * local * 3 * width * ff)
+        i2, w2_ = moe.route(z[:, :E], None, top, "softmax", False, 1.0)
+        pair("routed experts (like: with SwiGLU and combine)", f"{t} tokens, {top} of {E}",
+             (lambda: moe.experts_rows(h16, idx, ew.w13, ew.w2, 0, 7.0, kx.UNIT_SLOPE), *need),
+             (lambda: moe.experts_forward(h16, i2, w2_, ew.w13, ew.w2, 0), ebytes + t * width * 4, 2 * t * top * 3 * width * ff))
+        pair("routing (like: sigmoid, normalised)", f"{t} x {E + ident}",
+             (lambda: moe.route(z[:, :E + ident], ew.correction, top, "softmax", False, 1.0), t * (z.stride(0) * 4 + top * 8), 0),
+             (lambda: moe.route(z[:, :E], ew.correction[:E], top, "sigmoid", True, 1.0), t * (z.stride(0) * 4 + top * 8), 0))
+        # ---- latent attention around the attention itself
+        proj, q = rnd(t, aw.down.n), rnd(t, aw.uq.n)
+        cache = torch.zeros(max(t, 64) // bs + 1, bs, cw, dtype=torch.bfloat16, device=dev)
+        kvp, gam, qn = rnd(t, cw), torch.ones(c, device=dev, dtype=torch.bfloat16), rnd(t, qr)
+        gq = torch.ones(qr, device=dev, dtype=torch.bfloat16)
+        pair("latent prologue (like: query norm, cache append)", f"{t} tokens",
+             (lambda: latent.prep(proj, m, pos1, ar, cache), t * (qr + cw) * 4, 0),
+             (lambda: (basic.rmsnorm(qn, gq, 1e-5), mla.kv_append(kvp, gam, 1e-5, pos1, ar, 1e4, cache.view(-1, cw), c, r)), t * (qr + cw) * 4, 0))
+        if t > 32:
+            qs = torch.empty(t, H * (d + r), dtype=torch.bfloat16, device=dev)
+            pair("query rotation (like: split and rotate)", f"{t} tokens", (lambda: latent.rotate_heads(q, m, pos1), t * H * r * 4, 0),
+                 (lambda: mla.q_prepare(qs, pos1, 1e4, H, d, r), t * H * (d + r) * 4, 0))
+        else:
+            qa, ol = torch.empty(t, H, cw, dtype=torch.bfloat16, device=dev), rnd(t, H, c)
+            qh, oh, out = rnd(H, t, d), rnd(H, t, c), torch.empty(t, H * v, dtype=torch.bfloat16, device=dev)
+            wk = aw.uk.reshape(H * c, d)
+            pair("queries to the latent space", f"{t} tokens",
+                 (lambda: latent.head_linear(q, q.stride(0), d + r, aw.uk, qa, qa.stride(0), cw, t), (H * c * d + t * H * (d + c)) * 2, 2 * t * H * c * d),
+                 (lambda: mla.per_head_linear(qh, wk), (H * c * d + t * H * (d + c)) * 2, 2 * t * H * c * d))
+            wv = aw.uv.reshape(H * v, c)
+            pair("latents to values (like: with the transpose)", f"{t} tokens",
+                 (lambda: latent.head_linear(ol, ol.stride(0), c, aw.uv, out, out.stride(0), v, t), (H * v * c + t * H * (v + c)) * 2, 2 * t * H * c * v),
+                 (lambda: mla.transpose_heads(mla.per_head_linear(oh, wv)), (H * v * c + t * H * (v + c)) * 2, 2 * t * H * c * v))
+        # ---- recurrence: rows in and out, state read and written once per sequence
+        gp, st = rnd(t, gw.proj.n), torch.zeros(n_seq, gh, 128, 128, dtype=torch.float32, device=dev)
+        sbytes = t * (gh * 128 * 5 + gm.rank) * 2 + n_seq * gh * 128 * 128 * 8
+        mixed, gg = rnd(t, 3 * gh * 128), -torch.rand(t, gh, device=dev)
+        beta, gate = torch.rand(t, gh, device=dev), rnd(t * gh, 128)
+        gst = torch.zeros(n_seq, gh, 128, 128, dtype=torch.float32, device=dev)
+        nw = torch.ones(128, dtype=torch.bfloat16, device=dev)
+        like = (lambda: gdn.step(gst, ar, mixed, 0, gh * 128, 2 * gh * 128, gg, beta, gh, gh)) if t <= 32 else \
+            (lambda: gdn.chunked(mixed, 0, gh * 128, 2 * gh * 128, gg, beta, gst[0], gh, gh))
+        pair("recurrence with decay, norm and gate (like: Gated DeltaNet, gated norm)", f"{t} tokens, {gh} heads x 128 x 128",
+             (lambda: gla.recurrence(gp, gm, st, seg, pos1, gw.o.k), sbytes, 0),
+             (lambda: basic.gated_rmsnorm(like().view(t * gh, 128), gate, nw), sbytes, 0))
+    # ---- prompt attention, whole prompt: the products a pair needs with keys and values expanded; expansion included below
+    t = 8192
+    table = (torch.arange(t // bs, dtype=torch.int32, device=dev) + 1)[None]
+    cache, q, ql, qp = rnd(t // bs + 1, bs, cw), rnd(t, aw.uq.n), rnd(H, t, c), rnd(t, H, r)
+    out = torch.empty(t, H * v, dtype=torch.bfloat16, device=dev)
+    e0, et, pos = i32([0]), i32([t]), torch.arange(t, dtype=torch.int32, device=dev)
+    full = t * (t + 1) // 2
+    flops, absorbed = 2 * full * H * (d + r + v), 2 * full * H * (2 * c + r)
+    lat, key = latent.gather(cache, m, table, e0, et, e0, t)
+    kv = gemm.linear(lat, aw.ukv)
+    L, _lib, ptr = latent._lib.lib(), latent._lib, latent._lib.ptr
+    tiles = lambda: _lib.check(L.b200_attn_heads_prefill(
+        ptr(q), q.stride(0), ptr(kv), ptr(key), key.shape[1], ptr(out), out.stride(0), ptr(e0), ptr(et), ptr(et), ptr(e0), 1, t, t,
+        lat.shape[0], 0, H, m.d, m.r, m.v, latent._f(m.scale), ptr(_lib.status_word(dev)), _lib.stream()), "attn_heads_prefill")
+    like = lambda: mla.attention(ql, qp, cache.view(-1, cw), table, bs, pos, c, r, m.scale, max_keys=t)
+    pair("prompt attention, products executed (like: absorbed)", f"{t} tokens", (tiles, 0, flops), (like, 0, absorbed))
+    pair("prompt attention with expansion, expanded products counted for both", f"{t} tokens",
+         (lambda: latent.attend_tiles(q, m, *latent.gather(cache, m, table, e0, et, e0, t), aw.ukv, e0, et, et, e0, t, out), 0,
+          flops + 2 * t * H * c * (d + v)), (like, 0, flops))
+    for b in (1, 32):
+        tb = (torch.arange(b * pages, dtype=torch.int32, device=dev) + 1).view(b, pages)
+        cache = rnd(b * pages + 1, bs, cw)
+        qa, ql, qp, pos = rnd(b, H, cw), rnd(H, b, c), rnd(b, H, r), i32([ctx - 1] * b)
+        seq = torch.arange(b, dtype=torch.int32, device=dev)
+        need = (b * ctx * cw * 2, 2 * b * ctx * H * (2 * c + r))
+        pair("decode attention", f"batch {b}, {ctx} keys", (lambda: latent.attend_rows(qa, m, cache, tb, pos, ctx), *need),
+             (lambda: mla.attention(ql, qp, cache.view(-1, cw), tb, bs, pos, c, r, m.scale, seq_of_token=seq, max_keys=ctx), *need))
+    return rows_out
+
+
 def run(args) -> dict:
     from ..ops import _lib
     from .clocks import ClockSampler
@@ -317,21 +444,25 @@ def run(args) -> dict:
     out: dict = {"metric": f"{name} design: prefill and decode throughput", "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True,
                  "steps": timer.steps, "warmup": timer.warmup, "dtype": "bf16", "data": "synthetic", "designs": {}}
     slots = 32
-    sizes = SIZES if name == "rutulix" else ZG_SIZES
-    models, kernels = (_models, _kernels) if name == "rutulix" else (_zg_models, _zg_kernels)
+    sizes, models, kernels, closest = {
+        "rutulix": (SIZES, _models, _kernels, "full-attention decoder, fp8 weights"),
+        "zigasun": (ZG_SIZES, _zg_models, _zg_kernels, "Gated-DeltaNet / full-attention decoder, fp8 weights"),
+        "kemirax": (KX_SIZES, _kx_models, _kx_kernels, "latent-attention decoder with routed experts, bf16 weights")}[name]
     with torch.no_grad(), ClockSampler(0) as clk:
         for size in ([args.design_size] if args.design_size else list(sizes)):
             new, old = models(size, dev, prompt, slots)
             if name == "rutulix":
                 width, heads, kv, dim, inter, chunk = SIZES[size]
                 rec = {"layers": LAYERS, "width": width, "heads": heads, "kv_heads": kv, "dim": dim, "ff": inter * 3 // 2, "chunk": chunk}
-            else:
+            elif name == "zigasun":
                 keys = ("width", "heads", "kv_heads", "dim", "vdim", "ff", "inner", "state", "dt_rank")
                 rec = {"layers": LAYERS, **dict(zip(keys, ZG_SIZES[size]))}
+            else:
+                keys = ("width", "heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank", "gla_heads", "ff", "experts", "identity", "top")
+                rec = {"layers": KX_LAYERS, **dict(zip(keys, KX_SIZES[size]))}
             rec.update({"prompt": prompt, name: _throughput(new, dev, prompt, slots, timer)})
             torch.cuda.empty_cache()
-            rec["closest (" + ("full-attention decoder" if name == "rutulix" else "Gated-DeltaNet / full-attention decoder") + ", fp8 weights)"] = \
-                _throughput(old, dev, prompt, slots, timer)
+            rec[f"closest ({closest})"] = _throughput(old, dev, prompt, slots, timer)
             torch.cuda.empty_cache()
             rec["kernels"] = kernels(size, dev, timer, prompt)
             torch.cuda.empty_cache()
