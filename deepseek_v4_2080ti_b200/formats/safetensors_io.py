@@ -23,7 +23,7 @@ _RD = {v: k for k, v in _DT.items()}
 
 def _raw(t: torch.Tensor) -> bytes:
     t = t.detach().contiguous().cpu()
-    return t.view(torch.uint8).numpy().tobytes() if t.numel() else b""
+    return t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b""
 
 
 def write_file(path: str, tensors: dict[str, torch.Tensor], metadata: dict[str, str] | None = None) -> int:
