@@ -61,8 +61,9 @@ struct Ring {
   }
 };
 
-// VN: columns of a value slice rounded up to 32 (the accumulator's width in tensor memory and of the products).
-template <int VN>
+// VN: columns of a value slice rounded up to 32 (the accumulator's width in tensor memory and of the products).  SL: key slabs
+// where none has a ragged end (loops the issuer has unrolled), or 0.
+template <int VN, int SL>
 __global__ void __launch_bounds__(NTHREADS, 1)
 heads_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmKV,
                      const __grid_constant__ CUtensorMap tmR, Params p) {
@@ -71,7 +72,7 @@ heads_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   constexpr int VS = (VN + 63) / 64;                                     // slabs of the value slice
   extern __shared__ uint8_t smem_base[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_base) + 1023) & ~uintptr_t(1023));
-  const int slabs = p.slabs_d + p.slabs_r, stages = p.stages;
+  const int slabs = SL ? SL : p.slabs_d + p.slabs_r, stages = p.stages;
   uint8_t* sQ = smem;                                   // [2 streams][slabs] atoms
   uint8_t* sR = sQ + 2 * slabs * ATOM;                  // ring of slabs
   uint64_t* bars = reinterpret_cast<uint64_t*>(sR + stages * ATOM);
@@ -94,8 +95,8 @@ heads_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   const int q_row0 = p.q_start[b] + q0;
   const int pos0 = kv_len - q_len + q0;      // position of the first query row
   const bool two = q0 + BQ < q_len;          // the second stream has rows
-  const int n_tiles0 = (min(kv_len, pos0 + BQ) + BKV - 1) / BKV;
-  const int n_tiles1 = two ? (min(kv_len, pos0 + 2 * BQ) + BKV - 1) / BKV : 0;
+  const int n_tiles0 = __shfl_sync(0xffffffffu, (min(kv_len, pos0 + BQ) + BKV - 1) / BKV, 0);
+  const int n_tiles1 = __shfl_sync(0xffffffffu, two ? (min(kv_len, pos0 + 2 * BQ) + BKV - 1) / BKV : 0, 0);
   const int n_tiles = max(n_tiles0, n_tiles1);
 
   if (threadIdx.x == 0) {
@@ -119,7 +120,7 @@ heads_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem = *tmem_slot;
+  const uint32_t tmem = __shfl_sync(0xffffffffu, *tmem_slot, 0);
 
   // registers per thread at launch: 168 (3 x 168 = 2 x 216 + 72)
   if (warp >= 8) {
@@ -160,6 +161,7 @@ heads_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     } else if (warp == 9) {
       // The whole warp walks the loop, so that addresses and descriptors stay warp-uniform, and one elected lane issues.
       bool ok = true;
+      const uint32_t on = elect_one();
       auto wait = [&](uint64_t* bar, uint32_t parity) {
         ok = __all_sync(0xffffffffu, mbar_wait(bar, parity));
         return ok;
@@ -170,19 +172,18 @@ heads_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       // scores of a tile whose key slabs begin at ring position r (by value: both streams walk the same slabs); the tile's
       // last stream gives them back
       auto issue_s = [&](const int m, Ring r, bool last) {
-        for (int s = 0; s < slabs; ++s) {
+#pragma unroll
+        for (int s = 0; s < (SL ? SL : slabs); ++s) {
           if (!wait(&r_full[r.st], r.ph)) return;
           tc_fence_after();
           const uint64_t dk = ring + r.st * (ATOM >> 4), dq = dq0 + (m * slabs + s) * (ATOM >> 4);
-          const int steps = s == p.slabs_d - 1 ? steps_d : s == slabs - 1 ? steps_r : 4;
-          if (elect_one()) {
-            umma_bf16_ss(tmem + m * 128, dq, dk, idesc_qk, s ? 1u : 0u);
+          const int steps = SL ? 4 : s == p.slabs_d - 1 ? steps_d : s == slabs - 1 ? steps_r : 4;
+          umma_bf16_ss_warp(on, tmem + m * 128, dq, dk, idesc_qk, s ? 1u : 0u);
 #pragma unroll
-            for (int kk = 1; kk < 4; ++kk)
-              if (kk < steps) umma_bf16_ss(tmem + m * 128, dq + 2 * kk, dk + 2 * kk, idesc_qk, 1u);
-            if (last) umma_commit(&r_empty[r.st]);
-            if (s + 1 == slabs) umma_commit(&s_full[m]);
-          }
+          for (int kk = 1; kk < 4; ++kk)
+            if (kk < steps) umma_bf16_ss_warp(on, tmem + m * 128, dq + 2 * kk, dk + 2 * kk, idesc_qk, 1u);
+          if (last) umma_commit_warp(on, &r_empty[r.st]);
+          if (s + 1 == slabs) umma_commit_warp(on, &s_full[m]);
           r.next(stages);
         }
       };
@@ -194,7 +195,7 @@ heads_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         for (int s = 0; s < slabs; ++s) v.next(stages);
         if (VS == 2 && v.st == stages - 1) { // the stage that was left out
           if (!wait(&r_full[v.st], v.ph)) break;
-          if (elect_one()) mbar_arrive(&r_empty[v.st]);
+          if (on) mbar_arrive(&r_empty[v.st]);
           v.next(stages);
         }
         k = v;
@@ -213,15 +214,14 @@ heads_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
             if (!ok) break;
             tc_fence_after();
             const uint64_t dv = desc_mn_sw128(sR, ATOM, 1024) + v.st * (ATOM >> 4);
-            if (elect_one()) {
-              umma_bf16_ts(tmem + 256 + m * 128, tmem + m * 128, dv, idesc_pv, j ? 1u : 0u);
+            umma_bf16_ts_warp(on, tmem + 256 + m * 128, tmem + m * 128, dv, idesc_pv, j ? 1u : 0u);
 #pragma unroll
-              for (int kk = 1; kk < 8; ++kk) umma_bf16_ts(tmem + 256 + m * 128, tmem + m * 128 + kk * 8, dv + kk * 128, idesc_pv, 1u);
-              umma_commit(&pv_done[m]);
-              if (m == (two ? 1 : 0)) {
+            for (int kk = 1; kk < 8; ++kk)
+              umma_bf16_ts_warp(on, tmem + 256 + m * 128, tmem + m * 128 + kk * 8, dv + kk * 128, idesc_pv, 1u);
+            umma_commit_warp(on, &pv_done[m]);
+            if (m == (two ? 1 : 0)) {
 #pragma unroll
-                for (int s = 0; s < VS; ++s) umma_commit(&r_empty[v.st + s]);
-              }
+              for (int s = 0; s < VS; ++s) umma_commit_warp(on, &r_empty[v.st + s]);
             }
           }
           // the second stream sees at least as many tiles as the first, so it is the one that gives slabs back
@@ -360,18 +360,28 @@ heads_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   }
 }
 
-template <int VN>
-int launch(const CUtensorMap& q, const CUtensorMap& kv, const CUtensorMap& r, const Params& p, dim3 grid, size_t smem,
-           cudaStream_t stream) {
+template <int VN, int SL>
+int launch_as(const CUtensorMap& q, const CUtensorMap& kv, const CUtensorMap& r, const Params& p, dim3 grid, size_t smem,
+              cudaStream_t stream) {
   static PerDeviceOnce once_;
   bool& configured = once_.slot();
   if (!configured) {
-    const cudaError_t e = cudaFuncSetAttribute(heads_prefill_kernel<VN>, cudaFuncAttributeMaxDynamicSharedMemorySize, 232448);
+    const cudaError_t e = cudaFuncSetAttribute(heads_prefill_kernel<VN, SL>, cudaFuncAttributeMaxDynamicSharedMemorySize, 232448);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
-  heads_prefill_kernel<VN><<<grid, NTHREADS, smem, stream>>>(q, kv, r, p);
+  heads_prefill_kernel<VN, SL><<<grid, NTHREADS, smem, stream>>>(q, kv, r, p);
   return (int)cudaGetLastError();
+}
+
+template <int VN>
+int launch(const CUtensorMap& q, const CUtensorMap& kv, const CUtensorMap& r, const Params& p, dim3 grid, size_t smem,
+           cudaStream_t stream) {
+  if (p.D % 64 == 0 && p.R % 64 == 0) {
+    if (p.slabs_d + p.slabs_r == 2) return launch_as<VN, 2>(q, kv, r, p, grid, smem, stream);
+    if (p.slabs_d + p.slabs_r == 3) return launch_as<VN, 3>(q, kv, r, p, grid, smem, stream);
+  }
+  return launch_as<VN, 0>(q, kv, r, p, grid, smem, stream);
 }
 
 }  // namespace headsattn

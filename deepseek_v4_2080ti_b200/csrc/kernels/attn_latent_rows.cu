@@ -3,10 +3,11 @@
 //
 //   o[h] = softmax_j(scale q[h] . row(j)) latent(j)
 //
-// Used for decode batches and short portions, and for every row in fp32.  Sizes are run-time values.
+// Used for decode batches and short portions that attn_latent_decode.cu does not take, and for every row in fp32.  Sizes are
+// run-time values.
 //
-// bf16 (latent_rows_mma_kernel): a block takes one row, 16 MT heads (the M side of m16n8k16 products; 16 heads share a key
-// tile, so a 128-row tcgen05 tile would be an eighth full) and one slice of the row's keys.  Tiles of 32 cache rows are
+// bf16 (latent_rows_mma_kernel): a block takes one row, 16 MT heads (the M side of m16n8k16 products) and one slice of the
+// row's keys.  Tiles of 32 cache rows are
 // copied ahead with cp.async, once for all heads of the block.  Four warps share 16 heads: each scores 8 keys of a tile, the
 // probabilities travel through shared memory, and each sums its 16-column blocks of the latent.
 // fp32 and wider latents (latent_rows_kernel): CUDA cores, four heads per block, a warp per key for the dot products.
@@ -458,5 +459,15 @@ extern "C" int b200_attn_latent_rows(const void* q, const void* cache, void* out
   else if (heads == 32) rc = pick_mma<2>(q, cache, out, p, rows, stream);
   else rc = pick_mma<1>(q, cache, out, p, rows, stream);
   if (rc || splits == 1) return rc;
+  return f32 ? merge<float>(p, out, rows, stream) : merge<__nv_bfloat16>(p, out, rows, stream);
+}
+
+// The merge on its own: partial as above (sums, then maxima and weights), out [rows, H, C].
+extern "C" int b200_attn_latent_merge(const float* partial, void* out, int rows, int H, int C, int splits, int f32, cudaStream_t stream) {
+  if (rows <= 0 || rows > 65535 || H <= 0 || C <= 0 || (C & 15) || splits <= 1 || !partial) return -6;
+  Rows p = {};
+  p.H = H; p.C = C; p.splits = splits;
+  p.partial = const_cast<float*>(partial);
+  p.stats = p.partial + (size_t)rows * H * splits * C;
   return f32 ? merge<float>(p, out, rows, stream) : merge<__nv_bfloat16>(p, out, rows, stream);
 }

@@ -35,13 +35,13 @@ __global__ void bias_xielu_kernel(const T* __restrict__ in, const float* __restr
 }
 
 template <typename T>
-__global__ void glu_kernel(const T* __restrict__ in, T* __restrict__ out, long long nvec_total, int nvec, int tile, GluShape s) {
+__global__ void glu_kernel(const T* __restrict__ in, int ld, T* __restrict__ out, long long nvec_total, int nvec, int tile, GluShape s) {
   pdl_grid_trigger();
   pdl_grid_wait();
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < nvec_total; i += (long long)gridDim.x * blockDim.x) {
     const long long row = i / nvec;
     const int c = (int)(i - row * nvec) * 8;
-    const T* src = in + row * nvec * 16 + (c / tile) * 2 * tile + c % tile;
+    const T* src = in + row * ld + (c / tile) * 2 * tile + c % tile;
     float g[8], u[8];
     load8(src, g);
     load8(src + tile, u);
@@ -53,19 +53,19 @@ __global__ void glu_kernel(const T* __restrict__ in, T* __restrict__ out, long l
 
 }  // namespace
 
-// in [rows, 2 * inter], out [rows, inter]; inter a multiple of tile, tile a multiple of 8.
-extern "C" int b200_glu(const void* in, void* out, long long rows, int inter, int tile, float limit, float slope, int f32,
+// in: rows of 2 * inter columns, `ld` apart, out [rows, inter]; inter a multiple of tile, tile and ld multiples of 8.
+extern "C" int b200_glu(const void* in, int ld, void* out, long long rows, int inter, int tile, float limit, float slope, int f32,
                         cudaStream_t stream) {
-  if (rows <= 0 || inter <= 0 || tile <= 0 || (tile & 7) || inter % tile) return -6;
+  if (rows <= 0 || inter <= 0 || tile <= 0 || (tile & 7) || inter % tile || (ld & 7) || ld < 2 * inter) return -6;
   const int nvec = inter >> 3;
   const long long total = rows * nvec;
   const long long blocks = (total + 255) / 256;
   const dim3 grid((unsigned)(blocks < 148 * 16 ? blocks : 148 * 16));
   const GluShape s = {limit, slope};
   if (f32)
-    return (int)launch_pdl(glu_kernel<float>, grid, dim3(256), 0, stream, reinterpret_cast<const float*>(in),
+    return (int)launch_pdl(glu_kernel<float>, grid, dim3(256), 0, stream, reinterpret_cast<const float*>(in), ld,
                            reinterpret_cast<float*>(out), total, nvec, tile, s);
-  return (int)launch_pdl(glu_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, reinterpret_cast<const __nv_bfloat16*>(in),
+  return (int)launch_pdl(glu_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, reinterpret_cast<const __nv_bfloat16*>(in), ld,
                          reinterpret_cast<__nv_bfloat16*>(out), total, nvec, tile, s);
 }
 

@@ -245,13 +245,10 @@ __host__ __device__ constexpr size_t stage_bytes(int VB) {
 template <int DT, int CL>
 constexpr size_t scan_smem(int VB) { return 2 * stage_bytes<DT, CL>(VB) + (size_t)2 * VB * (DT + 8) * 2; }
 
-template <int DT>
-constexpr int SUBS = DT >= 128 ? 8 : 4;                 // warps per 16 value columns
-
-// grid (ceil(V / VB), H, entries), SUBS VB / 16 warps: SUBS of them own value columns 16 i .. 16 i + 15.
-template <int DT, int CL>
+// grid (ceil(V / VB), H, entries), W VB / 16 warps: W of them (4 or 8) own value columns 16 i .. 16 i + 15.
+template <int DT, int CL, int W>
 __global__ void __launch_bounds__(512) gla_chunk_scan_kernel(ChunkParams p) {
-  constexpr int LQ = DT + 8, LA = CL + 8, MT = CL / 16, W = SUBS<DT>, ND = DT / W, NS = ND / 8, NJ = W == 8 ? 1 : 2;
+  constexpr int LQ = DT + 8, LA = CL + 8, MT = CL / 16, ND = DT / W, NS = ND / 8, NJ = W == 8 ? 1 : 2;
   // channels, fragments of S^T and 8-column tiles of the output of a warp
   extern __shared__ __align__(16) uint8_t smem[];
   const int tid = threadIdx.x, nthr = blockDim.x, lane = tid & 31, g = lane >> 2, tig = lane & 3;
@@ -416,28 +413,39 @@ __global__ void __launch_bounds__(512) gla_chunk_scan_kernel(ChunkParams p) {
     }
 }
 
+template <int DT, int CL, int W>
+int launch_scan(const ChunkParams& p, int groups, cudaStream_t stream) {
+  static PerDeviceOnce once_;
+  bool& configured = once_.slot();
+  if (!configured) {
+    const cudaError_t e = cudaFuncSetAttribute(gla_chunk_scan_kernel<DT, CL, W>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    if (e != cudaSuccess) return (int)e;
+    configured = true;
+  }
+  return (int)launch_pdl(gla_chunk_scan_kernel<DT, CL, W>, dim3((p.V + 16 * groups - 1) / (16 * groups), p.H, p.entries),
+                         dim3(groups * W * 32), scan_smem<DT, CL>(16 * groups), stream, p);
+}
+
 template <int DT, int CL>
 int launch(ChunkParams p, int chunks, cudaStream_t stream) {
   static PerDeviceOnce once_;
   bool& configured = once_.slot();
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(gla_chunk_prep_kernel<DT, CL>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
-    if (e == cudaSuccess)
-      e = cudaFuncSetAttribute(gla_chunk_scan_kernel<DT, CL>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    const cudaError_t e = cudaFuncSetAttribute(gla_chunk_prep_kernel<DT, CL>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
   const size_t prep = (size_t)CL * (DT + 4) * 4 + (size_t)2 * CL * (DT + 8) * 2;
-  cudaError_t e = launch_pdl(gla_chunk_prep_kernel<DT, CL>, dim3(chunks, p.H), dim3(PT), prep, stream, p);
+  const cudaError_t e = launch_pdl(gla_chunk_prep_kernel<DT, CL>, dim3(chunks, p.H), dim3(PT), prep, stream, p);
   if (e != cudaSuccess) return (int)e;
   // 16 columns per block where one wave of blocks takes them, more otherwise
-  constexpr int W = SUBS<DT>;
   int groups = 1;
-  while (groups * W < 16 && (long long)p.entries * p.H * ((p.V + 16 * groups - 1) / (16 * groups)) > 148 && 16 * groups < p.V &&
+  while (groups < 4 && (long long)p.entries * p.H * ((p.V + 16 * groups - 1) / (16 * groups)) > 148 && 16 * groups < p.V &&
          scan_smem<DT, CL>(32 * groups) <= 227 * 1024)
     groups <<= 1;
-  return (int)launch_pdl(gla_chunk_scan_kernel<DT, CL>, dim3((p.V + 16 * groups - 1) / (16 * groups), p.H, p.entries), dim3(groups * W * 32),
-                         scan_smem<DT, CL>(16 * groups), stream, p);
+  if constexpr (DT >= 128)
+    if (groups <= 2) return launch_scan<DT, CL, 8>(p, groups, stream);
+  return launch_scan<DT, CL, 4>(p, groups, stream);
 }
 
 }  // namespace

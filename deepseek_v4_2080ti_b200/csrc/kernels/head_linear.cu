@@ -2,6 +2,9 @@
 // projections of latent attention around its absorbed form).  The weights are streamed once per 64 rows; operands go from
 // global memory straight into tensor-core fragments: the order of the dimensions inside a dot product is free, so a lane takes
 // 16 contiguous bytes of a row as its share of two k-steps.  Prompt-sized batches use the big GEMMs instead.
+//
+// rows_linear_f32: the same for one matrix with few rows of its own and fp32 results (a router): more warps share K, because
+// the features alone would occupy a handful of SMs.
 #include <cuda_bf16.h>
 #include <stdint.h>
 #include "launch.h"
@@ -16,14 +19,22 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1
                : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
-constexpr int WARPS = 4, NW = 16;          // features per block; the warps share K
+constexpr int NW = 16;                     // features per block; the warps share K
 
-// grid (features / 16, heads, rows / (16 MT)), 128 threads; K % 16 == 0 (32-wide chunks, the last may be half).  The warps'
+__device__ __forceinline__ void store2(__nv_bfloat16* p, int n, int N, float a, float b) {        // N is even
+  *reinterpret_cast<__nv_bfloat162*>(p + n) = __floats2bfloat162_rn(a, b);
+}
+__device__ __forceinline__ void store2(float* p, int n, int N, float a, float b) {
+  p[n] = a;
+  if (n + 1 < N) p[n + 1] = b;
+}
+
+// grid (features / 16, heads, rows / (16 MT)); K % 16 == 0 (32-wide chunks, the last may be half).  The warps'
 // sums are added up through shared memory.
-template <int MT>
+template <int MT, int WARPS, typename Out>
 __global__ void __launch_bounds__(WARPS * 32)
 head_linear_kernel(const __nv_bfloat16* __restrict__ x, int ldx, int x_head, const __nv_bfloat16* __restrict__ w,
-                   __nv_bfloat16* __restrict__ y, int ldy, int y_head, int T, int N, int K) {
+                   Out* __restrict__ y, int ldy, int y_head, int T, int N, int K) {
   __shared__ float red[WARPS][MT][2][4][32];
   pdl_grid_trigger();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gr = lane >> 2, kk = lane & 3;
@@ -70,8 +81,21 @@ head_linear_kernel(const __nv_bfloat16* __restrict__ x, int ldx, int x_head, con
       v1 += red[u][mt][nb][hf * 2 + 1][lane];
     }
     const int t = t0 + mt * 16 + gr + hf * 8, n = n0 + nb * 8 + kk * 2;
-    if (t < T && n < N) *reinterpret_cast<__nv_bfloat162*>(y + (size_t)t * ldy + h * y_head + n) = __floats2bfloat162_rn(v0, v1);
+    if (t < T && n < N) store2(y + (size_t)t * ldy + h * y_head, n, N, v0, v1);
   }
+}
+
+template <int WARPS, typename Out>
+int run(const void* x, int ldx, int x_head, const void* w, void* y, int ldy, int y_head, int T, int H, int N, int K, cudaStream_t stream) {
+  const int mt = T <= 16 ? 1 : T <= 32 ? 2 : 4;
+  if ((T + 16 * mt - 1) / (16 * mt) > 65535) return -6;
+  const dim3 grid((N + NW - 1) / NW, H, (T + 16 * mt - 1) / (16 * mt)), block(WARPS * 32);
+  auto xp = reinterpret_cast<const __nv_bfloat16*>(x);
+  auto wp = reinterpret_cast<const __nv_bfloat16*>(w);
+  auto yp = reinterpret_cast<Out*>(y);
+  if (mt == 1) return (int)launch_pdl(head_linear_kernel<1, WARPS, Out>, grid, block, 0, stream, xp, ldx, x_head, wp, yp, ldy, y_head, T, N, K);
+  if (mt == 2) return (int)launch_pdl(head_linear_kernel<2, WARPS, Out>, grid, block, 0, stream, xp, ldx, x_head, wp, yp, ldy, y_head, T, N, K);
+  return (int)launch_pdl(head_linear_kernel<4, WARPS, Out>, grid, block, 0, stream, xp, ldx, x_head, wp, yp, ldy, y_head, T, N, K);
 }
 
 }  // namespace
@@ -80,13 +104,12 @@ head_linear_kernel(const __nv_bfloat16* __restrict__ x, int ldx, int x_head, con
 extern "C" int b200_head_linear(const void* x, int ldx, int x_head, const void* w, void* y, int ldy, int y_head, int T, int H, int N,
                                 int K, cudaStream_t stream) {
   if (T <= 0 || H <= 0 || H > 65535 || N <= 0 || (N & 1) || K <= 0 || (K & 15) || ((ldx | x_head | ldy | y_head) & 7)) return -6;
-  const int mt = T <= 16 ? 1 : T <= 32 ? 2 : 4;
-  if ((T + 16 * mt - 1) / (16 * mt) > 65535) return -6;
-  const dim3 grid((N + NW - 1) / NW, H, (T + 16 * mt - 1) / (16 * mt)), block(WARPS * 32);
-  auto xp = reinterpret_cast<const __nv_bfloat16*>(x);
-  auto wp = reinterpret_cast<const __nv_bfloat16*>(w);
-  auto yp = reinterpret_cast<__nv_bfloat16*>(y);
-  if (mt == 1) return (int)launch_pdl(head_linear_kernel<1>, grid, block, 0, stream, xp, ldx, x_head, wp, yp, ldy, y_head, T, N, K);
-  if (mt == 2) return (int)launch_pdl(head_linear_kernel<2>, grid, block, 0, stream, xp, ldx, x_head, wp, yp, ldy, y_head, T, N, K);
-  return (int)launch_pdl(head_linear_kernel<4>, grid, block, 0, stream, xp, ldx, x_head, wp, yp, ldy, y_head, T, N, K);
+  return run<4, __nv_bfloat16>(x, ldx, x_head, w, y, ldy, y_head, T, H, N, K, stream);
+}
+
+// y [T, ldy] fp32 = x [T, ldx] W [N, K]^T; K % 16 == 0.
+extern "C" int b200_rows_linear_f32(const void* x, int ldx, const void* w, float* y, int ldy, int T, int N, int K,
+                                    cudaStream_t stream) {
+  if (T <= 0 || N <= 0 || K <= 0 || (K & 15) || (ldx & 7) || ldy < N) return -6;
+  return run<8, float>(x, ldx, 0, w, y, ldy, 0, T, 1, N, K, stream);
 }

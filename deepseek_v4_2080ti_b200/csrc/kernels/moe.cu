@@ -1,5 +1,4 @@
 // Routed-expert plumbing around the grouped GEMM (gemm_wdec.cu, grouped mode):
-//   moe_router_rows  - router logits of a short batch;
 //   moe_route        - scores (softmax | sigmoid | sqrt-softplus) + selection bias + top-k + weight normalisation;
 //   moe_plan         - counting sort of the (token, k) routes by local expert: per-expert offsets, the row of every
 //                      route in expert-sorted order, and the (expert, m_tile, row0, rows) work table of both grouped
@@ -15,7 +14,6 @@
 #include <cuda_bf16.h>
 #include <stdint.h>
 #include "glu.cuh"
-#include "launch.h"
 #include "ops.h"
 #include "vec8.cuh"
 
@@ -88,37 +86,6 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int ld, const
   }
   if (fn != 0 && norm_topk)
     for (int k = lane; k < K; k += 32) wts[(size_t)t * K + k] /= wsum;     // lane k & 31 wrote entry k
-}
-
-// z[t, n] = x[t] . w[n] in fp32 for a handful of rows: a warp per output feature, its weights read once for RT rows.
-constexpr int RT = 8;
-
-__global__ void __launch_bounds__(128) moe_router_rows_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w,
-                                                              float* __restrict__ z, int T, int N, int K) {
-  b200::pdl_grid_trigger();
-  b200::pdl_grid_wait();
-  const int n = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31, t0 = blockIdx.y * RT;
-  if (n >= N) return;
-  float acc[RT] = {};
-#pragma unroll 2
-  for (int k = lane * 8; k < K; k += 256) {
-    float f[8];
-    b200::load8(w + (size_t)n * K + k, f);
-#pragma unroll
-    for (int t = 0; t < RT; ++t) {
-      if (t0 + t < T) {
-        float a[8];
-        b200::load8(x + (size_t)(t0 + t) * K + k, a);
-#pragma unroll
-        for (int j = 0; j < 8; ++j) acc[t] = fmaf(f[j], a[j], acc[t]);
-      }
-    }
-  }
-#pragma unroll
-  for (int t = 0; t < RT; ++t) {
-    const float v = b200::warp_sum_all(acc[t]);
-    if (lane == 0 && t0 + t < T) z[(size_t)(t0 + t) * N + n] = v;
-  }
 }
 
 __device__ __forceinline__ int warp_scan(int v, int lane) {                // inclusive
@@ -299,13 +266,6 @@ int b200_moe_route(const float* logits, int ld, const float* bias, int T, int E,
   B200_ROUTE(1) B200_ROUTE(2) B200_ROUTE(4) B200_ROUTE(8) B200_ROUTE(16) B200_ROUTE(32)
 #undef B200_ROUTE
   return -6;
-}
-
-// fp32 logits z [T, N] of bf16 rows x [T, K] and router w [N, K] for short batches; K % 8 == 0.
-int b200_moe_router_rows(const void* x, const void* w, float* z, int T, int N, int K, cudaStream_t stream) {
-  if (T <= 0 || N <= 0 || K <= 0 || (K & 7)) return -6;
-  return (int)b200::launch_pdl(moe_router_rows_kernel, dim3((N + 3) / 4, (T + RT - 1) / RT), dim3(128), 0, stream,
-                               reinterpret_cast<const __nv_bfloat16*>(x), reinterpret_cast<const __nv_bfloat16*>(w), z, T, N, K);
 }
 
 // Plans the grouped GEMMs of this rank's experts [expert_lo, expert_hi).  All outputs are device buffers:

@@ -180,7 +180,7 @@ int b200_gemm_bf16_bias_xielu(const void* W, const void* X, const float* bias, f
                               cudaStream_t stream);
 int b200_bias_xielu(const void* in, const float* bias, void* out, long long rows, int ld, float ap, float an, int f32,
                     cudaStream_t stream);
-int b200_glu(const void* in, void* out, long long rows, int inter, int tile, float limit, float slope, int f32,
+int b200_glu(const void* in, int ld, void* out, long long rows, int inter, int tile, float limit, float slope, int f32,
              cudaStream_t stream);
 int b200_gemm_bf16_glu(const void* W, const void* X, void* out_bf16, int T, int N, int K, float limit, float slope, int* status,
                        cudaStream_t stream);

@@ -28,8 +28,9 @@ from .paged import PagedRuntime
 
 ARCH = "Kemirax"
 UNIT_SLOPE = 1.702
+SHORT_ROWS = 128              # batches up to this are bound by the weights' bytes and by launches
 # kernel sources the runtime launches (a partial build compiles only these)
-KERNEL_SOURCES = ("parallel_step.cu", "latent_prep.cu", "attn_latent_rows.cu", "attn_heads_prefill.cu",
+KERNEL_SOURCES = ("parallel_step.cu", "latent_prep.cu", "attn_latent_rows.cu", "attn_latent_decode.cu", "attn_heads_prefill.cu",
                   "head_linear.cu", "gated_linear.cu", "gla_chunk.cu", "moe.cu",
                   "bias_act.cu", "gemm_f32.cu", "gemm_wdec.cu", "gemm_bf16_2cta.cu", "elementwise.cu", "sampling.cu", "bounds.cu")
 
@@ -272,7 +273,7 @@ class ExpertsWeights:
     correction: torch.Tensor          # fp32 [experts + identity]
     w13: moe.ExpertWeights
     w2: moe.ExpertWeights
-    up: Projection | None = None      # shared expert: gate and up features interleaved in tiles
+    up: Projection | None = None      # shared expert: gate and up features interleaved in tiles (rows of the layer's ``wide``)
     down: Projection | None = None
 
 
@@ -281,7 +282,8 @@ class KemiraxLayer:
     mix: LatentWeights | LinearWeights
     norm: float
     shift: torch.Tensor               # fp32 [ld]
-    gates: Projection                 # rows [mixer's gate (ld) | feed-forward's gate (ld)]
+    wide: Projection                  # everything that reads the norm: rows [gates | shared expert's gate and up features]
+    gates: Projection                 # its rows [mixer's gate (ld) | feed-forward's gate (ld)]
     gate_b: torch.Tensor              # fp32 [2 ld]
     ff: ExpertsWeights | None = None
 
@@ -339,10 +341,18 @@ class KemiraxWeights:
             gate_b = torch.zeros(2, self.ld, dtype=torch.float32, device=self.device)
             for j, n in enumerate(names):
                 gate_b[j, :cfg.width] = t[f"{p}{n}.b"].to(self.device, torch.float32)
-            self.layers.append(KemiraxLayer(
-                mix, float(t[p + "norm1"]), self._row(t[p + "shift"], self.ld),
-                self._proj(_cat_rows([(t[p + n], self.ld) for n in names]), tile_n=True), gate_b.view(-1),
-                self._experts(L.mlp, sub("mlp")) if L.mlp else None))
+            ff = self._experts(L.mlp, sub("mlp")) if L.mlp else None
+            parts, ng = [(t[p + n], self.ld) for n in names], len(names) * self.ld
+            if ff is not None and L.mlp.shared_ff:
+                # rows in whole tiles of the pair GEMM, so that either part can be multiplied alone
+                up = decoder.interleave_glu(t[p + "mlp.shared.gate"], t[p + "mlp.shared.up"])
+                parts = [(_cat_rows(parts), (ng + 255) // 256 * 256), (up, up.shape[0])]
+            wide = self._proj(_cat_rows(parts), tile_n=True)
+            gates = wide
+            if ff is not None and L.mlp.shared_ff:
+                ng = parts[0][1]
+                gates, ff.up = wide.part(0, ng), wide.part(ng, ng + parts[1][1])
+            self.layers.append(KemiraxLayer(mix, float(t[p + "norm1"]), self._row(t[p + "shift"], self.ld), wide, gates, gate_b.view(-1), ff))
 
     def _proj(self, w: torch.Tensor, pad_n: bool = True, tile_n: bool = False) -> Projection:
         return Projection.make(w, self.dtype, self.device, pad_n, tile_n)
@@ -405,8 +415,7 @@ class KemiraxWeights:
         rows = [(t["router"], f.experts + f.identity)] + ([(t["shared.sg"], 1)] if f.shared_ff else [])
         ew = ExpertsWeights(f, self._proj(_cat_rows(rows)), self._row(t["correction"], f.experts + f.identity), pack(w13), pack(w2))
         if f.shared_ff:
-            ew.up = self._proj(decoder.interleave_glu(t["shared.gate"], t["shared.up"]))
-            down = torch.zeros(self.cfg.width, ew.up.n // 2, dtype=t["shared.down"].dtype, device=t["shared.down"].device)
+            down = torch.zeros(self.cfg.width, (f.shared_ff + decoder.GLU_TILE - 1) // decoder.GLU_TILE * decoder.GLU_TILE, dtype=t["shared.down"].dtype, device=t["shared.down"].device)
             down[:, :f.shared_ff] = t["shared.down"]
             ew.down = self._proj(down)
         return ew
@@ -416,12 +425,12 @@ class KemiraxWeights:
         n = size(self.embed) + self.head.nbytes()
         for L in self.layers:
             m = L.mix
-            n += L.gates.nbytes()
+            n += L.wide.nbytes()
             n += sum(p.nbytes() for p in ((m.down, m.uq, m.o) if isinstance(m, LatentWeights) else (m.proj, m.o)))
             n += sum(size(x) for x in ((m.uk, m.uv) if isinstance(m, LatentWeights) else (m.m.w2,)))
             n += m.ukv.nbytes() if isinstance(m, LatentWeights) and m.ukv is not None else 0
             if L.ff:
-                n += sum(p.nbytes() for p in (L.ff.router, L.ff.up, L.ff.down) if p is not None)
+                n += sum(p.nbytes() for p in (L.ff.router, L.ff.down) if p is not None)
                 n += size(L.ff.w13.weight) + size(L.ff.w2.weight)
         return n
 
@@ -487,7 +496,8 @@ class KemiraxRuntime(PagedRuntime):
     def _linear(self, i: int, lw: LinearWeights, y: torch.Tensor, positions, meta) -> torch.Tensor:
         return lw.o(gla.recurrence(lw.proj(y), lw.m, self.state[i], meta["segments"], positions, lw.o.k))
 
-    def _experts(self, ew: ExpertsWeights, h: torch.Tensor) -> dict:
+    def _experts(self, ew: ExpertsWeights, h: torch.Tensor, up: torch.Tensor | None = None) -> dict:
+        """``up``: the shared expert's gate and up features, where they are already there."""
         f = ew.spec
         total = f.experts + f.identity
         z = moe.router_logits(h, ew.router)
@@ -495,7 +505,8 @@ class KemiraxRuntime(PagedRuntime):
         y, row = moe.experts_rows(h, idx, ew.w13, ew.w2, 0, f.limit, UNIT_SLOPE)
         out = {"h": h, "routed": Routed(y, row, idx, weights, f.experts)}
         if ew.up is not None:
-            out.update(shared=ew.down(ew.up.glu(h, f.shared_limit, UNIT_SLOPE)), shared_gate=z[:, total:])
+            unit = ew.up.glu(h, f.shared_limit, UNIT_SLOPE) if up is None else decoder.glu(up, decoder.GLU_TILE, f.shared_limit, UNIT_SLOPE)
+            out.update(shared=ew.down(unit), shared_gate=z[:, total:])
         return out
 
     def _forward(self, ids, positions, kv_slots, meta, rows):
@@ -513,11 +524,14 @@ class KemiraxRuntime(PagedRuntime):
 
         for i, lw in enumerate(w.layers):
             h, m = boundary(lw.norm, x_out=x, shift=lw.shift, tail=self.tails[i], seg=meta["segments"], positions=positions)
-            pending = {"gates": lw.gates(h), "gate_b": lw.gate_b}
+            # short batches: one product for all that reads the norm; prompts: the gated unit in its GEMM's epilogue
+            short = lw.ff is not None and lw.ff.up is not None and n <= SHORT_ROWS
+            z = (lw.wide if short else lw.gates)(h)
+            pending = {"gates": z, "gate_b": lw.gate_b}
             pending["mix"] = (self._latent(i, lw.mix, m, positions, kv_slots, meta) if isinstance(lw.mix, LatentWeights)
                               else self._linear(i, lw.mix, m, positions, meta))
             if lw.ff is not None:
-                pending.update(self._experts(lw.ff, h))
+                pending.update(self._experts(lw.ff, h, z[:, lw.gates.n:lw.gates.n + lw.ff.up.n] if short else None))
             if self.residual_tap is not None:
                 boundary(1.0, x_out=x, norm=False)
                 self.residual_tap(i, x[:, :cfg.width].clone())

@@ -72,6 +72,13 @@ class Projection:
             return gemm.linear_bias_xielu(x, self.packed, bias, ap, an)
         return bias_xielu(gemm_f32(x, self.w32), bias, ap, an)
 
+    def part(self, lo: int, hi: int) -> "Projection":
+        """The features [lo, hi) as a projection of their own (the same memory)."""
+        from .gemm import PackedLinear
+        if self.w32 is not None:
+            return Projection(None, self.w32[lo:hi], hi - lo, self.k)
+        return Projection(PackedLinear(self.packed.wfmt, self.packed.weight[lo:hi], None, hi - lo, self.k), None, hi - lo, self.k)
+
     def nbytes(self) -> int:
         return self.n * self.k * (4 if self.packed is None else 2)
 
@@ -200,10 +207,10 @@ def bias_xielu(z: torch.Tensor, bias: torch.Tensor | None, ap: float, an: float)
 
 
 def glu(z: torch.Tensor, tile: int, limit: float, slope: float = 1.702) -> torch.Tensor:
-    """Gated unit over rows of gate and up features interleaved in tiles of ``tile`` columns: the clamped one-plus form
+    """Gated unit over rows (a stride is allowed) of gate and up features interleaved in tiles of ``tile`` columns: the clamped one-plus form
     ``min(g, limit) sigmoid(slope min(g, limit)) (clamp(u, -limit, limit) + 1)``, or ``silu(g) u`` with ``limit`` 0."""
     out = torch.empty(z.shape[0], z.shape[1] // 2, dtype=z.dtype, device=z.device)
-    rc = _lib.lib().b200_glu(_lib.ptr(z), _lib.ptr(out), _ll(z.shape[0]), out.shape[1], tile, _f(limit), _f(slope),
+    rc = _lib.lib().b200_glu(_lib.ptr(z), z.stride(0), _lib.ptr(out), _ll(z.shape[0]), out.shape[1], tile, _f(limit), _f(slope),
                              int(z.dtype == torch.float32), _lib.stream())
     _lib.check(rc, "glu")
     return out

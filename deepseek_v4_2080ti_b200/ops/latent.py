@@ -1,5 +1,6 @@
 """Front-ends of latent attention over a paged cache of one row per token, [latent | rotated key part], shared by all heads:
-prologue (csrc/kernels/latent_prep.cu), single rows in the absorbed form (attn_latent_rows.cu, head_linear.cu), prompt tiles on
+prologue (csrc/kernels/latent_prep.cu), single rows in the absorbed form (attn_latent_decode.cu on the tensor cores,
+attn_latent_rows.cu for other sizes and fp32; head_linear.cu), prompt tiles on
 the tensor cores over keys and values expanded from the latents (attn_heads_prefill.cu).
 
 All of it exists for bf16 and for fp32 activations; the tensors' dtype decides.  Widths are padded to multiples of 16 with
@@ -106,9 +107,10 @@ def pick_splits(blocks: int, keys: int) -> int:
 
 
 def attend_rows(q: torch.Tensor, m: LatentAttention, cache: torch.Tensor, block_table, positions, max_keys: int,
-                seq: torch.Tensor | None = None, splits: int | None = None) -> torch.Tensor:
+                seq: torch.Tensor | None = None, splits: int | None = None, tiles: bool = True) -> torch.Tensor:
     """Absorbed queries q [B, heads, c + r] of single rows, row i at position ``positions[i]`` of the sequence in table row
-    ``seq[i]`` (or i) -> summed latents [B, heads, c].  ``max_keys``: bound on the visible keys of a row."""
+    ``seq[i]`` (or i) -> summed latents [B, heads, c].  ``max_keys``: bound on the visible keys of a row.  ``tiles`` False:
+    not on the tcgen05 kernel, whatever the sizes."""
     b = q.shape[0]
     nb, bs, _ = cache.shape
     f32 = int(q.dtype == torch.float32)
@@ -116,9 +118,12 @@ def attend_rows(q: torch.Tensor, m: LatentAttention, cache: torch.Tensor, block_
     _lib.check_indices(block_table, 0, nb, 3)
     out = torch.empty(b, m.heads, m.c, dtype=q.dtype, device=q.device)
     L = _lib.lib()
+    group = 0 if f32 or not tiles else L.b200_attn_latent_decode_heads(m.heads, m.c, m.cache_width, bs)
     if splits is None:
-        per = L.b200_attn_latent_rows_heads(m.heads, m.c, m.cache_width, b, f32)
-        splits = pick_splits(b * ((m.heads + per - 1) // per), max_keys)
+        per = group or L.b200_attn_latent_rows_heads(m.heads, m.c, m.cache_width, b, f32)
+        blocks = b * ((m.heads + per - 1) // per)
+        # one tcgen05 CTA fills an SM; the other kernels want two blocks or more
+        splits = max(1, min(NUM_SMS // blocks, (max_keys + 127) // 128)) if group else pick_splits(blocks, max_keys)
     per_row = splits * m.heads * (m.c + 2) if splits > 1 else 0
     step = min(b, 65535, WS_LIMIT // per_row if per_row else b)
     ws = None
@@ -132,11 +137,20 @@ def attend_rows(q: torch.Tensor, m: LatentAttention, cache: torch.Tensor, block_
                                          name="latent attention partials")
     for lo in range(0, b, step):
         hi = min(b, lo + step)
-        rc = L.b200_attn_latent_rows(
-            _lib.ptr(q[lo:hi]), _lib.ptr(cache), _lib.ptr(out[lo:hi]), _lib.ptr(block_table if seq is not None else block_table[lo:hi]),
-            _lib.ptr(None if seq is None else seq[lo:hi]), _lib.ptr(positions[lo:hi]), _lib.ptr(ws), hi - lo, block_table.shape[1], bs,
-            m.heads, m.c, m.cache_width, int(splits), _f(m.scale), f32, _lib.stream())
-        _lib.check(rc, "attn_latent_rows", 2 if splits > 1 else 1)
+        qp, op, pos = _lib.ptr(q[lo:hi]), _lib.ptr(out[lo:hi]), _lib.ptr(positions[lo:hi])
+        table = _lib.ptr(block_table if seq is not None else block_table[lo:hi])
+        sq = _lib.ptr(None if seq is None else seq[lo:hi])
+        if group:
+            rc = L.b200_attn_latent_decode(qp, _lib.ptr(cache), op, table, sq, pos, _lib.ptr(ws), hi - lo, block_table.shape[1], nb, bs, m.heads,
+                                           m.c, m.cache_width, int(splits), _f(m.scale), _lib.ptr(_lib.status_word(q.device)), _lib.stream())
+            _lib.check(rc, "attn_latent_decode")
+            if splits > 1:
+                rc = L.b200_attn_latent_merge(_lib.ptr(ws), op, hi - lo, m.heads, m.c, int(splits), f32, _lib.stream())
+                _lib.check(rc, "attn_latent_merge")
+        else:
+            rc = L.b200_attn_latent_rows(qp, _lib.ptr(cache), op, table, sq, pos, _lib.ptr(ws), hi - lo, block_table.shape[1], bs, m.heads, m.c,
+                                         m.cache_width, int(splits), _f(m.scale), f32, _lib.stream())
+            _lib.check(rc, "attn_latent_rows", 2 if splits > 1 else 1)
     return out
 
 

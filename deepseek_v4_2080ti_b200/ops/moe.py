@@ -84,8 +84,8 @@ def router_logits(x: torch.Tensor, w) -> torch.Tensor:
     t, k = x.shape
     assert x.is_contiguous() and k == w.k
     z = torch.empty(t, w.n, dtype=torch.float32, device=x.device)
-    rc = _lib.lib().b200_moe_router_rows(_lib.ptr(x), _lib.ptr(w.packed.weight), _lib.ptr(z), t, w.n, k, _lib.stream())
-    _lib.check(rc, "moe_router_rows")
+    rc = _lib.lib().b200_rows_linear_f32(_lib.ptr(x), k, _lib.ptr(w.packed.weight), _lib.ptr(z), w.n, t, w.n, k, _lib.stream())
+    _lib.check(rc, "rows_linear")
     return z
 
 

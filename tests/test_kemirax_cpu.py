@@ -214,6 +214,7 @@ def test_weight_layouts():
     assert torch.equal(w13[3, 1, :22, :36], state["l0.mlp.e3.up"]) and not w13[:, :, 22:].any()
     assert torch.equal(f.w2.weight.view(5, w.ld, 32)[2, :36, :22], state["l0.mlp.e2.down"])
     t = decoder.GLU_TILE
+    assert lw.gates.n == 256 and lw.wide.n >= 256 + f.up.n and torch.equal(lw.wide.w32[256:256 + f.up.n], f.up.w32)
     up = x @ f.up.w32.t()
     assert near(up[:, :30], xs @ state["l0.mlp.shared.gate"].t()) and near(up[:, t:t + 30], xs @ state["l0.mlp.shared.up"].t())
     # latent attention: both forms of the up projections

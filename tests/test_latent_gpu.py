@@ -163,18 +163,22 @@ def _attend(m, q, c, kr, pos):
     return torch.softmax(s, -1) @ c[:pos + 1].double()
 
 
-@BOTH
+@pytest.mark.parametrize("dtype,tiles", [(torch.bfloat16, True), (torch.bfloat16, False), (torch.float32, False)])
 @pytest.mark.parametrize("sizes", SIZES)
 @pytest.mark.parametrize("splits", [None, 1, 7])
-def test_single_rows(dtype, sizes, splits):
+def test_single_rows(dtype, tiles, sizes, splits):
     """Rows of several sequences at positions around page and tile borders, first tokens included; one key per head stands out,
     wherever it lies, also when it is the row's own or the very first."""
-    _, lat = _mods()
+    _lib, lat = _mods()
     m, _ = _mixer(*sizes, scale=1.3, seed=5)
     ctx = Ctx(m, [300, 65, 1, 130], dtype, block=32, seed=6)
     where = [(0, 299), (0, 0), (0, 31), (0, 32), (1, 64), (2, 0), (3, 127), (3, 128), (0, 200)]
     q = _absorbed(m, len(where), dtype, 7)
-    got = lat.attend_rows(q.cuda(), m, ctx.gcache, ctx.gtable, _i32([p for _, p in where]), 301, seq=_i32([i for i, _ in where]), splits=splits)
+    got = lat.attend_rows(q.cuda(), m, ctx.gcache, ctx.gtable, _i32([p for _, p in where]), 301, seq=_i32([i for i, _ in where]), splits=splits,
+                          tiles=tiles)
+    _lib.check_status()
+    if tiles:
+        assert _lib.lib().b200_attn_latent_decode_heads(m.heads, m.c, m.cache_width, 32) > 0
     for r, (i, p) in enumerate(where):
         assert _rel(got[r, :, :m.kv_rank], _attend(m, q[r], ctx.c[i], ctx.kr[i], p)) < DT[dtype], (r, i, p)
     assert not got[:, :, m.kv_rank:].any()
@@ -183,12 +187,33 @@ def test_single_rows(dtype, sizes, splits):
         ctx.loud(0, far, q[0, m.heads - 1])
         rows = [p for p in (far - 1, far, 299) if p >= 0]
         qq = q[:1].expand(len(rows), -1, -1).contiguous()
-        got = lat.attend_rows(qq.cuda(), m, ctx.gcache, ctx.gtable[:1].expand(len(rows), -1).contiguous(), _i32(rows), 301, splits=splits)
+        got = lat.attend_rows(qq.cuda(), m, ctx.gcache, ctx.gtable[:1].expand(len(rows), -1).contiguous(), _i32(rows), 301, splits=splits, tiles=tiles)
         for r, p in enumerate(rows):
             want = _attend(m, qq[r], ctx.c[0], ctx.kr[0], p)
             assert _rel(got[r, :, :m.kv_rank], want) < 2 * DT[dtype], (far, p)
             seen = _rel(want[-1], ctx.c[0][far].double()) < 0.05
             assert seen == (p >= far)                        # the test itself tells a missed or a leaked key apart
+
+
+@pytest.mark.parametrize("block", [16, 32, 64, 128])
+@pytest.mark.parametrize("heads,kv_rank,rot", [(16, 512, 64), (5, 48, 32), (33, 208, 16), (50, 448, 64)])
+def test_single_rows_over_long_contexts(block, heads, kv_rank, rot):
+    """Growing scores (every tile moves the running maximum), all page sizes, one to four accumulators, several head groups."""
+    _lib, lat = _mods()
+    m, _ = _mixer(heads, 16, rot, 16, 16, kv_rank, scale=0.9, seed=15)
+    ctx = Ctx(m, [1500, 200], torch.bfloat16, block=block, seed=16)
+    q = _absorbed(m, 3, torch.bfloat16, 17)
+    ramp = torch.linspace(0.05, 4.0, 1500)[:, None]
+    for p in range(1500):
+        ctx.c[0][p] = (ctx.c[0][p].float() * 0.3 + q[0, p % heads, :kv_rank].float() * ramp[p] * kv_rank ** 0.5).bfloat16()
+        row = ctx.cache[ctx.table[0, p // block], p % block]
+        row[:kv_rank] = ctx.c[0][p]
+    ctx.gcache = ctx.cache.cuda()
+    for splits in (None, 1, 3, 40):
+        got = lat.attend_rows(q.cuda(), m, ctx.gcache, ctx.gtable, _i32([1499, 700, 199]), 1500, seq=_i32([0, 0, 1]), splits=splits)
+        _lib.check_status()
+        for r, (i, p) in enumerate(((0, 1499), (0, 700), (1, 199))):
+            assert _rel(got[r, :, :kv_rank], _attend(m, q[r], ctx.c[i], ctx.kr[i], p)) < 1e-2, (splits, r)
 
 
 @pytest.mark.parametrize("block", [16, 64])
