@@ -360,12 +360,14 @@ def _kx_kernels(size: str, dev, timer: _Timer, ctx: int) -> list[dict]:
              (lambda: decoder.parallel_step(x32, width, 1.0, 1e-5, **args), t * width * (8 + 2 + 4 + 2 + 2 + 2 + 2) + local * width * 2, 0),
              (lambda: basic.add_rmsnorm(x16, d16, g16, 1e-5), t * width * 8, 0))
         # ---- experts: routing, plan, gather, both products, unit; beside the same with SwiGLU and the combine
-        ebytes = min(E, t * top) * 3 * width * ff * 2
+        each = 3 * width * ff * 2
+        ebytes = int(torch.unique(idx[idx < E]).numel()) * each              # experts that have a token
         need = (ebytes + t * width * 2 + local * width * 2, 2 * local * 3 * width * ff)
         i2, w2_ = moe.route(z[:, :E], None, top, "softmax", False, 1.0)
+        ebytes2 = int(torch.unique(i2).numel()) * each
         pair("routed experts (like: with SwiGLU and combine)", f"{t} tokens, {top} of {E}",
              (lambda: moe.experts_rows(h16, idx, ew.w13, ew.w2, 0, 7.0, kx.UNIT_SLOPE), *need),
-             (lambda: moe.experts_forward(h16, i2, w2_, ew.w13, ew.w2, 0), ebytes + t * width * 4, 2 * t * top * 3 * width * ff))
+             (lambda: moe.experts_forward(h16, i2, w2_, ew.w13, ew.w2, 0), ebytes2 + t * width * 4, 2 * t * top * 3 * width * ff))
         pair("routing (like: sigmoid, normalised)", f"{t} x {E + ident}",
              (lambda: moe.route(z[:, :E + ident], ew.correction, top, "softmax", False, 1.0), t * (z.stride(0) * 4 + top * 8), 0),
              (lambda: moe.route(z[:, :E], ew.correction[:E], top, "sigmoid", True, 1.0), t * (z.stride(0) * 4 + top * 8), 0))
