@@ -380,7 +380,8 @@ class KemiraxWeights:
         ukv = PackedLinear.from_bf16(both.to(self.device)) if self.dtype == torch.bfloat16 else None
         return LatentWeights(m, self._proj(_cat_rows(parts), tile_n=True),
                              self._proj(_heads(t["uq"], a.heads, ((a.dim, d), (a.rot_dim, r))), tile_n=True),
-                             dev(uk.view(c, a.heads, d).permute(1, 0, 2)), dev(uv.view(a.heads, v, c)), ukv, self._proj(_heads(t["o"].t().contiguous(), a.heads, ((a.vdim, v),)).t()))
+                             dev(uk.view(c, a.heads, d).permute(1, 0, 2)), dev(uv.view(a.heads, v, c)), ukv,
+                             self._proj(_heads(t["o"].t().contiguous(), a.heads, ((a.vdim, v),)).t()))
 
     def _linear(self, s: LinearSpec, t: dict[str, torch.Tensor]) -> LinearWeights:
         rank = t["a1"].shape[0]
@@ -415,7 +416,8 @@ class KemiraxWeights:
         rows = [(t["router"], f.experts + f.identity)] + ([(t["shared.sg"], 1)] if f.shared_ff else [])
         ew = ExpertsWeights(f, self._proj(_cat_rows(rows)), self._row(t["correction"], f.experts + f.identity), pack(w13), pack(w2))
         if f.shared_ff:
-            down = torch.zeros(self.cfg.width, (f.shared_ff + decoder.GLU_TILE - 1) // decoder.GLU_TILE * decoder.GLU_TILE, dtype=t["shared.down"].dtype, device=t["shared.down"].device)
+            padded = (f.shared_ff + decoder.GLU_TILE - 1) // decoder.GLU_TILE * decoder.GLU_TILE
+            down = t["shared.down"].new_zeros(self.cfg.width, padded)
             down[:, :f.shared_ff] = t["shared.down"]
             ew.down = self._proj(down)
         return ew
@@ -458,7 +460,8 @@ class KemiraxRuntime(PagedRuntime):
             if isinstance(lw.mix, LatentWeights):
                 src = L.mixer.kv_from
                 c = self.cache[src] if src is not None else canary.zeros(
-                    self.num_blocks, block_size, lw.mix.m.cache_width, dtype=weights.dtype, device=self.device, name=f"paged latent cache of layer {i}")
+                    self.num_blocks, block_size, lw.mix.m.cache_width, dtype=weights.dtype, device=self.device,
+                    name=f"paged latent cache of layer {i}")
             else:
                 m = lw.mix.m
                 st = self.slot_state(m.heads, m.d, m.v, dtype=torch.float32, name=f"recurrent state of layer {i}")

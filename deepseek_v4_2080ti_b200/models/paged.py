@@ -130,8 +130,9 @@ class PagedRuntime(PagedSequences):
     ``meta["mode"]``: ``"decode"`` - one row per sequence, static buffers (``block_table`` row i belongs to row i,
     ``kv_len``, ``max_kv_len``); ``"mixed"`` - the first ``tile_rows`` rows are portions of several sequences
     (``q_start``, ``q_len``, ``kv_len``, ``max_q_len``, ``tile_seq``; ``kv_start`` / ``kv_total``: where their contexts begin
-    when they are laid out one after the other), the rest single rows (``row_seq``, ``max_kv_len``).  In both modes ``segments`` says which neighbouring rows form one
-    sequence's portion and which state slot it has, for mixers that carry a recurrent state.
+    when they are laid out one after the other), the rest single rows (``row_seq``, ``max_kv_len``).  In both modes
+    ``segments`` says which neighbouring rows form one sequence's portion and which state slot it has, for mixers that carry
+    a recurrent state.
 
     Recurrent state is held per request slot in tensors from ``slot_state``; a slot's content is meaningless until its
     sequence's first token, whose position 0 the kernels take as "start from zero".  The slot after the last one is scratch:
@@ -223,7 +224,8 @@ class PagedRuntime(PagedSequences):
                 "segments": Segments(start_d, seq_d, e_first, e_len, e_slot, max(lens), min(lens))}
         if tiles:
             n = len(tiles)
-            meta.update(q_start=e_first[:n], q_len=e_len[:n], kv_len=e_kv[:n], tile_seq=e_slot[:n], kv_start=e_start[:n], kv_total=kv_total)
+            meta.update(q_start=e_first[:n], q_len=e_len[:n], kv_len=e_kv[:n], tile_seq=e_slot[:n],
+                        kv_start=e_start[:n], kv_total=kv_total)
         # a pass has to run even when no logits are asked for: it fills the cache
         wanted = up[5 * n_rows + desc.numel():]
         logits = self._forward(ids, pos_d, slots_d, meta, wanted)

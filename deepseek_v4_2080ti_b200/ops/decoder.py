@@ -161,8 +161,8 @@ def parallel_step(x: torch.Tensor | None, cols: int, weight: float, eps: float, 
                   seg=None, positions: torch.Tensor | None = None, rows: torch.Tensor | None = None,
                   norm: bool = True) -> tuple[torch.Tensor | None, torch.Tensor | None]:
     """Step between layers whose sublayers run side by side (csrc/kernels/parallel_step.cu):
-    ``x + mix sigmoid(gates[:, :ld] + b) + ff sigmoid(gates[:, ld:] + b)`` goes to ``x_out`` (which may be ``x``), with ``ff`` the sum of the routed experts, of identity experts (``h``) and of ``shared`` behind its gate (a column of
-    logits).  Returns (RMS norm of it times ``weight``, that norm moved towards the row before it by ``shift``): the second
+    ``x + mix sigmoid(gates[:, :ld] + b) + ff sigmoid(gates[:, ld:] + b)`` goes to ``x_out`` (which may be ``x``), with ``ff``
+    the sum of the routed experts, of identity experts (``h``) and of ``shared`` behind its gate (a column of logits).  Returns (RMS norm of it times ``weight``, that norm moved towards the row before it by ``shift``): the second
     only with ``shift``, which also keeps the sequences' ``tail`` [slots, ld].  ``rows``: only these rows, norm only."""
     dev = (x if x is not None else ids).device
     assert x is None or (x.dtype == torch.float32 and x.shape[1] == ld and x.is_contiguous())
