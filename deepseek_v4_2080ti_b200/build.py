@@ -41,7 +41,7 @@ NVCC_FLAGS = ARCH + ["-lineinfo", "-O3", "-std=c++17", "--use_fast_math", "-Xcom
 # Kernels that also serve the fp32 runtimes: exact division, square root and exponentials instead of the fast variants.
 PRECISE = {"residual_norm.cu", "bias_act.cu", "qk_row_prep.cu", "attn_mix_rows.cu", "gemm_f32.cu", "qk_head_prep.cu",
            "attn_diff_rows.cu", "conv_rows.cu", "selective_scan.cu", "moe.cu", "parallel_step.cu", "latent_prep.cu",
-           "attn_latent_rows.cu", "gated_linear.cu"}
+           "attn_latent_rows.cu", "gated_linear.cu", "branch_step.cu", "row_act.cu", "decay_rule.cu", "attn_window_rows.cu"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-pthread"]
 # A compiler that links its C++ runtime statically would otherwise export that runtime's symbols from every module;
 # in a process that has already loaded another libstdc++ (torch) the dynamic linker then binds half of a stream or

@@ -6,7 +6,8 @@
 // positions[r] its position.  Inputs from before the batch come from the slot's tail (the last taps - 1 inputs, oldest
 // first); inputs from before position 0 are zero, so a slot needs no clearing.  A sequence that brings a single row has its
 // tail replaced right here (one thread holds all of it); the tail of a longer portion, which several blocks read, is replaced
-// by the kernel that runs the recurrence behind the convolution (selective_scan.cu).  One thread: 8 channels, `strip` rows.
+// by the kernel that runs the recurrence behind the convolution (selective_scan.cu), or by conv_tails.  One thread: 8
+// channels, `strip` rows.
 #include "launch.h"
 #include "ops.h"
 #include "vec8.cuh"
@@ -133,7 +134,38 @@ int run_conv_rows(const void* x, int ldx, const float* w, const float* bias, voi
   }
 }
 
+// New tails of the portions with more than one row: the inputs of their last taps - 1 positions.  A thread owns eight channels of
+// a tail; a portion shorter than the tail moves what stays of the old one.
+template <typename T>
+__global__ void conv_tails_kernel(const T* __restrict__ x, int ldx, T* __restrict__ tail, const int* __restrict__ first,
+                                  const int* __restrict__ length, const int* __restrict__ slot, int C, int keep) {
+  pdl_grid_trigger();
+  pdl_grid_wait();
+  const int e = blockIdx.y, n = length[e], c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+  if (n < 2 || c >= C) return;
+  T* dst = tail + (size_t)slot[e] * keep * C + c;
+  const T* src = x + (size_t)first[e] * ldx + c;
+  for (int j = 0; j < keep; ++j) {
+    const int at = n - keep + j;             // row of the portion, or behind its start: an entry of the old tail
+    float f[8];
+    load8(at >= 0 ? src + (size_t)at * ldx : dst + (size_t)(keep + at) * C, f);
+    store8(dst + (size_t)j * C, f);
+  }
+}
+
 }  // namespace
+
+// x [rows, >= C] the convolution's inputs; tails [slots, taps - 1, C] of the entries with more than one row are replaced.
+extern "C" int b200_conv_tails(const void* x, int ldx, void* tail, const int* first, const int* length, const int* slot, int entries,
+                               int C, int taps, int f32, cudaStream_t stream) {
+  if (entries <= 0 || entries > 65535 || C <= 0 || (C & 7) || (ldx & 7) || ldx < C || taps < 2 || taps > 64) return -6;
+  const dim3 grid((C / 8 + 127) / 128, entries);
+  if (f32)
+    return (int)launch_pdl(conv_tails_kernel<float>, grid, dim3(128), 0, stream, reinterpret_cast<const float*>(x), ldx,
+                           reinterpret_cast<float*>(tail), first, length, slot, C, taps - 1);
+  return (int)launch_pdl(conv_tails_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, reinterpret_cast<const __nv_bfloat16*>(x), ldx,
+                         reinterpret_cast<__nv_bfloat16*>(tail), first, length, slot, C, taps - 1);
+}
 
 // x rows of C channels (C, ldx, ldy multiples of 8); f32 != 0: x, tail, y are fp32, otherwise bf16.
 extern "C" int b200_conv_rows(const void* x, int ldx, const float* w, const float* bias, void* tail, const int* row_first,

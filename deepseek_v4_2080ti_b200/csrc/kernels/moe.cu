@@ -24,7 +24,7 @@ constexpr int MAX_EXPERTS = 1024;
 __device__ __forceinline__ float score_fn(float x, int fn) {
   if (fn == 1) return 1.f / (1.f + expf(-x));                         // sigmoid
   if (fn == 2) return sqrtf(x > 20.f ? x : log1pf(expf(x)));          // sqrt(softplus)
-  return x;                                                           // softmax handled by the caller
+  return x;                                                           // the softmaxes are handled by the caller
 }
 
 // One warp per token. logits fp32 [T, ld], the first E of a row; bias fp32 [E] or null; E <= 32 J.
@@ -53,12 +53,13 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int ld, const
     if (e < E) {
       sc[j] = fn == 0 ? expf(row[e] - mx) / den : score_fn(row[e], fn);
       sel[j] = sc[j] + (bias ? bias[e] : 0.f);
+      if (fn == 3) sc[j] = sel[j];                                    // the bias belongs to the logit
     } else {
       sc[j] = 0.f;
       sel[j] = -INFINITY;
     }
   }
-  float wsum = 0.f;
+  float wsum = 0.f, top = 0.f;
   for (int k = 0; k < K; ++k) {
     float best = -INFINITY;
     int be = 0x7fffffff;
@@ -78,6 +79,10 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int ld, const
     for (int j = 0; j < J; ++j)
       if (j * 32 + lane == be) { w = sc[j]; sel[j] = -INFINITY; }
     for (int o = 16; o > 0; o >>= 1) w += __shfl_xor_sync(0xffffffffu, w, o);
+    if (fn == 3) {                                                    // softmax over the chosen: the first is the largest
+      if (k == 0) top = w;
+      w = expf(w - top);
+    }
     wsum += w;
     if (lane == (k & 31)) {
       idx[(size_t)t * K + k] = be;

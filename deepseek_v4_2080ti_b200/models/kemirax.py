@@ -18,7 +18,7 @@ from typing import Any, Iterator
 import torch
 
 from ..ops import decoder, gla, latent, moe
-from ..ops.decoder import Projection, Routed, pad16
+from ..ops.decoder import Projection, Routed, cat_rows, pad16, pad_heads
 from ..ops.gemm import PackedLinear
 from ..ops.gla import GatedLinear
 from ..ops.latent import LatentAttention
@@ -292,27 +292,6 @@ def _fits(have: tuple[int, ...], want: tuple[int | None, ...]) -> bool:
     return len(have) == len(want) and all(w is None or h == w for h, w in zip(have, want))
 
 
-def _heads(w: torch.Tensor, n: int, parts: tuple[tuple[int, int], ...]) -> torch.Tensor:
-    """[n * sum(real), ...] -> [n * sum(padded), ...]: zero rows behind every (real, padded) part of every head."""
-    src = w.reshape(n, sum(r for r, _ in parts), *w.shape[1:])
-    out = torch.zeros(n, sum(p for _, p in parts), *w.shape[1:], dtype=w.dtype, device=w.device)
-    a = b = 0
-    for real, padded in parts:
-        out[:, b:b + real] = src[:, a:a + real]
-        a, b = a + real, b + padded
-    return out.reshape(-1, *w.shape[1:])
-
-
-def _cat_rows(parts: list[tuple[torch.Tensor, int]]) -> torch.Tensor:
-    """Matrices below one another, each padded to the given number of rows."""
-    out = torch.zeros(sum(n for _, n in parts), parts[0][0].shape[1], dtype=parts[0][0].dtype, device=parts[0][0].device)
-    at = 0
-    for w, n in parts:
-        out[at:at + w.shape[0]] = w
-        at += n
-    return out
-
-
 class KemiraxWeights:
     """Device-resident, padded, kernel-ready weights from (name, tensor) pairs."""
 
@@ -346,8 +325,8 @@ class KemiraxWeights:
             if ff is not None and L.mlp.shared_ff:
                 # rows in whole tiles of the pair GEMM, so that either part can be multiplied alone
                 up = decoder.interleave_glu(t[p + "mlp.shared.gate"], t[p + "mlp.shared.up"])
-                parts = [(_cat_rows(parts), (ng + 255) // 256 * 256), (up, up.shape[0])]
-            wide = self._proj(_cat_rows(parts), tile_n=True)
+                parts = [(cat_rows(parts), (ng + 255) // 256 * 256), (up, up.shape[0])]
+            wide = self._proj(cat_rows(parts), tile_n=True)
             gates = wide
             if ff is not None and L.mlp.shared_ff:
                 ng = parts[0][1]
@@ -373,15 +352,15 @@ class KemiraxWeights:
         if own:
             parts += [(t["dkv"][:a.kv_rank], c), (t["dkv"][a.kv_rank:], r)]
         dev = lambda w: w.to(self.device, self.dtype).contiguous()
-        uk = _cat_rows([(_heads(t["uk"], a.heads, ((a.dim, d),)).t(), c)])                         # [c, heads * d]
+        uk = cat_rows([(pad_heads(t["uk"], a.heads, ((a.dim, d),)).t(), c)])                         # [c, heads * d]
         uv = torch.zeros(a.heads * v, c, dtype=t["uv"].dtype, device=t["uv"].device)
-        uv[:, :a.kv_rank] = _heads(t["uv"], a.heads, ((a.vdim, v),))
+        uv[:, :a.kv_rank] = pad_heads(t["uv"], a.heads, ((a.vdim, v),))
         both = torch.cat([uk.t().reshape(a.heads, d, c), uv.view(a.heads, v, c)], 1).reshape(-1, c)
         ukv = PackedLinear.from_bf16(both.to(self.device)) if self.dtype == torch.bfloat16 else None
-        return LatentWeights(m, self._proj(_cat_rows(parts), tile_n=True),
-                             self._proj(_heads(t["uq"], a.heads, ((a.dim, d), (a.rot_dim, r))), tile_n=True),
+        return LatentWeights(m, self._proj(cat_rows(parts), tile_n=True),
+                             self._proj(pad_heads(t["uq"], a.heads, ((a.dim, d), (a.rot_dim, r))), tile_n=True),
                              dev(uk.view(c, a.heads, d).permute(1, 0, 2)), dev(uv.view(a.heads, v, c)), ukv,
-                             self._proj(_heads(t["o"].t().contiguous(), a.heads, ((a.vdim, v),)).t()))
+                             self._proj(pad_heads(t["o"].t().contiguous(), a.heads, ((a.vdim, v),)).t()))
 
     def _linear(self, s: LinearSpec, t: dict[str, torch.Tensor]) -> LinearWeights:
         rank = t["a1"].shape[0]
@@ -391,30 +370,19 @@ class KemiraxWeights:
             raise ValueError("the recurrence takes up to 512 key channels per head and a decay rank of 1024")
         d, v, rp = pad16(s.dim), pad16(s.vdim), pad16(rank)
         w2 = torch.zeros(s.heads * d, rp, dtype=t["a2"].dtype, device=t["a2"].device)
-        w2[:, :rank] = _heads(t["a2"], s.heads, ((s.dim, d),))
+        w2[:, :rank] = pad_heads(t["a2"], s.heads, ((s.dim, d),))
         m = GatedLinear(s.heads, s.dim, d, s.vdim, v, s.tau, self.cfg.eps, rp, w2.to(self.device, self.dtype).contiguous(),
-                        self._row(_heads(t["a2.b"], s.heads, ((s.dim, d),)), s.heads * d), self._row(t["norm"], v))
-        keys = [(_heads(t[n], s.heads, ((s.dim, d),)), s.heads * d) for n in ("q", "k")]
-        values = [(_heads(t[n], s.heads, ((s.vdim, v),)), s.heads * v) for n in ("v", "g")]
-        return LinearWeights(m, self._proj(_cat_rows(keys + values + [(t["a1"], rp)]), tile_n=True),
-                             self._proj(_heads(t["o"].t().contiguous(), s.heads, ((s.vdim, v),)).t()))
+                        self._row(pad_heads(t["a2.b"], s.heads, ((s.dim, d),)), s.heads * d), self._row(t["norm"], v))
+        keys = [(pad_heads(t[n], s.heads, ((s.dim, d),)), s.heads * d) for n in ("q", "k")]
+        values = [(pad_heads(t[n], s.heads, ((s.vdim, v),)), s.heads * v) for n in ("v", "g")]
+        return LinearWeights(m, self._proj(cat_rows(keys + values + [(t["a1"], rp)]), tile_n=True),
+                             self._proj(pad_heads(t["o"].t().contiguous(), s.heads, ((s.vdim, v),)).t()))
 
     def _experts(self, f: ExpertsSpec, t: dict[str, torch.Tensor]) -> ExpertsWeights:
-        f32 = self.dtype == torch.float32
-        ff = pad16(f.ff) if f32 else (f.ff + 63) // 64 * 64            # the grouped GEMM tiles features by 128, gate and up together
-        out = self.ld if f32 else (self.ld + 127) // 128 * 128
-        w13, w2 = [], []
-        for j in range(f.experts):
-            a = torch.zeros(2, ff, self.ld, dtype=self.dtype, device=self.device)
-            a[0, :f.ff, :self.cfg.width] = t[f"e{j}.gate"].to(self.device, self.dtype)
-            a[1, :f.ff, :self.cfg.width] = t[f"e{j}.up"].to(self.device, self.dtype)
-            b = torch.zeros(out, ff, dtype=self.dtype, device=self.device)
-            b[:self.cfg.width, :f.ff] = t[f"e{j}.down"].to(self.device, self.dtype)
-            w13.append(a.view(2 * ff, self.ld))
-            w2.append(b)
-        pack = moe.ExpertWeights.from_f32 if f32 else moe.ExpertWeights.from_bf16
+        w13, w2 = moe.pack_experts(*([t[f"e{j}.{n}"] for j in range(f.experts)] for n in ("gate", "up", "down")), self.cfg.width, self.ld,
+                                   self.dtype, self.device)
         rows = [(t["router"], f.experts + f.identity)] + ([(t["shared.sg"], 1)] if f.shared_ff else [])
-        ew = ExpertsWeights(f, self._proj(_cat_rows(rows)), self._row(t["correction"], f.experts + f.identity), pack(w13), pack(w2))
+        ew = ExpertsWeights(f, self._proj(cat_rows(rows)), self._row(t["correction"], f.experts + f.identity), w13, w2)
         if f.shared_ff:
             padded = (f.shared_ff + decoder.GLU_TILE - 1) // decoder.GLU_TILE * decoder.GLU_TILE
             down = t["shared.down"].new_zeros(self.cfg.width, padded)
@@ -481,13 +449,13 @@ class KemiraxRuntime(PagedRuntime):
             contexts = meta.setdefault("contexts", {})
             if src not in contexts:                  # layers that share a cache share its contiguous copy
                 contexts[src] = latent.gather(cache, m, self.block_table, meta["tile_seq"], meta["kv_len"], meta["kv_start"], meta["kv_total"])
-            latent.rotate_heads(q[:n], m, positions)
+            latent.rotatepad_heads(q[:n], m, positions)
             latent.attend_tiles(q[:n], m, *contexts[src], lw.ukv, meta["q_start"], meta["q_len"], meta["kv_len"], meta["kv_start"],
                                 meta["max_q_len"], out[:n])
         if n < t:                                    # single rows: queries are brought to the latents
             qr = q[n:]
             qa = torch.empty(t - n, m.heads, m.cache_width, dtype=y.dtype, device=y.device)
-            latent.rotate_heads(qr, m, positions[n:], qa, m.c)
+            latent.rotatepad_heads(qr, m, positions[n:], qa, m.c)
             latent.head_linear(qr, qr.stride(0), m.head_width, lw.uk, qa, qa.stride(0), qa.stride(1), t - n)
             if meta["mode"] == "decode":
                 o = latent.attend_rows(qa, m, cache, meta["block_table"], positions, meta["max_kv_len"])

@@ -506,3 +506,35 @@ def _kemirax_sources() -> tuple[str, ...]:
 register_checkpoint(CheckpointSpec("kemirax", "Kemirax (latent attention, gated linear attention, side-by-side sublayers, routed experts)",
                                    _kemirax_matches, _kemirax_build, dtypes=("bfloat16", "float32"),
                                    kernel_sources=_kemirax_sources(), tensor_shapes=_kemirax_shapes))
+
+
+def _nunosun_matches(raw) -> bool:
+    from .nunosun import NunosunConfig
+    return NunosunConfig.is_nunosun_json(raw)
+
+
+def _nunosun_build(raw, directory, device, rank=0, world=1, dtype=None, max_slots=1, max_context=4096, num_blocks=None,
+                   make_comm=None):
+    from ..formats import safetensors_io
+    from . import nunosun as ns
+    if world != 1:
+        raise ValueError("a Nunosun model runs on one rank")
+    cfg = ns.NunosunConfig.from_json(raw)
+    w = ns.NunosunWeights(cfg, safetensors_io.read_checkpoint(directory), device,
+                          _torch_dtype(dtype, ("bfloat16", "float32")))
+    return cfg, ns.NunosunRuntime(cfg, w, max_slots=max_slots, max_context=max_context, num_blocks=num_blocks)
+
+
+def _nunosun_shapes(raw) -> dict[str, tuple[int | None, ...]]:
+    from .nunosun import NunosunConfig
+    return NunosunConfig.from_json(raw).tensor_shapes()
+
+
+def _nunosun_sources() -> tuple[str, ...]:
+    from .nunosun import KERNEL_SOURCES
+    return KERNEL_SOURCES
+
+
+register_checkpoint(CheckpointSpec("nunosun", "Nunosun (delta rule, window attention beside retention, side embedding, dense or routed)",
+                                   _nunosun_matches, _nunosun_build, dtypes=("bfloat16", "float32"),
+                                   kernel_sources=_nunosun_sources(), tensor_shapes=_nunosun_shapes))

@@ -83,6 +83,27 @@ class Projection:
         return self.n * self.k * (4 if self.packed is None else 2)
 
 
+def pad_heads(w: torch.Tensor, n: int, parts: tuple[tuple[int, int], ...]) -> torch.Tensor:
+    """[n * sum(real), ...] -> [n * sum(padded), ...]: zero rows behind every (real, padded) part of every head."""
+    src = w.reshape(n, sum(r for r, _ in parts), *w.shape[1:])
+    out = torch.zeros(n, sum(p for _, p in parts), *w.shape[1:], dtype=w.dtype, device=w.device)
+    a = b = 0
+    for real, padded in parts:
+        out[:, b:b + real] = src[:, a:a + real]
+        a, b = a + real, b + padded
+    return out.reshape(-1, *w.shape[1:])
+
+
+def cat_rows(parts: list[tuple[torch.Tensor, int]]) -> torch.Tensor:
+    """Matrices below one another, each padded to the given number of rows."""
+    out = torch.zeros(sum(n for _, n in parts), parts[0][0].shape[1], dtype=parts[0][0].dtype, device=parts[0][0].device)
+    at = 0
+    for w, n in parts:
+        out[at:at + w.shape[0]] = w
+        at += n
+    return out
+
+
 GLU_TILE = 128          # features per gate / up tile of an interleaved projection
 
 
@@ -195,6 +216,76 @@ def parallel_step(x: torch.Tensor | None, cols: int, weight: float, eps: float, 
                                         _lib.ptr(seg.slot), seg.first.numel(), n, ld, f32, _lib.stream())
         _lib.check(rc, "shift_rows", 2)
     return out, m
+
+
+def branch_step(x: torch.Tensor | None, cols: int, eps: float, *, ld: int, n: int, dtype: torch.dtype, x_out: torch.Tensor | None = None,
+                ids: torch.Tensor | None = None, table: torch.Tensor | None = None,
+                normed: tuple[tuple[torch.Tensor | None, torch.Tensor], ...] = (), plain: tuple[torch.Tensor, ...] = (),
+                routed: Routed | None = None, copy: bool = False, weight: torch.Tensor | None = None, conv: torch.Tensor | None = None,
+                tail: torch.Tensor | None = None, seg=None, positions: torch.Tensor | None = None,
+                rows: torch.Tensor | None = None) -> tuple[torch.Tensor | None, torch.Tensor | None, torch.Tensor | None]:
+    """Step of a residual that takes several sublayer results at once (csrc/kernels/branch_step.cu): ``x`` (zero without it) plus up
+    to two ``normed`` branches (result, weight), up to two ``plain`` ones and the ``routed`` experts' sum goes to ``x_out`` (which may
+    be ``x``).  ``ids`` / ``table``: the first normed branch is an embedding row (its result is None).  Returns (that sum in ``dtype``
+    with ``copy``, its RMS norm times ``weight``, that norm plus its causal convolution with ``conv`` [taps, ld]): the last keeps the
+    sequences' ``tail`` [slots, taps - 1, ld]; ``conv``'s last row has the 1 of the norm itself in it.  ``rows``: only these rows."""
+    from . import scan
+    dev = (x if x is not None else ids).device
+    assert x is None or (x.dtype == torch.float32 and x.shape[1] == ld and x.is_contiguous())
+    assert len(normed) <= 2 and len(plain) <= 2
+    for t in [r for r, _ in normed] + list(plain) + [table]:
+        assert t is None or (t.dtype == dtype and t.shape[1] == ld and t.is_contiguous())
+    for w in [w for _, w in normed] + [weight]:
+        assert w is None or (w.dtype == torch.float32 and w.numel() == ld)
+    if ids is not None:
+        _lib.check_indices(ids, 0, table.shape[0], 1)
+    if rows is not None:
+        _lib.check_indices(rows, 0, x.shape[0], 7)
+    if conv is not None:
+        _lib.check_indices(seg.row_slot, 0, tail.shape[0], 4)
+    count = rows.numel() if rows is not None else n
+    new = lambda m: torch.empty(m, ld, dtype=dtype, device=dev)
+    c, h = new(n) if copy else None, new(count) if weight is not None else None
+    single = conv is not None and seg.max_length == 1      # no row needs its neighbour: convolution and tails in the same launch
+    m = new(n) if single else None
+    taps = 0 if conv is None else conv.shape[0]
+    b = list(normed) + [(None, None)] * (2 - len(normed))
+    p = list(plain) + [None] * (2 - len(plain))
+    r, f32 = routed, int(dtype == torch.float32)
+    rc = _lib.lib().b200_branch_step(
+        _lib.ptr(x), _lib.ptr(x_out), _lib.ptr(ids), _lib.ptr(table), 0 if table is None else table.shape[0], _lib.ptr(b[0][0]),
+        _lib.ptr(b[0][1]), _lib.ptr(b[1][0]), _lib.ptr(b[1][1]), _lib.ptr(p[0]), _lib.ptr(p[1]), _lib.ptr(r.y if r else None),
+        r.y.stride(0) if r else 0, _lib.ptr(r.row if r else None), _lib.ptr(r.weights if r else None), r.idx.shape[1] if r else 0,
+        _lib.ptr(c), _lib.ptr(weight), _f(eps), _lib.ptr(h), _lib.ptr(m), _lib.ptr(conv if single else None),
+        _lib.ptr(tail if single else None), _lib.ptr(seg.row_slot if single else None), _lib.ptr(positions if single else None), taps,
+        _lib.ptr(rows), count, ld, cols, f32, _lib.stream())
+    _lib.check(rc, "branch_step")
+    if conv is not None and not single:
+        m = scan.conv_rows(h, conv, None, tail, seg, positions, silu=False)
+        if taps > 1:
+            scan.conv_tails(h, tail, seg)
+    return c, h, m
+
+
+def poly_norm(z: torch.Tensor, cols: int, coef: tuple[float, float, float, float], eps: float, ldo: int) -> torch.Tensor:
+    """``a N(z) + b N(z^2) + c N(z^3) + e`` with N over the root mean square of a row's first ``cols`` columns: [T, ldo]."""
+    out = torch.empty(z.shape[0], ldo, dtype=z.dtype, device=z.device)
+    a, b, c, e = coef
+    rc = _lib.lib().b200_poly_norm(_lib.ptr(z), z.stride(0), _lib.ptr(out), ldo, z.shape[0], cols, _f(a), _f(b), _f(c), _f(e),
+                                   _f(eps), int(z.dtype == torch.float32), _lib.stream())
+    _lib.check(rc, "poly_norm")
+    return out
+
+
+def token_gate(z: torch.Tensor, table: torch.Tensor, col: int, ids: torch.Tensor) -> torch.Tensor:
+    """``gelu_tanh(z) * table[ids, col:col + columns of z]``."""
+    assert table.dtype == z.dtype and table.is_contiguous()
+    _lib.check_indices(ids, 0, table.shape[0], 1)
+    out = torch.empty(z.shape, dtype=z.dtype, device=z.device)
+    rc = _lib.lib().b200_token_gate(_lib.ptr(z), z.stride(0), _lib.ptr(table), table.shape[1], col, table.shape[0], _lib.ptr(ids),
+                                    _lib.ptr(out), z.shape[1], z.shape[0], int(z.dtype == torch.float32), _lib.stream())
+    _lib.check(rc, "token_gate")
+    return out
 
 
 def bias_xielu(z: torch.Tensor, bias: torch.Tensor | None, ap: float, an: float) -> torch.Tensor:

@@ -13,7 +13,8 @@ from .gemm import WF_BF16, WF_FP8_B128
 
 WF_FP4 = 2
 WF_F32 = 100                   # not a GEMM format: plain fp32 matrices on the CUDA cores (gemm_f32.cu)
-SCORE_FN = {"softmax": 0, "sigmoid": 1, "sqrtsoftplus": 2}
+# softmax_chosen: softmax over the chosen logits only, the bias belongs to the logits
+SCORE_FN = {"softmax": 0, "sigmoid": 1, "sqrtsoftplus": 2, "softmax_chosen": 3}
 
 
 def prepack_fp4(packed: torch.Tensor, scale_e8m0: torch.Tensor) -> torch.Tensor:
@@ -100,6 +101,25 @@ def route(logits: torch.Tensor, bias: torch.Tensor | None, k: int, score_func: s
                                    int(norm_topk), ctypes.c_float(route_scale), _lib.ptr(idx), _lib.ptr(wts), _lib.stream())
     _lib.check(rc, "moe_route")
     return idx, wts
+
+
+def pack_experts(gate: list[torch.Tensor], up: list[torch.Tensor], down: list[torch.Tensor], width: int, ld: int, dtype: torch.dtype,
+                 device) -> tuple[ExpertWeights, ExpertWeights]:
+    """Gate, up [ff, width] and down [width, ff] of every expert, padded for the grouped GEMM on rows of ``ld`` columns."""
+    f32, real = dtype == torch.float32, gate[0].shape[0]
+    ff = (real + 15) // 16 * 16 if f32 else (real + 63) // 64 * 64     # the grouped GEMM tiles features by 128, gate and up together
+    out = ld if f32 else (ld + 127) // 128 * 128
+    w13, w2 = [], []
+    for g, u, d in zip(gate, up, down):
+        a = torch.zeros(2, ff, ld, dtype=dtype, device=device)
+        a[0, :real, :width] = g.to(device, dtype)
+        a[1, :real, :width] = u.to(device, dtype)
+        b = torch.zeros(out, ff, dtype=dtype, device=device)
+        b[:width, :real] = d.to(device, dtype)
+        w13.append(a.view(2 * ff, ld))
+        w2.append(b)
+    pack = ExpertWeights.from_f32 if f32 else ExpertWeights.from_bf16
+    return pack(w13), pack(w2)
 
 
 F32_TILE = 64                   # rows and features of a tile of the fp32 grouped GEMM

@@ -32,7 +32,7 @@ class Segments:
 def conv_rows(x: torch.Tensor, w_t: torch.Tensor, bias: torch.Tensor | None, tail: torch.Tensor, seg: Segments,
               positions: torch.Tensor, silu: bool = True) -> torch.Tensor:
     """x [T, >= C] (row stride allowed), w_t fp32 [taps, C], tail [slots, taps - 1, C] -> [T, C].  The tails of sequences with a
-    single row are replaced here, those of longer portions by ``selective_scan``."""
+    single row are replaced here, those of longer portions by ``selective_scan`` or ``conv_tails``."""
     taps, c = w_t.shape
     t = x.shape[0]
     assert x.stride(1) == 1 and tail.dtype == x.dtype and tail.shape[1:] == (max(taps - 1, 1), c)
@@ -43,6 +43,15 @@ def conv_rows(x: torch.Tensor, w_t: torch.Tensor, bias: torch.Tensor | None, tai
                                    int(x.dtype == torch.float32), _lib.stream())
     _lib.check(rc, "conv_rows")
     return y
+
+
+def conv_tails(x: torch.Tensor, tail: torch.Tensor, seg: Segments) -> None:
+    """The tails [slots, taps - 1, C] of sequences that bring more than one row, from the convolution's inputs x [T, >= C]."""
+    keep, c = tail.shape[1:]
+    assert x.stride(1) == 1 and tail.dtype == x.dtype and tail.is_contiguous()
+    rc = _lib.lib().b200_conv_tails(_lib.ptr(x), x.stride(0), _lib.ptr(tail), _lib.ptr(seg.first), _lib.ptr(seg.length), _lib.ptr(seg.slot),
+                                    seg.first.numel(), c, keep + 1, int(x.dtype == torch.float32), _lib.stream())
+    _lib.check(rc, "conv_tails")
 
 
 _ws: dict[int, torch.Tensor] = {}

@@ -3,8 +3,8 @@ for this rank, open the rank-0 -> workers command channel.
 
 Model strings:
   ``synthetic:qwen-tiny`` / ``synthetic:qwen-27b``  random-init models generated on the device
-  ``synthetic:rutulix-tiny`` / ``zigasun-tiny`` / ``kemirax-tiny``  likewise, the Rutulix, Zigasun and Kemirax decoders
-  a directory with ``config.json`` + safetensors      a family of ``models.registry`` (MLA + experts, Rutulix, Zigasun, Kemirax), else a
+  ``synthetic:rutulix-tiny`` / ``zigasun-tiny`` / ``kemirax-tiny`` / ``nunosun-tiny``  likewise, the decoders of those names
+  a directory with ``config.json`` + safetensors      a family of ``models.registry`` (MLA + experts, Rutulix, Zigasun, Kemirax, Nunosun), else a
                                                       Qwen-style hybrid FP8 checkpoint
   a ``.gguf`` file or bundle                          MoE families (routed by ``general.architecture``)
 """
@@ -321,7 +321,7 @@ class CppRuntimeAdapter:
 
 
 class GgufRuntimeAdapter:
-    """The same surface over a registry family's runtime (``models.registry`` builds it: GQA-MoE, Rutulix, Zigasun and Kemirax with paged
+    """The same surface over a registry family's runtime (``models.registry`` builds it: GQA-MoE, Rutulix, Zigasun, Kemirax and Nunosun with paged
     slots and a mixed-batch step, or the MLA runtimes): sequences admitted up to the runtime's slot count; greedy, and
     sampled where the runtime leaves its logits on the device."""
     supports_sampling = False
@@ -518,7 +518,7 @@ def _load_host(args):
         if spec is not None:
             raise ConfigurationError(f"the {spec.name} family needs a GPU")
     if model.startswith("synthetic:"):
-        if "tiny" not in model or any(f in model for f in ("rutulix", "zigasun", "kemirax")):
+        if "tiny" not in model or any(f in model for f in ("rutulix", "zigasun", "kemirax", "nunosun")):
             raise ConfigurationError("the host path generates only the tiny synthetic hybrid model")
         cfg = qh.QwenHybridConfig.tiny()
         state = qh.synth_state(cfg, 0, "cpu", std=0.05)
@@ -606,13 +606,14 @@ def load_runtime(args):
     raw_cfg, family_spec = None, None
     if model.startswith("synthetic:"):
         name = model.split(":", 1)[1]
-        if name in ("rutulix-tiny", "zigasun-tiny", "kemirax-tiny"):
+        if name in ("rutulix-tiny", "zigasun-tiny", "kemirax-tiny", "nunosun-tiny"):
             from ..models import kemirax as kx
+            from ..models import nunosun as ns
             from ..models import rutulix as rx
             from ..models import zigasun as zg
             from pocketllm.backends.native_backend import NullChannel
             mod, config = {"rutulix-tiny": (rx, rx.RutulixConfig), "zigasun-tiny": (zg, zg.ZigasunConfig),
-                           "kemirax-tiny": (kx, kx.KemiraxConfig)}[name]
+                           "kemirax-tiny": (kx, kx.KemiraxConfig), "nunosun-tiny": (ns, ns.NunosunConfig)}[name]
             rt = mod.build_synthetic(config.tiny(), dev, max_slots=slots, max_context=max_ctx)
             return GgufRuntimeAdapter(rt, max_ctx, slots, dev), None, channel or NullChannel()
     else:

@@ -100,7 +100,7 @@ class NativeBackend(BackendBase):
     def capabilities(self) -> BackendCapabilities:
         rt = self.runtime
         return BackendCapabilities(
-            name=self.name, models=("qwen3_5", "minimax_m2", "deepseek_v4", "glm_dsa", "rutulix", "zigasun", "kemirax"),
+            name=self.name, models=("qwen3_5", "minimax_m2", "deepseek_v4", "glm_dsa", "rutulix", "zigasun", "kemirax", "nunosun"),
             model_formats=("safetensors", "gguf", "synthetic"), devices=("cuda:sm_100a",),
             supports_batch=True, supports_streaming=True, supports_cancellation=True,
             supports_prefix_caching=bool(getattr(rt, "supports_prefix_cache", False)),
