@@ -26,7 +26,7 @@ from .paged import PagedRuntime
 
 ARCH = "Nunosun"
 # kernel sources the runtime launches (a partial build compiles only these)
-KERNEL_SOURCES = ("branch_step.cu", "row_act.cu", "conv_rows.cu", "qk_head_prep.cu", "attn_window_rows.cu", "decay_rule.cu",
+KERNEL_SOURCES = ("branch_step.cu", "row_act.cu", "conv_rows.cu", "qk_head_prep.cu", "attn_window_rows.cu", "attn_window_prefill.cu", "decay_rule.cu",
                   "gated_linear.cu", "head_linear.cu", "moe.cu", "bias_act.cu", "gemm_f32.cu", "gemm_wdec.cu", "gemm_bf16_2cta.cu",
                   "elementwise.cu", "sampling.cu", "bounds.cu")
 
@@ -433,6 +433,7 @@ class NunosunWeights:
 # ---------------------------------------------------------------------------------------------- runtime
 class NunosunRuntime(PagedRuntime):
     exposes_logits = True
+    tile_min_rows = winattn.TILE_MIN_ROWS
 
     def __init__(self, cfg: NunosunConfig, weights: NunosunWeights, max_slots: int = 1, max_context: int = 4096,
                  block_size: int = 64, num_blocks: int | None = None, comm=None):
@@ -440,7 +441,10 @@ class NunosunRuntime(PagedRuntime):
         if self.comm.world != 1:
             raise ValueError("a Nunosun model runs on one rank")
         self.cfg, self.w = cfg, weights
-        self.tile_min_rows = 1 << 30
+        tiles = weights.dtype == torch.bfloat16 and all(winattn.tiles_supported(lw.mix.left, block_size) for lw in weights.layers
+                                                        if isinstance(lw.mix, PairWeights))
+        if not tiles:
+            self.tile_min_rows = 1 << 30              # every row on the row kernel (fp32, or heads wider than the tile kernel takes)
         self.window = max([L.mixer.left.size for L in cfg.layers if isinstance(L.mixer, PairSpec)], default=0)
         self.k_cache: list[torch.Tensor | None] = []
         self.v_cache: list[torch.Tensor | None] = []
@@ -474,10 +478,14 @@ class NunosunRuntime(PagedRuntime):
         proj = pw.proj(y)
         q = winattn.head_prep(proj, m, positions, kv_slots, k, v)
         out = torch.empty(t, pw.left_o.k, dtype=y.dtype, device=y.device)
+        n = meta["tile_rows"] if meta["mode"] == "mixed" else 0
+        if n:
+            winattn.prefill(q[:n], m, k, v, self.block_table, meta["q_start"], meta["q_len"], meta["kv_len"], meta["max_q_len"], out[:n],
+                            seq=meta["tile_seq"])
         if meta["mode"] == "decode":
             winattn.rows(q, m, k, v, meta["block_table"], positions, meta["max_kv_len"], out)
-        else:
-            winattn.rows(q, m, k, v, self.block_table, positions, meta["max_kv_len"], out, seq=meta["row_seq"])
+        elif n < t:
+            winattn.rows(q[n:], m, k, v, self.block_table, positions[n:], meta["max_kv_len"], out[n:], seq=meta["row_seq"][n:])
         left = pw.left_o(out)
         right = pw.right_o(decay.retention(proj[:, pw.right_off:], pw.right, self.state[i], meta["segments"], positions, pw.right_o.k))
         return (left, pw.left_w), (right, pw.right_w)

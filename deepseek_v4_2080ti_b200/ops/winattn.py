@@ -1,5 +1,5 @@
 """Front-ends of attention with a sliding window and a learned bias per head and distance: per-head query / key norm prologue
-(csrc/kernels/qk_head_prep.cu) and single rows (attn_window_rows.cu).  Vectors are padded to multiples of 16 with zero rows of
+(csrc/kernels/qk_head_prep.cu), prompt tiles on the tensor cores (attn_window_prefill.cu) and single rows (attn_window_rows.cu).  Vectors are padded to multiples of 16 with zero rows of
 the projections.
 """
 from __future__ import annotations
@@ -15,6 +15,8 @@ from . import _lib
 
 _f = ctypes.c_float
 NUM_SMS = 148
+# entries with fewer new rows than this take the row kernel (keys of one row split over the SMs) instead of a 128-row tile
+TILE_MIN_ROWS = 16
 
 
 @dataclass
@@ -74,6 +76,26 @@ def head_prep(proj: torch.Tensor, m: WindowAttention, positions, slots, k_cache,
         _lib.ptr(v_cache), t, int(proj.dtype == torch.float32), _lib.stream())
     _lib.check(rc, "qk_head_prep")
     return q
+
+
+def tiles_supported(m: WindowAttention, block_size: int) -> bool:
+    return bool(_lib.lib().b200_attn_window_prefill_supported(m.heads, m.groups, m.d, m.v, block_size))
+
+
+def prefill(q: torch.Tensor, m: WindowAttention, k_cache, v_cache, block_table, q_start, q_len, kv_len, max_q_len: int,
+            out: torch.Tensor, seq: torch.Tensor | None = None) -> torch.Tensor:
+    """Rows of several sequences' portions (tensor-core tiles).  ``out`` [rows, ldo] bf16 in place; ``seq`` names each entry's row
+    of ``block_table``."""
+    nb, bs, _ = k_cache.shape
+    assert q.is_contiguous() and out.stride(1) == 1
+    _lib.check_indices(block_table, 0, nb, 3)
+    rc = _lib.lib().b200_attn_window_prefill(
+        _lib.ptr(q), _lib.ptr(k_cache), _lib.ptr(v_cache), _lib.ptr(m.bias), _lib.ptr(out), out.stride(0), _lib.ptr(block_table),
+        _lib.ptr(seq), _lib.ptr(q_start), _lib.ptr(q_len), _lib.ptr(kv_len), q_len.numel(), int(max_q_len), q.shape[0],
+        block_table.shape[1], nb, bs, m.heads, m.groups, m.d, m.v, m.size, _f(m.scale), _lib.ptr(_lib.status_word(out.device)),
+        _lib.stream())
+    _lib.check(rc, "attn_window_prefill")
+    return out
 
 
 _ws: dict[int, torch.Tensor] = {}
