@@ -27,7 +27,7 @@ from .paged import PagedRuntime
 ARCH = "Nunosun"
 # kernel sources the runtime launches (a partial build compiles only these)
 KERNEL_SOURCES = ("branch_step.cu", "row_act.cu", "conv_rows.cu", "qk_head_prep.cu", "attn_window_rows.cu", "attn_window_prefill.cu", "decay_rule.cu",
-                  "gated_linear.cu", "head_linear.cu", "moe.cu", "bias_act.cu", "gemm_f32.cu", "gemm_wdec.cu", "gemm_bf16_2cta.cu",
+                  "decay_chunk.cu", "gated_linear.cu", "head_linear.cu", "moe.cu", "bias_act.cu", "gemm_f32.cu", "gemm_wdec.cu", "gemm_bf16_2cta.cu",
                   "elementwise.cu", "sampling.cu", "bounds.cu")
 
 

@@ -1,6 +1,7 @@
-"""Front-ends of the recurrences with one decay per head (csrc/kernels/decay_rule.cu): retention (a fixed decay, rotated
-queries and keys) and the gated delta rule, each over a batch of rows of several sequences (``ops.scan.Segments``), with
-per-head norm and gate.  Batches of single rows are one launch."""
+"""Front-ends of the recurrences with one decay per head (csrc/kernels/decay_rule.cu, decay_chunk.cu): retention (a fixed decay,
+rotated queries and keys) and the gated delta rule, each over a batch of rows of several sequences (``ops.scan.Segments``),
+with per-head norm and gate.  Batches of single rows are one launch; bf16 portions run in chunks on the tensor cores, fp32 and
+very short portions token by token."""
 from __future__ import annotations
 
 import ctypes
@@ -11,6 +12,7 @@ import torch
 from . import _lib, scan
 
 _f = ctypes.c_float
+CHUNK_MIN_ROWS = 16             # bf16 portions with fewer rows run token by token
 STEP_MAX_V = 2048               # widest value head of the single-row kernel
 
 
@@ -56,12 +58,26 @@ class DeltaRule:
 
 def _portions(q, k, v, log_decay, decay, beta, heads: int, groups: int, d: int, vw: int, state, seg, positions) -> torch.Tensor:
     """Prepared rows -> read-outs fp32 [T, heads * vw]; ``state`` in place."""
-    t, f32 = v.shape[0], int(v.dtype == torch.float32)
-    o = torch.empty(t, heads * vw, dtype=torch.float32, device=v.device)
-    rc = _lib.lib().b200_decay_scan(_lib.ptr(q), _lib.ptr(k), _lib.ptr(v), v.stride(0), _lib.ptr(log_decay), _lib.ptr(decay), _lib.ptr(beta),
-                                    _lib.ptr(state), _lib.ptr(o), _lib.ptr(seg.first), _lib.ptr(seg.length), _lib.ptr(seg.slot),
-                                    _lib.ptr(positions), seg.first.numel(), 0, heads, groups, d, vw, f32, _lib.stream())
-    _lib.check(rc, "decay_scan")
+    t, f32, dev, L = v.shape[0], int(v.dtype == torch.float32), v.device, _lib.lib()
+    entries = seg.first.numel()
+    o = torch.empty(t, heads * vw, dtype=torch.float32, device=dev)
+    rows = 0 if f32 else L.b200_decay_chunk_rows(d)
+    chunked = rows > 0 and seg.max_length >= CHUNK_MIN_ROWS
+    if chunked:
+        chunks, delta = t // rows + entries, int(beta is not None)
+        ws = torch.empty(chunks * heads * L.b200_decay_chunk_ws(d, delta), dtype=torch.bfloat16, device=dev)
+        u0 = torch.empty(chunks * heads * rows * vw, dtype=torch.float32, device=dev) if delta else None
+        end = torch.empty(chunks * heads, dtype=torch.float32, device=dev)
+        rc = L.b200_decay_chunk(_lib.ptr(q), _lib.ptr(k), _lib.ptr(v), v.stride(0), _lib.ptr(log_decay), _lib.ptr(decay), _lib.ptr(beta),
+                                _lib.ptr(state), _lib.ptr(o), _lib.ptr(seg.first), _lib.ptr(seg.length), _lib.ptr(seg.slot),
+                                _lib.ptr(positions), entries, CHUNK_MIN_ROWS, chunks, _lib.ptr(ws), _lib.ptr(u0), _lib.ptr(end), heads,
+                                groups, d, vw, _lib.stream())
+        _lib.check(rc, "decay_chunk", 2)
+    if not chunked or seg.min_length < CHUNK_MIN_ROWS:
+        rc = L.b200_decay_scan(_lib.ptr(q), _lib.ptr(k), _lib.ptr(v), v.stride(0), _lib.ptr(log_decay), _lib.ptr(decay), _lib.ptr(beta),
+                               _lib.ptr(state), _lib.ptr(o), _lib.ptr(seg.first), _lib.ptr(seg.length), _lib.ptr(seg.slot),
+                               _lib.ptr(positions), entries, CHUNK_MIN_ROWS - 1 if chunked else 0, heads, groups, d, vw, f32, _lib.stream())
+        _lib.check(rc, "decay_scan")
     return o
 
 
