@@ -42,7 +42,7 @@ def parse():
                     help="config 2: also run greedy speculative decoding after the timed steps (mtp: a random-init "
                          "multi-token-prediction head is added to the synthetic checkpoint) and report acceptance")
     ap.add_argument("--spec-tokens", type=int, default=2)
-    ap.add_argument("--design", choices=["rutulix", "zigasun", "kemirax"], default=None,
+    ap.add_argument("--design", choices=["rutulix", "zigasun", "kemirax", "nunosun"], default=None,
                     help="instead of the headline workload: one decoder design at model-like layer sizes beside the closest "
                          "existing model, with the kernels' roofline fractions (utils/design_bench.py; one GPU)")
     ap.add_argument("--design-size", choices=["small", "large"], default=None, help="--design: only this size")

@@ -9,7 +9,7 @@
 //   delta_prep      unit queries and keys, log decays and step sizes of every row, fp32
 //   rotate_prep     rotated queries and keys of every row, fp32
 //   decay_scan      one token after the other: eight lanes share a column of the state.  For fp32, and for bf16 portions too
-//                   short for decay_chunk.cu
+//                   short for retention_chunk.cu and delta_chunk.cu
 //   decay_step      one token of many sequences: a block per head and sequence reads, updates and writes the state once,
 //                   with the row's preparation in front and norm and gate behind
 // The norm and the gate of prepared rows are gla_finish (gated_linear.cu).
@@ -74,7 +74,8 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(DeltaPrepParams<T> p, i
   }
 }
 
-// A block per row.  Pairs (i, i + rot / 2) of every query and key vector are rotated, the rest passes; keys are scaled.
+// A block per row.  Pairs (i, i + rot / 2) of every query and key vector are rotated, the rest passes; keys are scaled.  A thread
+// takes eight neighbouring channels (and their partners where those are eight neighbours as well).
 template <typename T>
 __global__ void __launch_bounds__(256) rotate_prep_kernel(const T* __restrict__ q, const T* __restrict__ k, int ld,
                                                           const int* __restrict__ positions, const double* __restrict__ freq, int rot,
@@ -88,14 +89,33 @@ __global__ void __launch_bounds__(256) rotate_prep_kernel(const T* __restrict__ 
   const int pos = positions[row];
   for (int i = threadIdx.x; i < half; i += blockDim.x) rotary_angle(pos, freq[i], 1.f, cs[i].x, cs[i].y);
   __syncthreads();
-  for (int i = threadIdx.x; i < 2 * n; i += blockDim.x) {
+  const bool vectors = half % 8 == 0;
+  for (int i = threadIdx.x * 8; i < 2 * n; i += blockDim.x * 8) {
     const bool is_k = i >= n;
     const int c = is_k ? i - n : i, d = c % D;
     const T* src = (is_k ? k : q) + row * ld + c;
-    float f = (float)*src;
-    if (d < half) f = f * cs[d].x - (float)src[half] * cs[d].y;
-    else if (d < rot) f = f * cs[d - half].x + (float)src[-half] * cs[d - half].y;
-    (is_k ? k_out : q_out)[row * n + c] = is_k ? f * k_scale : f;
+    float f[8];
+    load8(src, f);
+    if (vectors) {
+      if (d < rot) {
+        const bool low = d < half;
+        float o[8];
+        load8(src + (low ? half : -half), o);
+        const float2* a = cs + (low ? d : d - half);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) f[j] = f[j] * a[j].x + (low ? -o[j] : o[j]) * a[j].y;
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        if (d + j < half) f[j] = f[j] * cs[d + j].x - (float)src[j + half] * cs[d + j].y;
+        else if (d + j < rot) f[j] = f[j] * cs[d + j - half].x + (float)src[j - half] * cs[d + j - half].y;
+      }
+    }
+    const float s = is_k ? k_scale : 1.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) f[j] *= s;
+    store8((is_k ? k_out : q_out) + row * n + c, f);
   }
 }
 
@@ -448,7 +468,7 @@ extern "C" int b200_delta_prep(const void* qk, int ld_qk, const void* a, const v
 // q, k: H heads of D channels in rows `ld` apart, the first `rot` (even) rotated in pairs (i, i + rot / 2); fp32 out [rows, H, D].
 extern "C" int b200_rotate_prep(const void* q, const void* k, int ld, const int* positions, const double* freq, int rot, float k_scale,
                                 float* q_out, float* k_out, int rows, int H, int D, int f32, cudaStream_t stream) {
-  if (rows <= 0 || H <= 0 || D <= 0 || rot < 0 || (rot & 1) || rot > D || rot > 4096 || ld < H * D) return -6;
+  if (rows <= 0 || H <= 0 || D <= 0 || (D & 7) || (ld & 7) || rot < 0 || (rot & 1) || rot > D || rot > 4096 || ld < H * D) return -6;
   const size_t smem = (size_t)(rot / 2) * 8;
   if (f32)
     return (int)launch_pdl(rotate_prep_kernel<float>, dim3(rows), dim3(256), smem, stream, reinterpret_cast<const float*>(q),

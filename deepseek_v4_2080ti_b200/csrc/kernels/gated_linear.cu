@@ -239,23 +239,23 @@ __global__ void __launch_bounds__(STEP_THREADS) gla_step_kernel(GlaStepParams<T>
 __device__ __forceinline__ float silu_of(float z, __nv_bfloat16) { return __fdividef(z, 1.f + __expf(-z)); }
 __device__ __forceinline__ float silu_of(float z, float) { return z / (1.f + expf(-z)); }
 
-// A warp per (row, head): out[row, h * V + c] = o / rms over the head's vdim values * weight * silu(gate).
-template <typename T, int KEEP>             // KEEP: 256-column rounds held in registers
+// LANES lanes per (row, head): out[row, h * V + c] = o / rms over the head's vdim values * weight * silu(gate).
+template <typename T, int KEEP, int LANES>  // KEEP: rounds of 8 LANES columns held in registers
 __global__ void gla_finish_kernel(const float* __restrict__ o, const T* __restrict__ gate, int ld_gate, const float* __restrict__ w,
                                   T* __restrict__ out, int ldo, int rows, int H, int V, int vdim, float eps) {
   pdl_grid_trigger();
   pdl_grid_wait();
-  const int lane = threadIdx.x & 31;
-  const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  const size_t row = item / H;
-  const int h = (int)(item - (long long)row * H);
-  if (row >= (size_t)rows) return;
-  const float* src = o + item * V;
+  const int lane = threadIdx.x % LANES;
+  const long long item = (long long)blockIdx.x * (blockDim.x / LANES) + threadIdx.x / LANES;
+  const bool on = item < (long long)rows * H;               // the sums below are shuffles of whole warps
+  const size_t row = on ? item / H : 0;
+  const int h = on ? (int)(item - (long long)row * H) : 0;
+  const float* src = o + (on ? item : 0) * V;
   const T* gsrc = gate + row * ld_gate + h * V;
   float f[KEEP][8], g[KEEP][8], ss = 0.f;
 #pragma unroll
   for (int i = 0; i < KEEP; ++i) {
-    const int c = i * 256 + lane * 8;
+    const int c = i * 8 * LANES + lane * 8;
     if (c < V) {
       load8(src + c, f[i]);
       load8(gsrc + c, g[i]);
@@ -263,13 +263,16 @@ __global__ void gla_finish_kernel(const float* __restrict__ o, const T* __restri
       for (int j = 0; j < 8; ++j) ss += f[i][j] * f[i][j];               // padded columns are zero
     }
   }
-  for (int c = KEEP * 256 + lane * 8; c < V; c += 256) {
+  for (int c = KEEP * 8 * LANES + lane * 8; c < V; c += 8 * LANES) {
     float t[8];
     load8(src + c, t);
 #pragma unroll
     for (int j = 0; j < 8; ++j) ss += t[j] * t[j];
   }
-  const float inv = 1.f / sqrtf(warp_sum_all(ss) / (float)vdim + eps);
+#pragma unroll
+  for (int x = LANES / 2; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
+  if (!on) return;
+  const float inv = 1.f / sqrtf(ss / (float)vdim + eps);
   auto finish = [&](int c, float (&v)[8], const float (&gv)[8]) {
     float ww[8];
     load8(w + c, ww);
@@ -279,15 +282,15 @@ __global__ void gla_finish_kernel(const float* __restrict__ o, const T* __restri
   };
 #pragma unroll
   for (int i = 0; i < KEEP; ++i)
-    if (i * 256 + lane * 8 < V) finish(i * 256 + lane * 8, f[i], g[i]);
-  for (int c = KEEP * 256 + lane * 8; c < V; c += 256) {
+    if (i * 8 * LANES + lane * 8 < V) finish(i * 8 * LANES + lane * 8, f[i], g[i]);
+  for (int c = KEEP * 8 * LANES + lane * 8; c < V; c += 8 * LANES) {
     float v[8], gv[8];
     load8(src + c, v);
     load8(gsrc + c, gv);
     finish(c, v, gv);
   }
   if (h == H - 1)
-    for (int c = H * V + lane; c < ldo; c += 32) out[row * ldo + c] = (T)0.f;
+    for (int c = H * V + lane; c < ldo; c += LANES) out[row * ldo + c] = (T)0.f;
 }
 
 template <typename T, int RD>
@@ -334,11 +337,14 @@ template <typename T>
 int run_finish(const float* o, const void* gate, int ld_gate, const float* w, void* out, int ldo, int rows, int H, int V, int vdim,
                float eps, cudaStream_t stream) {
   const long long items = (long long)rows * H;
-  const dim3 grid((unsigned)((items + 7) / 8)), block(256);
+  const int lanes = V <= 64 ? 8 : V <= 128 ? 16 : 32, per = 256 / lanes;
+  const dim3 grid((unsigned)((items + per - 1) / per)), block(256);
   auto gp = reinterpret_cast<const T*>(gate);
   auto op = reinterpret_cast<T*>(out);
-  if (V <= 256) return (int)launch_pdl(gla_finish_kernel<T, 1>, grid, block, 0, stream, o, gp, ld_gate, w, op, ldo, rows, H, V, vdim, eps);
-  return (int)launch_pdl(gla_finish_kernel<T, 2>, grid, block, 0, stream, o, gp, ld_gate, w, op, ldo, rows, H, V, vdim, eps);
+  if (lanes == 8) return (int)launch_pdl(gla_finish_kernel<T, 1, 8>, grid, block, 0, stream, o, gp, ld_gate, w, op, ldo, rows, H, V, vdim, eps);
+  if (lanes == 16) return (int)launch_pdl(gla_finish_kernel<T, 1, 16>, grid, block, 0, stream, o, gp, ld_gate, w, op, ldo, rows, H, V, vdim, eps);
+  if (V <= 256) return (int)launch_pdl(gla_finish_kernel<T, 1, 32>, grid, block, 0, stream, o, gp, ld_gate, w, op, ldo, rows, H, V, vdim, eps);
+  return (int)launch_pdl(gla_finish_kernel<T, 2, 32>, grid, block, 0, stream, o, gp, ld_gate, w, op, ldo, rows, H, V, vdim, eps);
 }
 
 template <typename T>

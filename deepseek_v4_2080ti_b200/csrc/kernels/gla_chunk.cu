@@ -20,6 +20,7 @@
 #include "launch.h"
 #include "ops.h"
 #include "per_device.h"
+#include "split_mma.cuh"
 
 namespace {
 using namespace b200;
@@ -37,43 +38,6 @@ struct ChunkParams {
   int ld, H, D, V, entries, min_len;
   float scale;
 };
-
-__device__ __forceinline__ float pow2(float v) {
-  float e;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(v));
-  return e;
-}
-__device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
-  return *reinterpret_cast<const uint32_t*>(&h);
-}
-// Two values as two bf16 terms each.
-__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
-  const float2 f = __bfloat1622float2(h);
-  hi = *reinterpret_cast<const uint32_t*>(&h);
-  lo = pack_bf16(a - f.x, b - f.y);
-}
-__device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], const void* p) {
-  const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
-}
-__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], const void* p) {
-  const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
-}
-__device__ __forceinline__ void cp16(void* dst, const void* src, bool ok) {
-  const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
-  const int n = ok ? 16 : 0;                                     // 0 source bytes: the 16 bytes are zero-filled
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(n) : "memory");
-}
 
 __device__ __forceinline__ int chunks_of(const ChunkParams& p, int e, int CL) {
   const int n = p.length[e];
@@ -285,7 +249,7 @@ __global__ void __launch_bounds__(512) gla_chunk_scan_kernel(ChunkParams p) {
     }
     float* end = reinterpret_cast<float*>(dst + CL * LV);
     for (int i = tid; i < DT / 4; i += nthr) cp16(end + i * 4, p.end + at * DT + i * 4, true);
-    asm volatile("cp.async.commit_group;" ::: "memory");
+    cp_commit();
   };
   fetch(0, 0);
   const int vw = v0 + vg * 16, d_own = sub * ND;
@@ -317,7 +281,7 @@ __global__ void __launch_bounds__(512) gla_chunk_scan_kernel(ChunkParams p) {
   const int brow = (lane & 7) + (lane >> 4) * 8, bcol = ((lane >> 3) & 1) * 8;   // right operand stored by column; left, transposed
   const int trow = (lane & 7) + ((lane >> 3) & 1) * 8;                       // right operand, transposed
   for (int c = 0; c < chunks; ++c) {
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    cp_wait<0>();
     __syncthreads();                                    // chunk and state landed; the other buffer's readers are done
     if (c + 1 < chunks) fetch(c + 1, (c + 1) & 1);
     const __nv_bfloat16* sq = reinterpret_cast<const __nv_bfloat16*>(smem + (c & 1) * stage);
@@ -402,7 +366,7 @@ __global__ void __launch_bounds__(512) gla_chunk_scan_kernel(ChunkParams p) {
     __syncthreads();                                    // everyone has read the state of before the chunk
     publish();
   }
-  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  cp_wait<0>();
   if (!live) return;
 #pragma unroll
   for (int i = 0; i < NS; ++i)

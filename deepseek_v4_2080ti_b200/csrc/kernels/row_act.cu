@@ -108,9 +108,9 @@ __global__ void token_gate_kernel(const T* __restrict__ z, int ldz, const T* __r
 
 template <typename T>
 int run_poly_norm(const void* z, int ldz, void* y, int ldy, int cols, const PolyShape& s, int rows, cudaStream_t stream) {
-  const int nvec = ldy >> 3;
-  int threads = (nvec + 31) / 32 * 32;
-  if (threads > 256) threads = nvec > 1024 ? 512 : 256;
+  const int nvec = ldy >> 3, want = nvec <= 256 ? 1 : nvec <= 512 ? 2 : 4;          // vectors of a thread
+  int threads = ((nvec + want - 1) / want + 31) / 32 * 32;
+  if (threads > 512) threads = 512;
   const int vec = (nvec + threads - 1) / threads;
   const T* zp = reinterpret_cast<const T*>(z);
   T* yp = reinterpret_cast<T*>(y);

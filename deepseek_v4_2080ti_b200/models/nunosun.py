@@ -27,7 +27,7 @@ from .paged import PagedRuntime
 ARCH = "Nunosun"
 # kernel sources the runtime launches (a partial build compiles only these)
 KERNEL_SOURCES = ("branch_step.cu", "row_act.cu", "conv_rows.cu", "qk_head_prep.cu", "attn_window_rows.cu", "attn_window_prefill.cu", "decay_rule.cu",
-                  "decay_chunk.cu", "gated_linear.cu", "head_linear.cu", "moe.cu", "bias_act.cu", "gemm_f32.cu", "gemm_wdec.cu", "gemm_bf16_2cta.cu",
+                  "retention_chunk.cu", "delta_chunk.cu", "gated_linear.cu", "head_linear.cu", "moe.cu", "bias_act.cu", "gemm_f32.cu", "gemm_wdec.cu", "gemm_bf16_2cta.cu",
                   "elementwise.cu", "sampling.cu", "bounds.cu")
 
 
@@ -383,9 +383,9 @@ class NunosunWeights:
         left = WindowAttention(a.heads, a.kv_heads, a.dim, d, a.vdim, v, a.scale, a.size, self.cfg.eps, self._row(t["left.q.norm"], d),
                                self._row(t["left.k.norm"], d), winattn.distance_bias(rel.to(self.device), a.size, a.reach))
         freq = r.rot_base ** (-torch.arange(0, r.rot_dims, 2, dtype=torch.float64) / max(r.rot_dims, 1))
-        right = Retention(r.heads, r.dim, rd, r.vdim, rv, self.cfg.eps, r.rot_dims, freq.to(self.device),
-                          torch.tensor(r.decay, dtype=torch.float64).to(self.device, torch.float32),
-                          torch.ones(rv, dtype=torch.float32, device=self.device))
+        fixed = torch.tensor(r.decay, dtype=torch.float64)
+        right = Retention(r.heads, r.dim, rd, r.vdim, rv, self.cfg.eps, r.rot_dims, freq.to(self.device), fixed.float().to(self.device),
+                          torch.log2(fixed).float().to(self.device), torch.ones(rv, dtype=torch.float32, device=self.device))
         rows = [(pad_heads(t["left." + n], h, ((real, pad),)), h * pad)
                 for n, h, real, pad in (("q", a.heads, a.dim, d), ("k", a.kv_heads, a.dim, d), ("v", a.kv_heads, a.vdim, v))]
         off = sum(n for _, n in rows)

@@ -1,5 +1,5 @@
-"""Front-ends of the recurrences with one decay per head (csrc/kernels/decay_rule.cu, decay_chunk.cu): retention (a fixed decay,
-rotated queries and keys) and the gated delta rule, each over a batch of rows of several sequences (``ops.scan.Segments``),
+"""Front-ends of the recurrences with one decay per head (csrc/kernels/decay_rule.cu, retention_chunk.cu,
+delta_chunk.cu): retention (a fixed decay, rotated queries and keys) and the gated delta rule, each over a batch of rows of several sequences (``ops.scan.Segments``),
 with per-head norm and gate.  Batches of single rows are one launch; bf16 portions run in chunks on the tensor cores, fp32 and
 very short portions token by token."""
 from __future__ import annotations
@@ -9,6 +9,7 @@ from dataclasses import dataclass
 
 import torch
 
+from ..utils import canary
 from . import _lib, scan
 
 _f = ctypes.c_float
@@ -28,6 +29,7 @@ class Retention:
     rot: int
     freq: torch.Tensor          # fp64 [rot / 2]
     decay: torch.Tensor         # fp32 [heads]
+    log2_decay: torch.Tensor    # fp32 [heads]
     norm_w: torch.Tensor        # fp32 [v]
 
     @property
@@ -56,28 +58,64 @@ class DeltaRule:
         return 2 * self.groups * self.d + self.heads * self.v
 
 
-def _portions(q, k, v, log_decay, decay, beta, heads: int, groups: int, d: int, vw: int, state, seg, positions) -> torch.Tensor:
-    """Prepared rows -> read-outs fp32 [T, heads * vw]; ``state`` in place."""
-    t, f32, dev, L = v.shape[0], int(v.dtype == torch.float32), v.device, _lib.lib()
-    entries = seg.first.numel()
-    o = torch.empty(t, heads * vw, dtype=torch.float32, device=dev)
-    rows = 0 if f32 else L.b200_decay_chunk_rows(d)
-    chunked = rows > 0 and seg.max_length >= CHUNK_MIN_ROWS
+_ws: dict[int, torch.Tensor] = {}
+
+
+def _workspace(sizes: list[int], device) -> list[int]:
+    """Addresses of buffers of the given bytes in the device's workspace (used within one call; grown on demand)."""
+    sizes = [(n + 255) // 256 * 256 for n in sizes]
+    dev = device.index or 0
+    ws = _ws.get(dev)
+    if ws is None or ws.numel() < sum(sizes):
+        ws = _ws[dev] = canary.empty(max(sum(sizes), 1 << 20), dtype=torch.uint8, device=device, name="recurrence chunks")
+    out, at = [], ws.data_ptr()
+    for n in sizes:
+        out.append(ctypes.c_void_p(at))
+        at += n
+    return out
+
+
+def _scan(q, k, v, log_decay, decay, beta, m, groups: int, state, o, seg, positions, max_len: int) -> None:
+    rc = _lib.lib().b200_decay_scan(_lib.ptr(q), _lib.ptr(k), _lib.ptr(v), v.stride(0), _lib.ptr(log_decay), _lib.ptr(decay), _lib.ptr(beta),
+                                    _lib.ptr(state), _lib.ptr(o), _lib.ptr(seg.first), _lib.ptr(seg.length), _lib.ptr(seg.slot),
+                                    _lib.ptr(positions), seg.first.numel(), max_len, m.heads, groups, m.d, m.v,
+                                    int(v.dtype == torch.float32), _lib.stream())
+    _lib.check(rc, "decay_scan")
+
+
+def _delta_portions(q, k, v, log_decay, beta, m: "DeltaRule", state, seg, positions) -> torch.Tensor:
+    """Prepared rows -> read-outs fp32 [T, heads * v]; ``state`` in place."""
+    t, dev, L, entries = v.shape[0], v.device, _lib.lib(), seg.first.numel()
+    o = torch.empty(t, m.heads * m.v, dtype=torch.float32, device=dev)
+    n = 0 if v.dtype == torch.float32 else L.b200_delta_chunk_rows(m.d)
+    chunked = n > 0 and seg.max_length >= CHUNK_MIN_ROWS
     if chunked:
-        chunks, delta = t // rows + entries, int(beta is not None)
-        ws = torch.empty(chunks * heads * L.b200_decay_chunk_ws(d, delta), dtype=torch.bfloat16, device=dev)
-        u0 = torch.empty(chunks * heads * rows * vw, dtype=torch.float32, device=dev) if delta else None
-        end = torch.empty(chunks * heads, dtype=torch.float32, device=dev)
-        rc = L.b200_decay_chunk(_lib.ptr(q), _lib.ptr(k), _lib.ptr(v), v.stride(0), _lib.ptr(log_decay), _lib.ptr(decay), _lib.ptr(beta),
-                                _lib.ptr(state), _lib.ptr(o), _lib.ptr(seg.first), _lib.ptr(seg.length), _lib.ptr(seg.slot),
-                                _lib.ptr(positions), entries, CHUNK_MIN_ROWS, chunks, _lib.ptr(ws), _lib.ptr(u0), _lib.ptr(end), heads,
-                                groups, d, vw, _lib.stream())
-        _lib.check(rc, "decay_chunk", 2)
+        chunks, w = t // n + entries, L.b200_delta_chunk_width(m.d)
+        rows, mats, fade = _workspace([chunks * m.groups * 8 * n * w, chunks * m.heads * 8 * n * n, chunks * m.heads * 8 * n], dev)
+        rc = L.b200_delta_chunk(_lib.ptr(q), _lib.ptr(k), _lib.ptr(v), v.stride(0), _lib.ptr(log_decay), _lib.ptr(beta), _lib.ptr(state),
+                                _lib.ptr(o), _lib.ptr(seg.first), _lib.ptr(seg.length), _lib.ptr(seg.slot), _lib.ptr(positions), entries,
+                                CHUNK_MIN_ROWS, chunks, rows, mats, fade, m.heads, m.groups, m.d, m.v, _lib.stream())
+        _lib.check(rc, "delta_chunk", 2)
     if not chunked or seg.min_length < CHUNK_MIN_ROWS:
-        rc = L.b200_decay_scan(_lib.ptr(q), _lib.ptr(k), _lib.ptr(v), v.stride(0), _lib.ptr(log_decay), _lib.ptr(decay), _lib.ptr(beta),
-                               _lib.ptr(state), _lib.ptr(o), _lib.ptr(seg.first), _lib.ptr(seg.length), _lib.ptr(seg.slot),
-                               _lib.ptr(positions), entries, CHUNK_MIN_ROWS - 1 if chunked else 0, heads, groups, d, vw, f32, _lib.stream())
-        _lib.check(rc, "decay_scan")
+        _scan(q, k, v, log_decay, None, beta, m, m.groups, state, o, seg, positions, CHUNK_MIN_ROWS - 1 if chunked else 0)
+    return o
+
+
+def _retention_portions(q, k, v, m: "Retention", state, seg, positions) -> torch.Tensor:
+    """Prepared rows -> read-outs fp32 [T, heads * v]; ``state`` in place."""
+    t, dev, L, entries = v.shape[0], v.device, _lib.lib(), seg.first.numel()
+    o = torch.empty(t, m.heads * m.v, dtype=torch.float32, device=dev)
+    n = 0 if v.dtype == torch.float32 else L.b200_retention_chunk_rows(m.d)
+    chunked = n > 0 and seg.max_length >= CHUNK_MIN_ROWS
+    if chunked:
+        chunks = t // n + entries
+        ws, end = _workspace([chunks * m.heads * L.b200_retention_chunk_ws(m.d) * 2, chunks * m.heads * 4], dev)
+        rc = L.b200_retention_chunk(_lib.ptr(q), _lib.ptr(k), _lib.ptr(v), v.stride(0), _lib.ptr(m.log2_decay), _lib.ptr(state), _lib.ptr(o),
+                                    _lib.ptr(seg.first), _lib.ptr(seg.length), _lib.ptr(seg.slot), _lib.ptr(positions), entries,
+                                    CHUNK_MIN_ROWS, chunks, ws, end, m.heads, m.d, m.v, _lib.stream())
+        _lib.check(rc, "retention_chunk", 2)
+    if not chunked or seg.min_length < CHUNK_MIN_ROWS:
+        _scan(q, k, v, None, m.decay, None, m, m.heads, state, o, seg, positions, CHUNK_MIN_ROWS - 1 if chunked else 0)
     return o
 
 
@@ -115,7 +153,7 @@ def retention(proj: torch.Tensor, m: Retention, state: torch.Tensor, seg, positi
     rc = _lib.lib().b200_rotate_prep(_lib.ptr(q), _lib.ptr(k), ld, _lib.ptr(positions), _lib.ptr(m.freq), m.rot, _f(scale), _lib.ptr(qf),
                                      _lib.ptr(kf), t, m.heads, m.d, f32, _lib.stream())
     _lib.check(rc, "rotate_prep")
-    return _finish(_portions(qf, kf, v, None, m.decay, None, m.heads, m.heads, m.d, m.v, state, seg, positions), g, m, ldo)
+    return _finish(_retention_portions(qf, kf, v, m, state, seg, positions), g, m, ldo)
 
 
 def delta_rule(proj: torch.Tensor, m: DeltaRule, state: torch.Tensor, tail: torch.Tensor, seg, positions, ldo: int) -> torch.Tensor:
@@ -143,4 +181,4 @@ def delta_rule(proj: torch.Tensor, m: DeltaRule, state: torch.Tensor, tail: torc
     rc = _lib.lib().b200_delta_prep(_lib.ptr(x), c, _lib.ptr(a), _lib.ptr(b), ldg, _lib.ptr(m.neg_a), _lib.ptr(m.dt), _lib.ptr(qf),
                                     _lib.ptr(kf), _lib.ptr(ld_), _lib.ptr(beta), t, m.heads, m.groups, m.d, _f(scale), f32, _lib.stream())
     _lib.check(rc, "delta_prep")
-    return _finish(_portions(qf, kf, x[:, 2 * gd:], ld_, None, beta, m.heads, m.groups, m.d, m.v, state, seg, positions), g, m, ldo)
+    return _finish(_delta_portions(qf, kf, x[:, 2 * gd:], ld_, beta, m, state, seg, positions), g, m, ldo)

@@ -1,12 +1,14 @@
 """Prefill and decode throughput of one decoder design at sizes of real models' layers (random weights), beside the
 framework's closest existing model at equal size, and the kernels of both beside their rooflines.
 
-    python bench.py --design rutulix|zigasun|kemirax [--design-size small|large] [--steps K] [--warmup W]
+    python bench.py --design rutulix|zigasun|kemirax|nunosun [--design-size small|large] [--steps K] [--warmup W]
 
 Closest model of Rutulix: the Qwen-style decoder with full-attention layers only (per-head QK norm, grouped attention, SwiGLU
 with FP8 weights) of the same width, heads and feed-forward parameters.  Of Zigasun: the same decoder with Gated-DeltaNet and
 full-attention layers in turn (both recurrent states as wide as the scan's channels).  Of Kemirax: the latent-attention
-decoder with routed experts, equal width, heads, latents and experts; its recurrence stands beside Gated DeltaNet.  Whole-model numbers: CUDA events around a prompt of
+decoder with routed experts, equal width, heads, latents and experts; its recurrence stands beside Gated DeltaNet.  Of Nunosun:
+the Qwen-style decoder with Gated-DeltaNet and full-attention layers in turn, equal width, heads, recurrent channels and
+feed-forward parameters per token.  Whole-model numbers: CUDA events around a prompt of
 ``--prompt`` tokens and around replayed decode steps.  Kernel numbers: CUDA events around single launches, L2 flushed
 before each; fractions of the measured copy bandwidth / bf16 GEMM burst of MEASURED_PEAKS.json.
 """
@@ -26,6 +28,11 @@ ZG_SIZES = {"small": (2048, 16, 4, 64, 128, 5632, 4096, 16, 128), "large": (4096
 # width, experts, identity experts, experts per token
 KX_SIZES = {"small": (2048, 16, 128, 64, 128, 768, 512, 16, 1024, 64, 8, 6), "large": (4096, 32, 128, 64, 128, 1536, 512, 32, 1536, 128, 16, 8)}
 KX_LAYERS = "gaba"
+# Nunosun: width, heads, kv heads (128 x 128), window, retention heads (128 x 128), delta-rule heads and query / key heads
+# (128 x 128), SwiGLU width of the closest model (the two-matrix feed-forward gets 3/2 of it, the experts of a token together
+# as much), experts, experts per token, side embedding
+NS_SIZES = {"small": (2048, 16, 4, 2048, 16, 32, 16, 5632, 64, 8, 256), "large": (4096, 32, 8, 4096, 32, 64, 16, 10752, 128, 8, 256)}
+NS_LAYERS = "dpdp"
 LAYERS, VOCAB = 4, 32768
 
 
@@ -436,6 +443,148 @@ def _kx_kernels(size: str, dev, timer: _Timer, ctx: int) -> list[dict]:
     return rows_out
 
 
+def _ns_config(size: str, kinds: str, vocab: int):
+    from ..models import nunosun as ns
+    width, H, G, window, rh, dh, dg, inter, E, top, side = NS_SIZES[size]
+    return ns.NunosunConfig.pattern(kinds, width, H, G, 128, 128, window, rh, 128, 128, dh, dg, 128, 128, inter * 3 // 2, inter // top, E, top,
+                                    side, vocab)
+
+
+def _ns_models(size: str, dev, prompt: int, slots: int):
+    from ..models import nunosun as ns
+    from ..models import qwen_hybrid as qh
+    width, H, G, _, _, dh, dg, inter, *_ = NS_SIZES[size]
+    cfg = _ns_config(size, NS_LAYERS, VOCAB)
+    new = lambda: ns.build_synthetic(cfg, dev, max_slots=slots, max_context=prompt + 192)
+    qcfg = qh.QwenHybridConfig(vocab_size=VOCAB, hidden_size=width, intermediate_size=inter, num_hidden_layers=LAYERS,
+                               num_attention_heads=H, num_key_value_heads=G, attn_output_gate=False, linear_num_key_heads=dg,
+                               linear_num_value_heads=dh, layer_types=["linear_attention", "full_attention"] * (LAYERS // 2))
+    old = lambda: qh.build_synthetic(qcfg, dev, max_slots=slots, max_context=prompt + 192)
+    return new, old
+
+
+def _ns_kernels(size: str, dev, timer: _Timer, ctx: int) -> list[dict]:
+    from ..models import nunosun as ns
+    from ..ops import attention, basic, decay, decoder, gdn, gemm, moe, scan, winattn
+    width, H, G, window, rh, dh, dg, inter, E, top, side = NS_SIZES[size]
+    ff, eff = inter * 3 // 2, inter // top
+    rnd = lambda *s, dt=torch.bfloat16: torch.randn(*s, device=dev, dtype=torch.float32).to(dt)
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    cfg = _ns_config(size, "dp", 64)
+    w = ns.NunosunWeights(cfg, ns.synth_state(cfg, 0, dev), dev)
+    dl, pl = w.layers
+    dw, pw, ew, dense = dl.mix, pl.mix, pl.ff, dl.ff
+    m = pw.left
+    rows_out, pair = _recorder(timer)
+    bs, pages = 64, (ctx + 63) // 64
+    for t in (8192, 32):
+        ar, one, zero = torch.arange(t, dtype=torch.int32, device=dev), torch.ones(t, dtype=torch.int32, device=dev), torch.zeros(t, dtype=torch.int32, device=dev)
+        seg = scan.Segments(ar, ar, ar, one, ar, 1) if t <= 32 else scan.Segments(zero, zero, i32([0]), i32([t]), i32([0]), t)
+        n_seq, pos1 = seg.first.numel(), ar + 5
+        # ---- the two residual steps of a layer, beside the plain residual add + norm
+        x32, x16, h16, d16 = rnd(t, width, dt=torch.float32), rnd(t, width), rnd(t, width), rnd(t, width)
+        xo, g16 = torch.empty_like(x32), torch.ones(width, device=dev, dtype=torch.bfloat16)
+        z = moe.router_logits(h16, ew.router)[:, :E]
+        idx, wts = moe.route(z, ew.router_b, top, "softmax_chosen", True, 1.0)
+        y, row = moe.experts_rows(h16, idx, ew.w13, ew.w2)
+        common = dict(ld=width, n=t, dtype=torch.bfloat16, x_out=xo)
+        like_step = (lambda: basic.add_rmsnorm(x16, d16, g16, 1e-5), t * width * 8, 0)
+        pair("step behind the pair and the experts (like: residual + norm)", f"{t} x {width}",
+             (lambda: decoder.branch_step(x32, width, 1e-5, normed=((d16, pw.left_w), (x16, pw.right_w)),
+                                          routed=decoder.Routed(y, row, idx, wts, E), copy=True, **common), t * width * (8 + 4 + 2 + 2 * top), 0),
+             like_step)
+        pair("step behind the delta rule and the dense unit (like: residual + norm)", f"{t} x {width}",
+             (lambda: decoder.branch_step(x32, width, 1e-5, plain=(d16, x16), copy=True, **common), t * width * (8 + 4 + 2), 0), like_step)
+        tails = torch.zeros(n_seq, 3, width, dtype=torch.bfloat16, device=dev)
+        pair("step in front of a layer, with the row convolution (like: residual + norm)", f"{t} x {width}",
+             (lambda: decoder.branch_step(x32, width, 1e-5, normed=((d16, dl.side_norm),), weight=dl.norm, conv=dl.conv, tail=tails, seg=seg,
+                                          positions=pos1, **common), t * width * (8 + 2 + 2 + (4 if t > 32 else 2)), 0), like_step)
+        # ---- activations and the side input
+        zu, gu = rnd(t, ff), rnd(t, 2 * inter)
+        pair("polynomial of row norms (like: SwiGLU unit)", f"{t} x {ff}", (lambda: decoder.poly_norm(zu, ff, dense.act, 1e-5, ff), t * ff * 4, 0),
+             (lambda: basic.silu_mul(gu), t * inter * 6, 0))
+        zs, gs, ids = rnd(t, side), rnd(t, 2 * side), ar % 64
+        pair("side gate (like: SwiGLU unit)", f"{t} x {side}", (lambda: decoder.token_gate(zs, w.side_embed, 0, ids), t * side * 6, 0),
+             (lambda: basic.silu_mul(gs), t * side * 6, 0))
+        # ---- experts
+        each = 3 * width * eff * 2
+        ebytes = int(torch.unique(idx).numel()) * each
+        i2, w2_ = moe.route(z, None, top, "softmax", False, 1.0)
+        ebytes2 = int(torch.unique(i2).numel()) * each
+        pair("routed experts (like: with combine)", f"{t} tokens, {top} of {E}",
+             (lambda: moe.experts_rows(h16, idx, ew.w13, ew.w2), ebytes + t * width * 2 * (1 + top), 2 * t * top * 3 * width * eff),
+             (lambda: moe.experts_forward(h16, i2, w2_, ew.w13, ew.w2, 0), ebytes2 + t * width * 4, 2 * t * top * 3 * width * eff))
+        pair("routing (like: sigmoid, normalised)", f"{t} x {E}",
+             (lambda: moe.route(z, ew.router_b, top, "softmax_chosen", True, 1.0), t * (z.stride(0) * 4 + top * 8), 0),
+             (lambda: moe.route(z, ew.router_b, top, "sigmoid", True, 1.0), t * (z.stride(0) * 4 + top * 8), 0))
+        # ---- attention prologue
+        proj, qkv = rnd(t, pw.proj.n), rnd(t, (H + 2 * G) * 128)
+        kc, vc = (torch.zeros(max(t, 64) // bs + 1, bs, G * 128, dtype=torch.bfloat16, device=dev) for _ in range(2))
+        k4, v4 = (torch.zeros(max(t, 64) // bs + 1, G, bs, 128, dtype=torch.bfloat16, device=dev) for _ in range(2))
+        qn, inv = torch.ones(128, device=dev, dtype=torch.bfloat16), attention.rope_inv_freq(64, 5e5, dev)
+        nb = t * (H + 2 * G) * 128 * 4
+        pair("attention prologue", f"{t} tokens", (lambda: winattn.head_prep(proj, m, ar, ar, kc, vc), nb, 0),
+             (lambda: attention.qk_norm_rope_append(qkv, 0, 128, False, qkv, H * 128, qkv, (H + G) * 128, qn, qn, True, 1e-5, inv, 64,
+                                                    ar, ar, k4, v4, H, G), nb, 0))
+        # ---- recurrences: projected rows in, gated rows out, state read and written once per sequence
+        dp, st = rnd(t, dw.proj.n), torch.zeros(n_seq, dh, 128, 128, dtype=torch.float32, device=dev)
+        ch = (2 * dg + dh) * 128
+        tail = torch.zeros(n_seq, 3, ch, dtype=torch.bfloat16, device=dev)
+        sbytes = t * (ch + 2 * dh * 128) * 2 + n_seq * (dh * 128 * 128 * 8 + 3 * ch * 4)
+        cw, ab, nw = rnd(ch, 4), rnd(t, 2 * dh), torch.ones(128, dtype=torch.bfloat16, device=dev)
+        gst, gtail = torch.zeros_like(st), torch.zeros_like(tail)
+        a_log, dtb = torch.zeros(dh, device=dev), torch.zeros(dh, device=dev)
+        if t <= 32:
+            w_ab = rnd(2 * dh, width)
+            like = lambda: gdn.decode_fused(dp[:, :ch + dh * 128], x16, w_ab, a_log, dtb, cw, gtail, gst, ar, nw, dh, dg)
+        else:
+            def like():
+                mixed = basic.conv_silu(dp[:, :ch], cw, gtail[0])
+                g, beta = basic.gdn_gates(ab, 0, dh, a_log, dtb, dh)
+                o = gdn.chunked(mixed, 0, dg * 128, 2 * dg * 128, g, beta, gst[0], dh, dg)
+                return basic.gated_rmsnorm(o.view(t * dh, 128), gate, nw)
+            gate = rnd(t * dh, 128)
+        pair("delta rule with convolution, decay, norm and gate", f"{t} tokens, {dh} heads x 128 x 128",
+             (lambda: decay.delta_rule(dp, dw.m, st, tail, seg, pos1, dw.o.k), sbytes, 0), (like, sbytes, 0))
+        del st, gst
+        rst, gst = (torch.zeros(n_seq, rh, 128, 128, dtype=torch.float32, device=dev) for _ in range(2))
+        rbytes = t * rh * 128 * 5 * 2 + n_seq * rh * 128 * 128 * 8
+        mixed, gg, beta, gate2 = rnd(t, 3 * rh * 128), -torch.rand(t, rh, device=dev), torch.rand(t, rh, device=dev), rnd(t * rh, 128)
+        core = (lambda: gdn.step(gst, ar, mixed, 0, rh * 128, 2 * rh * 128, gg, beta, rh, rh)) if t <= 32 else \
+            (lambda: gdn.chunked(mixed, 0, rh * 128, 2 * rh * 128, gg, beta, gst[0], rh, rh))
+        pair("retention with rotation, norm and gate (like: Gated DeltaNet, gated norm)", f"{t} tokens, {rh} heads x 128 x 128",
+             (lambda: decay.retention(proj[:, pw.right_off:], pw.right, rst, seg, pos1, pw.right_o.k), rbytes, 0),
+             (lambda: basic.gated_rmsnorm(core().view(t * rh, 128), gate2, nw), rbytes, 0))
+        del rst, gst
+        # ---- projections (like: none; all of them are the framework's GEMM)
+        for what, pr in (("pair projection", pw.proj), ("delta projection", dw.proj), ("up projection", dense.up), ("down projection", dense.down),
+                         ("side gate projection", dl.side_gate), ("side projection", dl.side_proj)):
+            xk = rnd(t, pr.k)
+            pair(what, f"{t} x {pr.n} x {pr.k}", (lambda: pr(xk), (pr.n * pr.k + t * pr.k + t * pr.n) * 2, 2 * t * pr.n * pr.k), None)
+    # ---- prompt attention
+    t = 8192
+    table = (torch.arange(t // bs, dtype=torch.int32, device=dev) + 1)[None]
+    q = rnd(t, H, 128)
+    kc, vc = (rnd(t // bs + 1, bs, G * 128) for _ in range(2))
+    k4, v4 = kc.view(-1, G, bs, 128), vc.view(-1, G, bs, 128)
+    out = torch.empty(t, H * 128, dtype=torch.bfloat16, device=dev)
+    pairs_n = sum(min(p + 1, window) for p in range(t))
+    args = (i32([0]), i32([t]), i32([t]), t)
+    pair("prompt attention (like: without bias)", f"{t} tokens, window {window}",
+         (lambda: winattn.prefill(q, m, kc, vc, table, *args, out), 0, 2 * pairs_n * H * 256),
+         (lambda: attention.prefill(q, k4, v4, table, *args, window=window), 0, 2 * pairs_n * H * 256))
+    for b in (1, 32):
+        tb = (torch.arange(b * pages, dtype=torch.int32, device=dev) + 1).view(b, pages)
+        kc, vc = (rnd(b * pages + 1, bs, G * 128) for _ in range(2))
+        k4, v4 = kc.view(-1, G, bs, 128), vc.view(-1, G, bs, 128)
+        q, ob = rnd(b, H, 128), torch.empty(b, H * 128, dtype=torch.bfloat16, device=dev)
+        pos, kvl, seen = i32([ctx - 1] * b), i32([ctx] * b), min(ctx, window)
+        pair("decode attention (like: without bias)", f"batch {b}, window {seen}",
+             (lambda: winattn.rows(q, m, kc, vc, tb, pos, ctx, ob), b * seen * G * 128 * 4, 0),
+             (lambda: attention.decode(q, k4, v4, tb, kvl, max_kv_len=seen, window=window), b * seen * G * 128 * 4, 0))
+    return rows_out
+
+
 def run(args) -> dict:
     from ..ops import _lib
     from .clocks import ClockSampler
@@ -449,7 +598,8 @@ def run(args) -> dict:
     sizes, models, kernels, closest = {
         "rutulix": (SIZES, _models, _kernels, "full-attention decoder, fp8 weights"),
         "zigasun": (ZG_SIZES, _zg_models, _zg_kernels, "Gated-DeltaNet / full-attention decoder, fp8 weights"),
-        "kemirax": (KX_SIZES, _kx_models, _kx_kernels, "latent-attention decoder with routed experts, bf16 weights")}[name]
+        "kemirax": (KX_SIZES, _kx_models, _kx_kernels, "latent-attention decoder with routed experts, bf16 weights"),
+        "nunosun": (NS_SIZES, _ns_models, _ns_kernels, "Gated-DeltaNet / full-attention decoder, fp8 weights")}[name]
     with torch.no_grad(), ClockSampler(0) as clk:
         for size in ([args.design_size] if args.design_size else list(sizes)):
             new, old = models(size, dev, prompt, slots)
@@ -459,6 +609,9 @@ def run(args) -> dict:
             elif name == "zigasun":
                 keys = ("width", "heads", "kv_heads", "dim", "vdim", "ff", "inner", "state", "dt_rank")
                 rec = {"layers": LAYERS, **dict(zip(keys, ZG_SIZES[size]))}
+            elif name == "nunosun":
+                keys = ("width", "heads", "kv_heads", "window", "retention_heads", "delta_heads", "delta_kv_heads", "swiglu_ff", "experts", "top", "side")
+                rec = {"layers": NS_LAYERS, **dict(zip(keys, NS_SIZES[size]))}
             else:
                 keys = ("width", "heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank", "gla_heads", "ff", "experts", "identity", "top")
                 rec = {"layers": KX_LAYERS, **dict(zip(keys, KX_SIZES[size]))}

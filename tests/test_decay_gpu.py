@@ -40,7 +40,8 @@ class Mixer:
             self.decay = 1.0 - 2.0 ** (-torch.linspace(0.1 if strong else 1.0, 9.0, heads, dtype=torch.float64))
             self.rot = dim if rot is None else rot
             f = 500.0 ** (-torch.arange(0, self.rot, 2, dtype=torch.float64) / max(self.rot, 1))
-            self.m = decay.Retention(heads, dim, d, vdim, v, EPS, self.rot, f.to(DEV), self.decay.float().to(DEV), torch.ones(v, device=DEV))
+            self.m = decay.Retention(heads, dim, d, vdim, v, EPS, self.rot, f.to(DEV), self.decay.float().to(DEV), torch.log2(self.decay).float().to(DEV),
+                                     torch.ones(v, device=DEV))
             self.parts = [("q", heads, dim, d), ("k", heads, dim, d), ("v", heads, vdim, v), ("g", heads, vdim, v)]
         else:
             self.a_log, self.dt = torch.randn(heads, generator=gen) * (2.0 if strong else 0.7), torch.randn(heads, generator=gen) - 2.0
