@@ -4,9 +4,10 @@
 // 16 contiguous bytes of a row as its share of two k-steps.  Prompt-sized batches use the big GEMMs instead.
 //
 // rows_linear_f32: the same for one matrix with few rows of its own and fp32 results (a router): more warps share K, because
-// the features alone would occupy a handful of SMs.
+// the features alone would occupy a handful of SMs.  rows_token_gate: that with gelu and the token's side embedding as epilogue.
 #include <cuda_bf16.h>
 #include <stdint.h>
+#include "gelu.cuh"
 #include "launch.h"
 #include "ops.h"
 
@@ -29,12 +30,32 @@ __device__ __forceinline__ void store2(float* p, int n, int N, float a, float b)
   if (n + 1 < N) p[n + 1] = b;
 }
 
+// Where a pair of features of a row goes: stored as it is, or behind gelu and times the row's token's embedding.
+template <typename Out>
+struct Plain {
+  Out* y;
+  int ldy, y_head;
+  __device__ __forceinline__ void put(int t, int h, int n, int N, float a, float b) const { store2(y + (size_t)t * ldy + h * y_head, n, N, a, b); }
+};
+struct TokenGate {
+  __nv_bfloat16* y;
+  const __nv_bfloat16* table;      // [vocab, ld_table], this projection's part from column `col` on
+  const int* ids;
+  int ldy, ld_table, col, vocab;
+  __device__ __forceinline__ void put(int t, int, int n, int N, float a, float b) const {
+    const int id = ids[t];
+    float2 e = make_float2(0.f, 0.f);
+    if (id >= 0 && id < vocab) e = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(table + (size_t)id * ld_table + col + n));
+    store2(y + (size_t)t * ldy, n, N, gelu_tanh(a) * e.x, gelu_tanh(b) * e.y);
+  }
+};
+
 // grid (features / 16, heads, rows / (16 MT)); K % 16 == 0 (32-wide chunks, the last may be half).  The warps'
 // sums are added up through shared memory.
-template <int MT, int WARPS, typename Out>
+template <int MT, int WARPS, typename Sink>
 __global__ void __launch_bounds__(WARPS * 32)
 head_linear_kernel(const __nv_bfloat16* __restrict__ x, int ldx, int x_head, const __nv_bfloat16* __restrict__ w,
-                   Out* __restrict__ y, int ldy, int y_head, int T, int N, int K) {
+                   Sink sink, int T, int N, int K) {
   __shared__ float red[WARPS][MT][2][4][32];
   pdl_grid_trigger();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gr = lane >> 2, kk = lane & 3;
@@ -81,21 +102,20 @@ head_linear_kernel(const __nv_bfloat16* __restrict__ x, int ldx, int x_head, con
       v1 += red[u][mt][nb][hf * 2 + 1][lane];
     }
     const int t = t0 + mt * 16 + gr + hf * 8, n = n0 + nb * 8 + kk * 2;
-    if (t < T && n < N) store2(y + (size_t)t * ldy + h * y_head, n, N, v0, v1);
+    if (t < T && n < N) sink.put(t, h, n, N, v0, v1);
   }
 }
 
-template <int WARPS, typename Out>
-int run(const void* x, int ldx, int x_head, const void* w, void* y, int ldy, int y_head, int T, int H, int N, int K, cudaStream_t stream) {
+template <int WARPS, typename Sink>
+int run(const void* x, int ldx, int x_head, const void* w, const Sink& sink, int T, int H, int N, int K, cudaStream_t stream) {
   const int mt = T <= 16 ? 1 : T <= 32 ? 2 : 4;
   if ((T + 16 * mt - 1) / (16 * mt) > 65535) return -6;
   const dim3 grid((N + NW - 1) / NW, H, (T + 16 * mt - 1) / (16 * mt)), block(WARPS * 32);
   auto xp = reinterpret_cast<const __nv_bfloat16*>(x);
   auto wp = reinterpret_cast<const __nv_bfloat16*>(w);
-  auto yp = reinterpret_cast<Out*>(y);
-  if (mt == 1) return (int)launch_pdl(head_linear_kernel<1, WARPS, Out>, grid, block, 0, stream, xp, ldx, x_head, wp, yp, ldy, y_head, T, N, K);
-  if (mt == 2) return (int)launch_pdl(head_linear_kernel<2, WARPS, Out>, grid, block, 0, stream, xp, ldx, x_head, wp, yp, ldy, y_head, T, N, K);
-  return (int)launch_pdl(head_linear_kernel<4, WARPS, Out>, grid, block, 0, stream, xp, ldx, x_head, wp, yp, ldy, y_head, T, N, K);
+  if (mt == 1) return (int)launch_pdl(head_linear_kernel<1, WARPS, Sink>, grid, block, 0, stream, xp, ldx, x_head, wp, sink, T, N, K);
+  if (mt == 2) return (int)launch_pdl(head_linear_kernel<2, WARPS, Sink>, grid, block, 0, stream, xp, ldx, x_head, wp, sink, T, N, K);
+  return (int)launch_pdl(head_linear_kernel<4, WARPS, Sink>, grid, block, 0, stream, xp, ldx, x_head, wp, sink, T, N, K);
 }
 
 }  // namespace
@@ -104,12 +124,22 @@ int run(const void* x, int ldx, int x_head, const void* w, void* y, int ldy, int
 extern "C" int b200_head_linear(const void* x, int ldx, int x_head, const void* w, void* y, int ldy, int y_head, int T, int H, int N,
                                 int K, cudaStream_t stream) {
   if (T <= 0 || H <= 0 || H > 65535 || N <= 0 || (N & 1) || K <= 0 || (K & 15) || ((ldx | x_head | ldy | y_head) & 7)) return -6;
-  return run<4, __nv_bfloat16>(x, ldx, x_head, w, y, ldy, y_head, T, H, N, K, stream);
+  return run<4>(x, ldx, x_head, w, Plain<__nv_bfloat16>{reinterpret_cast<__nv_bfloat16*>(y), ldy, y_head}, T, H, N, K, stream);
 }
 
 // y [T, ldy] fp32 = x [T, ldx] W [N, K]^T; K % 16 == 0.
 extern "C" int b200_rows_linear_f32(const void* x, int ldx, const void* w, float* y, int ldy, int T, int N, int K,
                                     cudaStream_t stream) {
   if (T <= 0 || N <= 0 || K <= 0 || (K & 15) || (ldx & 7) || ldy < N) return -6;
-  return run<8, float>(x, ldx, 0, w, y, ldy, 0, T, 1, N, K, stream);
+  return run<8>(x, ldx, 0, w, Plain<float>{y, ldy, 0}, T, 1, N, K, stream);
+}
+
+// y [T, ldy] bf16 = gelu(x [T, ldx] W [N, K]^T) * table[ids, col:col + N]; K % 16 == 0, N, ld_table and col even.
+extern "C" int b200_rows_token_gate(const void* x, int ldx, const void* w, const void* table, int ld_table, int col, int vocab,
+                                    const int* ids, void* y, int ldy, int T, int N, int K, cudaStream_t stream) {
+  if (T <= 0 || N <= 0 || (N & 1) || K <= 0 || (K & 15) || (ldx & 7) || (ldy & 1) || ldy < N || ((ld_table | col) & 1) || col < 0 ||
+      col + N > ld_table || vocab <= 0 || !ids)
+    return -6;
+  const TokenGate sink = {reinterpret_cast<__nv_bfloat16*>(y), reinterpret_cast<const __nv_bfloat16*>(table), ids, ldy, ld_table, col, vocab};
+  return run<8>(x, ldx, 0, w, sink, T, 1, N, K, stream);
 }

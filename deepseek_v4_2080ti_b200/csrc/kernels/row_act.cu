@@ -1,9 +1,11 @@
 // Activations that look at a whole row, or at the row's token.
 //
 //   poly_norm    y = a N(z) + b N(z^2) + c N(z^3) + e,   N: over the root mean square of the row's `cols` values
-//   token_gate   y = gelu_tanh(z) * table[token, part]   a layer's part of the token's side embedding
+//   token_gate   y = gelu_tanh(z) * table[token, part]   a layer's part of the token's side embedding (short batches take it
+//                in the epilogue of their projection, head_linear.cu)
 //
 // bf16 or fp32 data, fp32 arithmetic.  Rows are `ld` wide (a multiple of 8); columns past `cols` are written as zero.
+#include "gelu.cuh"
 #include "launch.h"
 #include "ops.h"
 #include "vec8.cuh"
@@ -80,10 +82,6 @@ __global__ void __launch_bounds__(512) poly_norm_kernel(const T* __restrict__ z,
       finish(r, v);
     }
   }
-}
-
-__device__ __forceinline__ float gelu_tanh(float z) {
-  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z)));
 }
 
 // table rows `ld_table` apart, the layer's part at column `col`.

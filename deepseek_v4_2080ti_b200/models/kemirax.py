@@ -449,13 +449,13 @@ class KemiraxRuntime(PagedRuntime):
             contexts = meta.setdefault("contexts", {})
             if src not in contexts:                  # layers that share a cache share its contiguous copy
                 contexts[src] = latent.gather(cache, m, self.block_table, meta["tile_seq"], meta["kv_len"], meta["kv_start"], meta["kv_total"])
-            latent.rotatepad_heads(q[:n], m, positions)
+            latent.rotate_heads(q[:n], m, positions)
             latent.attend_tiles(q[:n], m, *contexts[src], lw.ukv, meta["q_start"], meta["q_len"], meta["kv_len"], meta["kv_start"],
                                 meta["max_q_len"], out[:n])
         if n < t:                                    # single rows: queries are brought to the latents
             qr = q[n:]
             qa = torch.empty(t - n, m.heads, m.cache_width, dtype=y.dtype, device=y.device)
-            latent.rotatepad_heads(qr, m, positions[n:], qa, m.c)
+            latent.rotate_heads(qr, m, positions[n:], qa, m.c)
             latent.head_linear(qr, qr.stride(0), m.head_width, lw.uk, qa, qa.stride(0), qa.stride(1), t - n)
             if meta["mode"] == "decode":
                 o = latent.attend_rows(qa, m, cache, meta["block_table"], positions, meta["max_kv_len"])

@@ -524,7 +524,7 @@ class NunosunRuntime(PagedRuntime):
                 routed = self._experts(lw.ff, h)
             pending = {"normed": normed, "plain": plain, "routed": routed}
             c = step(x_out=x, copy=not exact)[0]
-            g = decoder.token_gate(lw.side_gate(x if exact else c), w.side_embed, i * w.side, ids)
+            g = decoder.token_gate(x if exact else c, lw.side_gate, w.side_embed, i * w.side, ids)
             pending = {"normed": ((lw.side_proj(g), lw.side_norm),)}
             if self.residual_tap is not None:
                 step(x_out=x)

@@ -277,13 +277,23 @@ def poly_norm(z: torch.Tensor, cols: int, coef: tuple[float, float, float, float
     return out
 
 
-def token_gate(z: torch.Tensor, table: torch.Tensor, col: int, ids: torch.Tensor) -> torch.Tensor:
-    """``gelu_tanh(z) * table[ids, col:col + columns of z]``."""
-    assert table.dtype == z.dtype and table.is_contiguous()
+TOKEN_GATE_MAX_ROWS = 64        # bf16 batches up to this take the row kernel: a GEMM tile would leave all but a few SMs idle
+
+
+def token_gate(x: torch.Tensor, w: Projection, table: torch.Tensor, col: int, ids: torch.Tensor) -> torch.Tensor:
+    """``gelu_tanh(x W^T) * table[ids, col:col + features of W]``; short bf16 batches in one launch."""
+    assert table.dtype == x.dtype and table.is_contiguous() and x.is_contiguous()
     _lib.check_indices(ids, 0, table.shape[0], 1)
-    out = torch.empty(z.shape, dtype=z.dtype, device=z.device)
-    rc = _lib.lib().b200_token_gate(_lib.ptr(z), z.stride(0), _lib.ptr(table), table.shape[1], col, table.shape[0], _lib.ptr(ids),
-                                    _lib.ptr(out), z.shape[1], z.shape[0], int(z.dtype == torch.float32), _lib.stream())
+    t, L = x.shape[0], _lib.lib()
+    out = torch.empty(t, w.n, dtype=x.dtype, device=x.device)
+    if w.w32 is None and t <= TOKEN_GATE_MAX_ROWS:
+        rc = L.b200_rows_token_gate(_lib.ptr(x), x.shape[1], _lib.ptr(w.packed.weight), _lib.ptr(table), table.shape[1], col, table.shape[0],
+                                    _lib.ptr(ids), _lib.ptr(out), w.n, t, w.n, w.k, _lib.stream())
+        _lib.check(rc, "rows_token_gate")
+        return out
+    z = w(x)
+    rc = L.b200_token_gate(_lib.ptr(z), z.stride(0), _lib.ptr(table), table.shape[1], col, table.shape[0], _lib.ptr(ids), _lib.ptr(out), w.n,
+                           t, int(x.dtype == torch.float32), _lib.stream())
     _lib.check(rc, "token_gate")
     return out
 

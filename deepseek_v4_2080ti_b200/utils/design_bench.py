@@ -503,9 +503,10 @@ def _ns_kernels(size: str, dev, timer: _Timer, ctx: int) -> list[dict]:
         zu, gu = rnd(t, ff), rnd(t, 2 * inter)
         pair("polynomial of row norms (like: SwiGLU unit)", f"{t} x {ff}", (lambda: decoder.poly_norm(zu, ff, dense.act, 1e-5, ff), t * ff * 4, 0),
              (lambda: basic.silu_mul(gu), t * inter * 6, 0))
-        zs, gs, ids = rnd(t, side), rnd(t, 2 * side), ar % 64
-        pair("side gate (like: SwiGLU unit)", f"{t} x {side}", (lambda: decoder.token_gate(zs, w.side_embed, 0, ids), t * side * 6, 0),
-             (lambda: basic.silu_mul(gs), t * side * 6, 0))
+        ids, wg = ar % 64, gemm.PackedLinear.from_bf16(rnd(2 * side, width))
+        pair("side gate with its projection (like: SwiGLU unit with its projection)", f"{t} x {side} x {width}",
+             (lambda: decoder.token_gate(h16, dl.side_gate, w.side_embed, 0, ids), (side * width + t * width + 2 * t * side) * 2, 2 * t * side * width),
+             (lambda: basic.silu_mul(gemm.linear(h16, wg)), (2 * side * width + t * width + t * side) * 2, 4 * t * side * width))
         # ---- experts
         each = 3 * width * eff * 2
         ebytes = int(torch.unique(idx).numel()) * each
@@ -558,7 +559,7 @@ def _ns_kernels(size: str, dev, timer: _Timer, ctx: int) -> list[dict]:
         del rst, gst
         # ---- projections (like: none; all of them are the framework's GEMM)
         for what, pr in (("pair projection", pw.proj), ("delta projection", dw.proj), ("up projection", dense.up), ("down projection", dense.down),
-                         ("side gate projection", dl.side_gate), ("side projection", dl.side_proj)):
+                         ("side projection", dl.side_proj)):
             xk = rnd(t, pr.k)
             pair(what, f"{t} x {pr.n} x {pr.k}", (lambda: pr(xk), (pr.n * pr.k + t * pr.k + t * pr.n) * 2, 2 * t * pr.n * pr.k), None)
     # ---- prompt attention
