@@ -115,7 +115,15 @@ int run(const void* x, int ldx, int x_head, const void* w, const Sink& sink, int
   auto wp = reinterpret_cast<const __nv_bfloat16*>(w);
   if (mt == 1) return (int)launch_pdl(head_linear_kernel<1, WARPS, Sink>, grid, block, 0, stream, xp, ldx, x_head, wp, sink, T, N, K);
   if (mt == 2) return (int)launch_pdl(head_linear_kernel<2, WARPS, Sink>, grid, block, 0, stream, xp, ldx, x_head, wp, sink, T, N, K);
-  return (int)launch_pdl(head_linear_kernel<4, WARPS, Sink>, grid, block, 0, stream, xp, ldx, x_head, wp, sink, T, N, K);
+  if constexpr (WARPS <= 8)
+    return (int)launch_pdl(head_linear_kernel<4, WARPS, Sink>, grid, block, 0, stream, xp, ldx, x_head, wp, sink, T, N, K);
+  return -6;
+}
+
+// One matrix: few blocks, so many warps share K (their sums fit into shared memory for up to 32 rows at a time).
+template <typename Sink>
+int run_rows(const void* x, int ldx, const void* w, const Sink& sink, int T, int N, int K, cudaStream_t stream) {
+  return T <= 32 && K >= 1024 ? run<16>(x, ldx, 0, w, sink, T, 1, N, K, stream) : run<8>(x, ldx, 0, w, sink, T, 1, N, K, stream);
 }
 
 }  // namespace
@@ -131,7 +139,7 @@ extern "C" int b200_head_linear(const void* x, int ldx, int x_head, const void* 
 extern "C" int b200_rows_linear_f32(const void* x, int ldx, const void* w, float* y, int ldy, int T, int N, int K,
                                     cudaStream_t stream) {
   if (T <= 0 || N <= 0 || K <= 0 || (K & 15) || (ldx & 7) || ldy < N) return -6;
-  return run<8>(x, ldx, 0, w, Plain<float>{y, ldy, 0}, T, 1, N, K, stream);
+  return run_rows(x, ldx, w, Plain<float>{y, ldy, 0}, T, N, K, stream);
 }
 
 // y [T, ldy] bf16 = gelu(x [T, ldx] W [N, K]^T) * table[ids, col:col + N]; K % 16 == 0, N, ld_table and col even.
@@ -141,5 +149,5 @@ extern "C" int b200_rows_token_gate(const void* x, int ldx, const void* w, const
       col + N > ld_table || vocab <= 0 || !ids)
     return -6;
   const TokenGate sink = {reinterpret_cast<__nv_bfloat16*>(y), reinterpret_cast<const __nv_bfloat16*>(table), ids, ldy, ld_table, col, vocab};
-  return run<8>(x, ldx, 0, w, sink, T, 1, N, K, stream);
+  return run_rows(x, ldx, w, sink, T, N, K, stream);
 }

@@ -9,6 +9,7 @@ Activations are bf16 (serving) or fp32 (``dtype``).
 """
 from __future__ import annotations
 
+import contextlib
 import json
 import math
 import os
@@ -17,7 +18,7 @@ from typing import Any, Iterator
 
 import torch
 
-from ..ops import decay, decoder, moe, winattn
+from ..ops import decay, decoder, gemm, moe, winattn
 from ..ops.decay import DeltaRule, Retention
 from ..ops.decoder import Projection, Routed, cat_rows, pad16, pad_heads
 from ..ops.winattn import WindowAttention
@@ -123,8 +124,8 @@ class NunosunConfig:
                     raise ValueError(f"layer {i}: heads must be a multiple of kv_heads")
                 if left.size < 1:
                     raise ValueError(f"layer {i}: the window holds at least the position itself")
-                if len(right.decay) != right.heads or not all(0.0 < d <= 1.0 for d in right.decay):
-                    raise ValueError(f"layer {i}: one decay in (0, 1] per retention head")
+                if len(right.decay) != right.heads or not all(0.0 <= d <= 1.0 for d in right.decay):
+                    raise ValueError(f"layer {i}: one decay in [0, 1] per retention head")
                 if right.rot_dims % 2 or right.rot_dims > right.dim:
                     raise ValueError(f"layer {i}: rot.dims must be even and at most dim")
                 mix: PairSpec | DeltaSpec = PairSpec(left, right)
@@ -465,6 +466,7 @@ class NunosunRuntime(PagedRuntime):
             self.conv_tail.append(tail)
             self.state.append(self.slot_state(m.heads, m.d, m.v, dtype=torch.float32, name=f"recurrent state of layer {i}"))
             self.row_tail.append(self.slot_state(max(cfg.taps - 1, 1), weights.ld, dtype=weights.dtype, name=f"row tail of layer {i}"))
+        self._side_stream: torch.cuda.Stream | None = None
         self.residual_tap = None                      # debugging: called with (layer, residual [T, width]) after every layer
 
     def history_floor(self, length: int) -> int:
@@ -496,6 +498,25 @@ class NunosunRuntime(PagedRuntime):
         y, row = moe.experts_rows(h, idx, ew.w13, ew.w2)
         return Routed(y, row, idx, weights, f.experts)
 
+    def _feed_forward(self, ff: DenseWeights | ExpertsWeights, h: torch.Tensor) -> dict:
+        if isinstance(ff, DenseWeights):
+            return {"dense": ff.down(decoder.poly_norm(ff.up(h), ff.ff, ff.act, self.cfg.eps, ff.down.k))}
+        return {"routed": self._experts(ff, h)}
+
+    @contextlib.contextmanager
+    def _beside(self, on: bool):
+        """Work inside runs on a second stream, beside what the caller launches until it leaves ``join`` (yielded) behind.
+        Tensors made inside are read after the join only, and the next work on that stream waits for those readers."""
+        if not on:
+            yield lambda: None
+            return
+        if self._side_stream is None:
+            self._side_stream = torch.cuda.Stream(self.device)
+        main, side = torch.cuda.current_stream(self.device), self._side_stream
+        side.wait_event(main.record_event())
+        with torch.cuda.stream(side), gemm.scratch(1):
+            yield lambda: main.wait_event(side.record_event())
+
     def _forward(self, ids, positions, kv_slots, meta, rows):
         cfg, w, n = self.cfg, self.w, ids.numel()
         x = torch.empty(n, w.ld, dtype=torch.float32, device=self.device)
@@ -512,17 +533,21 @@ class NunosunRuntime(PagedRuntime):
 
         for i, lw in enumerate(w.layers):
             _, h, m = step(x_out=x, weight=lw.norm, conv=lw.conv, tail=self.row_tail[i], seg=meta["segments"], positions=positions)
-            normed, plain, routed = (), (), None
+            # a decoding step is bound by launches and by the weights' stream: the sublayers run beside each other
+            join, extra = lambda: None, {}
+            if lw.ff is not None:
+                with self._beside(meta["mode"] == "decode") as join:
+                    extra = self._feed_forward(lw.ff, h)
             if isinstance(lw.mix, PairWeights):
-                normed = self._pair(i, lw.mix, m, positions, kv_slots, meta)
+                pending = {"normed": self._pair(i, lw.mix, m, positions, kv_slots, meta), "plain": ()}
             else:
                 d = lw.mix
-                plain = (d.o(decay.delta_rule(d.proj(m), d.m, self.state[i], self.conv_tail[i], meta["segments"], positions, d.o.k)),)
-            if isinstance(lw.ff, DenseWeights):
-                plain += (lw.ff.down(decoder.poly_norm(lw.ff.up(h), lw.ff.ff, lw.ff.act, cfg.eps, lw.ff.down.k)),)
-            elif lw.ff is not None:
-                routed = self._experts(lw.ff, h)
-            pending = {"normed": normed, "plain": plain, "routed": routed}
+                y = d.o(decay.delta_rule(d.proj(m), d.m, self.state[i], self.conv_tail[i], meta["segments"], positions, d.o.k))
+                pending = {"plain": (y,)}
+            join()
+            if "dense" in extra:
+                pending["plain"] += (extra["dense"],)
+            pending["routed"] = extra.get("routed")
             c = step(x_out=x, copy=not exact)[0]
             g = decoder.token_gate(x if exact else c, lw.side_gate, w.side_embed, i * w.side, ids)
             pending = {"normed": ((lw.side_proj(g), lw.side_norm),)}

@@ -7,6 +7,7 @@ and bf16 matvec/matmul (cpp_engine/backends/cuda/kernels/bf16_ops.cu:30-167).
 """
 from __future__ import annotations
 
+import contextlib
 import ctypes
 import os
 from dataclasses import dataclass
@@ -74,15 +75,27 @@ class PackedLinear:
         return self.weight.numel() * self.weight.element_size() + (0 if self.scales is None else self.scales.numel() * 4)
 
 
-_workspaces: dict[int, tuple[torch.Tensor, torch.Tensor]] = {}
+_workspaces: dict[tuple[int, int], tuple[torch.Tensor, torch.Tensor]] = {}
+_scratch = 0
 _outgrown: list[torch.Tensor] = []      # smaller scratch buffers stay alive: captured graphs hold their addresses
 MAX_TILE_COUNTERS = 1 << 16
+
+
+@contextlib.contextmanager
+def scratch(number: int):
+    """Products inside use this split-K scratch: those on a stream beside another need one of their own."""
+    global _scratch
+    old, _scratch = _scratch, number
+    try:
+        yield
+    finally:
+        _scratch = old
 
 
 def _workspace(nfloats: int, device) -> tuple[torch.Tensor, torch.Tensor]:
     """(fp32 split-K scratch, zeroed int32 tile counters) of the device; grown on demand, never shrunk.
     The kernel leaves the counters at zero, so they are cleared only when allocated."""
-    key = torch.device(device).index or 0
+    key = (torch.device(device).index or 0, _scratch)
     ws = _workspaces.get(key)
     if ws is None or ws[0].numel() < nfloats:
         if ws is not None:
